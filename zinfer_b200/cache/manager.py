@@ -1,8 +1,9 @@
 """The cache manager: which pages and which state slot each request holds.
 
 Keys and values live in pages of ``page_size`` tokens.  Caches with the same need
-(kv heads, key and value size, window and kept first tokens, with or without values) form a *group*: a group has a page pool of its own
-and one block table per request, valid for every cache of the group.  A request's
+(kv heads, key and value size, window and kept first tokens, with or without values, tokens per entry) form a *group*: a group has a page pool of its own
+and one block table per request, valid for every cache of the group.  A group may keep one entry per several tokens (means over
+blocks of tokens): its pages hold ``page_size`` entries, and an entry gets its place with the last of its tokens.  A request's
 pages are given back when it ends, and, in a group with a window, as soon as the
 window has passed them (except those that hold the first tokens the group keeps visible).  Beside the pages, each request holds one slot for
 per-request state of fixed size (used by mixers that keep a state instead of keys;
@@ -27,6 +28,7 @@ from typing import Hashable, Optional
 
 from ..csrc import host
 from .pages import GroupPool, OutOfPages
+from .sizing import entry_pages
 
 
 @dataclass(frozen=True)
@@ -37,6 +39,7 @@ class KVNeedKey:
     values: bool = True        # False: pages of keys only
     value_dim: Optional[int] = None   # size of a value where it differs from a key's
     keep_first: int = 0        # with a window: the request's first tokens whose pages are never given back
+    tokens_per_entry: int = 1  # above 1: one key and value stands for this many tokens
 
 
 @dataclass
@@ -74,7 +77,9 @@ class CacheManager:
     def __init__(self, kv_needs: dict[str, "KVNeedKey"], state_caches: list[str], page_size: int,
                  num_pages: int | dict[KVNeedKey, int], max_requests: int):
         """``kv_needs`` maps a cache name to what it needs; ``num_pages`` is the size
-        of each group's pool (one number for all groups, or one per need)."""
+        of each group's pool (one number for all groups, or one per need).  With one number, a group whose entries
+        stand for several tokens gets as many pages as those tokens need (and one more per request, for the page
+        each request has only begun)."""
         if page_size <= 0:
             raise ValueError("page_size must be positive")
         self.page_size = page_size
@@ -87,11 +92,14 @@ class CacheManager:
             vd = getattr(need, "value_dim", None)
             key = KVNeedKey(need.num_kv_heads, need.head_dim, need.window, getattr(need, "values", True),
                             None if vd is None or vd == need.head_dim else int(vd),
-                            int(getattr(need, "keep_first", 0) or 0) if need.window is not None else 0)
+                            int(getattr(need, "keep_first", 0) or 0) if need.window is not None else 0,
+                            int(getattr(need, "tokens_per_entry", 1) or 1))
             if key.window is not None and key.window <= 0:
                 raise ValueError(f"cache {name!r}: window must be positive")
             if key.keep_first < 0:
                 raise ValueError(f"cache {name!r}: the kept first tokens cannot be fewer than none")
+            if key.tokens_per_entry < 1 or (key.tokens_per_entry > 1 and key.window is not None):
+                raise ValueError(f"cache {name!r}: an entry stands for at least one token, and entries of several tokens have no window")
             if key in keys:
                 gi = keys.index(key)
                 self.group_of[name] = (gi, len(members[gi]))
@@ -99,7 +107,8 @@ class CacheManager:
             else:
                 keys.append(key)
                 members.append([name])
-                sizes.append(int(num_pages[key] if isinstance(num_pages, dict) else num_pages))
+                sizes.append(int(num_pages[key]) if isinstance(num_pages, dict)
+                             else entry_pages(int(num_pages), key.tokens_per_entry, max_requests))
                 self.group_of[name] = (len(keys) - 1, 0)
         if any(n < 0 for n in sizes):
             raise ValueError("num_pages must be >= 0")
@@ -113,6 +122,8 @@ class CacheManager:
         for gi, k in enumerate(keys):
             if k.keep_first:
                 self._lib.zi_cache_keep_first(self._handle, gi, k.keep_first)
+            if k.tokens_per_entry > 1:
+                self._lib.zi_cache_tokens_per_entry(self._handle, gi, k.tokens_per_entry)
         self.groups: list[KVGroup] = [
             KVGroup(key, names, GroupPool(self._handle, gi, f"kv pages of group {gi}"))
             for gi, (key, names) in enumerate(zip(keys, members))]
@@ -246,17 +257,17 @@ class CacheManager:
         self._lib.zi_cache_table(self._handle, nid, group, out, n)
         return list(out[:n])
 
-    def blocks_held(self, request_id: Hashable) -> int:
-        """Blocks (pages, released ones included) that the request's shortest block table spans."""
-        nid = self._live(request_id).native_id
-        return min((self._lib.zi_cache_table_len(self._handle, nid, gi) for gi in range(len(self.groups))), default=0)
+    def room(self, request_id: Hashable) -> int:
+        """The most tokens that could be reserved for the request right now (in every group, with the pages that are free)."""
+        return int(self._lib.zi_cache_room(self._handle, self._live(request_id).native_id))
 
     # ---------------------------------------------------------------- accounting
     def free_pages(self) -> list[int]:
         return [g.pool.num_free for g in self.groups]
 
-    def min_free_pages(self) -> int:
-        return min((g.pool.num_free for g in self.groups), default=0)
+    def fullest_group(self) -> KVGroup:
+        """The group with the smallest share of free pages (the first of them)."""
+        return min(self.groups, key=lambda g: g.pool.num_free / max(1, g.pool.num_pages))
 
     def check(self) -> None:
         """No page lost, held twice or freed twice; no slot either."""

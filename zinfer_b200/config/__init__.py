@@ -4,6 +4,7 @@ from .luvavik import LuvavikConfig, luvavik_model_spec
 from .rogosun import RogosunConfig, rogosun_model_spec
 from .vumezen import VumezenConfig, vumezen_model_spec
 from .sepitar import SepitarConfig, sepitar_model_spec
+from .kesitar import KesitarConfig, kesitar_model_spec
 from .registry import (Family, UnknownArchitecture, family_for, load_config, register_family, registered,
                        unregister_family)
 
@@ -22,7 +23,11 @@ register_family(Family(name="Vumezen", model_type="vumezen", config_class=Vumeze
 register_family(Family(name="Sepitar", model_type="sepitar", config_class=SepitarConfig,
                        model_spec=sepitar_model_spec), replace=True)
 
+register_family(Family(name="Kesitar", model_type="kesitar", config_class=KesitarConfig,
+                       model_spec=kesitar_model_spec), replace=True)
+
 __all__ = [
+    "KesitarConfig", "kesitar_model_spec",
     "SepitarConfig", "sepitar_model_spec",
     "VumezenConfig", "vumezen_model_spec",
     "ConfigError", "Family", "LayerSpec", "LuvavikConfig", "ModelSpec", "PartSpec", "Qwen3Config", "luvavik_model_spec", "ScheduleEntry",

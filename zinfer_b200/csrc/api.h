@@ -11,7 +11,7 @@ extern "C" {
 
 const char* zi_last_error();
 
-int zi_embed_gather(float* h, const void* table, int table_dtype, const int* ids, int T, int H, int V,
+int zi_embed_gather(float* h, const void* table, int table_dtype, const int* ids, int T, int H, int V, float scale,
                     cudaStream_t stream);
 // h[t] = scale * table[ids[t]] + bigram[row], row = (previous token * mul_prev + token * mul_cur) mod buckets, or row
 // `buckets` for a request's first token (position 0).  The token before a step's first token of a request comes from
@@ -137,7 +137,8 @@ int zi_paged_attention_mods(void* out, int out_stride, const void* q, int q_stri
                             const int* kv_lens, const int* tile_seq, const int* tile_q0, int n_tiles, int nq, int nkv,
                             int d, int dv, int v_row, int page_size, int window, int keep_first, float scale,
                             int skip_from, int skip_single, float sink, const float* sink_logit, float softcap,
-                            const float* dist_bias, int n_dist, cudaStream_t stream);
+                            const float* dist_bias, int n_dist, const void* kpool, const void* vpool, const int* pool_tables,
+                            int pool_bt_stride, int pool_per, cudaStream_t stream);
 // The tensor-core kernels (mma.sync, softmax weights as two bfloat16 parts) with the same changes to the score.
 int zi_attention_prefill_mma_mods(void* out, int out_stride, const void* q, int q_stride, const void* kcache,
                                   const void* vcache, const int* block_tables, int bt_stride, const int* cu_q,
@@ -157,6 +158,26 @@ int zi_qkv_rows_prepare(const void* src, int src_dtype, int src_stride, const fl
                         const float* qw, const float* kw, float eps, int rot_dims, const float* cos_t, const float* sin_t,
                         int n_table_pos, const int* positions, void* kcache, void* vcache, const int* slots, int page_size,
                         cudaStream_t stream);
+// What follows a projection row [q heads | k heads | v heads] whose q and k heads are normed one by one: biases, an RMS norm
+// per head (weight [d], shared by the heads), rotation of the first rot_dims dimensions, values mixed with v_in
+// (float32 [T, nkv * dv]: v <- (1 - v_lambda) v + v_lambda v_in) and copied to v_out where given, q into a tensor of its
+// own, k and v into the token's page slot.  The rows come whole or as partial sums part[splits][T][src_stride].
+int zi_qkv_heads_prepare(const void* src, int src_dtype, int src_stride, const float* part, int splits, long long zstride,
+                         const float* bias, void* q_out, int q_stride, int out_dtype, int T, int nq, int nkv, int d, int dv,
+                         const float* qw, const float* kw, float eps, int rot_dims, const float* cos_t, const float* sin_t,
+                         int n_table_pos, const int* positions, void* kcache, void* vcache, const int* slots, int page_size,
+                         const float* v_in, float v_lambda, float* v_out, cudaStream_t stream);
+// The pooled entry (means of keys and values) of every block of `per` tokens that this step's tokens complete:
+// entry_slots[t] is where the entry goes that token t completes, or -1.
+int zi_pool_blocks(const void* kcache, const void* vcache, int dtype, const int* block_tables, int bt_stride, void* kpool,
+                   void* vpool, const int* entry_slots, const int* positions, const int* cu_q, int n_seqs, int T, int nkv, int d,
+                   int dv, int per, int page_size, cudaStream_t stream);
+// The seam of a block that norms its sublayers' inputs and outputs: h += N_post(scale * a) * w_post, x_out = N_pre(h) * w_pre;
+// norms: 0 RMS, 1 layer norm (mean taken off).  a comes whole or as partial sums, or not at all; w_post null: no norm of
+// the update; w_pre null: no second norm; rows: picked rows' x, h left as it is.
+int zi_sandwich_norm(float* h, const void* a, int a_dtype, const float* part, int splits, long long zstride, float scale,
+                     const float* w_post, int post_kind, float post_eps, const float* w_pre, int pre_kind, float pre_eps,
+                     void* x_out, int out_dtype, const int* rows, int n_rows, int H, cudaStream_t stream);
 // RMS norm of rows of activations: out[t] = x[t] * w / sqrt(mean(x[t]^2) + eps).
 int zi_rmsnorm_rows(void* out, int ldo, int out_dtype, const void* x, int ldx, int x_dtype, const float* w, float eps, int T,
                     int n, cudaStream_t stream);
@@ -207,6 +228,12 @@ int zi_linear_recurrence(float* out, int ldo, const void* q, int ldq, const void
                          int ldv, int v_dtype, const float* decay, int ldg, const float* beta, int ldb, float q_scale,
                          float* state, long long slot_stride, int H, int G, int D, int V, int delta, const int* cu_q,
                          const int* state_slots, int n_seqs, cudaStream_t stream);
+// The form whose forget gate decides what is written: g = l + (1 - l) sigmoid(z + b), k = 1 - g, q = silu(raw q); q, z, v
+// float32 projections, whole (splits 1) or split-K partial sums zstride apart.
+int zi_linear_recurrence_gated(float* out, int ldo, const float* q, int ldq, const float* z, int ldz, const float* v, int ldv,
+                               int splits, long long zstride, const float* f_bias, const float* lower, float* state,
+                               long long slot_stride, int H, int D, int V, const int* cu_q, const int* state_slots, int n_seqs,
+                               cudaStream_t stream);
 int zi_head_norm_gate(void* out, int out_dtype, int ldo, const float* o, int ldi, const float* w, float eps,
                       const void* gate, int gate_dtype, int ldgate, int act, int T, int heads, int V, cudaStream_t stream);
 int zi_moe_router_grouped(int* chosen, float* weight, const void* x, int x_dtype, int ldx, const void* w, int w_dtype, int T,

@@ -19,7 +19,9 @@ constexpr int BQ = 16, BK = 32, THREADS = 128, ROWS_PER_WARP = BQ / (THREADS / 3
 // Values may have another size than keys and may lie in the key rows themselves (a latent cache whose row
 // serves as key and, in its first dv columns, as value): dv value columns are read from rows of
 // v_row elements in `vcache`; the output has dv columns per head.  MAXJ * 32 bounds dv.
-// With a window, query i sees key j <= i if i - j < window or j < keep_first.
+// With a window, query i sees key j <= i if i - j < window or j < keep_first.  With pooled blocks (pool.per > 0) it also
+// sees one key and value for every block of `per` tokens that lies wholly before its window: entry b of the request's
+// pooled pages, if b per + per - 1 <= i - window.  They are walked first; all keys share one softmax.
 // Changes to the score, each off unless given: softcap c (s <- c tanh(s / c) after the scale), dist_bias
 // [heads][n_dist] (a bias by the distance i - j, distances from n_dist - 1 on share the last entry; added after
 // the cap), sink_logit [heads] (exp(sink_logit[h]) joins head h's denominator; it has no value).
@@ -32,7 +34,7 @@ paged_attention_kernel(T* __restrict__ out, int out_stride, const T* __restrict_
                        const int* __restrict__ tile_q0, int nq, int nkv, int d, int page_size, int window,
                        float scale, int dv, int v_row, int skip_from, int skip_single, float sink, int keep_first,
                        const float* __restrict__ sink_logit, float softcap, const float* __restrict__ dist_bias,
-                       int n_dist) {
+                       int n_dist, const PooledKeys pool) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float smem[];
@@ -69,8 +71,15 @@ paged_attention_kernel(T* __restrict__ out, int out_stride, const T* __restrict_
     for (int j = 0; j < MAXJ; ++j) acc[i][j] = 0.f;
   }
 
-  for (int kt = keep_end > 0 ? 0 : (kv_begin / BK) * BK; kt < kv_end; kt += BK) {
-    if (kt >= keep_end && kt + BK <= kv_begin) {   // a tile wholly between the kept first tokens and the window
+  const int n_pooled = pooled_visible(pool, last_pos, window);          // what the tile's last query sees
+  const T* kpool = static_cast<const T*>(pool.k);
+  const T* vpool = static_cast<const T*>(pool.v);
+  const int* pbt = pool.block_tables + (size_t)seq * pool.bt_stride;
+  // tiles of pooled entries first (ahead > 0), then the tokens'
+  int ahead = (n_pooled + BK - 1) / BK, kt = ahead > 0 ? 0 : (keep_end > 0 ? 0 : (kv_begin / BK) * BK);
+  for (; ahead > 0 || kt < kv_end; kt += BK) {
+    const bool of_blocks = ahead > 0;
+    if (!of_blocks && kt >= keep_end && kt + BK <= kv_begin) {   // a tile wholly between the kept first tokens and the window
       kt = (kv_begin / BK) * BK - BK;
       continue;
     }
@@ -79,7 +88,10 @@ paged_attention_kernel(T* __restrict__ out, int out_stride, const T* __restrict_
       const int kk = e / d, c = e % d;
       const int j = kt + kk;
       float kval = 0.f;
-      if ((j >= kv_begin || j < keep_end) && j < kv_end) {
+      if (of_blocks) {
+        const int page = j < n_pooled ? pbt[j / page_size] : -1;
+        if (page >= 0) kval = to_f32(kpool[(((size_t)page * nkv + kvh) * page_size + (j % page_size)) * d + c]);
+      } else if ((j >= kv_begin || j < keep_end) && j < kv_end) {
         const int page = bt[j / page_size];
         if (page >= 0) kval = to_f32(kcache[(((size_t)page * nkv + kvh) * page_size + (j % page_size)) * d + c]);
       }
@@ -89,7 +101,10 @@ paged_attention_kernel(T* __restrict__ out, int out_stride, const T* __restrict_
       const int kk = e / dv, c = e % dv;
       const int j = kt + kk;
       float vval = 0.f;
-      if ((j >= kv_begin || j < keep_end) && j < kv_end) {
+      if (of_blocks) {
+        const int page = j < n_pooled ? pbt[j / page_size] : -1;
+        if (page >= 0) vval = to_f32(vpool[(((size_t)page * nkv + kvh) * page_size + (j % page_size)) * dv + c]);
+      } else if ((j >= kv_begin || j < keep_end) && j < kv_end) {
         const int page = bt[j / page_size];
         if (page >= 0) vval = to_f32(vcache[(((size_t)page * nkv + kvh) * page_size + (j % page_size)) * v_row + c]);
       }
@@ -110,7 +125,8 @@ paged_attention_kernel(T* __restrict__ out, int out_stride, const T* __restrict_
       for (int c = 0; c < d; ++c) s = fmaf(qr[c], kr[c], s);
       s *= scale;
       if (softcap > 0.f) s = softcap * tanhf(s / softcap);
-      const bool visible = j <= pos && (window <= 0 || j > pos - window || j < keep_first);
+      const bool visible = of_blocks ? j < pooled_visible(pool, pos, window)
+                                     : j <= pos && (window <= 0 || j > pos - window || j < keep_first);
       if (!visible) s = -INFINITY;
       else if (dist_bias) s += dist_bias[(size_t)h * n_dist + min(pos - j, n_dist - 1)];   // not scaled, not capped
       const float m_new = fmaxf(m[i], warp_max(s));
@@ -139,6 +155,7 @@ paged_attention_kernel(T* __restrict__ out, int out_stride, const T* __restrict_
         }
       }
     }
+    if (of_blocks && --ahead == 0) kt = (keep_end > 0 ? 0 : (kv_begin / BK) * BK) - BK;   // on with the tokens
   }
 #pragma unroll
   for (int i = 0; i < ROWS_PER_WARP; ++i) {
@@ -198,17 +215,19 @@ extern "C" int zi_paged_attention_mask(void* out, int out_stride, const void* q,
                                        cudaStream_t stream) {
   return zi_paged_attention_mods(out, out_stride, q, q_stride, dtype, kcache, vcache, block_tables, bt_stride, cu_q, kv_lens,
                                  tile_seq, tile_q0, n_tiles, nq, nkv, d, dv, v_row, page_size, window, keep_first, scale,
-                                 skip_from, skip_single, sink, nullptr, 0.f, nullptr, 0, stream);
+                                 skip_from, skip_single, sink, nullptr, 0.f, nullptr, 0, nullptr, nullptr, nullptr, 0, 0, stream);
 }
 
-// The same with the changes to the score: a learned sink per head, a cap, a bias by distance.
+// The same with the changes to the score (a learned sink per head, a cap, a bias by distance), and with pooled keys and
+// values: pages of one entry per pool_per tokens beside the window's tokens (0: none).
 extern "C" int zi_paged_attention_mods(void* out, int out_stride, const void* q, int q_stride, int dtype,
                                        const void* kcache, const void* vcache, const int* block_tables, int bt_stride,
                                        const int* cu_q, const int* kv_lens, const int* tile_seq, const int* tile_q0,
                                        int n_tiles, int nq, int nkv, int d, int dv, int v_row, int page_size, int window,
                                        int keep_first, float scale, int skip_from, int skip_single, float sink,
                                        const float* sink_logit, float softcap, const float* dist_bias, int n_dist,
-                                       cudaStream_t stream) {
+                                       const void* kpool, const void* vpool, const int* pool_tables, int pool_bt_stride,
+                                       int pool_per, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (!(softcap >= 0.f)) return zi_refuse("paged_attention: the cap on the scores must not be negative");
   if (dist_bias && n_dist <= 0) return zi_refuse("paged_attention: a bias by distance needs a table");
@@ -220,6 +239,9 @@ extern "C" int zi_paged_attention_mods(void* out, int out_stride, const void* q,
   if (dv <= 0 || dv > 32 * WIDE || v_row < dv) return zi_refuse("paged_attention: %d value columns of rows of %d, keys of %d", dv, v_row, d);
   if (nkv <= 0 || nq % nkv) return zi_refuse("paged_attention: %d query heads do not divide into %d kv heads", nq, nkv);
   if (page_size <= 0) return zi_refuse("paged_attention: page_size %d", page_size);
+  if (pool_per > 0 && (!kpool || !vpool || !pool_tables || window <= 0 || dist_bias || v_row != dv))
+    return zi_refuse("paged_attention: pooled keys go with a window, pages of their own and no bias by distance");
+  const PooledKeys pool = {kpool, vpool, pool_tables, pool_bt_stride, pool_per};
   const size_t smem = (size_t)(BQ * d + BK * (d + 1) + BK * dv + BQ * BK) * sizeof(float);
   dim3 grid(n_tiles, nq);
 #define ZI_LAUNCH_ATTN(J)                                                                                          \
@@ -232,7 +254,7 @@ extern "C" int zi_paged_attention_mods(void* out, int out_stride, const void* q,
     zi_launch(kern, dim3(grid), dim3(THREADS), smem, stream, (TT*)out, out_stride, (const TT*)q, q_stride,         \
               (const TT*)kcache, (const TT*)vcache, block_tables, bt_stride, cu_q, kv_lens, tile_seq, tile_q0, nq, \
               nkv, d, page_size, window, scale, dv, v_row, skip_from, skip_single, sink, keep_first, sink_logit,    \
-              softcap, dist_bias, n_dist);                                                                         \
+              softcap, dist_bias, n_dist, pool);                                                                       \
   } while (0)
   ZI_DISPATCH_DTYPE(dtype, TT, {
     if (dv <= 256) ZI_LAUNCH_ATTN(8);

@@ -61,6 +61,20 @@ __device__ __forceinline__ void rotate_pair(float& x, float& y, float c, float s
   y = ry;
 }
 
+// Pages of pooled keys and values: entry b of a request stands for its positions b per .. b per + per - 1 (their means).
+// A query at position i with a window of `window` tokens sees the entries whose positions all lie before the window.
+struct PooledKeys {
+  const void* k;
+  const void* v;
+  const int* block_tables;
+  int bt_stride;
+  int per;                 // tokens per entry; 0: no pooled keys
+};
+__device__ __forceinline__ int pooled_visible(const PooledKeys& p, int pos, int window) {
+  const int before = pos - window + 1;                       // positions 0 .. before - 1 lie before the window
+  return p.per > 0 && before > 0 ? before / p.per : 0;
+}
+
 // Sum over a block of up to 1024 threads; every thread receives the result.  The
 // order of additions depends only on blockDim, never on the data's place in a batch.
 __device__ __forceinline__ float block_sum(float v, float* scratch /* >= 33 floats */) {

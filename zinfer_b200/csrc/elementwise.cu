@@ -8,7 +8,7 @@
 // ---------------------------------------------------------------- embedding gather
 template <typename T>
 __global__ void embed_gather_kernel(float* __restrict__ h, const T* __restrict__ table,
-                                    const int* __restrict__ ids, int H, int V) {
+                                    const int* __restrict__ ids, int H, int V, float scale) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -19,14 +19,14 @@ __global__ void embed_gather_kernel(float* __restrict__ h, const T* __restrict__
     return;
   }
   const T* row = table + (size_t)id * H;
-  for (int i = threadIdx.x; i < H; i += blockDim.x) out[i] = to_f32(row[i]);
+  for (int i = threadIdx.x; i < H; i += blockDim.x) out[i] = to_f32(row[i]) * scale;
 }
 
 extern "C" int zi_embed_gather(float* h, const void* table, int table_dtype, const int* ids, int T, int H,
-                               int V, cudaStream_t stream) {
+                               int V, float scale, cudaStream_t stream) {
   if (T <= 0) return 0;
   ZI_DISPATCH_DTYPE(table_dtype, TT,
-                    zi_launch(embed_gather_kernel<TT>, dim3(T), dim3(256), 0, stream, h, (const TT*)table, ids, H, V));
+                    zi_launch(embed_gather_kernel<TT>, dim3(T), dim3(256), 0, stream, h, (const TT*)table, ids, H, V, scale));
   return zi_check_launch("embed_gather");
 }
 

@@ -23,6 +23,8 @@ _SIGNATURES = {
     "zi_pool_check": (_I, [_P]),
     "zi_cache_create": (_P, [_I, _P, _P, _I, _I]),
     "zi_cache_keep_first": (_I, [_P, _I, _I]),
+    "zi_cache_tokens_per_entry": (_I, [_P, _I, _I]),
+    "zi_cache_room": (_LL, [_P, _LL]),
     "zi_cache_destroy": (None, [_P]),
     "zi_cache_add": (_I, [_P, _LL]),
     "zi_cache_free": (_I, [_P, _LL, _P, _I]),

@@ -104,6 +104,7 @@ struct Pool {
 struct Group {
   int window = 0;   // 0: every key stays visible
   int keep_first = 0;   // with a window: this many tokens at a request's start stay visible too
+  int tokens_per_entry = 1;   // an entry (a key and a value) stands for this many tokens: one is complete with the last of them
   Pool pool;
 };
 
@@ -119,15 +120,20 @@ struct Cache {
   Pool slots;
   std::unordered_map<long long, Request> requests;
 
-  int blocks_for(long long tokens) const { return (int)((tokens + page_size - 1) / page_size); }
+  // pages that hold the complete entries of a request of `tokens` tokens
+  int blocks_for(const Group& g, long long tokens) const {
+    return (int)((tokens / g.tokens_per_entry + page_size - 1) / page_size);
+  }
   Request* find(long long id) {
     auto it = requests.find(id);
     return it == requests.end() ? nullptr : &it->second;
   }
+  int pages_needed(const Request& r, long long n_new, size_t g) const {
+    return std::max(0, blocks_for(groups[g], r.length + n_new) - (int)r.tables[g].size());
+  }
   // pages each group must still take so that n_new more tokens fit
   void pages_needed(const Request& r, long long n_new, int* out) const {
-    const int want = blocks_for(r.length + n_new);
-    for (size_t g = 0; g < groups.size(); ++g) out[g] = std::max(0, want - (int)r.tables[g].size());
+    for (size_t g = 0; g < groups.size(); ++g) out[g] = pages_needed(r, n_new, g);
   }
 };
 
@@ -195,6 +201,15 @@ extern "C" int zi_cache_keep_first(void* h, int group, int tokens) {
   return 0;
 }
 
+// A group whose entries stand for `tokens` tokens each (means over blocks of tokens): entry e belongs to positions
+// e * tokens .. (e + 1) * tokens - 1 and is written with the last of them.  Such a group has no window.
+extern "C" int zi_cache_tokens_per_entry(void* h, int group, int tokens) {
+  Cache* c = as_cache(h);
+  if (group < 0 || group >= (int)c->groups.size() || tokens < 1 || (tokens > 1 && c->groups[group].window > 0)) return ERR_ARGUMENT;
+  c->groups[group].tokens_per_entry = tokens;
+  return 0;
+}
+
 // The request's state slot, or a negative code.
 extern "C" int zi_cache_add(void* h, long long id) {
   Cache* c = as_cache(h);
@@ -258,10 +273,22 @@ extern "C" int zi_cache_can_reserve(void* h, long long id, long long n_new) {
   Cache* c = as_cache(h);
   Request* r = c->find(id);
   if (!r) return ERR_NOT_LIVE;
-  const int want = c->blocks_for(r->length + n_new);
   for (size_t g = 0; g < c->groups.size(); ++g)
-    if (std::max(0, want - (int)r->tables[g].size()) > c->groups[g].pool.num_free()) return 0;
+    if (c->pages_needed(*r, n_new, g) > c->groups[g].pool.num_free()) return 0;
   return 1;
+}
+// The most tokens that would still fit the request: what its pages and every group's free pages hold, less its length.
+extern "C" long long zi_cache_room(void* h, long long id) {
+  Cache* c = as_cache(h);
+  Request* r = c->find(id);
+  if (!r) return ERR_NOT_LIVE;
+  long long room = 1ll << 40;
+  for (size_t g = 0; g < c->groups.size(); ++g) {
+    const Group& gr = c->groups[g];
+    const long long entries = ((long long)r->tables[g].size() + gr.pool.num_free()) * c->page_size;
+    room = std::min(room, (entries + 1) * gr.tokens_per_entry - 1 - r->length);   // the tokens of an incomplete entry need no place
+  }
+  return std::max(0ll, room);
 }
 // Pages for positions length .. length + n_new - 1 in every group, or ERR_OUT_OF_PAGES with
 // nothing taken (info: the group that ran out, pages wanted there, pages free there).
@@ -269,9 +296,8 @@ extern "C" int zi_cache_reserve(void* h, long long id, long long n_new, int* inf
   Cache* c = as_cache(h);
   Request* r = c->find(id);
   if (!r) return ERR_NOT_LIVE;
-  const int want = c->blocks_for(r->length + n_new);
   for (size_t g = 0; g < c->groups.size(); ++g) {
-    const int need = std::max(0, want - (int)r->tables[g].size());
+    const int need = c->pages_needed(*r, n_new, g);
     if (need > c->groups[g].pool.num_free()) {
       if (info) {
         info[0] = (int)g;
@@ -282,7 +308,7 @@ extern "C" int zi_cache_reserve(void* h, long long id, long long n_new, int* inf
     }
   }
   for (size_t g = 0; g < c->groups.size(); ++g) {
-    const int need = std::max(0, want - (int)r->tables[g].size());
+    const int need = c->pages_needed(*r, n_new, g);
     const size_t old = r->tables[g].size();
     r->tables[g].resize(old + need);
     c->groups[g].pool.alloc(need, r->tables[g].data() + old);
@@ -296,8 +322,7 @@ extern "C" int zi_cache_reserve_all(void* h, int n, const long long* ids, const 
   for (int i = 0; i < n; ++i) {
     Request* r = c->find(ids[i]);
     if (!r) return ERR_NOT_LIVE;
-    const int want = c->blocks_for(r->length + n_new[i]);
-    for (size_t g = 0; g < c->groups.size(); ++g) need[g] += std::max(0, want - (int)r->tables[g].size());
+    for (size_t g = 0; g < c->groups.size(); ++g) need[g] += c->pages_needed(*r, n_new[i], g);
   }
   for (size_t g = 0; g < c->groups.size(); ++g)
     if (need[g] > c->groups[g].pool.num_free()) {
@@ -326,7 +351,7 @@ extern "C" int zi_cache_commit(void* h, long long id, long long n_new, int* rele
     const long long first_needed = r->length - window + 1;
     const long long n_dead = first_needed > 0 ? first_needed / c->page_size : 0;
     std::vector<int>& table = r->tables[g];
-    const long long kept = c->blocks_for(c->groups[g].keep_first);   // blocks that hold tokens every query still reads
+    const long long kept = c->blocks_for(c->groups[g], c->groups[g].keep_first);   // blocks that hold tokens every query still reads
     for (long long b = kept; b < n_dead && b < (long long)table.size(); ++b) {
       if (table[b] < 0) continue;
       const int p = table[b];
@@ -357,7 +382,8 @@ extern "C" int zi_cache_table(void* h, long long id, int group, int* out, int ca
   if (n > 0) memcpy(out, r->tables[group].data(), (size_t)n * sizeof(int));
   return (int)r->tables[group].size();
 }
-// Flat slot (page * page_size + offset) of positions start .. start + n - 1.
+// Flat slot (page * page_size + offset) of entries start .. start + n - 1 (an entry is a token's, unless the group's
+// entries stand for several tokens).
 extern "C" int zi_cache_slots_for(void* h, long long id, int group, long long start, int n, int* out) {
   Cache* c = as_cache(h);
   Request* r = c->find(id);
@@ -469,9 +495,10 @@ extern "C" long long zi_step_build(void* h, int n_entries, const long long* ids,
   std::vector<int> width(G, 1);
   for (int g = 0; g < G; ++g) {
     if (is_static) {
-      width[g] = static_width;
+      // a bucket's tables hold static_width pages of tokens; a group whose entries stand for several tokens needs fewer
+      width[g] = std::max(1, c->blocks_for(c->groups[g], (long long)static_width * c->page_size));
       for (int i = 0; i < n_entries; ++i)
-        if ((int)reqs[i]->tables[g].size() > static_width)
+        if ((int)reqs[i]->tables[g].size() > width[g])
           return zi_refuse("step_build: a request is longer than its bucket's block tables"), ERR_ARGUMENT;
     } else {
       for (int i = 0; i < n_entries; ++i) width[g] = std::max(width[g], (int)reqs[i]->tables[g].size());
@@ -586,7 +613,12 @@ extern "C" long long zi_step_build(void* h, int n_entries, const long long* ids,
       const std::vector<int>& table = reqs[i]->tables[g];
       if (!table.empty()) memcpy(bt + (long long)i * W, table.data(), table.size() * sizeof(int));
       for (int j = 0; j < ql[i]; ++j) {
-        const long long p = ctx[i] + j;
+        long long p = ctx[i] + j;
+        const int per = c->groups[g].tokens_per_entry;
+        if (per > 1) {                      // only the token that completes an entry writes it; the others keep slot -1
+          if ((p + 1) % per != 0) continue;
+          p /= per;
+        }
         const long long b = p / c->page_size;
         if (b >= (long long)table.size()) return zi_refuse("step_build: entry %d: no page was reserved for position %lld", i, p), ERR_ARGUMENT;
         if (table[b] < 0) return zi_refuse("step_build: entry %d: a token would be written to a page already given back", i), ERR_RELEASED;

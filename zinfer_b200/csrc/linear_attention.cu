@@ -7,6 +7,9 @@
 //     u_t = v_t                             plain form
 //     u_t = beta_t (v_t - S^T k_t)          delta rule
 //     S <- S + k_t u_t^T ;  o_t = S^T (q_scale q_t)
+// In a third form (HGRN2: "HGRN2: Gated Linear RNNs with State Expansion", Qin et al., 2024) the forget gate also decides
+// what is written: g = l + (1 - l) sigmoid(z + b) with a lower bound l per channel, k = 1 - g, u_t = v_t, q = silu(raw q).
+// The kernel makes g, k and q from the projections as it stages them.
 // Everything here is 32-bit arithmetic.  A request's tokens of this step are rows cu_q[s] ..
 // cu_q[s+1]-1 of the flat batch and continue the request from slot state_slots[s].  Each column of S
 // is visited by one group of lanes, token after token, in an order that depends on D alone, so a
@@ -125,13 +128,28 @@ __global__ void sigmoid_rows_kernel(float* __restrict__ out, int ldo, const T* _
 // into registers while these are worked on and stored afterwards (one barrier per TB tokens).
 constexpr int LR_WARPS = 8, LR_THREADS = LR_WARPS * 32, TB = 16, NC = 2;
 
-template <typename TQ, typename TV, int R, bool DELTA>
+// What the third form (GATE) makes its gate from: `k` of the kernel is the raw forget projection z.  With splits > 1
+// q, z and v are split-K partial sums, zstride apart, added in order as they are fetched.
+struct ForgetGate {
+  const float* lower;      // [H * D]
+  const float* bias;       // [H * D] or null
+  int splits;
+  long long zstride;
+};
+__device__ __forceinline__ void forget_gate(float z, float lower, float& g, float& k) {
+  const float e = expf(-fabsf(z)), r = 1.0f / (1.0f + e);      // sigmoid(|z|) = r, sigmoid(-|z|) = e r
+  const float up = z >= 0.f ? r : e * r, down = z >= 0.f ? e * r : r;
+  g = fmaf(1.0f - lower, up, lower);
+  k = (1.0f - lower) * down;                                   // 1 - g without cancellation
+}
+
+template <typename TQ, typename TV, int R, bool DELTA, bool GATE = false>
 __global__ void __launch_bounds__(LR_THREADS)
 linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict__ q, int ldq, const TQ* __restrict__ k,
                          int ldk, const TV* __restrict__ v, int ldv, const float* __restrict__ decay, int ldg,
                          const float* __restrict__ beta, int ldb, float q_scale, float* __restrict__ state,
                          long long slot_stride, int H, int G, int D, int V, int P, const int* __restrict__ cu_q,
-                         const int* __restrict__ state_slots) {
+                         const int* __restrict__ state_slots, const ForgetGate fgate) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
@@ -177,7 +195,7 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
         const size_t row = (size_t)(tok0 + t0 + tt);
         fq[u] = q[row * ldq + (size_t)kvh * D + i];
         fk[u] = k[row * ldk + (size_t)kvh * D + i];
-        fg[u] = decay[row * ldg + (size_t)h * D + i];
+        if (!GATE) fg[u] = decay[row * ldg + (size_t)h * D + i];
       } else {
         fq[u] = from_f32<TQ>(0.f);
         fk[u] = from_f32<TQ>(0.f);
@@ -191,6 +209,49 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
       fv[u] = (e < (nt << lgCB) && c < V) ? v[(size_t)(tok0 + t0 + (e >> lgCB)) * ldv + (size_t)h * V + c] : from_f32<TV>(0.f);
     }
     if (DELTA && tid < nt) fb = beta[(size_t)(tok0 + t0 + tid) * ldb + h];
+    if constexpr (GATE) {
+      for (int z = 1; z < fgate.splits; ++z) {
+        const size_t zo = (size_t)z * fgate.zstride;
+#pragma unroll
+        for (int u = 0; u < NPF; ++u) {
+          const int e = tid + u * LR_THREADS;
+          const int tt = e >> lgDP, i = e & (DP - 1);
+          if (e < total && i < D) {
+            const size_t row = (size_t)(tok0 + t0 + tt);
+            fq[u] += q[zo + row * ldq + (size_t)kvh * D + i];
+            fk[u] += k[zo + row * ldk + (size_t)kvh * D + i];
+          }
+        }
+#pragma unroll
+        for (int u = 0; u < NPV; ++u) {
+          const int e = tid + u * LR_THREADS;
+          const int c = j0 + (e & (CB - 1));
+          if (e < (nt << lgCB) && c < V) fv[u] += v[zo + (size_t)(tok0 + t0 + (e >> lgCB)) * ldv + (size_t)h * V + c];
+        }
+      }
+    }
+  };
+  // element i of a token's q, k and g into the staging buffer at `at`
+  auto stage = [&](float* buf, int at, int i, float qv, float kv, float gv) {
+    if constexpr (GATE) {
+      if (i < D) {
+        const int ch = h * D + i;
+        forget_gate(kv + (fgate.bias ? fgate.bias[ch] : 0.f), fgate.lower[ch], gv, kv);
+        qv = qv * sigmoid_f32(qv);
+      } else {
+        kv = gv = 0.f;
+      }
+    }
+    buf[at] = qv * q_scale;
+    buf[TB * DP + at] = kv;
+    buf[2 * TB * DP + at] = gv;
+  };
+  // a value that was not fetched into a register: whole, or the sum of its partial sums
+  auto whole = [&](const auto* p) {
+    float x = to_f32(*p);
+    if constexpr (GATE)
+      for (int z = 1; z < fgate.splits; ++z) x += to_f32(p[(size_t)z * fgate.zstride]);
+    return x;
   };
   auto put = [&](int t0, int nt, float* buf) {
     const int total = nt << lgDP;
@@ -198,20 +259,15 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
     for (int u = 0; u < NPF; ++u) {
       const int e = tid + u * LR_THREADS;
       if (e < total) {
-        const int at = (e & ~(DP - 1)) + place(e & (DP - 1));
-        buf[at] = to_f32(fq[u]) * q_scale;
-        buf[TB * DP + at] = to_f32(fk[u]);
-        buf[2 * TB * DP + at] = fg[u];
+        stage(buf, (e & ~(DP - 1)) + place(e & (DP - 1)), e & (DP - 1), to_f32(fq[u]), to_f32(fk[u]), GATE ? 0.f : fg[u]);
       }
     }
     for (int e = tid + NPF * LR_THREADS; e < total; e += LR_THREADS) {      // beyond the registers (DP > 128)
       const int tt = e >> lgDP, i = e & (DP - 1);
       const size_t row = (size_t)(tok0 + t0 + tt);
       const bool in = i < D;
-      const int at = (e & ~(DP - 1)) + place(i);
-      buf[at] = in ? to_f32(q[row * ldq + (size_t)kvh * D + i]) * q_scale : 0.f;
-      buf[TB * DP + at] = in ? to_f32(k[row * ldk + (size_t)kvh * D + i]) : 0.f;
-      buf[2 * TB * DP + at] = in ? decay[row * ldg + (size_t)h * D + i] : 0.f;
+      stage(buf, (e & ~(DP - 1)) + place(i), i, in ? whole(q + row * ldq + (size_t)kvh * D + i) : 0.f,
+            in ? whole(k + row * ldk + (size_t)kvh * D + i) : 0.f, in && !GATE ? decay[row * ldg + (size_t)h * D + i] : 0.f);
     }
 #pragma unroll
     for (int u = 0; u < NPV; ++u) {
@@ -220,7 +276,7 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
     }
     for (int e = tid + NPV * LR_THREADS; e < (nt << lgCB); e += LR_THREADS) {
       const int c = j0 + (e & (CB - 1));
-      buf[3 * TB * DP + e] = c < V ? to_f32(v[(size_t)(tok0 + t0 + (e >> lgCB)) * ldv + (size_t)h * V + c]) : 0.f;
+      buf[3 * TB * DP + e] = c < V ? whole(v + (size_t)(tok0 + t0 + (e >> lgCB)) * ldv + (size_t)h * V + c) : 0.f;
     }
     if (tid < nt) buf[3 * TB * DP + TB * CB + tid] = fb;
   };
@@ -292,7 +348,7 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
 }
 
 // ----------------------------------------------------------------------- gated per-head norm
-// out[t, head, :] = o / sqrt(mean(o^2) + eps) * w * act(gate[t, head, :]); act: 0 silu, 1 sigmoid.
+// out[t, head, :] = o / sqrt(mean(o^2) + eps) * w * act(gate[t, head, :]); act: 0 silu, 1 sigmoid, 2 no gate.
 // One warp per (token, head).
 template <typename TG, typename TO>
 __global__ void head_norm_gate_kernel(TO* __restrict__ out, int ldo, const float* __restrict__ o, int ldi,
@@ -309,8 +365,8 @@ __global__ void head_norm_gate_kernel(TO* __restrict__ out, int ldo, const float
   ss = warp_sum(ss);
   const float inv = 1.0f / sqrtf(ss / (float)V + eps);
   for (int i = lane; i < V; i += 32) {
-    const float g = to_f32(gate[(size_t)t * ldgate + (size_t)h * V + i]);
-    const float a = act == 0 ? g * sigmoid_f32(g) : sigmoid_f32(g);
+    const float g = act == 2 ? 1.f : to_f32(gate[(size_t)t * ldgate + (size_t)h * V + i]);
+    const float a = act == 2 ? 1.f : (act == 0 ? g * sigmoid_f32(g) : sigmoid_f32(g));
     out[(size_t)t * ldo + (size_t)h * V + i] = from_f32<TO>(p[i] * inv * w[i] * a);
   }
 }
@@ -386,7 +442,7 @@ extern "C" int zi_linear_recurrence(float* out, int ldo, const void* q, int ldq,
         return zi_refuse("linear_recurrence: cannot get %zu bytes of shared memory", smem);                            \
     }                                                                                                                  \
     zi_launch(kern, dim3(grid), dim3(block), smem, stream, out, ldo, (const TQ*)q, ldq, (const TQ*)k, ldk, (const TV*)v, \
-              ldv, decay, ldg, beta, ldb, q_scale, state, slot_stride, H, G, D, V, P, cu_q, state_slots);              \
+              ldv, decay, ldg, beta, ldb, q_scale, state, slot_stride, H, G, D, V, P, cu_q, state_slots, ForgetGate{}); \
   } while (0)
 #define ZI_LR_R(TQ, TV)                                          \
   do {                                                           \
@@ -402,11 +458,35 @@ extern "C" int zi_linear_recurrence(float* out, int ldo, const void* q, int ldq,
   return zi_check_launch("linear_recurrence");
 }
 
+// The third form: q, z and v are float32 projections (rows may be views of wider rows), whole or split-K partial sums.
+extern "C" int zi_linear_recurrence_gated(float* out, int ldo, const float* q, int ldq, const float* z, int ldz, const float* v,
+                                          int ldv, int splits, long long zstride, const float* f_bias, const float* lower,
+                                          float* state, long long slot_stride, int H, int D, int V, const int* cu_q,
+                                          const int* state_slots, int n_seqs, cudaStream_t stream) {
+  if (n_seqs <= 0) return 0;
+  if (H <= 0 || H > 65535) return zi_refuse("linear_recurrence_gated: %d heads", H);
+  if (D <= 0 || D > 512 || V <= 0) return zi_refuse("linear_recurrence_gated: %d key channels (1..512), %d value channels", D, V);
+  if (!lower || splits < 1) return zi_refuse("linear_recurrence_gated: needs the gate's lower bound and whole rows or partial sums");
+  const int R = D <= 256 ? 8 : 16;
+  int P = 1;
+  while (P * R < D) P <<= 1;
+  const int CB = LR_WARPS * (32 / P) * NC;
+  const size_t smem = (size_t)2 * (3 * TB * P * R + TB * CB + TB) * sizeof(float);
+  dim3 grid(n_seqs, H, (V + CB - 1) / CB), block(LR_THREADS);
+  const ForgetGate gate = {lower, f_bias, splits, zstride};
+  auto kern = R == 8 ? linear_recurrence_kernel<float, float, 8, false, true> : linear_recurrence_kernel<float, float, 16, false, true>;
+  if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    return zi_refuse("linear_recurrence_gated: cannot get %zu bytes of shared memory", smem);
+  zi_launch(kern, grid, block, smem, stream, out, ldo, q, ldq, z, ldz, v, ldv, (const float*)nullptr, 0, (const float*)nullptr, 0, 1.0f,
+            state, slot_stride, H, H, D, V, P, cu_q, state_slots, gate);
+  return zi_check_launch("linear_recurrence_gated");
+}
+
 extern "C" int zi_head_norm_gate(void* out, int out_dtype, int ldo, const float* o, int ldi, const float* w, float eps,
                                  const void* gate, int gate_dtype, int ldgate, int act, int T, int heads, int V,
                                  cudaStream_t stream) {
   if (T <= 0 || heads <= 0) return 0;
-  if (act != 0 && act != 1) return zi_refuse("head_norm_gate: unknown gate %d", act);
+  if (act < 0 || act > 2 || (act != 2 && !gate)) return zi_refuse("head_norm_gate: unknown gate %d", act);
   const int warps = 4;
   dim3 grid((unsigned)(((size_t)T * heads + warps - 1) / warps));
   ZI_DISPATCH_DTYPE(gate_dtype, TG, ZI_DISPATCH_DTYPE(out_dtype, TO,

@@ -62,6 +62,7 @@ class StepContext:
     patch_dst: Optional[torch.Tensor] = None   # flat token positions to fill from the previous step's tokens
     patch_src: Optional[torch.Tensor] = None   # rows of the previous step's sampled tokens
     n_patch: int = 0
+    carried: dict = field(default_factory=dict)   # what a layer hands to later layers of the same step, by name
 
 
 class PinnedStaging:

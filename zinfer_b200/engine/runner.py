@@ -58,7 +58,7 @@ class ModelRunner:
                 budget = int(free * gpu_memory_fraction) - workspace_bytes
             if budget is None and max_tokens is None:
                 raise ValueError("give num_pages, kv_cache_bytes, gpu_memory_fraction or max_tokens")
-            num_pages = pages_for(kv_needs, page_size, elt, budget_bytes=budget, tokens=max_tokens)
+            num_pages = pages_for(kv_needs, page_size, elt, budget_bytes=budget, tokens=max_tokens, requests=max_requests)
         self.manager = CacheManager(kv_needs, list(state_needs), page_size, num_pages, max_requests)
         self.storage = CacheStorage(self.manager, state_needs, model.dtype, self.device)
         if poison_freed_pages:

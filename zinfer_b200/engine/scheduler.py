@@ -179,10 +179,7 @@ class Scheduler:
         """The most tokens <= want whose pages are free right now."""
         if self.cache.can_reserve(r.request_id, want):
             return want
-        ps = self.cache.page_size
-        have = self.cache.blocks_held(r.request_id) * ps if self.cache.groups else 1 << 30
-        room = have + self.cache.min_free_pages() * ps - self.cache.length(r.request_id)
-        return max(0, min(want, room))
+        return max(0, min(want, self.cache.room(r.request_id)))
 
     # ------------------------------------------------------------------- schedule
     def schedule(self) -> StepPlan:
@@ -263,8 +260,8 @@ class Scheduler:
         st.steps += 1
         st.step_tokens, st.running, st.waiting = plan.num_tokens, len(self.running), len(self.waiting)
         if self.cache.groups:
-            st.pages_total = self.cache.groups[0].pool.num_pages
-            st.pages_used = st.pages_total - self.cache.min_free_pages()
+            fullest = self.cache.fullest_group().pool
+            st.pages_total, st.pages_used = fullest.num_pages, fullest.num_used
         return plan
 
     # --------------------------------------------------------------------- update

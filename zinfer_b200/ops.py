@@ -168,6 +168,20 @@ class Carried:
         self.x = x
 
 
+class PostNormed:
+    """An update of the residual stream that is normed before it is added (a block that norms its sublayers' outputs as
+    well as their inputs): ``delta`` is a tensor, :class:`Partials`, or either inside :class:`Scaled`; ``norm`` is the norm
+    part (its ``weight``, ``eps`` and ``kind``)."""
+
+    def __init__(self, delta, norm):
+        self.delta = delta
+        self.norm = norm
+
+    @property
+    def shape(self):
+        return self.delta.shape
+
+
 class Several:
     """Updates of the residual stream that are still to be added, in this order (a block whose sublayers read the
     same stream leaves one per sublayer): each a tensor, :class:`Partials`, or either inside :class:`Scaled`.
@@ -266,8 +280,8 @@ def _unscaled(delta):
 
 
 # ------------------------------------------------------------------ elementwise
-def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """Rows ``ids`` of ``table`` [V, H] as the 32-bit residual stream [T, H]."""
+def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: Optional[torch.Tensor] = None, scale: float = 1.0) -> torch.Tensor:
+    """Rows ``ids`` of ``table`` [V, H], times ``scale``, as the 32-bit residual stream [T, H]."""
     V, H = table.shape
     T = ids.shape[0]
     _need(table.is_contiguous(), "embedding table must be contiguous")
@@ -275,7 +289,8 @@ def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: Optional[torch.Ten
     if out is None:
         out = torch.empty((T, H), dtype=torch.float32, device=table.device)
     with _prof.region("embed_gather", lambda: T * H * table.element_size() + _nb(out, ids)):
-        _check(lib().zi_embed_gather(_ptr(out), _ptr(table), _tag(table), _ptr(ids), T, H, V, _stream()), "embed_gather")
+        _check(lib().zi_embed_gather(_ptr(out), _ptr(table), _tag(table), _ptr(ids), T, H, V, ctypes.c_float(scale), _stream()),
+               "embed_gather")
     return out
 
 
@@ -470,6 +485,78 @@ def qkv_rows_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], num_heads
             rot_dims if cos is not None else 0, _ptr(cos), _ptr(sin), n_table, _ptr(_i32(positions, "positions")),
             _ptr(k_cache), _ptr(v_cache), _ptr(_i32(slots, "slots")), page_size, _stream()), "qkv_rows_prepare")
     return q, gate
+
+
+def qkv_heads_prepare(proj, bias: Optional[torch.Tensor], num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int,
+                      q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float, rot_dims: int,
+                      cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], positions: torch.Tensor, k_cache: torch.Tensor,
+                      v_cache: torch.Tensor, slots: torch.Tensor, page_size: int, out_dtype: torch.dtype,
+                      mix_with: Optional[torch.Tensor] = None, mix_lambda: float = 0.0, keep_values: bool = False):
+    """What follows a fused projection row [q heads | k heads | v heads] (a tensor, or :class:`Partials` whose splits the
+    kernel adds in order) when the q and k heads are normed one by one: ``bias`` (float32, the row's width) is added; an
+    RMS norm per head (``q_weight``, ``k_weight`` float32 [head_dim]); the first ``rot_dims`` dimensions rotate; values
+    become ``(1 - mix_lambda) v + mix_lambda * mix_with`` where ``mix_with`` (float32 [T, kv heads * value_dim]) is given; k
+    and v go into the token's page slot.  Returns (q [T, heads * head_dim] in ``out_dtype``, the values float32
+    [T, kv heads * value_dim] if ``keep_values`` else None)."""
+    T, width = proj.shape
+    _need(width == num_heads * head_dim + num_kv_heads * (head_dim + value_dim), "qkv_heads_prepare: rows as wide as their heads")
+    part, splits, src = (proj.data, proj.splits, None) if isinstance(proj, Partials) else (None, 0, proj)
+    _need(src is None or src.stride(1) == 1, "qkv_heads_prepare: dense rows")
+    if bias is not None:
+        _need(bias.dtype == torch.float32 and bias.numel() == width and bias.is_contiguous(), "the bias is float32 of the row's width")
+    for wt in (q_weight, k_weight):
+        _need(wt is None or (wt.dtype == torch.float32 and wt.numel() == head_dim and wt.is_contiguous()), "q/k norm weights are float32 [head_dim]")
+    n_table = 0
+    if cos is not None:
+        _need(cos.shape == sin.shape and cos.shape[1] == rot_dims // 2 and cos.dtype == torch.float32,
+              "rotary tables are float32 [positions, rot_dims/2]")
+        n_table = cos.shape[0]
+    _need(k_cache.dtype == out_dtype and v_cache.dtype == out_dtype and k_cache.is_contiguous() and v_cache.is_contiguous(),
+          "cache pages have the activations' dtype")
+    _need(tuple(k_cache.shape[1:]) == (num_kv_heads, page_size, head_dim)
+          and tuple(v_cache.shape[1:]) == (num_kv_heads, page_size, value_dim), "cache pages are [pages, kv heads, page, size]")
+    if mix_with is not None:
+        _need(mix_with.dtype == torch.float32 and tuple(mix_with.shape) == (T, num_kv_heads * value_dim) and mix_with.is_contiguous(),
+              "the values to mix with are float32 [T, kv heads * value size]")
+    dev = proj.data.device if part is not None else proj.device
+    q = torch.empty((T, num_heads * head_dim), dtype=out_dtype, device=dev)
+    values = torch.empty((T, num_kv_heads * value_dim), dtype=torch.float32, device=dev) if keep_values else None
+    with _prof.region("qkv heads (bias, head norms, rotation, value mix, page write)",
+                      lambda: _nb(part) + (T * width * src.element_size() if src is not None else 0) + T * width * q.element_size()
+                      + _nb(mix_with, values)):
+        _check(lib().zi_qkv_heads_prepare(
+            _ptr(src), _tag(src) if src is not None else F32, src.stride(0) if src is not None else width, _ptr(part), splits,
+            _ll(T * width), _ptr(bias), _ptr(q), q.stride(0), _tag(q), T, num_heads, num_kv_heads, head_dim, value_dim, _ptr(q_weight),
+            _ptr(k_weight), ctypes.c_float(eps), rot_dims if cos is not None else 0, _ptr(cos), _ptr(sin), n_table,
+            _ptr(_i32(positions, "positions")), _ptr(k_cache), _ptr(v_cache), _ptr(_i32(slots, "slots")), page_size, _ptr(mix_with),
+            ctypes.c_float(mix_lambda), _ptr(values), _stream()), "qkv_heads_prepare")
+    return q, values
+
+
+class PooledKeys:
+    """Pages that hold one key and value per block of ``per`` tokens, beside the tokens' own pages: ``k``, ``v`` [pages,
+    kv heads, page_size, size], ``block_tables`` [n, W].  A query at position i with a window sees the blocks that lie
+    wholly before the window."""
+
+    def __init__(self, k: torch.Tensor, v: torch.Tensor, block_tables: torch.Tensor, per: int):
+        self.k, self.v, self.block_tables, self.per = k, v, block_tables, int(per)
+
+
+def pool_blocks(k_cache: torch.Tensor, v_cache: torch.Tensor, block_tables: torch.Tensor, pooled: PooledKeys, entry_slots: torch.Tensor,
+                step, page_size: int) -> None:
+    """Writes the pooled entry (means of keys and values, summed in 32-bit) of every block that this step's tokens
+    complete: ``entry_slots[t]`` is the slot of the entry that token t completes, or -1."""
+    nkv, d, dv = k_cache.shape[1], k_cache.shape[3], v_cache.shape[3]
+    _need(tuple(pooled.k.shape[1:]) == tuple(k_cache.shape[1:]) and tuple(pooled.v.shape[1:]) == tuple(v_cache.shape[1:])
+          and pooled.k.dtype == k_cache.dtype and pooled.v.dtype == v_cache.dtype and pooled.k.is_contiguous()
+          and pooled.v.is_contiguous(), "pooled pages are laid out like the tokens'")
+    T = step.n_tokens
+    with _prof.region("pooled keys and values",
+                      lambda: (sum((c + q) // pooled.per - c // pooled.per for q, c in zip(step.q_lens, step.ctx_lens))
+                               * (pooled.per + 1) * nkv * (d + dv) * k_cache.element_size())):
+        _check(lib().zi_pool_blocks(_ptr(k_cache), _ptr(v_cache), _tag(k_cache), _ptr(block_tables), block_tables.stride(0), _ptr(pooled.k),
+                                    _ptr(pooled.v), _ptr(_i32(entry_slots, "entry_slots")), _ptr(step.positions), _ptr(step.cu_q),
+                                    step.n_seqs, T, nkv, d, dv, pooled.per, page_size, _stream()), "pool_blocks")
 
 
 ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
@@ -1138,7 +1225,7 @@ def latent_attention(q_eff: torch.Tensor, cache: torch.Tensor, block_tables: tor
             _ptr(_i32(block_tables, "block_tables")), block_tables.stride(0), _ptr(step.cu_q), _ptr(step.kv_lens),
             _ptr(step.tile_seq), _ptr(step.tile_q0), step.tile_seq.shape[0], heads, 1, D, rank, D, page_size,
             int(window or 0), 0, ctypes.c_float(scale), skip_from, skip_single, ctypes.c_float(0.0), _ptr(sink_logit),
-            ctypes.c_float(0.0), None, 0, _stream()), "latent_attention")
+            ctypes.c_float(0.0), None, 0, None, None, None, 0, 0, _stream()), "latent_attention")
     return out
 
 
@@ -1205,14 +1292,15 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                     num_heads: int, num_kv_heads: int, head_dim: int, page_size: int, window: Optional[int],
                     scale: float, out: Optional[torch.Tensor] = None, sink: float = 0.0, keep_first: int = 0,
                     value_dim: Optional[int] = None, sink_logit: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                    dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    dist_bias: Optional[torch.Tensor] = None, pooled: Optional[PooledKeys] = None) -> torch.Tensor:
     """Causal attention of the step's query tokens over their requests' pages.  Changes to the score, each off unless
     given: ``softcap`` c (s <- c tanh(s / c) after the scale); ``dist_bias`` (float32 [heads, n]: entry [h, i - j] is
     added for a key i - j tokens back, distances from n - 1 on share the last entry; neither scaled nor capped);
     ``sink_logit`` (float32 [heads]: exp(sink_logit[h]) joins head h's denominator and has no value).  ``sink``: that many keys of
     score 0 without a value are counted in the softmax's denominator (p_j = exp(s_j) / (sink + sum exp(s))).
     ``keep_first``: with a window, a request's first tokens that stay visible beyond it (query i sees key j <= i if
-    i - j < window or j < keep_first).  ``value_dim``: the values' size where it differs from the keys'.
+    i - j < window or j < keep_first).  ``pooled``: with a window, one key and value per block of tokens that lies wholly
+    before it, in pages of their own; they share the softmax with the tokens.  ``value_dim``: the values' size where it differs from the keys'.
 
     ``q`` [T, >= num_heads*head_dim] (row stride free), caches [pages, kv heads,
     page_size, head_dim], ``block_tables`` [n, W], ``cu_q`` [n+1] token offsets,
@@ -1238,7 +1326,9 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
             block_tables.stride(0), _ptr(cu_q), _ptr(kv_lens), _ptr(tile_seq), _ptr(tile_q0), tile_seq.shape[0],
             num_heads, num_kv_heads, head_dim, dv, dv, page_size, int(window or 0), int(keep_first or 0),
             ctypes.c_float(scale), 0, 0, ctypes.c_float(sink), _ptr(sink_logit), ctypes.c_float(softcap), _ptr(dist_bias),
-            dist_bias.shape[1] if dist_bias is not None else 0, _stream()), "paged_attention")
+            dist_bias.shape[1] if dist_bias is not None else 0, _ptr(pooled.k) if pooled else None, _ptr(pooled.v) if pooled else None,
+            _ptr(pooled.block_tables) if pooled else None, pooled.block_tables.stride(0) if pooled else 0, pooled.per if pooled else 0,
+            _stream()), "paged_attention")
     return out
 
 
@@ -1286,7 +1376,7 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, blo
               num_heads: int, num_kv_heads: int, head_dim: int, page_size: int, window: Optional[int],
               scale: float, sink: float = 0.0, keep_first: int = 0, value_dim: Optional[int] = None,
               sink_logit: Optional[torch.Tensor] = None, softcap: float = 0.0,
-              dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+              dist_bias: Optional[torch.Tensor] = None, pooled: Optional[PooledKeys] = None) -> torch.Tensor:
     """Attention of a step's query tokens over their pages, by the fastest kernel that
     takes the shape: in bfloat16 with head sizes 64/128 (decode also 256) the
     tensor-core kernels (requests that bring one token go to the split-key decode
@@ -1299,7 +1389,7 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, blo
     # the tensor-core kernels take values of the keys' size; kept first tokens only in the form with a sink
     changed = sink_logit is not None or bool(softcap) or dist_bias is not None
     fast = ATTENTION_BACKEND != "generic" and q.dtype == torch.bfloat16 and same_size and (not keep_first or bool(sink)) \
-        and not (changed and (sink or keep_first))
+        and not (changed and (sink or keep_first)) and pooled is None
     dec_ok = fast and step.n_dec > 0 and L.zi_attention_mma_supported(num_heads, num_kv_heads, head_dim, 1)
     pf_ok = fast and step.n_pf_tiles > 0 and L.zi_attention_mma_supported(num_heads, num_kv_heads, head_dim, 0) \
         and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
@@ -1307,7 +1397,7 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, blo
         return paged_attention(q, k_cache, v_cache, block_tables, step.cu_q, step.kv_lens, step.tile_seq, step.tile_q0,
                                num_heads, num_kv_heads, head_dim, page_size, window, scale, sink=sink,
                                keep_first=keep_first, value_dim=value_dim, sink_logit=sink_logit, softcap=softcap,
-                               dist_bias=dist_bias)
+                               dist_bias=dist_bias, pooled=pooled)
     _need(q.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous(), "attention: dense operands")
     _need(tuple(k_cache.shape[1:]) == (num_kv_heads, page_size, head_dim) and k_cache.dtype == q.dtype,
           "cache pages are [pages, kv heads, page, d] in the activations' dtype")
@@ -1521,6 +1611,47 @@ def norm_residual(h: torch.Tensor, a, weight: torch.Tensor, eps: float, out_dtyp
     return h if x is None else x
 
 
+NORM_KINDS = {"rms": 0, "layer": 1}
+
+
+def sandwich_norm(h: torch.Tensor, delta, pre_weight: Optional[torch.Tensor], pre_eps: float, pre_kind: str, out_dtype: torch.dtype,
+                  rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """The seam between two sublayers in one kernel: ``h += delta`` in place (32-bit), where a :class:`PostNormed` update is
+    normed first, then the norm of ``h`` times ``pre_weight`` in ``out_dtype`` (None: no second norm, nothing returned).
+    Norm kinds: ``rms``, ``layer`` (mean taken off).  With ``rows`` the picked rows' norms are returned and ``h`` is left
+    as it is."""
+    T, H = h.shape
+    _need(h.dtype == torch.float32 and h.is_contiguous(), "the residual stream is contiguous float32")
+    if isinstance(delta, Several):          # all but the last update go in by themselves, in order
+        _need(delta.row_bias is None and (rows is None or len(delta.terms) < 2), "several updates with a vector, or for picked rows, are not built here")
+        for term in delta.terms[:-1]:
+            sandwich_norm(h, term, None, 0.0, "rms", out_dtype)
+        delta = delta.terms[-1] if delta.terms else None
+    post_w, post_eps, post_kind = None, 0.0, "rms"
+    if isinstance(delta, PostNormed):
+        post_w, post_eps, post_kind = delta.norm.weight, delta.norm.eps, delta.norm.kind
+        delta = delta.delta
+    delta, scale = _unscaled(delta)
+    for w in (post_w, pre_weight):
+        _need(w is None or (w.dtype == torch.float32 and w.numel() == H and w.is_contiguous()), "norm weights are float32 of the row's width")
+    part, splits = None, 0
+    if isinstance(delta, Partials):
+        _need(tuple(delta.shape) == (T, H), "an update must match the residual stream")
+        part, splits, delta = delta.data, delta.splits, None
+    elif delta is not None:
+        _need(tuple(delta.shape) == (T, H) and delta.is_contiguous(), "an update must match the residual stream")
+    n = T if rows is None else _i32(rows, "rows").shape[0]
+    out = torch.empty((n, H), dtype=out_dtype, device=h.device) if pre_weight is not None else None
+    with _prof.region("norm of the output + residual add + norm",
+                      lambda: (2 if rows is None else 1) * n * H * 4 + _nb(out) + splits * n * H * 4
+                      + (n * H * delta.element_size() if delta is not None else 0)):
+        _check(lib().zi_sandwich_norm(_ptr(h), _ptr(delta), _tag(delta) if delta is not None else F32, _ptr(part), splits, _ll(T * H),
+                                      ctypes.c_float(scale), _ptr(post_w), NORM_KINDS[post_kind], ctypes.c_float(post_eps),
+                                      _ptr(pre_weight), NORM_KINDS[pre_kind], ctypes.c_float(pre_eps), _ptr(out),
+                                      _tag(out) if out is not None else F32, _ptr(rows), n, H, _stream()), "sandwich_norm")
+    return out
+
+
 def cast_rows(h: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
     """The 32-bit residual stream in the activations' type (itself for float32)."""
     if dtype == torch.float32:
@@ -1653,18 +1784,47 @@ def linear_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: 
     return out
 
 
-def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, eps: float, gate: torch.Tensor, gate_kind: str, heads: int, vdim: int,
-                   out_dtype: torch.dtype) -> torch.Tensor:
+def linear_recurrence_gated(proj, lower: torch.Tensor, f_bias: Optional[torch.Tensor], state: torch.Tensor, heads: int, dim: int,
+                            vdim: int, step) -> torch.Tensor:
+    """The recurrence whose forget gate decides what is written, from and to ``state`` [slots, heads, dim, vdim] (float32):
+    with the projection's columns [q | z | v], ``f = lower + (1 - lower) sigmoid(z + f_bias)``,
+    ``S = diag(f) S + (1 - f) v^T``, ``o = S^T silu(q)``.  ``proj`` is float32 [T, heads * (2 dim + vdim)], or
+    :class:`Partials` of it whose splits the kernel adds in order.  Returns float32 [T, heads * vdim]."""
+    qk, hv = heads * dim, heads * vdim
+    data, splits = (proj.data, proj.splits) if isinstance(proj, Partials) else (proj, 1)
+    T, W = proj.shape
+    _need(data.dtype == torch.float32 and data.is_contiguous() and W == 2 * qk + hv, "linear_recurrence_gated: float32 [T, heads * (2 dim + vdim)]")
+    for t in (lower, f_bias):
+        _need(t is None or (t.dtype == torch.float32 and t.numel() == qk and t.is_contiguous()), "the gate's vectors are float32 [heads * dim]")
+    state, stride = _slot_view(state, "linear_recurrence_gated")
+    _need(state[0].numel() == heads * dim * vdim, "linear_recurrence_gated: state [slots, heads, dim, vdim]")
+    out = torch.empty((T, hv), dtype=torch.float32, device=data.device)
+    base = data.data_ptr()
+    at = lambda cols: ctypes.c_void_p(base + 4 * cols)
+    with _prof.region("linear recurrence (gate writes)",
+                      lambda: _nb(data, out) + 2 * step.n_seqs * heads * dim * vdim * 4, 6 * T * heads * dim * vdim):
+        _check(lib().zi_linear_recurrence_gated(
+            _ptr(out), out.stride(0), at(0), W, at(qk), W, at(2 * qk), W, splits, _ll(T * W), _ptr(f_bias), _ptr(lower), _ptr(state),
+            _ll(stride), heads, dim, vdim, _ptr(step.cu_q), _ptr(step.state_slots), step.n_seqs, _stream()), "linear_recurrence_gated")
+    return out
+
+
+def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, eps: float, gate: Optional[torch.Tensor], gate_kind: str, heads: int,
+                   vdim: int, out_dtype: torch.dtype) -> torch.Tensor:
     """Every head of float32 ``o`` [T, heads * vdim] divided by its root mean square (``eps`` inside the root), times
-    ``weight`` [vdim], times ``silu(gate)`` or ``sigmoid(gate)`` (``gate`` [T, heads * vdim], rows may be views)."""
+    ``weight`` [vdim], times ``silu(gate)`` or ``sigmoid(gate)`` (``gate`` [T, heads * vdim], rows may be views; kind
+    ``none``: no gate)."""
     T = o.shape[0]
-    _need(o.dtype == torch.float32 and o.is_contiguous() and gate.stride(1) == 1 and gate.shape[1] == heads * vdim
+    _need((gate is None) == (gate_kind == "none"), "head_norm_gate: a gate and its kind go together")
+    _need(o.dtype == torch.float32 and o.is_contiguous() and (gate is None or (gate.stride(1) == 1 and gate.shape[1] == heads * vdim))
           and weight.dtype == torch.float32 and weight.numel() == vdim, "head_norm_gate: shapes")
-    _need(gate_kind in ("silu", "sigmoid"), f"head_norm_gate: unknown gate {gate_kind!r}")
+    kinds = {"silu": 0, "sigmoid": 1, "none": 2}
+    _need(gate_kind in kinds, f"head_norm_gate: unknown gate {gate_kind!r}")
     out = torch.empty((T, heads * vdim), dtype=out_dtype, device=o.device)
-    with _prof.region("head norm + gate", lambda: _nb(o, out) + T * heads * vdim * gate.element_size()):
+    with _prof.region("head norm + gate", lambda: _nb(o, out) + (T * heads * vdim * gate.element_size() if gate is not None else 0)):
         _check(lib().zi_head_norm_gate(_ptr(out), _tag(out), out.stride(0), _ptr(o), o.stride(0), _ptr(weight), ctypes.c_float(eps),
-                                       _ptr(gate), _tag(gate), gate.stride(0), 0 if gate_kind == "silu" else 1, T, heads, vdim,
+                                       _ptr(gate), _tag(gate) if gate is not None else F32, gate.stride(0) if gate is not None else 0,
+                                       kinds[gate_kind], T, heads, vdim,
                                        _stream()), "head_norm_gate")
     return out
 

@@ -32,6 +32,16 @@ and min(rows - 1, rows/2 + floor(ln(n / (rows/2)) / ln(far / (rows/2)) * (rows -
 "Exploring the Limits of Transfer Learning with a Unified Text-to-Text Transformer", Raffel et al., 2020, for one
 direction); ``output_gate`` multiplies the heads' outputs by sigmoid(W_g x) before the output projection, ``channel``
 with one gate value per output channel, ``head`` with one per head (tensor ``g``).
+
+Options of the "heads" form (one product [q | k | v] with 32-bit results, one kernel that finishes the row head by
+head): ``bias: "qkv"`` adds biases to q, k and v and none to the output; ``value_mix`` {tensor, first} replaces a token's
+value by (1 - lambda) v + lambda v_first, with the scalar lambda in ``tensor`` and v_first the same token's values of the
+layer whose ``first`` is true (which hands its own on, unmixed, and does not use its lambda); the mixed value is what is
+cached; ``pool`` P, with ``window`` w, lets a query at position i see, beside the window's tokens, ONE key and value for
+each block of P tokens that lies wholly before the window (b P + P - 1 <= i - w): the means of the block's keys and values as
+the cache holds them.  Those live in pages of their own, one entry per P tokens, written with the block's last token; the
+tokens' own pages are given back once the window has passed them and their block is complete.  ``sink`` and per-head
+``qk_norm_eps`` go with this form.
 """
 from __future__ import annotations
 
@@ -86,7 +96,7 @@ class GQAttention(Mixer):
                             or (self.position is not None and self.rot_dims != self.d and hasattr(self.position, "head_dim")))
         self.w_qkv = self.w_o = self.q_norm = self.k_norm = None
         # ---- the rows form
-        self.has_bias = bool(params.get("bias", False))
+        self.has_bias = params.get("bias", False) is True
         wn = params.get("whole_norm_eps")
         self.whole_norm_eps = None if wn is None else float(wn)
         self.softcap = float(params.get("softcap") or 0.0)
@@ -110,6 +120,22 @@ class GQAttention(Mixer):
             names.setdefault("sink", "sink")
             if self.whole_norm_eps is not None and "q_norm" not in (params.get("names") or {}):
                 names["q_norm"], names["k_norm"] = names["q"] + ".norm", names["k"] + ".norm"
+        # ---- the heads form
+        if params.get("bias", False) not in (True, False, None, "qkv"):
+            raise ValueError(f"biases are on all projections (True) or on q, k and v ('qkv'), not {params['bias']!r}")
+        self.qkv_bias = params.get("bias") == "qkv"
+        self.value_mix = dict(params["value_mix"]) if params.get("value_mix") else None
+        self.pool = int(params.get("pool") or 0)
+        self.heads_form = bool(self.qkv_bias or self.value_mix or self.pool)
+        if self.pool < 0 or (self.pool and not self.window):
+            raise ValueError("pooled blocks go with a window and hold at least one token")
+        if self.heads_form:
+            if self.rows_form or self.values_from_keys or self.keep_first or not self.projects_kv:
+                raise ValueError("the heads form of attention goes with none of: the rows form's options, values from the keys, "
+                                 "kept first tokens, another layer's cache")
+            if getattr(self.position, "pairing", "halves") != "halves":
+                raise ValueError("this mixer rotates pairs (i, i + dims/2) only")
+        self.mix_lambda = 0.0
         self.output_bias = None
         self.row_bias = self.sink_logit = self.dist_table = self.w_rows = None
 
@@ -125,6 +151,12 @@ class GQAttention(Mixer):
         if self.qk_norm_eps is not None:
             specs[n["q_norm"]] = TensorSpec((self.d,), init="norm")
             specs[n["k_norm"]] = TensorSpec((self.d,), init="norm")
+        if self.qkv_bias:
+            specs[n["q"] + ".b"] = TensorSpec((q,), init="around_zero")
+            specs[n["k"] + ".b"] = TensorSpec((kv,), init="around_zero")
+            specs[n["v"] + ".b"] = TensorSpec((self.nkv * self.dv,), init="around_zero")
+        if self.value_mix:
+            specs[str(self.value_mix["tensor"])] = TensorSpec((), init="unit")
         if self.rows_form:
             if self.has_bias:
                 specs[n["q"] + ".b"] = TensorSpec((q,), init="around_zero")
@@ -157,6 +189,10 @@ class GQAttention(Mixer):
         if self.qk_norm_eps is not None:
             self.q_norm = tensors[n["q_norm"]].to(torch.float32).contiguous()
             self.k_norm = tensors[n["k_norm"]].to(torch.float32).contiguous()
+        if self.qkv_bias:
+            self.row_bias = torch.cat([tensors[n[x] + ".b"].to(torch.float32) for x in ("q", "k", "v")]).contiguous()
+        if self.value_mix:
+            self.mix_lambda = float(tensors[str(self.value_mix["tensor"])])
         if self.rows_form:
             self._bind_rows(tensors, parts)
 
@@ -188,6 +224,11 @@ class GQAttention(Mixer):
 
     # -------------------------------------------------------------------- cache
     def cache_need(self):
+        if self.pool:
+            vd = self.dv if self.dv != self.d else None
+            # a block's tokens stay until it is complete, also when the window is shorter than a block
+            return {"tokens": KVCacheNeed(num_kv_heads=self.nkv, head_dim=self.d, window=max(int(self.window), self.pool), value_dim=vd),
+                    "pooled": KVCacheNeed(num_kv_heads=self.nkv, head_dim=self.d, value_dim=vd, tokens_per_entry=self.pool)}
         return KVCacheNeed(num_kv_heads=self.nkv, head_dim=self.d, window=self.window,
                            value_dim=self.dv if self.dv != self.d else None, keep_first=self.keep_first)
 
@@ -227,7 +268,38 @@ class GQAttention(Mixer):
             heads = ops.sigmoid_gate(heads, gate, out=heads, group=self.dv if self.output_gate == "head" else 1)
         return ops.linear(heads, self.w_o, out_dtype=self.ctx.dtype, allow_partials=True)
 
+    VALUES_CARRIED = "first values"      # under this name the first mixing layer hands its values on
+
+    def _forward_heads(self, x, step, cache):
+        pooled_cache = None
+        if self.pool:
+            cache, pooled_cache = cache["tokens"], cache["pooled"]
+        if not cache.writes:
+            raise ValueError("the heads form of attention fills its own cache")
+        # 32-bit results of the product: biases, norms and the mix of values meet the unrounded sums
+        proj = ops.linear(x, self.w_qkv, out_dtype=torch.float32, allow_partials=True)
+        group = step.kv_groups[cache.group]
+        cos, sin = self.position.tables() if self.position is not None else (None, None)
+        first = bool(self.value_mix and self.value_mix.get("first"))
+        mix_with = step.carried[self.VALUES_CARRIED] if self.value_mix and not first else None
+        q, values = ops.qkv_heads_prepare(
+            proj, self.row_bias, self.nq, self.nkv, self.d, self.dv, self.q_norm, self.k_norm, self.qk_norm_eps or 0.0, self.rot_dims,
+            cos, sin, step.positions, cache.k, cache.v, group.slot_mapping, cache.page_size, self.ctx.dtype, mix_with=mix_with,
+            mix_lambda=self.mix_lambda if mix_with is not None else 0.0, keep_values=first)
+        if first:
+            step.carried[self.VALUES_CARRIED] = values
+        pooled = None
+        if pooled_cache is not None:
+            pgroup = step.kv_groups[pooled_cache.group]
+            pooled = ops.PooledKeys(pooled_cache.k, pooled_cache.v, pgroup.block_tables, self.pool)
+            ops.pool_blocks(cache.k, cache.v, group.block_tables, pooled, pgroup.slot_mapping, step, cache.page_size)
+        heads = ops.attention(q, cache.k, cache.v, group.block_tables, step, self.nq, self.nkv, self.d, cache.page_size, self.window,
+                              self.scale, sink=self.sink, value_dim=self.dv, pooled=pooled)
+        return ops.linear(heads, self.w_o, out_dtype=self.ctx.dtype, allow_partials=True)
+
     def forward(self, x, step, cache):
+        if self.heads_form:
+            return self._forward_heads(x, step, cache)
         if self.rows_form:
             if not cache.writes:
                 raise ValueError("the rows form of attention fills its own cache")

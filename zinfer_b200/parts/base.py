@@ -9,14 +9,15 @@ Kinds of part and what each must provide:
 
 ``Norm``            ``forward(h, delta, rows=None, bias=None)``: adds ``delta`` (may be None;
                     a tensor, split-K partial sums, or either with a multiplier as
-                    ``ops.Scaled``) and the vector ``bias`` into the 32-bit residual ``h``
+                    ``ops.Scaled``, or normed first as ``ops.PostNormed``) and the vector ``bias`` into the 32-bit residual ``h``
                     in place and returns the normed rows in the activation dtype; with
                     ``rows`` it returns the norm of the picked rows of ``h + delta`` and
                     leaves ``h`` alone.
 ``PositionEncoding````tables()``: what the mixer's kernels need to place a token.
 ``Mixer``           ``cache_need()``: a :class:`KVCacheNeed`, a :class:`StateNeed`
-                    or None; ``forward(x, step, cache)`` mixes tokens of the same
-                    request, reading and writing only its own cache.
+                    or None, or several by name; ``forward(x, step, cache)`` mixes tokens of the same
+                    request, reading and writing only its own cache; what it hands to later layers
+                    of the same step (per token) goes into ``step.carried``.
 ``FeedForward``     ``forward(x)``: works on each token alone.
 ``Block``           ``mixer`` attribute and ``forward(h, pending, step, cache, bias=None)``:
                     arranges norms, mixer, feed-forward and residual sums; returns
@@ -37,7 +38,7 @@ from ..config.spec import PartSpec
 @dataclass(frozen=True)
 class TensorSpec:
     """A tensor a part needs.  ``init`` says how the random-weights mode fills it:
-    ``matrix`` normal(0, 0.02), ``norm`` 1 + U(-0.1, 0.1), ``around_zero`` U(-0.1, 0.1), ``zeros``; ``integer``
+    ``matrix`` normal(0, 0.02), ``norm`` 1 + U(-0.1, 0.1), ``around_zero`` U(-0.1, 0.1), ``unit`` U(0, 1), ``zeros``; ``integer``
     tensors are kept as int32, others in the run's dtype (bfloat16 or float32)
     unless the file stores them in 32-bit, in which case they stay so.
 
@@ -67,7 +68,9 @@ class KVCacheNeed:
     whose values are part of its key rows, such as a latent shared by keys and values).
     ``value_dim``: the size of a value when it differs from a key's (None: ``head_dim``).  ``keep_first``:
     with a window, the request's first tokens that stay visible to every later query, so that the pages
-    which hold them are never given back.  Runs that share a cache may want different windows; the cache
+    which hold them are never given back.  ``tokens_per_entry`` P: the pages hold ONE key and value per P tokens (means over
+    blocks of tokens): entry e belongs to positions e P .. e P + P - 1, has its place from the step that brings the last
+    of them, and is never given back before the request ends (no window).  Runs that share a cache may want different windows; the cache
     then keeps what the most demanding of them reads (:meth:`merged`)."""
 
     num_kv_heads: int
@@ -76,17 +79,18 @@ class KVCacheNeed:
     values: bool = True
     value_dim: Optional[int] = None
     keep_first: int = 0
+    tokens_per_entry: int = 1
 
     def same_pages(self, other: "KVCacheNeed") -> bool:
         """Whether both describe pages of the same layout (whatever they keep of them)."""
-        return (self.num_kv_heads, self.head_dim, self.values, self.value_dim or self.head_dim) == \
-            (other.num_kv_heads, other.head_dim, other.values, other.value_dim or other.head_dim)
+        return (self.num_kv_heads, self.head_dim, self.values, self.value_dim or self.head_dim, self.tokens_per_entry) == \
+            (other.num_kv_heads, other.head_dim, other.values, other.value_dim or other.head_dim, other.tokens_per_entry)
 
     def merged(self, other: "KVCacheNeed") -> "KVCacheNeed":
         """The need of a cache that serves both: the wider window (none if either has none), the longer kept start."""
         window = None if self.window is None or other.window is None else max(self.window, other.window)
         keep = 0 if window is None else max(self.keep_first, other.keep_first)
-        return KVCacheNeed(self.num_kv_heads, self.head_dim, window, self.values, self.value_dim, keep)
+        return KVCacheNeed(self.num_kv_heads, self.head_dim, window, self.values, self.value_dim, keep, self.tokens_per_entry)
 
 
 @dataclass(frozen=True)

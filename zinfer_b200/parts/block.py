@@ -122,3 +122,42 @@ class ParallelBlock(PreNormBlock):
             return self._update(a) if row_bias is None else ops.Several([self._update(a)], row_bias=row_bias)
         out = self.feed_forward.forward(x2)
         return ops.Several([self._update(t) for t in (a, *(out if isinstance(out, tuple) else (out,)))], row_bias=row_bias)
+
+
+class SandwichBlock(PreNormBlock):
+    """The arrangement that norms a sublayer's input AND its output: h1 = h + post1(mixer(norm1(h)));
+    h2 = h1 + post2(ffn(norm2(h1))).  Parameters and tensor names as :class:`PreNormBlock`, and ``mixer_post_norm`` and
+    ``ffn_post_norm`` (names ``mixer_post_norm_name``, ``ffn_post_norm_name``) for the norms of the outputs.
+
+    A sublayer's output stays pending as :class:`ops.PostNormed`: the next norm's kernel norms it, adds it and norms the
+    sum in one pass, within the block and from a block to the next (or to the model's last norm)."""
+
+    def __init__(self, params, ctx):
+        super().__init__(params, ctx)
+        if self.residual_scale != 1.0:
+            raise ValueError("a block that norms its sublayers' outputs takes no residual multiplier")
+        if self.feed_forward is not None and self.ffn_norm is None:
+            raise ValueError("this arrangement needs a norm before its feed-forward")
+        self.mixer_post_norm = make_part(params["mixer_post_norm"], ctx)
+        self.ffn_post_norm = make_part(params["ffn_post_norm"], ctx) if self.feed_forward is not None else None
+        dot = "" if params.get("verbatim_names") else "."
+        self._names["mixer_post_norm"] = params.get("mixer_post_norm_name", "mixer_post_norm") + dot
+        self._names["ffn_post_norm"] = params.get("ffn_post_norm_name", "ffn_post_norm") + dot
+
+    def _parts(self):
+        return super()._parts() + [(self._names[k], getattr(self, k)) for k in ("mixer_post_norm", "ffn_post_norm")
+                                   if getattr(self, k) is not None]
+
+    def forward(self, h, pending, step, cache, bias=None):
+        if bias is not None:
+            raise ValueError("a block that norms its sublayers' outputs takes no per-pass vector")
+        a = self.mixer.forward(self.mixer_norm.forward(h, pending), step, cache)
+        if isinstance(a, tuple) or getattr(self.mixer, "output_bias", None) is not None:
+            raise ValueError("this arrangement takes mixers of one output without a bias")
+        pending = ops.PostNormed(a, self.mixer_post_norm)
+        if self.feed_forward is None:
+            return pending
+        out = self.feed_forward.forward(self.ffn_norm.forward(h, pending))
+        if isinstance(out, tuple):
+            raise ValueError("this arrangement takes feed-forwards of one output")
+        return ops.PostNormed(out, self.ffn_post_norm)

@@ -9,13 +9,14 @@ from .base import Part, TensorSpec
 
 
 class TokenEmbedding(Part):
-    """h0 = table[token]; no scaling.  Gives the 32-bit residual stream."""
+    """h0 = ``scale`` * table[token] (``scale`` 1 unless the model gives one).  Gives the 32-bit residual stream."""
 
     def __init__(self, params, ctx):
         super().__init__(params, ctx)
         self.vocab = int(params["vocab_size"])
         self.hidden = int(params["hidden_size"])
         self.name = params.get("name", "embed_tokens") + params.get("suffix", ".weight")
+        self.scale = float(params.get("scale", 1.0))
         self.weight = None
 
     def tensor_specs(self):
@@ -25,7 +26,7 @@ class TokenEmbedding(Part):
         self.weight = tensors[self.name].contiguous()
 
     def forward(self, token_ids):
-        return ops.embed_gather(self.weight, token_ids)
+        return ops.embed_gather(self.weight, token_ids, scale=self.scale)
 
 
 class HashedBigramEmbedding(TokenEmbedding):
@@ -39,7 +40,6 @@ class HashedBigramEmbedding(TokenEmbedding):
 
     def __init__(self, params, ctx):
         super().__init__(params, ctx)
-        self.scale = float(params.get("scale", 1.0))
         pairs = params.get("pairs")
         self.pairs_name = None if pairs is None else str(pairs["name"])
         self.buckets = int(pairs["buckets"]) if pairs is not None else 0

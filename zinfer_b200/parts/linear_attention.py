@@ -1,7 +1,7 @@
 """Mixers that keep a matrix-valued state per head instead of keys: linear attention with a decay per key
-channel, in two forms.
+channel, in three forms.
 
-Both carry, per request and head, S [dim key channels, vdim value channels] in 32-bit and update it token by token:
+All carry, per request and head, S [dim key channels, vdim value channels] in 32-bit and update it token by token:
 
     S <- diag(g_t) S ;  u_t = v_t  or  beta_t (v_t - S^T k_t) ;  S <- S + k_t u_t^T ;  o_t = S^T q_t
 
@@ -17,6 +17,10 @@ Yang et al., 2024, is the family): q, k (``kv_heads`` heads, shared by groups of
 causal convolution per channel and silu; q and k are made unit vectors per head (x / sqrt(sum x^2 + 1e-6)), q also
 times dim^(-1/2); beta = sigmoid(W_b h); g = exp(-exp(A_log_h) * softplus(W_a2 (W_a1 h) + dt_bias)) per head and key
 channel; gate sigmoid(W_g2 (W_g1 h)).  The convolutions' last taps-1 inputs are state too.
+
+:class:`HGRN2` (the form whose forget gate decides what is written; "HGRN2: Gated Linear RNNs with State Expansion",
+Qin et al., 2024, is the family): q = silu(W_q h), v = W_v h, f = l + (1 - l) sigmoid(W_f h + b) with a lower bound l
+per head and channel, g = f, k = 1 - f, u = v; no scale on q and no gate on the output.
 
 Decays, beta, unit norms, the recurrence, the state and the head norm are 32-bit; the projections run in the
 model's dtype.  The ranks of the low-rank pairs (a1/a2, g1/g2) are read from the tensors.
@@ -83,6 +87,44 @@ class GatedLinearAttention(Mixer):
         o = ops.linear_recurrence(q, k, v, decay, None, self.dim ** -0.5, cache.state, self.heads, self.heads, self.dim,
                                   self.vdim, step)
         y = ops.head_norm_gate(o, self.norm, self.eps, g, "silu", self.heads, self.vdim, self.ctx.dtype)
+        return ops.linear(y, self.w_o, out_dtype=self.ctx.dtype, allow_partials=True)
+
+
+class HGRN2(Mixer):
+    graph_safe = True
+
+    def __init__(self, params, ctx):
+        super().__init__(params, ctx)
+        self.hidden = int(params["hidden_size"])
+        self.heads = int(params["num_heads"])
+        self.dim = int(params["dim"])
+        self.vdim = int(params["vdim"])
+        self.eps = float(params["norm_eps"])
+        if min(self.heads, self.dim, self.vdim) <= 0:
+            raise ValueError("heads, dim and vdim must be positive")
+
+    def tensor_specs(self):
+        qk, hv, hid = self.heads * self.dim, self.heads * self.vdim, self.hidden
+        return {
+            "q": TensorSpec((qk, hid)), "f": TensorSpec((qk, hid)), "f.b": TensorSpec((qk,), init="zeros"),
+            "lower": TensorSpec((qk,), init="unit"), "v": TensorSpec((hv, hid)),
+            "norm": TensorSpec((self.vdim,), init="norm"), "o": TensorSpec((hid, hv)),
+        }
+
+    def bind(self, tensors):
+        f32 = lambda name: tensors[name].to(torch.float32).contiguous()
+        self.w_in = _cat([tensors[n] for n in ("q", "f", "v")])       # one product feeds all three
+        self.f_bias, self.lower, self.norm = f32("f.b"), f32("lower"), f32("norm")
+        self.w_o = tensors["o"].contiguous()
+
+    def cache_need(self):
+        return StateNeed((self.heads, self.dim, self.vdim), torch.float32)
+
+    def forward(self, x, step, cache):
+        # 32-bit results of the product: the gate and the recurrence read the unrounded sums (and add its K splits)
+        proj = ops.linear(x, self.w_in, out_dtype=torch.float32, allow_partials=True)
+        o = ops.linear_recurrence_gated(proj, self.lower, self.f_bias, cache.state, self.heads, self.dim, self.vdim, step)
+        y = ops.head_norm_gate(o, self.norm, self.eps, None, "none", self.heads, self.vdim, self.ctx.dtype)
         return ops.linear(y, self.w_o, out_dtype=self.ctx.dtype, allow_partials=True)
 
 
