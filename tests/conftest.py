@@ -80,7 +80,8 @@ def cpu_kernels(monkeypatch):
                  "latent_attention", "Carried", "norm_residual", "cast_rows", "relu2_", "qk_prepare", "short_conv", "short_conv_carry",
                  "decay_sigmoid_root_", "decay_exp_softplus_", "unit_norm_", "sigmoid_rows", "linear_recurrence", "head_norm_gate",
                  "moe_route_grouped", "moe_router_grouped", "Several", "sum_norm", "add_rmsnorm_pair", "embed_bigram",
-                 "clamped_gate", "rmsnorm_rows", "rope_table_freqs", "qkv_rows_prepare", "latent_prepare_rows", "moe_router_top_logits"):
+                 "clamped_gate", "rmsnorm_rows", "rope_table_freqs", "qkv_rows_prepare", "latent_prepare_rows", "moe_router_top_logits",
+                 "PostNormed", "PooledKeys", "sandwich_norm", "qkv_heads_prepare", "pool_blocks", "linear_recurrence_gated"):
         monkeypatch.setattr(ops, name, getattr(kernel_refs, name))
     monkeypatch.setattr(ops, "lib", lambda: None)
     monkeypatch.setattr(runner, "_require_cuda", lambda device: None)

@@ -10,8 +10,8 @@ import numpy as np
 import torch
 
 
-def embed_gather(table, ids, out=None):
-    return table[ids.long()].to(torch.float32)
+def embed_gather(table, ids, out=None, scale=1.0):
+    return table[ids.long()].to(torch.float32) * scale
 
 
 class Scaled:
@@ -418,7 +418,7 @@ def attention_prefill_tile_rows():
 
 def paged_attention(q, k_cache, v_cache, block_tables, cu_q, kv_lens, tile_seq, tile_q0, num_heads, num_kv_heads,
                     head_dim, page_size, window, scale, out=None, sink=0.0, keep_first=0, value_dim=None, sink_logit=None,
-                    softcap=0.0, dist_bias=None):
+                    softcap=0.0, dist_bias=None, pooled=None):
     T = q.shape[0]
     nq, nkv, d = num_heads, num_kv_heads, head_dim
     dv = int(value_dim or d)
@@ -439,6 +439,12 @@ def paged_attention(q, k_cache, v_cache, block_tables, cu_q, kv_lens, tile_seq, 
             offs = js % page_size
             K = k_cache[pages, :, offs, :].to(torch.float32)   # [keys, nkv, d]
             V = v_cache[pages, :, offs, :].to(torch.float32)
+            seen = max(0, (pos - window + 1) // pooled.per) if pooled is not None else 0     # blocks wholly before the window
+            if seen > 0:
+                bs = torch.arange(seen, device=q.device)
+                pp = pooled.block_tables[s, (bs // page_size)].long()
+                K = torch.cat([pooled.k[pp, :, bs % page_size, :].to(torch.float32), K])
+                V = torch.cat([pooled.v[pp, :, bs % page_size, :].to(torch.float32), V])
             qt = q[t, :nq * d].to(torch.float32).reshape(nq, d)
             for h in range(nq):
                 sc = (K[:, h // g, :] @ qt[h]) * scale
@@ -469,10 +475,10 @@ def linear_argmax(x, weight):
 
 
 def attention(q, k_cache, v_cache, block_tables, step, num_heads, num_kv_heads, head_dim, page_size, window, scale, sink=0.0,
-              keep_first=0, value_dim=None, sink_logit=None, softcap=0.0, dist_bias=None):
+              keep_first=0, value_dim=None, sink_logit=None, softcap=0.0, dist_bias=None, pooled=None):
     return paged_attention(q, k_cache, v_cache, block_tables, step.cu_q, step.kv_lens, step.tile_seq, step.tile_q0,
                            num_heads, num_kv_heads, head_dim, page_size, window, scale, sink=sink, keep_first=keep_first,
-                           value_dim=value_dim, sink_logit=sink_logit, softcap=softcap, dist_bias=dist_bias)
+                           value_dim=value_dim, sink_logit=sink_logit, softcap=softcap, dist_bias=dist_bias, pooled=pooled)
 
 
 def patch_tokens(ids, prev, dst, src):
@@ -658,6 +664,8 @@ def linear_recurrence(q, k, v, decay, beta, q_scale, state, heads, key_heads, di
 def head_norm_gate(o, weight, eps, gate, gate_kind, heads, vdim, out_dtype):
     T = o.shape[0]
     x = o.reshape(T, heads, vdim)
+    if gate_kind == "none":
+        return (x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * weight).reshape(T, heads * vdim).to(out_dtype)
     g = gate.to(torch.float32).reshape(T, heads, vdim)
     act = g * torch.sigmoid(g) if gate_kind == "silu" else torch.sigmoid(g)
     return (x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * weight * act).reshape(T, heads * vdim).to(out_dtype)
@@ -764,3 +772,84 @@ def moe_router_top_logits(x, w_router, bias, top):
     order = torch.sort(z, dim=-1, descending=True, stable=True).indices[:, :top]
     weight = torch.softmax(torch.gather(z, 1, order), dim=-1)
     return order.to(torch.int32), weight
+
+
+# ------------------------- norms before and after a sublayer, pooled keys, gates that decide what is written
+class PostNormed:
+    def __init__(self, delta, norm):
+        self.delta, self.norm = delta, norm
+
+
+class PooledKeys:
+    def __init__(self, k, v, block_tables, per):
+        self.k, self.v, self.block_tables, self.per = k, v, block_tables, int(per)
+
+
+def _norm_kind(x, w, eps, kind):
+    c = x - x.mean(-1, keepdim=True) if kind == "layer" else x
+    return c / torch.sqrt((c * c).mean(-1, keepdim=True) + eps) * w
+
+
+def sandwich_norm(h, delta, pre_weight, pre_eps, pre_kind, out_dtype, rows=None):
+    post = None
+    if isinstance(delta, PostNormed):
+        delta, post = delta.delta, delta.norm
+    y = _terms_sum(delta)
+    if y is not None and post is not None:
+        y = _norm_kind(y, post.weight, post.eps, post.kind)
+    total = h if y is None else h + y
+    if rows is None and y is not None:
+        h.copy_(total)
+    if pre_weight is None:
+        return None
+    x = _norm_kind(total, pre_weight, pre_eps, pre_kind)
+    return (x if rows is None else x[rows.long()]).to(out_dtype)
+
+
+def qkv_heads_prepare(proj, bias, num_heads, num_kv_heads, head_dim, value_dim, q_weight, k_weight, eps, rot_dims, cos, sin, positions,
+                      k_cache, v_cache, slots, page_size, out_dtype, mix_with=None, mix_lambda=0.0, keep_values=False):
+    T = proj.shape[0]
+    qn, kn = num_heads * head_dim, num_kv_heads * head_dim
+    row = proj.to(torch.float32) + (bias if bias is not None else 0.0)
+
+    def finish(x, w, heads):
+        x = x.reshape(T, heads, head_dim)
+        if w is not None:
+            x = x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * w
+        if cos is not None:
+            pos = positions.long()
+            x = _rotate_first(x, cos[pos][:, None, :], sin[pos][:, None, :], rot_dims)
+        return x
+
+    q, k = finish(row[:, :qn], q_weight, num_heads), finish(row[:, qn:qn + kn], k_weight, num_kv_heads)
+    v = row[:, qn + kn:]
+    if mix_with is not None:
+        v = (1.0 - mix_lambda) * v + mix_lambda * mix_with
+    for t in range(T):
+        slot = int(slots[t])
+        if slot >= 0:
+            k_cache[slot // page_size, :, slot % page_size] = k[t].to(out_dtype)
+            v_cache[slot // page_size, :, slot % page_size] = v[t].reshape(num_kv_heads, value_dim).to(out_dtype)
+    return q.reshape(T, qn).to(out_dtype), (v.clone() if keep_values else None)
+
+
+def pool_blocks(k_cache, v_cache, block_tables, pooled, entry_slots, step, page_size):
+    cu = [int(c) for c in step.cu_q[:step.n_seqs + 1]]
+    for s in range(step.n_seqs):
+        for t in range(cu[s], cu[s + 1]):
+            entry = int(entry_slots[t])
+            if entry < 0:
+                continue
+            last = int(step.positions[t])
+            for src, dst in ((k_cache, pooled.k), (v_cache, pooled.v)):
+                rows = [src[int(block_tables[s, p // page_size]), :, p % page_size].to(torch.float32)
+                        for p in range(last - pooled.per + 1, last + 1)]
+                dst[entry // page_size, :, entry % page_size] = torch.stack(rows).mean(0).to(dst.dtype)
+
+
+def linear_recurrence_gated(proj, lower, f_bias, state, heads, dim, vdim, step):
+    qk = heads * dim
+    q, z, v = proj[:, :qk], proj[:, qk:2 * qk], proj[:, 2 * qk:]
+    f = lower + (1.0 - lower) * torch.sigmoid(z + (f_bias if f_bias is not None else 0.0))
+    k = (1.0 - lower) * torch.sigmoid(-(z + (f_bias if f_bias is not None else 0.0)))
+    return linear_recurrence(q * torch.sigmoid(q), k, v, f, None, 1.0, state, heads, heads, dim, vdim, step)

@@ -330,6 +330,20 @@ int zi_attention_decode_mma_mask(void* out, int out_stride, float* workspace, co
                                  const int* cu_q, const int* kv_lens, const int* dec_seq, int n_dec, int nq, int nkv, int d,
                                  int page_size, int window, int keep_first, float scale, int splits, float sink,
                                  cudaStream_t stream);
+// Whether they take these sizes (multiples of 8 up to 128, decode up to 256), and the tile width they run with.
+int zi_attention_mma_sized_supported(int nq, int nkv, int d, int dv, int decode);
+int zi_attention_mma_sized_tile(int d, int dv);
+// The two kernels with a window, one key and value per `per` tokens for the blocks of tokens before it, and a sink.
+int zi_attention_prefill_mma_pooled(void* out, int out_stride, const void* q, int q_stride, const void* kcache,
+                                    const void* vcache, const int* block_tables, int bt_stride, const void* kpool,
+                                    const void* vpool, const int* pool_tables, int pool_bt_stride, int per, const int* cu_q,
+                                    const int* kv_lens, const int* tile_seq, const int* tile_q0, int n_tiles, int nq, int nkv,
+                                    int d, int dv, int page_size, int window, float scale, float sink, cudaStream_t stream);
+int zi_attention_decode_mma_pooled(void* out, int out_stride, float* workspace, const void* q, int q_stride, const void* kcache,
+                                   const void* vcache, long long n_pages, const int* block_tables, int bt_stride,
+                                   const void* kpool, const void* vpool, const int* pool_tables, int pool_bt_stride, int per,
+                                   const int* cu_q, const int* kv_lens, const int* dec_seq, int n_dec, int nq, int nkv, int d,
+                                   int dv, int page_size, int window, float scale, int splits, float sink, cudaStream_t stream);
 long long zi_attention_decode_workspace_floats(int n_dec, int nq, int nkv, int d, int splits);
 int zi_attention_decode_mma(void* out, int out_stride, float* workspace, const void* q, int q_stride,
                             const void* kcache, const void* vcache, long long n_pages, const int* block_tables, int bt_stride,

@@ -241,7 +241,7 @@ extern "C" int zi_paged_attention_mods(void* out, int out_stride, const void* q,
   if (page_size <= 0) return zi_refuse("paged_attention: page_size %d", page_size);
   if (pool_per > 0 && (!kpool || !vpool || !pool_tables || window <= 0 || dist_bias || v_row != dv))
     return zi_refuse("paged_attention: pooled keys go with a window, pages of their own and no bias by distance");
-  const PooledKeys pool = {kpool, vpool, pool_tables, pool_bt_stride, pool_per};
+  const PooledKeys pool = {kpool, vpool, pool_tables, pool_bt_stride, pool_per, d, dv};
   const size_t smem = (size_t)(BQ * d + BK * (d + 1) + BK * dv + BQ * BK) * sizeof(float);
   dim3 grid(n_tiles, nq);
 #define ZI_LAUNCH_ATTN(J)                                                                                          \

@@ -32,14 +32,17 @@ constexpr int PF_BQ = 128, PF_BK = 64, PF_THREADS = 256;
 // With a window, a request's first keep_first keys stay visible (query i sees key j <= i if i - j < window or
 // j < keep_first): the tiles of those keys that lie before the window's first tile are walked first.
 // MD (with XP): the scores are changed as ScoreMods says (a cap, a bias by distance, a learned sink per head).
-template <int D, bool XP, bool MD = false>
+// PL (with XP, no kept first tokens): one key and value for every block of tokens that lies wholly before a query's window
+// (PooledKeys; none if pool.per is 0); their tiles are walked first.  Keys and values may be narrower than D (multiples of
+// 8): the tiles' columns beyond them are zero.
+template <int D, bool XP, bool MD = false, bool PL = false>
 __global__ void __launch_bounds__(PF_THREADS, 2)
 attn_prefill_mma_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restrict__ q, int q_stride,
                         const bf16* __restrict__ kcache, const bf16* __restrict__ vcache,
                         const int* __restrict__ block_tables, int bt_stride, const int* __restrict__ cu_q,
                         const int* __restrict__ kv_lens, const int* __restrict__ tile_seq,
                         const int* __restrict__ tile_q0, int nq, int nkv, int page_size, int page_shift,
-                        int window, float scale_log2, float sink, int keep_first, const ScoreMods md) {
+                        int window, float scale_log2, float sink, int keep_first, const ScoreMods md, const PooledKeys pool) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(128) uint8_t smem[];
@@ -64,13 +67,20 @@ attn_prefill_mma_kernel(bf16* __restrict__ out, int out_stride, const bf16* __re
   for (int e = tid; e < PF_BQ * (D / 8); e += PF_THREADS) {
     const int r = e / (D / 8), c = e % (D / 8);
     const bool valid = r < nqv;
+    if constexpr (PL) {
+      const bool in = valid && c * 8 < pool.d;
+      cp_async16(qs + swz<D>(r, c), q + (in ? (size_t)(tok0 + q0 + r) * q_stride + (size_t)h * pool.d + c * 8 : 0), in);
+      continue;
+    }
     const bf16* src = q + (size_t)(tok0 + q0 + (valid ? r : 0)) * q_stride + (size_t)h * D + c * 8;
     cp_async16(qs + swz<D>(r, c), src, valid);
   }
   const int kt0 = (kv_lo / PF_BK) * PF_BK;
   // (only in the form with a sink; the plain form's code stays as it was: everything below folds away)
-  const int keep_end = XP && window > 0 ? min(keep_first, kv_lo) : 0;      // keys [0, keep_end) lie before the window and stay visible
-  const int n_keep = (min(keep_end, kt0) + PF_BK - 1) / PF_BK;       // their tiles before the window's first tile
+  const int keep_end = XP && !PL && window > 0 ? min(keep_first, kv_lo) : 0;      // keys [0, keep_end) lie before the window and stay visible
+  const int n_pooled = PL ? pooled_visible(pool, last_pos, window) : 0;      // the pooled entries that the block's last query sees
+  const int n_keep = ((PL ? n_pooled : min(keep_end, kt0)) + PF_BK - 1) / PF_BK;       // their tiles before the window's first tile
+  const int* pbt = PL ? pool.block_tables + (size_t)seq * pool.bt_stride : nullptr;
   const int n_tiles = n_keep + (kv_hi - kt0 + PF_BK - 1) / PF_BK;
   auto tile_kt = [&](int t) { return t < n_keep ? t * PF_BK : kt0 + (t - n_keep) * PF_BK; };
 
@@ -80,29 +90,45 @@ attn_prefill_mma_kernel(bf16* __restrict__ out, int out_stride, const bf16* __re
   constexpr int CH = D / 8, NPER = PF_BK * CH / PF_THREADS, RSTEP = PF_THREADS / CH;
   const int my_r = tid / CH, my_c = tid % CH;
   int pg[NPER];
-  auto lookup = [&](int kt) {
+  auto lookup = [&](int t) {
+    const int kt = tile_kt(t);
 #pragma unroll
     for (int i = 0; i < NPER; ++i) {
       const int j = kt + my_r + i * RSTEP;
+      if (PL && t < n_keep) {
+        pg[i] = j < n_pooled ? __ldg(pbt + (page_shift >= 0 ? (j >> page_shift) : (j / page_size))) : -1;
+        continue;
+      }
       pg[i] = ((j >= kv_lo || j < keep_end) && j < kv_hi) ? __ldg(bt + (page_shift >= 0 ? (j >> page_shift) : (j / page_size))) : -1;
     }
   };
-  auto issue = [&](int kt, int buf) {
+  auto issue = [&](int t, int buf) {
+    const int kt = tile_kt(t);
+    const bool of_blocks = PL && t < n_keep;
+    const bf16* kb = of_blocks ? static_cast<const bf16*>(pool.k) : kcache;
+    const bf16* vb = of_blocks ? static_cast<const bf16*>(pool.v) : vcache;
 #pragma unroll
     for (int i = 0; i < NPER; ++i) {
       const int r = my_r + i * RSTEP, j = kt + r;
       const bool valid = pg[i] >= 0;
       const int in_page = page_shift >= 0 ? (j & (page_size - 1)) : (j % page_size);
-      const size_t off = valid ? (((size_t)pg[i] * nkv + kvh) * page_size + in_page) * D + my_c * 8 : 0;
       const uint32_t so = swz<D>(r, my_c);
-      cp_async16(kbuf + buf * TILE_BYTES + so, kcache + off, valid);
-      cp_async16(vbuf + buf * TILE_BYTES + so, vcache + off, valid);
+      if constexpr (PL) {
+        const bool kin = valid && my_c * 8 < pool.d, vin = valid && my_c * 8 < pool.dv;
+        const size_t row = valid ? ((size_t)pg[i] * nkv + kvh) * page_size + in_page : 0;
+        cp_async16(kbuf + buf * TILE_BYTES + so, kb + (kin ? row * pool.d + my_c * 8 : 0), kin);
+        cp_async16(vbuf + buf * TILE_BYTES + so, vb + (vin ? row * pool.dv + my_c * 8 : 0), vin);
+        continue;
+      }
+      const size_t off = valid ? (((size_t)pg[i] * nkv + kvh) * page_size + in_page) * D + my_c * 8 : 0;
+      cp_async16(kbuf + buf * TILE_BYTES + so, kb + off, valid);
+      cp_async16(vbuf + buf * TILE_BYTES + so, vb + off, valid);
     }
   };
-  lookup(tile_kt(0));
-  issue(tile_kt(0), 0);
+  lookup(0);
+  issue(0, 0);
   cp_async_commit();
-  if (n_tiles > 1) lookup(tile_kt(1));
+  if (n_tiles > 1) lookup(1);
 
   float o[D / 8][4];
 #pragma unroll
@@ -117,9 +143,9 @@ attn_prefill_mma_kernel(bf16* __restrict__ out, int out_stride, const bf16* __re
     const int kt = tile_kt(t);
     const int buf = t & 1;
     if (t + 1 < n_tiles) {
-      issue(tile_kt(t + 1), buf ^ 1);
+      issue(t + 1, buf ^ 1);
       cp_async_commit();
-      if (t + 2 < n_tiles) lookup(tile_kt(t + 2));
+      if (t + 2 < n_tiles) lookup(t + 2);
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
@@ -127,7 +153,8 @@ attn_prefill_mma_kernel(bf16* __restrict__ out, int out_stride, const bf16* __re
     __syncthreads();
     // a warp whose rows all lie before this tile (causal) or after it (window, unless the tile holds kept first
     // keys: those of the window's own first tiles count too, for the block's later rows) has nothing to do
-    const bool tile_visible = warp_active && kt <= warp_last_pos &&
+    const bool of_blocks = PL && t < n_keep;
+    const bool tile_visible = of_blocks ? warp_active && kt < pooled_visible(pool, warp_last_pos, window) : warp_active && kt <= warp_last_pos &&
                               (window <= 0 || kt + PF_BK - 1 > warp_first_pos - window || (XP && kt < keep_first));
     if (tile_visible) {
       const uint32_t ks_addr = smem_addr(kbuf + buf * TILE_BYTES), vs_addr = smem_addr(vbuf + buf * TILE_BYTES);
@@ -150,6 +177,8 @@ attn_prefill_mma_kernel(bf16* __restrict__ out, int out_stride, const bf16* __re
         }
       }
       const bool need_mask = kt + PF_BK - 1 > warp_first_pos || window > 0 || kt < kv_lo;
+      const int seen[2] = {of_blocks ? pooled_visible(pool, first_pos + row_lo, window) : 0,          // entries that this thread's
+                           of_blocks ? pooled_visible(pool, first_pos + row_lo + 8, window) : 0};     // two rows see
 #pragma unroll
       for (int nt = 0; nt < PF_BK / 8; ++nt) {
 #pragma unroll
@@ -160,7 +189,8 @@ attn_prefill_mma_kernel(bf16* __restrict__ out, int out_stride, const bf16* __re
           if (need_mask) {
             const int j = kt + nt * 8 + 2 * (lane & 3) + (c & 1);
             const int pos = first_pos + row_lo + (c >> 1) * 8;
-            const bool vis = j <= pos && (window <= 0 || j > pos - window || (XP && j < keep_first));
+            const bool vis = PL && of_blocks ? j < seen[c >> 1]
+                                             : j <= pos && (window <= 0 || j > pos - window || (XP && !PL && j < keep_first));
             if (!vis) v = -INFINITY;
           }
           s[nt][c] = v;
@@ -194,9 +224,11 @@ attn_prefill_mma_kernel(bf16* __restrict__ out, int out_stride, const bf16* __re
         if (md.sink_logit) sum += exp2f(md.sink_logit[h] * ZI_LOG2E - m[i]);      // a learned sink of this head
       }
       const float inv = 1.0f / sum;
-      bf16* orow = out + (size_t)(tok0 + q0 + r) * out_stride + (size_t)h * D + 2 * (lane & 3);
+      const int od = PL ? pool.dv : D;
+      bf16* orow = out + (size_t)(tok0 + q0 + r) * out_stride + (size_t)h * od + 2 * (lane & 3);
 #pragma unroll
       for (int t = 0; t < D / 8; ++t)
+        if (!PL || t * 8 < od)
         *reinterpret_cast<uint32_t*>(orow + t * 8) = pack_bf16(o[t][2 * i] * inv, o[t][2 * i + 1] * inv);
     }
   }
@@ -207,7 +239,7 @@ struct BlockSync {
   static __device__ __forceinline__ void sync() { __syncthreads(); }
 };
 
-template <int D, bool FUSED, bool TR, bool TMA, bool XP = false, bool MD = false>
+template <int D, bool FUSED, bool TR, bool TMA, bool XP = false, bool MD = false, bool PL = false>
 __global__ void __launch_bounds__(DC_THREADS)
 attn_decode_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                        int* __restrict__ status, bf16* __restrict__ out, int out_stride, float* __restrict__ partial,
@@ -215,7 +247,8 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                        const bf16* __restrict__ vcache, const int* __restrict__ block_tables, int bt_stride,
                        const int* __restrict__ cu_q, const int* __restrict__ kv_lens,
                        const int* __restrict__ dec_seq, int nq, int nkv, int page_size, int page_shift, int window,
-                       float scale_log2, int splits, const FusedQK fq, float sink, int keep_first, const ScoreMods md) {
+                       float scale_log2, int splits, const FusedQK fq, float sink, int keep_first, const ScoreMods md,
+                       const PooledKeys pool) {
   pdl_launch_dependents();
   // (the unit waits for the kernel before this one itself, after it has asked for its first keys)
   extern __shared__ __align__(128) uint8_t smem_raw[];
@@ -224,23 +257,23 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
   constexpr int RING_BYTES = DC_WARPS * DecodeCfg<D>::STAGES * 2 * DC_KEYS * D * 2;
   constexpr int FUSED_BYTES = FUSED ? 16 * D * 2 + (2 * D + 16) * (int)sizeof(float) : 0;
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + RING_BYTES + ((FUSED_BYTES + 15) & ~15));
-  attn_decode_unit<D, FUSED, BlockSync, DecodeCfg<D>::STAGES, TR, TMA, XP, MD>(
+  attn_decode_unit<D, FUSED, BlockSync, DecodeCfg<D>::STAGES, TR, TMA, XP, MD, PL>(
       smem, threadIdx.x, blockIdx.x, blockIdx.y, blockIdx.z, out, out_stride, partial, q, q_stride, kcache, vcache,
       block_tables, bt_stride, cu_q, kv_lens, dec_seq, nq, nkv, page_size, page_shift, window, scale_log2, splits, fq,
-      nullptr, &map_k, &map_v, bars, status, sink, keep_first, &md);
+      nullptr, &map_k, &map_v, bars, status, sink, keep_first, &md, &pool);
 }
 
 template <int D>
 __global__ void attn_decode_combine_kernel(bf16* __restrict__ out, int out_stride, const float* __restrict__ partial,
                                            const int* __restrict__ cu_q, const int* __restrict__ dec_seq, int nq,
-                                           int nkv, int splits, float sink, const float* __restrict__ sink_logit) {
+                                           int nkv, int splits, float sink, const float* __restrict__ sink_logit, int dv) {
   pdl_launch_dependents();
   // which token this is comes from the step's own arrays (copied before any kernel of the step):
   // these two dependent loads need not wait for the attention kernel
   const int token = cu_q[dec_seq[blockIdx.x]];
   pdl_wait();
   attn_decode_combine_item<D>(blockIdx.x, blockIdx.y, threadIdx.x, blockDim.x, out, out_stride, partial, token, nq, nkv,
-                              splits, sink, sink_logit);
+                              splits, sink, sink_logit, dv);
 }
 
 
@@ -248,8 +281,10 @@ template <int D>
 int launch_prefill(void* out, int out_stride, const void* q, int q_stride, const void* kc, const void* vc,
                    const int* bt, int bt_stride, const int* cu_q, const int* kv_lens, const int* tile_seq,
                    const int* tile_q0, int n_tiles, int nq, int nkv, int page_size, int window, float scale,
-                   cudaStream_t stream, bool xp = false, float sink = 0.f, int keep_first = 0, const ScoreMods* mods = nullptr) {
-  auto kern = mods ? attn_prefill_mma_kernel<D, true, true> : (xp ? attn_prefill_mma_kernel<D, true> : attn_prefill_mma_kernel<D, false>);
+                   cudaStream_t stream, bool xp = false, float sink = 0.f, int keep_first = 0, const ScoreMods* mods = nullptr,
+                   const PooledKeys* pool = nullptr) {
+  auto kern = pool ? attn_prefill_mma_kernel<D, true, false, true>
+                   : mods ? attn_prefill_mma_kernel<D, true, true> : (xp ? attn_prefill_mma_kernel<D, true> : attn_prefill_mma_kernel<D, false>);
   ScoreMods md = {};
   if (mods) md = *mods;
   md.scale = scale;
@@ -260,7 +295,7 @@ int launch_prefill(void* out, int out_stride, const void* q, int q_stride, const
   zi_launch(kern, dim3(grid), dim3(PF_THREADS), smem, stream, (bf16*)out, out_stride, (const bf16*)q, q_stride, (const bf16*)kc,
                                            (const bf16*)vc, bt, bt_stride, cu_q, kv_lens, tile_seq, tile_q0, nq, nkv,
                                            page_size, log2_or_minus1(page_size), window, scale * 1.4426950408889634f, sink,
-                                           keep_first, md);
+                                           keep_first, md, pool ? *pool : PooledKeys{});
   return zi_check_launch("attention_prefill");
 }
 
@@ -268,13 +303,13 @@ int g_decode_transposed = 1;   // zi_attention_decode_transposed(0) switches the
 
 int g_decode_tma = 1;          // see zi_attention_decode_tma
 
-template <int D, bool FUSED, bool TR, bool TMA, bool XP = false, bool MD = false>
+template <int D, bool FUSED, bool TR, bool TMA, bool XP = false, bool MD = false, bool PL = false>
 int launch_decode_as(void* out, int out_stride, float* partial, const void* q, int q_stride, const void* kc,
                      const void* vc, long long n_pages, const int* bt, int bt_stride, const int* cu_q,
                      const int* kv_lens, const int* dec_seq, int n_dec, int nq, int nkv, int page_size, int window,
                      float scale, int splits, const FusedQK& fq, cudaStream_t stream, float sink = 0.f, int keep_first = 0,
-                     const ScoreMods* mods = nullptr) {
-  auto kern = attn_decode_mma_kernel<D, FUSED, TR, TMA, XP, MD>;
+                     const ScoreMods* mods = nullptr, const PooledKeys* pool = nullptr) {
+  auto kern = attn_decode_mma_kernel<D, FUSED, TR, TMA, XP, MD, PL>;
   ScoreMods md = {};
   if (mods) md = *mods;
   md.scale = scale;
@@ -299,7 +334,7 @@ int launch_decode_as(void* out, int out_stride, float* partial, const void* q, i
   zi_launch(kern, dim3(grid), dim3(DC_THREADS), smem, stream, map_k, map_v, status, (bf16*)out, out_stride,
             splits > 1 ? partial : nullptr, (const bf16*)q, q_stride, (const bf16*)kc, (const bf16*)vc, bt, bt_stride, cu_q,
             kv_lens, dec_seq, nq, nkv, page_size, log2_or_minus1(page_size), window, scale * 1.4426950408889634f, splits, fq, sink,
-            keep_first, md);
+            keep_first, md, pool ? *pool : PooledKeys{});
   return 0;
 }
 
@@ -308,7 +343,7 @@ int launch_decode(void* out, int out_stride, float* partial, const void* q, int 
                   const void* vc, long long n_pages, const int* bt, int bt_stride, const int* cu_q, const int* kv_lens,
                   const int* dec_seq, int n_dec, int nq, int nkv, int page_size, int window, float scale, int splits,
                   const FusedQK& fq, cudaStream_t stream, bool xp = false, float sink = 0.f, int keep_first = 0,
-                  const ScoreMods* mods = nullptr) {
+                  const ScoreMods* mods = nullptr, const PooledKeys* pool = nullptr) {
   // Groups of at most 8 query heads take the transposed tile (keys on the MMA's rows).  Keys and values come by
   // TMA (page boxes, pages of 8, 16, 32, ... tokens whose rows a tensor map can address) while the requests
   // are few, and by cp.async from every lane when they are many.  Measured per 36-layer step (Qwen3-8B
@@ -330,9 +365,15 @@ int launch_decode(void* out, int out_stride, float* partial, const void* q, int 
   launch_decode_as<D, false, TR_, TMA_, true, true>(out, out_stride, partial, q, q_stride, kc, vc, n_pages, bt, bt_stride, cu_q, \
                                                     kv_lens, dec_seq, n_dec, nq, nkv, page_size, window, scale, splits, fq, stream, \
                                                     sink, keep_first, mods)
+#define ZI_DECODE_PL(TR_)                                                                                              \
+  launch_decode_as<D, false, TR_, false, true, false, true>(out, out_stride, partial, q, q_stride, kc, vc, n_pages, bt, bt_stride, \
+                                                            cu_q, kv_lens, dec_seq, n_dec, nq, nkv, page_size, window, scale,      \
+                                                            splits, fq, stream, sink, 0, nullptr, pool)
   int rc0;
   if constexpr (!FUSED) {
-    if (mods)   // changed scores (a cap, a bias by distance, a learned sink), exact weights
+    if (pool)   // pooled entries beside a window's tokens, exact weights
+      rc0 = tr ? ZI_DECODE_PL(true) : ZI_DECODE_PL(false);
+    else if (mods)   // changed scores (a cap, a bias by distance, a learned sink), exact weights
       rc0 = tr ? (tma ? ZI_DECODE_MD(true, true) : ZI_DECODE_MD(true, false)) : (tma ? ZI_DECODE_MD(false, true) : ZI_DECODE_MD(false, false));
     else if (xp)     // exact weights and a sink: the kernel that only reads q (the fused form makes whole-head rotations)
       rc0 = tr ? (tma ? ZI_DECODE_XP(true, true) : ZI_DECODE_XP(true, false)) : (tma ? ZI_DECODE_XP(false, true) : ZI_DECODE_XP(false, false));
@@ -341,6 +382,7 @@ int launch_decode(void* out, int out_stride, float* partial, const void* q, int 
   } else {
     rc0 = tr ? (tma ? ZI_DECODE_AS(true, true) : ZI_DECODE_AS(true, false)) : (tma ? ZI_DECODE_AS(false, true) : ZI_DECODE_AS(false, false));
   }
+#undef ZI_DECODE_PL
 #undef ZI_DECODE_MD
 #undef ZI_DECODE_XP
 #undef ZI_DECODE_AS
@@ -349,7 +391,7 @@ int launch_decode(void* out, int out_stride, float* partial, const void* q, int 
   if (rc) return rc;
   if (splits > 1) {
     zi_launch(attn_decode_combine_kernel<D>, dim3(n_dec, nq), dim3(D >= 128 ? 128 : 64), 0, stream, (bf16*)out,
-              out_stride, partial, cu_q, dec_seq, nq, nkv, splits, sink, mods ? mods->sink_logit : (const float*)nullptr);
+              out_stride, partial, cu_q, dec_seq, nq, nkv, splits, sink, mods ? mods->sink_logit : (const float*)nullptr, pool ? pool->dv : D);
     rc = zi_check_launch("attention_decode_combine");
   }
   return rc;
@@ -360,15 +402,15 @@ int dispatch_decode(int d, void* out, int out_stride, float* partial, const void
                     const void* vc, long long n_pages, const int* bt, int bt_stride, const int* cu_q, const int* kv_lens,
                     const int* dec_seq, int n_dec, int nq, int nkv, int page_size, int window, float scale, int splits,
                     const FusedQK& fq, cudaStream_t stream, bool xp = false, float sink = 0.f, int keep_first = 0,
-                    const ScoreMods* mods = nullptr) {
+                    const ScoreMods* mods = nullptr, const PooledKeys* pool = nullptr) {
   if (d == 64)
     return launch_decode<64, FUSED>(out, out_stride, partial, q, q_stride, kc, vc, n_pages, bt, bt_stride, cu_q, kv_lens, dec_seq,
-                                    n_dec, nq, nkv, page_size, window, scale, splits, fq, stream, xp, sink, keep_first, mods);
+                                    n_dec, nq, nkv, page_size, window, scale, splits, fq, stream, xp, sink, keep_first, mods, pool);
   if (d == 128)
     return launch_decode<128, FUSED>(out, out_stride, partial, q, q_stride, kc, vc, n_pages, bt, bt_stride, cu_q, kv_lens,
-                                     dec_seq, n_dec, nq, nkv, page_size, window, scale, splits, fq, stream, xp, sink, keep_first, mods);
+                                     dec_seq, n_dec, nq, nkv, page_size, window, scale, splits, fq, stream, xp, sink, keep_first, mods, pool);
   return launch_decode<256, FUSED>(out, out_stride, partial, q, q_stride, kc, vc, n_pages, bt, bt_stride, cu_q, kv_lens, dec_seq,
-                                   n_dec, nq, nkv, page_size, window, scale, splits, fq, stream, xp, sink, keep_first, mods);
+                                   n_dec, nq, nkv, page_size, window, scale, splits, fq, stream, xp, sink, keep_first, mods, pool);
 }
 }  // namespace
 
@@ -395,6 +437,14 @@ extern "C" int zi_attention_mma_supported(int nq, int nkv, int d, int decode) {
   if (nkv <= 0 || nq % nkv) return 0;
   if (decode) return (d == 64 || d == 128 || d == 256) && nq / nkv <= 16;
   return d == 64 || d == 128;
+}
+
+// The same for the form with pooled keys, which takes any sizes (multiples of 8) that a tile holds; and that tile.
+extern "C" int zi_attention_mma_sized_tile(int d, int dv) { return d <= 64 && dv <= 64 ? 64 : (d <= 128 && dv <= 128 ? 128 : 256); }
+extern "C" int zi_attention_mma_sized_supported(int nq, int nkv, int d, int dv, int decode) {
+  if (nkv <= 0 || nq % nkv || d <= 0 || dv <= 0 || d % 8 || dv % 8) return 0;
+  if (decode) return d <= 256 && dv <= 256 && nq / nkv <= 16;
+  return d <= 128 && dv <= 128;
 }
 
 extern "C" int zi_attention_prefill_mma(void* out, int out_stride, const void* q, int q_stride, const void* kcache,
@@ -504,6 +554,47 @@ extern "C" int zi_attention_decode_mma_mask(void* out, int out_stride, float* wo
   FusedQK none = {};
   return dispatch_decode<false>(d, out, out_stride, workspace, q, q_stride, kcache, vcache, n_pages, block_tables, bt_stride, cu_q,
                                 kv_lens, dec_seq, n_dec, nq, nkv, page_size, window, scale, splits, none, stream, true, sink, keep_first);
+}
+
+// The two kernels with a window, pooled keys and values of the tokens before it (pages of one entry per `per` tokens, with
+// their own block tables) and a sink.
+extern "C" int zi_attention_prefill_mma_pooled(void* out, int out_stride, const void* q, int q_stride, const void* kcache,
+                                               const void* vcache, const int* block_tables, int bt_stride, const void* kpool,
+                                               const void* vpool, const int* pool_tables, int pool_bt_stride, int per,
+                                               const int* cu_q, const int* kv_lens, const int* tile_seq, const int* tile_q0,
+                                               int n_tiles, int nq, int nkv, int d, int dv, int page_size, int window,
+                                               float scale, float sink, cudaStream_t stream) {
+  if (n_tiles <= 0) return 0;
+  if (!zi_attention_mma_sized_supported(nq, nkv, d, dv, 0)) return zi_refuse("attention_prefill: keys of %d and values of %d", d, dv);
+  if (q_stride % 8 || ((uintptr_t)q % 16) || ((uintptr_t)out % 4) || out_stride % 2) return zi_refuse("attention_prefill: q rows must be 16-byte aligned");
+  if (!(sink >= 0.f)) return zi_refuse("attention_prefill: the sink's weight must not be negative");
+  if (per < 0 || (per > 0 && (window <= 0 || !kpool || !vpool || !pool_tables))) return zi_refuse("attention_prefill: pooled keys go with a window and pages");
+  const PooledKeys pool = {kpool, vpool, pool_tables, pool_bt_stride, per, d, dv};
+  auto launch = d <= 64 && dv <= 64 ? launch_prefill<64> : launch_prefill<128>;
+  return launch(out, out_stride, q, q_stride, kcache, vcache, block_tables, bt_stride, cu_q, kv_lens, tile_seq, tile_q0, n_tiles, nq,
+                nkv, page_size, window, scale, stream, true, sink, 0, nullptr, &pool);
+}
+
+extern "C" int zi_attention_decode_mma_pooled(void* out, int out_stride, float* workspace, const void* q, int q_stride,
+                                              const void* kcache, const void* vcache, long long n_pages,
+                                              const int* block_tables, int bt_stride, const void* kpool, const void* vpool,
+                                              const int* pool_tables, int pool_bt_stride, int per, const int* cu_q,
+                                              const int* kv_lens, const int* dec_seq, int n_dec, int nq, int nkv, int d,
+                                              int dv, int page_size, int window, float scale, int splits, float sink,
+                                              cudaStream_t stream) {
+  if (n_dec <= 0) return 0;
+  if (!zi_attention_mma_sized_supported(nq, nkv, d, dv, 1))
+    return zi_refuse("attention_decode: keys of %d, values of %d or groups of %d (<= 16) are not supported", d, dv, nq / nkv);
+  if (splits < 1 || (splits > 1 && !workspace)) return zi_refuse("attention_decode: %d splits need a workspace", splits);
+  if (q_stride % 2) return zi_refuse("attention_decode: q rows must be 4-byte aligned");
+  if (!(sink >= 0.f)) return zi_refuse("attention_decode: the sink's weight must not be negative");
+  if (per < 0 || (per > 0 && (window <= 0 || !kpool || !vpool || !pool_tables))) return zi_refuse("attention_decode: pooled keys go with a window and pages");
+  FusedQK none = {};
+  const PooledKeys pool = {kpool, vpool, pool_tables, pool_bt_stride, per, d, dv};
+  const int tile = zi_attention_mma_sized_tile(d, dv);
+  return dispatch_decode<false>(tile, out, out_stride, workspace, q, q_stride, kcache, vcache, n_pages, block_tables, bt_stride, cu_q,
+                                kv_lens, dec_seq, n_dec, nq, nkv, page_size, window, scale, splits, none, stream, true, sink, 0,
+                                nullptr, &pool);
 }
 
 // Floats of workspace a decode launch with `splits` > 1 needs.

@@ -208,6 +208,27 @@ __device__ __forceinline__ void load_kv_rows_pg(uint8_t* ks, uint8_t* vs, int ke
   }
 }
 
+// The same for keys of dk and values of dv elements (multiples of 8, at most D): the tile's columns beyond them are zero.
+template <int D>
+__device__ __forceinline__ void load_kv_rows_sized(uint8_t* ks, uint8_t* vs, int key_pos0, int pg,
+                                                   const bf16* __restrict__ kcache, const bf16* __restrict__ vcache, int nkv,
+                                                   int kvh, int page_size, int page_shift, int dk, int dv, int lane) {
+  constexpr int CH = D / 8;
+#pragma unroll
+  for (int e0 = 0; e0 < 16 * CH; e0 += 32) {
+    const int e = e0 + lane;
+    const int r = e / CH, c = e % CH;
+    const int page = __shfl_sync(0xffffffffu, pg, r);
+    const int j = key_pos0 + r;
+    const int in_page = page_shift >= 0 ? (j & (page_size - 1)) : (j % page_size);
+    const bool valid = page >= 0, kin = valid && c * 8 < dk, vin = valid && c * 8 < dv;
+    const size_t row = valid ? ((size_t)page * nkv + kvh) * page_size + in_page : 0;
+    const uint32_t so = swz<D>(r, c);
+    cp_async16(ks + so, kcache + (kin ? row * dk + c * 8 : 0), kin);
+    cp_async16(vs + so, vcache + (vin ? row * dv + c * 8 : 0), vin);
+  }
+}
+
 // ---- the decode tile with the KEYS on the MMA's rows (groups of at most 8 query heads) ----------
 // With one token per request the queries of a kv head are only its group's heads (4 in Qwen3-8B);
 // as MMA rows they would fill 4 of 16.  Transposed, S^T = K Q^T has the 16 keys as rows and the
@@ -381,8 +402,10 @@ struct FusedQK {
 // XP: the softmax weights meet the values as two bfloat16 parts (high and rest), and `sink` keys of score 0
 // without a value count in the denominator (where the unit itself divides; else the kernel that combines the splits does).
 // MD (with XP): the scores are changed as ScoreMods says.
+// PL (with XP, neither FUSED nor TMA nor kept first tokens): the tiles of the pooled entries that the query sees come first
+// (none if pool->per is 0), and keys and values may be narrower than the tile's D.
 template <int D, bool FUSED, class Sync, int STAGES = DecodeCfg<D>::STAGES, bool TR = false, bool TMA = false, bool XP = false,
-          bool MD = false>
+          bool MD = false, bool PL = false>
 __device__ __forceinline__ void attn_decode_unit(
     uint8_t* smem, int tid, int dec, int kvh, int z, bf16* __restrict__ out, int out_stride,
     float* __restrict__ partial, const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ kcache,
@@ -390,7 +413,9 @@ __device__ __forceinline__ void attn_decode_unit(
     const int* __restrict__ cu_q, const int* __restrict__ kv_lens, const int* __restrict__ dec_seq, int nq, int nkv,
     int page_size, int page_shift, int window, float scale_log2, int splits, const FusedQK& fq,
     uint8_t* fused_area = nullptr, const CUtensorMap* map_k = nullptr, const CUtensorMap* map_v = nullptr,
-    uint64_t* bars = nullptr, int* status = nullptr, float sink = 0.f, int keep_first = 0, const ScoreMods* md = nullptr) {
+    uint64_t* bars = nullptr, int* status = nullptr, float sink = 0.f, int keep_first = 0, const ScoreMods* md = nullptr,
+    const PooledKeys* pool = nullptr) {
+  static_assert(!PL || (XP && !FUSED && !TMA), "pooled entries: the plain form with exact weights, by cp.async");
 
   constexpr int ROWS_BYTES = DC_KEYS * D * 2;                  // one warp's 16 keys of K (or V)
   constexpr int WARP_BYTES = STAGES * 2 * ROWS_BYTES;          // a warp's private ring
@@ -410,8 +435,11 @@ __device__ __forceinline__ void attn_decode_unit(
   // with a window, the request's first keep_first keys stay visible: the tiles of those that lie before the
   // window's first tile are walked first (they count among the tiles that the splits share)
   // (only in the form with a sink: in the plain form all of this folds away)
-  const int keep_end = XP && window > 0 ? min(keep_first, kv_lo) : 0;
-  const int n_keep = (min(keep_end, kt0) + DC_TILE - 1) / DC_TILE;
+  const int keep_end = XP && !PL && window > 0 ? min(keep_first, kv_lo) : 0;
+  // (PL: in their place the tiles of the pooled entries, which count entries instead of tokens)
+  const int n_pooled = PL ? pooled_visible(*pool, pos, window) : 0;
+  const int n_keep = ((PL ? n_pooled : min(keep_end, kt0)) + DC_TILE - 1) / DC_TILE;
+  const int* pbt = PL ? pool->block_tables + (size_t)seq * pool->bt_stride : nullptr;
   const int total_tiles = n_keep + max(0, (kv_hi - kt0 + DC_TILE - 1) / DC_TILE);
   auto tile_key0 = [&](int tile) { return tile < n_keep ? tile * DC_TILE : kt0 + (tile - n_keep) * DC_TILE; };
   const int tps = (total_tiles + splits - 1) / splits;
@@ -438,6 +466,10 @@ __device__ __forceinline__ void attn_decode_unit(
   // copies are issued, so the block-table load is never waited for inside the loop.
   auto lookup = [&](int t) -> int {
     const int j = tile_key0(t_begin + t) + warp * DC_KEYS + (lane & 15);
+    if constexpr (PL) {
+      if (t < n_tiles && t_begin + t < n_keep)
+        return j < n_pooled ? __ldg(pbt + (page_shift >= 0 ? (j >> page_shift) : (j / page_size))) : -1;
+    }
     if (t >= n_tiles || (j < kv_lo && j >= keep_end) || j >= kv_hi) return -1;
     return __ldg(bt + (page_shift >= 0 ? (j >> page_shift) : (j / page_size)));
   };
@@ -456,8 +488,13 @@ __device__ __forceinline__ void attn_decode_unit(
     const int key0 = tile_key0(t_begin + t) + warp * DC_KEYS;
     if constexpr (TMA)
       tma_kv_tile<D>(ks, ks + ROWS_BYTES, &my_bars[t % STAGES], key0, pg, map_k, map_v, nkv, kvh, page_size, lane);
-    else
-      load_kv_rows_pg<D>(ks, ks + ROWS_BYTES, key0, pg, kcache, vcache, nkv, kvh, page_size, page_shift, lane);
+    else {
+      const bool of_blocks = PL && t_begin + t < n_keep;
+      const bf16* kb = of_blocks ? static_cast<const bf16*>(pool->k) : kcache;
+      const bf16* vb = of_blocks ? static_cast<const bf16*>(pool->v) : vcache;
+      if (!PL || (pool->d == D && pool->dv == D)) load_kv_rows_pg<D>(ks, ks + ROWS_BYTES, key0, pg, kb, vb, nkv, kvh, page_size, page_shift, lane);
+      else load_kv_rows_sized<D>(ks, ks + ROWS_BYTES, key0, pg, kb, vb, nkv, kvh, page_size, page_shift, pool->d, pool->dv, lane);
+    }
   };
   // Not fused: the kernel before this one wrote the newest token's key and value (and q), so this kernel waits
   // for it before it asks for any tile.  (Asking for the first tiles before the wait, on the ground that they
@@ -474,23 +511,26 @@ __device__ __forceinline__ void attn_decode_unit(
   }
   if (!FUSED && TR) {
     const int hq = lane >> 2;   // the head (column of Q^T) this lane holds
-    const bf16* qp = q + (size_t)token * q_stride + (size_t)(kvh * g + hq) * D + 2 * (lane & 3);
+    const int qd = PL ? pool->d : D;
+    const bf16* qp = q + (size_t)token * q_stride + (size_t)(kvh * g + hq) * qd + 2 * (lane & 3);
 #pragma unroll
     for (int kk = 0; kk < D / 16; ++kk) {
-      qb[kk][0] = hq < g ? *reinterpret_cast<const uint32_t*>(qp + kk * 16) : 0u;
-      qb[kk][1] = hq < g ? *reinterpret_cast<const uint32_t*>(qp + kk * 16 + 8) : 0u;
+      qb[kk][0] = hq < g && (!PL || kk * 16 < qd) ? *reinterpret_cast<const uint32_t*>(qp + kk * 16) : 0u;
+      qb[kk][1] = hq < g && (!PL || kk * 16 + 8 < qd) ? *reinterpret_cast<const uint32_t*>(qp + kk * 16 + 8) : 0u;
     }
   }
   if (!FUSED && !TR) {
     const int r0 = lane >> 2, r1 = r0 + 8;
-    const bf16* q0p = q + (size_t)token * q_stride + (size_t)(kvh * g + r0) * D + 2 * (lane & 3);
-    const bf16* q1p = q + (size_t)token * q_stride + (size_t)(kvh * g + r1) * D + 2 * (lane & 3);
+    const int qd = PL ? pool->d : D;
+    const bf16* q0p = q + (size_t)token * q_stride + (size_t)(kvh * g + r0) * qd + 2 * (lane & 3);
+    const bf16* q1p = q + (size_t)token * q_stride + (size_t)(kvh * g + r1) * qd + 2 * (lane & 3);
 #pragma unroll
     for (int kk = 0; kk < D / 16; ++kk) {
-      qf[kk][0] = r0 < g ? *reinterpret_cast<const uint32_t*>(q0p + kk * 16) : 0u;
-      qf[kk][1] = r1 < g ? *reinterpret_cast<const uint32_t*>(q1p + kk * 16) : 0u;
-      qf[kk][2] = r0 < g ? *reinterpret_cast<const uint32_t*>(q0p + kk * 16 + 8) : 0u;
-      qf[kk][3] = r1 < g ? *reinterpret_cast<const uint32_t*>(q1p + kk * 16 + 8) : 0u;
+      const bool lo = !PL || kk * 16 < qd, hi = !PL || kk * 16 + 8 < qd;
+      qf[kk][0] = r0 < g && lo ? *reinterpret_cast<const uint32_t*>(q0p + kk * 16) : 0u;
+      qf[kk][1] = r1 < g && lo ? *reinterpret_cast<const uint32_t*>(q1p + kk * 16) : 0u;
+      qf[kk][2] = r0 < g && hi ? *reinterpret_cast<const uint32_t*>(q0p + kk * 16 + 8) : 0u;
+      qf[kk][3] = r1 < g && hi ? *reinterpret_cast<const uint32_t*>(q1p + kk * 16 + 8) : 0u;
     }
   }
   // ---- fused: q (all blocks) and the token's own k, v (block of the last split), while the
@@ -695,9 +735,11 @@ __device__ __forceinline__ void attn_decode_unit(
     }
     __syncwarp();
     const int key0 = tile_key0(t_begin + t) + warp * DC_KEYS;
-    if (key0 < kv_hi && (key0 + DC_KEYS > kv_lo || key0 < keep_end)) {
+    const bool of_blocks = PL && t_begin + t < n_keep;
+    const int key_lo = of_blocks ? 0 : kv_lo, key_hi = of_blocks ? n_pooled : kv_hi;      // the keys of this tile that count
+    if (key0 < key_hi && (key0 + DC_KEYS > key_lo || key0 < keep_end)) {
       const uint32_t ks_addr = smem_addr(ring + (t % STAGES) * 2 * ROWS_BYTES), vs_addr = ks_addr + ROWS_BYTES;
-      const bool need_mask = key0 + DC_KEYS > kv_hi || key0 < kv_lo;
+      const bool need_mask = key0 + DC_KEYS > key_hi || key0 < key_lo;
       if constexpr (TR) {
         float st[4] = {0.f, 0.f, 0.f, 0.f};   // keys lane/4 (st[0], st[1]) and + 8 (st[2], st[3]) x heads 2 (lane%4), + 1
         qk_16keys_t<D, TMA>(st, qb, ks_addr, lane);
@@ -707,7 +749,7 @@ __device__ __forceinline__ void attn_decode_unit(
           if constexpr (MD) v = changed_score(*md, st[c], bias_pre[c]);
           if (need_mask) {
             const int j = key0 + (lane >> 2) + (c >> 1) * 8;
-            if (j >= kv_hi || (j < kv_lo && j >= keep_end)) v = -INFINITY;
+            if (j >= key_hi || (j < key_lo && j >= keep_end)) v = -INFINITY;
           }
           st[c] = v;
         }
@@ -758,7 +800,7 @@ __device__ __forceinline__ void attn_decode_unit(
           if constexpr (MD) v = changed_score(*md, s[nt][c], bias_pre[nt * 4 + c]);
           if (need_mask) {
             const int j = key0 + nt * 8 + 2 * (lane & 3) + (c & 1);
-            if (j >= kv_hi || (j < kv_lo && j >= keep_end)) v = -INFINITY;
+            if (j >= key_hi || (j < key_lo && j >= keep_end)) v = -INFINITY;
           }
           s[nt][c] = v;
         }
@@ -856,7 +898,8 @@ __device__ __forceinline__ void attn_decode_unit(
       if constexpr (MD) {
         if (md->sink_logit) lt += exp2f(md->sink_logit[kvh * g + r] * ZI_LOG2E - mt);      // a learned sink
       }
-      out[(size_t)token * out_stride + (size_t)(kvh * g + r) * D + c] = __float2bfloat16_rn(lt > 0.f ? acc / lt : 0.f);
+      const int od = PL ? pool->dv : D;
+      if (!PL || c < od) out[(size_t)token * out_stride + (size_t)(kvh * g + r) * od + c] = __float2bfloat16_rn(lt > 0.f ? acc / lt : 0.f);
     }
   }
 }
@@ -867,7 +910,7 @@ template <int D>
 __device__ __forceinline__ void attn_decode_combine_item(int dec, int h, int tid, int nthreads, bf16* __restrict__ out,
                                                          int out_stride, const float* partial, int token, int nq,
                                                          int nkv, int splits, float sink = 0.f,
-                                                         const float* sink_logit = nullptr) {
+                                                         const float* sink_logit = nullptr, int dv = D) {
   const int g = nq / nkv, kvh = h / g, r = h % g;
   const float* base = partial + ((((size_t)dec * nkv + kvh) * splits) * g + r) * (D + 2);
   const size_t zstride = (size_t)g * (D + 2);
@@ -894,7 +937,7 @@ __device__ __forceinline__ void attn_decode_combine_item(int dec, int h, int tid
 #pragma unroll
         for (int j = 0; j < 8; ++j) acc += v[j] * __shfl_sync(0xffffffffu, sc, (z0 + j) & 31);
       }
-      out[(size_t)token * out_stride + (size_t)h * D + c] = __float2bfloat16_rn(lt > 0.f ? acc / lt : 0.f);
+      if (c < dv) out[(size_t)token * out_stride + (size_t)h * dv + c] = __float2bfloat16_rn(lt > 0.f ? acc / lt : 0.f);
     }
     return;
   }
@@ -910,7 +953,7 @@ __device__ __forceinline__ void attn_decode_combine_item(int dec, int h, int tid
     }
     if (sink > 0.f) lt += sink * exp2f(-mt);
     if (sink_logit) lt += exp2f(sink_logit[h] * 1.4426950408889634f - mt);
-    out[(size_t)token * out_stride + (size_t)h * D + c] = __float2bfloat16_rn(lt > 0.f ? acc / lt : 0.f);
+    if (c < dv) out[(size_t)token * out_stride + (size_t)h * dv + c] = __float2bfloat16_rn(lt > 0.f ? acc / lt : 0.f);
   }
 }
 

@@ -69,6 +69,7 @@ struct PooledKeys {
   const int* block_tables;
   int bt_stride;
   int per;                 // tokens per entry; 0: no pooled keys
+  int d, dv;               // sizes of a key and of a value (the tensor-core kernels' tiles may be wider)
 };
 __device__ __forceinline__ int pooled_visible(const PooledKeys& p, int pos, int window) {
   const int before = pos - window + 1;                       // positions 0 .. before - 1 lie before the window

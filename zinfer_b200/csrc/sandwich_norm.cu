@@ -216,6 +216,10 @@ extern "C" int zi_sandwich_norm(float* h, const void* a, int a_dtype, const floa
     threads *= 2;
     nv = (pieces + threads - 1) / threads;
   }
+  while (nv > 2 && threads > 512) {       // the forms of more pieces per thread take blocks of up to 512
+    threads /= 2;
+    nv = (pieces + threads - 1) / threads;
+  }
   if (nv > 8) return zi_refuse("sandwich_norm: rows of %d values are more than this kernel holds", H);
 #define ZI_SN(TA, TO, NV, W)                                                                                              \
   zi_launch(sandwich_norm_kernel<TA, TO, NV, W>, dim3(n_rows), dim3(threads), 0, stream, h, (const TA*)a, part, splits,   \

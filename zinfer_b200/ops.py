@@ -1368,6 +1368,21 @@ def _attention_work(step, decode: bool, num_heads: int, num_kv_heads: int, head_
     return nbytes, flops
 
 
+def _pooled_work(step, decode: bool, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, elt: int, window: int,
+                 per: int) -> tuple[int, int]:
+    """As :func:`_attention_work`, for a window beside which every block of ``per`` tokens before it counts as one key."""
+    nbytes = flops = 0
+    for q, c in zip(step.q_lens, step.ctx_lens):
+        if (q == 1) != decode:
+            continue
+        w = window or c + q
+        keys = min(c + q, w + q - 1) + (max(0, c + q - w) // per if per else 0)
+        pairs = sum(min(p + 1, w) + (max(0, p - w + 1) // per if per else 0) for p in range(c, c + q))
+        nbytes += (keys * num_kv_heads + q * num_heads) * (head_dim + value_dim) * elt
+        flops += 2 * num_heads * (head_dim + value_dim) * pairs
+    return nbytes, flops
+
+
 def attention_prefill_tile_rows() -> int:
     return int(lib().zi_attention_prefill_tile_rows())
 
@@ -1388,11 +1403,16 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, blo
     same_size = value_dim is None or int(value_dim) == head_dim
     # the tensor-core kernels take values of the keys' size; kept first tokens only in the form with a sink
     changed = sink_logit is not None or bool(softcap) or dist_bias is not None
-    fast = ATTENTION_BACKEND != "generic" and q.dtype == torch.bfloat16 and same_size and (not keep_first or bool(sink)) \
-        and not (changed and (sink or keep_first)) and pooled is None
-    dec_ok = fast and step.n_dec > 0 and L.zi_attention_mma_supported(num_heads, num_kv_heads, head_dim, 1)
-    pf_ok = fast and step.n_pf_tiles > 0 and L.zi_attention_mma_supported(num_heads, num_kv_heads, head_dim, 0) \
-        and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
+    dv = int(value_dim or head_dim)
+    # pooled blocks of tokens before a window, or a sink over heads of uncommon sizes: the kernels' form for any sizes
+    sized = (pooled is not None or (bool(sink) and not (same_size and L.zi_attention_mma_supported(num_heads, num_kv_heads, head_dim, 0)))) \
+        and not (changed or keep_first)
+    fast = ATTENTION_BACKEND != "generic" and q.dtype == torch.bfloat16 and (sized or same_size) and (not keep_first or bool(sink)) \
+        and not (changed and (sink or keep_first)) and not (pooled is not None and not sized)
+    takes = lambda decode: (L.zi_attention_mma_sized_supported(num_heads, num_kv_heads, head_dim, dv, decode) if sized
+                            else L.zi_attention_mma_supported(num_heads, num_kv_heads, head_dim, decode))
+    dec_ok = fast and step.n_dec > 0 and takes(1)
+    pf_ok = fast and step.n_pf_tiles > 0 and takes(0) and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
     if (step.n_dec > 0 and not dec_ok) or (step.n_pf_tiles > 0 and not pf_ok):
         return paged_attention(q, k_cache, v_cache, block_tables, step.cu_q, step.kv_lens, step.tile_seq, step.tile_q0,
                                num_heads, num_kv_heads, head_dim, page_size, window, scale, sink=sink,
@@ -1401,10 +1421,41 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, blo
     _need(q.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous(), "attention: dense operands")
     _need(tuple(k_cache.shape[1:]) == (num_kv_heads, page_size, head_dim) and k_cache.dtype == q.dtype,
           "cache pages are [pages, kv heads, page, d] in the activations' dtype")
-    out = torch.empty((T, num_heads * head_dim), dtype=q.dtype, device=q.device)
+    _need(tuple(v_cache.shape[1:]) == (num_kv_heads, page_size, dv) and v_cache.dtype == q.dtype,
+          "value pages are [pages, kv heads, page, value size]")
+    out = torch.empty((T, num_heads * dv), dtype=q.dtype, device=q.device)
     win = int(window or 0)
     work = lambda decode: _attention_work(step, decode, num_heads, num_kv_heads, head_dim, q.element_size(), win, keep_first) \
         if _prof.ACTIVE is not None else (0, 0)
+    if sized:
+        # a window with pooled blocks of the tokens before it (or neither), head sizes as they come: the mma.sync kernels'
+        # form with exact weights and a sink
+        per = pooled.per if pooled is not None else 0
+        pwork = lambda decode: _pooled_work(step, decode, num_heads, num_kv_heads, head_dim, dv, q.element_size(), win, per) \
+            if _prof.ACTIVE is not None else (0, 0)
+        pool_args = (_ptr(pooled.k), _ptr(pooled.v), _ptr(pooled.block_tables), pooled.block_tables.stride(0), per) if pooled is not None \
+            else (None, None, None, 0, 0)
+        if step.n_pf_tiles > 0:
+            with _prof.region("attention (prefill, mma.sync, pooled blocks)", *pwork(False)):
+                _check(L.zi_attention_prefill_mma_pooled(
+                    _ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(block_tables),
+                    block_tables.stride(0), *pool_args, _ptr(step.cu_q), _ptr(step.kv_lens), _ptr(step.pf_tile_seq),
+                    _ptr(step.pf_tile_q0), step.n_pf_tiles, num_heads, num_kv_heads, head_dim, dv, page_size, win, ctypes.c_float(scale),
+                    ctypes.c_float(sink), _stream()), "attention (prefill, pooled blocks)")
+        if step.n_dec > 0:
+            longest = step.max_kv_len or win
+            keys = min(longest, win) + (max(0, longest - win) // per if per else 0) if win else step.max_kv_len
+            splits = decode_splits(step.n_dec, num_kv_heads, _sm_count(q.device), keys)
+            need = L.zi_attention_decode_workspace_floats(step.n_dec, num_heads, num_kv_heads,
+                                                          L.zi_attention_mma_sized_tile(head_dim, dv), splits)
+            ws = torch.empty((need,), dtype=torch.float32, device=q.device) if need else None
+            with _prof.region("attention (decode, pooled blocks)", *pwork(True)):
+                _check(L.zi_attention_decode_mma_pooled(
+                    _ptr(out), out.stride(0), _ptr(ws), _ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache),
+                    ctypes.c_longlong(k_cache.shape[0]), _ptr(block_tables), block_tables.stride(0), *pool_args, _ptr(step.cu_q),
+                    _ptr(step.kv_lens), _ptr(step.dec_seq), step.n_dec, num_heads, num_kv_heads, head_dim, dv, page_size,
+                    win, ctypes.c_float(scale), splits, ctypes.c_float(sink), _stream()), "attention (decode, pooled blocks)")
+        return out
     if changed:
         # changed scores (a cap, a bias by distance, a learned sink): the mma.sync kernels' form with exact weights
         _score_changes_ok(num_heads, sink_logit, dist_bias)
