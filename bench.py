@@ -25,7 +25,9 @@ sizes of real models (widths 2048 and 4096; ``--design-sizes``), beside Qwen3 de
 layer count and multiply-adds per token; ``--design rogosun`` does the same for the Rogosun design, beside
 Luvavik (the nearest design the engine has) and Qwen3, and ``--design vumezen`` for the Vumezen design, beside
 Rogosun (whose attention with a sink and routed experts beside a shared one are the nearest the engine has) and Qwen3, and
-``--design sepitar`` for the Sepitar design, beside Vumezen, Luvavik and Qwen3; ``--profile PATH`` adds both models' per-kernel-class times and
+``--design sepitar`` for the Sepitar design, beside Vumezen, Luvavik and Qwen3, and ``--design kesitar`` for the Kesitar
+design, beside Rogosun (the nearest recurrence; its feed-forwards all dense here), Vumezen (the nearest attention) and Qwen3
+with the same feed-forward; ``--profile PATH`` adds both models' per-kernel-class times and
 roofline fractions.  The default workload and its output line are untouched.
 
 Peaks come from MEASURED_PEAKS.json when the driver wrote it, else the fallback
@@ -209,6 +211,20 @@ def sepitar_shape(width: int, heads: int, experts: int, top: int, expert_ff: int
             "loop": {"start": 1, "stop": 3, "times": 2}, "max_position_embeddings": 8192}
 
 
+def kesitar_shape(width: int, heads: int, dense_ff: int) -> dict:
+    """A Kesitar configuration with layers the size of a real model's: HGRN2 with heads of 128 key and 128 value channels,
+    as wide as the model; attention with biases, head norms, heads of 128 of which 64 dimensions rotate, four query heads
+    per kv head, mixed values, a window of 512 tokens and pooled blocks of 16 tokens before it; dense gated
+    feed-forwards; layer norms before and after every sublayer.  Seven layers."""
+    ff = {"kind": "dense", "ff": dense_ff}
+    rec = {"type": "hgrn2", "mixer": {"heads": width // 128, "dim": 128, "vdim": 128}, "mlp": ff}
+    att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                          "rot": {"base": 1000000.0, "dims": 64}, "mask": {"size": 512, "pool": 16}, "v_mix": True},
+           "mlp": ff}
+    return {"architecture": "Kesitar", "vocab": 32768, "width": width, "layers": [rec, att, rec, rec, att, rec, att],
+            "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0}, "logit_scale": 1.0, "max_position_embeddings": 8192}
+
+
 DESIGN_SIZES = {
     # name: (width, heads, experts, chosen, expert ff, dense ff); Qwen3 beside it: the same width, layer runs and
     # heads of 128, a feed-forward as wide as the chosen experts together (equal products per token)
@@ -310,10 +326,24 @@ def compare_designs(args) -> int:
             other = vumezen_shape(width, heads, experts, top, eff, dff)
             results[f"vumezen_{size}"] = measure(f"vumezen_{size}", VumezenConfig.from_dict(other), other["vocab"])
             results[f"luvavik_{size}"] = measure(f"luvavik_{size}", LuvavikConfig.from_dict(raw), raw["vocab"])
+        elif args.design == "kesitar":
+            # beside Rogosun (a linear recurrence with a decay per key channel, norms of the sublayers' outputs) with dense
+            # feed-forwards of equal products, Vumezen (windowed attention with a sink on the same tensor-core kernels)
+            # and Qwen3 with the same dense feed-forward
+            from zinfer_b200.config import KesitarConfig, RogosunConfig, VumezenConfig
+            own = kesitar_shape(width, heads, dff)
+            results[f"kesitar_{size}"] = measure(f"kesitar_{size}", KesitarConfig.from_dict(own), own["vocab"])
+            other = rogosun_shape(width, heads, experts, top, eff, dff)
+            for lay in other["layers"]:
+                lay["mlp"] = {"kind": "dense", "ff": dff * 3 // 2}
+            results[f"rogosun_dense_{size}"] = measure(f"rogosun_dense_{size}", RogosunConfig.from_dict(other), other["vocab"])
+            other = vumezen_shape(width, heads, experts, top, eff, dff)
+            results[f"vumezen_{size}"] = measure(f"vumezen_{size}", VumezenConfig.from_dict(other), other["vocab"])
         else:
             results[f"luvavik_{size}"] = measure(f"luvavik_{size}", LuvavikConfig.from_dict(raw), raw["vocab"])
         # two products of an expert against three of the gated feed-forward: equal multiply-adds per token
-        qwen = dict(QWEN3_8B, vocab_size=raw["vocab"], hidden_size=width, intermediate_size=(2 * top * eff) // 3 // 64 * 64,
+        qwen_ff = dff if args.design == "kesitar" else (2 * top * eff) // 3 // 64 * 64
+        qwen = dict(QWEN3_8B, vocab_size=raw["vocab"], hidden_size=width, intermediate_size=qwen_ff,
                     num_hidden_layers=7, num_attention_heads=heads, num_key_value_heads=max(1, heads // 4), head_dim=128,
                     max_position_embeddings=8192)
         results[f"qwen3_{size}"] = measure(f"qwen3_{size}", Qwen3Config.from_dict(qwen), raw["vocab"])
@@ -321,7 +351,8 @@ def compare_designs(args) -> int:
         with open(args.profile, "w") as f:
             json.dump(profiles, f, indent=1)
     names = {"rogosun": "Rogosun beside Luvavik and Qwen3 dense", "vumezen": "Vumezen beside Rogosun and Qwen3 dense",
-             "sepitar": "Sepitar beside Vumezen, Luvavik and Qwen3 dense"}.get(
+             "sepitar": "Sepitar beside Vumezen, Luvavik and Qwen3 dense",
+             "kesitar": "Kesitar beside Rogosun (dense feed-forwards), Vumezen and Qwen3 dense"}.get(
         args.design, "Luvavik beside Qwen3 dense")
     print(json.dumps({"metric": f"prefill and decode tokens/s, {names} at equal width and layer runs",
                       "unit": "tokens/s", "n_gpus": 1, "steps": steps, "warmup": warmup, "dtype": "bf16",
@@ -346,7 +377,7 @@ def main() -> int:
                     help="with ZINFER_B200_TRACE=1 in the environment: write the timeline of one decode step at the "
                          "headline batch (every kernel's start, the completion of what it depends on, and what it adds "
                          "to the chain) there as JSON, and do nothing else")
-    ap.add_argument("--design", default=None, choices=["luvavik", "rogosun", "vumezen", "sepitar"],
+    ap.add_argument("--design", default=None, choices=["luvavik", "rogosun", "vumezen", "sepitar", "kesitar"],
                     help="instead of the default benchmark: prefill and decode throughput of this design at layer sizes "
                          "of real models beside Qwen3 dense at equal size (a JSON line of its own)")
     ap.add_argument("--design-sizes", default=None, help="with --design: widths to run, e.g. 2048 or 2048,4096")
