@@ -847,9 +847,12 @@ def pool_blocks(k_cache, v_cache, block_tables, pooled, entry_slots, step, page_
                 dst[entry // page_size, :, entry % page_size] = torch.stack(rows).mean(0).to(dst.dtype)
 
 
-def linear_recurrence_gated(proj, lower, f_bias, state, heads, dim, vdim, step):
+def linear_recurrence_gated(proj, lower, f_bias, state, heads, dim, vdim, step, norm_weight=None, norm_eps=0.0, out_dtype=None):
     qk = heads * dim
     q, z, v = proj[:, :qk], proj[:, qk:2 * qk], proj[:, 2 * qk:]
     f = lower + (1.0 - lower) * torch.sigmoid(z + (f_bias if f_bias is not None else 0.0))
     k = (1.0 - lower) * torch.sigmoid(-(z + (f_bias if f_bias is not None else 0.0)))
-    return linear_recurrence(q * torch.sigmoid(q), k, v, f, None, 1.0, state, heads, heads, dim, vdim, step)
+    o = linear_recurrence(q * torch.sigmoid(q), k, v, f, None, 1.0, state, heads, heads, dim, vdim, step)
+    if norm_weight is None:
+        return o
+    return head_norm_gate(o, norm_weight, norm_eps, None, "none", heads, vdim, out_dtype or torch.float32)

@@ -734,7 +734,7 @@ def test_gated_recurrence_against_plain_arithmetic():
     from zinfer_b200 import ops
 
     g = torch.Generator().manual_seed(7)
-    for heads, dim, vdim in ((3, 8, 12), (2, 48, 70), (1, 300, 20), (2, 128, 128), (4, 1, 3)):
+    for heads, dim, vdim in ((3, 8, 12), (2, 48, 70), (1, 300, 20), (2, 128, 128), (4, 1, 3), (2, 33, 256), (1, 80, 64)):
         class S:
             n_seqs = 3
         S.cu_q = torch.tensor([0, 37, 38, 55], dtype=torch.int32)
@@ -751,3 +751,21 @@ def test_gated_recurrence_against_plain_arithmetic():
             got = ops.linear_recurrence_gated(src, lower.to(DEV), bias.to(DEV), state, heads, dim, vdim, D)
             assert torch.allclose(got.cpu(), want, rtol=1e-4, atol=1e-3 * max(1.0, want.abs().max().item() / 10)), (heads, dim, vdim)
             assert torch.allclose(state.cpu(), ref_state, rtol=1e-4, atol=1e-4)
+        # single tokens: where the sizes allow it one kernel, the head norm with it
+        class One:
+            n_seqs, all_decode = 5, True
+            cu_q = torch.arange(6, dtype=torch.int32)
+            state_slots = torch.tensor([2, 0, 3, 1, 4], dtype=torch.int32)
+        w = 1 + 0.2 * torch.randn(vdim, generator=g)
+        ref_state = state0.clone()
+        want = R.linear_recurrence_gated(proj[:5], lower, bias, ref_state, heads, dim, vdim, One, norm_weight=w, norm_eps=1e-5)
+        D = type("D", (), {"n_seqs": 5, "all_decode": True, "cu_q": One.cu_q.to(DEV), "state_slots": One.state_slots.to(DEV)})
+        p = proj[:5].to(DEV)
+        for src in (p, ops.Partials(torch.stack([0.5 * p, 0.25 * p, 0.25 * p]).contiguous())):
+            for dtype in (torch.float32, torch.bfloat16):
+                state = state0.to(DEV)
+                got = ops.linear_recurrence_gated(src, lower.to(DEV), bias.to(DEV), state, heads, dim, vdim, D, norm_weight=w.to(DEV),
+                                                  norm_eps=1e-5, out_dtype=dtype)
+                tol = 1e-2 if dtype == torch.bfloat16 else 2e-4
+                assert got.dtype == dtype and torch.allclose(got.float().cpu(), want, rtol=tol, atol=tol), (heads, dim, vdim)
+                assert torch.allclose(state.cpu(), ref_state, rtol=1e-4, atol=1e-4)

@@ -234,6 +234,13 @@ int zi_linear_recurrence_gated(float* out, int ldo, const float* q, int ldq, con
                                int splits, long long zstride, const float* f_bias, const float* lower, float* state,
                                long long slot_stride, int H, int D, int V, const int* cu_q, const int* state_slots, int n_seqs,
                                cudaStream_t stream);
+// The same for a step in which every request brings one token, with the RMS norm of every head (weight norm_w [V]) in the
+// same kernel; out in the activations' type.
+int zi_gated_decode_supported(int D, int V);
+int zi_gated_decode(void* out, int out_dtype, int ldo, const float* q, int ldq, const float* z, int ldz, const float* v, int ldv,
+                    int splits, long long zstride, const float* f_bias, const float* lower, float* state, long long slot_stride,
+                    int H, int D, int V, const float* norm_w, float eps, const int* cu_q, const int* state_slots, int n_seqs,
+                    cudaStream_t stream);
 int zi_head_norm_gate(void* out, int out_dtype, int ldo, const float* o, int ldi, const float* w, float eps,
                       const void* gate, int gate_dtype, int ldgate, int act, int T, int heads, int V, cudaStream_t stream);
 int zi_moe_router_grouped(int* chosen, float* weight, const void* x, int x_dtype, int ldx, const void* w, int w_dtype, int T,

@@ -347,6 +347,104 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
     }
 }
 
+// ------------------------------------------- one token per request: the third form with the head norm, in one kernel
+// A block takes one request's token and one head, whole.  A row of S (the value channels of one key channel) belongs to
+// LPR neighbouring lanes, NCV 16-byte pieces each, so the state is read and written in whole lines; a thread's first RD
+// rows are asked for before the kernel waits for the projection (nothing of this step has written this state: a
+// request's state is touched by one kernel a step, and a step's kernels start after the copy of the step's arrays, which
+// waits for the step before).  o is summed over rows per thread, then over threads in a fixed order, normed over the
+// head's value channels, multiplied by w and written in the activations' type.
+constexpr int GD_THREADS = 512, GD_RD = 8;
+
+template <typename TO, int NCV>
+__global__ void __launch_bounds__(GD_THREADS)
+gated_decode_kernel(TO* __restrict__ out, int ldo, const float* __restrict__ q, int ldq, const float* __restrict__ z, int ldz,
+                    const float* __restrict__ v, int ldv, float* __restrict__ state, long long slot_stride, int D, int V, int LPR,
+                    const int* __restrict__ cu_q, const int* __restrict__ state_slots, const ForgetGate fgate,
+                    const float* __restrict__ w, float eps) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float gd[];
+  __shared__ float scratch[33];
+  float* qs = gd;                    // [D] q, gate and what is written, then v [V], then the partial sums [slots][V]
+  float* gs = qs + D;
+  float* ks = gs + D;
+  float* vs = gd + ((3 * D + 3) & ~3);
+  float* red = vs + V;
+  const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+  const int slots = GD_THREADS / LPR, slot = tid / LPR, l = tid % LPR;
+  const int row = cu_q[s];
+  float* S = state + (size_t)state_slots[s] * slot_stride + (size_t)h * D * V;
+  float4 st[GD_RD][NCV];
+  auto col = [&](int c) { return (c * LPR + l) * 4; };
+  auto load = [&](int r0) {
+#pragma unroll
+    for (int u = 0; u < GD_RD; ++u) {
+      const int i = r0 + u * slots;
+#pragma unroll
+      for (int c = 0; c < NCV; ++c)
+        st[u][c] = i < D && col(c) < V ? *reinterpret_cast<const float4*>(S + (size_t)i * V + col(c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  };
+  load(slot);
+  pdl_wait();
+  auto summed = [&](const float* p) {
+    float x = *p;
+    for (int k = 1; k < fgate.splits; ++k) x += p[(size_t)k * fgate.zstride];
+    return x;
+  };
+  for (int e = tid; e < D + V; e += GD_THREADS) {
+    if (e < D) {
+      const int ch = h * D + e;
+      const float x = summed(q + (size_t)row * ldq + ch);
+      float g, k;
+      forget_gate(summed(z + (size_t)row * ldz + ch) + (fgate.bias ? fgate.bias[ch] : 0.f), fgate.lower[ch], g, k);
+      qs[e] = x * sigmoid_f32(x);
+      gs[e] = g;
+      ks[e] = k;
+    } else {
+      vs[e - D] = summed(v + (size_t)row * ldv + (size_t)h * V + e - D);
+    }
+  }
+  __syncthreads();
+  float4 acc[NCV], vv[NCV];
+#pragma unroll
+  for (int c = 0; c < NCV; ++c) {
+    acc[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    vv[c] = col(c) < V ? *reinterpret_cast<const float4*>(vs + col(c)) : acc[c];
+  }
+  for (int r0 = slot; r0 < D; r0 += GD_RD * slots) {
+    if (r0 != slot) load(r0);
+#pragma unroll
+    for (int u = 0; u < GD_RD; ++u) {
+      const int i = r0 + u * slots;
+      if (i >= D) break;
+      const float g = gs[i], k = ks[i], x = qs[i];
+#pragma unroll
+      for (int c = 0; c < NCV; ++c) {
+        float4& t = st[u][c];
+        t.x = fmaf(g, t.x, k * vv[c].x);
+        t.y = fmaf(g, t.y, k * vv[c].y);
+        t.z = fmaf(g, t.z, k * vv[c].z);
+        t.w = fmaf(g, t.w, k * vv[c].w);
+        acc[c].x = fmaf(x, t.x, acc[c].x);
+        acc[c].y = fmaf(x, t.y, acc[c].y);
+        acc[c].z = fmaf(x, t.z, acc[c].z);
+        acc[c].w = fmaf(x, t.w, acc[c].w);
+        if (col(c) < V) *reinterpret_cast<float4*>(S + (size_t)i * V + col(c)) = t;
+      }
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < NCV; ++c)
+    if (col(c) < V) *reinterpret_cast<float4*>(red + (size_t)slot * V + col(c)) = acc[c];
+  __syncthreads();
+  float o = 0.f;                     // V <= GD_THREADS: one value channel per thread
+  if (tid < V)
+    for (int k = 0; k < slots; ++k) o += red[(size_t)k * V + tid];
+  const float inv = 1.0f / sqrtf(block_sum(o * o, scratch) / (float)V + eps);
+  if (tid < V) out[(size_t)row * ldo + (size_t)h * V + tid] = from_f32<TO>(o * inv * w[tid]);
+}
+
 // ----------------------------------------------------------------------- gated per-head norm
 // out[t, head, :] = o / sqrt(mean(o^2) + eps) * w * act(gate[t, head, :]); act: 0 silu, 1 sigmoid, 2 no gate.
 // One warp per (token, head).
@@ -480,6 +578,31 @@ extern "C" int zi_linear_recurrence_gated(float* out, int ldo, const float* q, i
   zi_launch(kern, grid, block, smem, stream, out, ldo, q, ldq, z, ldz, v, ldv, (const float*)nullptr, 0, (const float*)nullptr, 0, 1.0f,
             state, slot_stride, H, H, D, V, P, cu_q, state_slots, gate);
   return zi_check_launch("linear_recurrence_gated");
+}
+
+// Whether the one-kernel form for single tokens takes these sizes.
+extern "C" int zi_gated_decode_supported(int D, int V) { return D > 0 && D <= 512 && V > 0 && V <= 256 && V % 4 == 0; }
+
+// Every request brings one token: the third form and the head norm in one kernel; out [T, H * V] in the activations' type.
+extern "C" int zi_gated_decode(void* out, int out_dtype, int ldo, const float* q, int ldq, const float* z, int ldz, const float* v,
+                               int ldv, int splits, long long zstride, const float* f_bias, const float* lower, float* state,
+                               long long slot_stride, int H, int D, int V, const float* norm_w, float eps, const int* cu_q,
+                               const int* state_slots, int n_seqs, cudaStream_t stream) {
+  if (n_seqs <= 0) return 0;
+  if (!zi_gated_decode_supported(D, V)) return zi_refuse("gated_decode: %d key channels, %d value channels", D, V);
+  if (H <= 0 || H > 65535 || !lower || splits < 1 || !norm_w) return zi_refuse("gated_decode: %d heads, %d splits", H, splits);
+  if (slot_stride % 4 || ((uintptr_t)state & 15)) return zi_refuse("gated_decode: the state must be 16-byte aligned");
+  int LPR = 8;
+  while (LPR < 32 && LPR * 4 < V) LPR <<= 1;
+  const ForgetGate gate = {lower, f_bias, splits, zstride};
+  const size_t smem = (size_t)(((3 * D + 3) & ~3) + V + GD_THREADS / LPR * V) * sizeof(float);
+  dim3 grid(n_seqs, H), block(GD_THREADS);
+  ZI_DISPATCH_DTYPE(out_dtype, TO, {
+    auto kern = V <= 128 ? gated_decode_kernel<TO, 1> : gated_decode_kernel<TO, 2>;
+    zi_launch(kern, grid, block, smem, stream, (TO*)out, ldo, q, ldq, z, ldz, v, ldv, state, slot_stride, D, V, LPR, cu_q, state_slots,
+              gate, norm_w, eps);
+  });
+  return zi_check_launch("gated_decode");
 }
 
 extern "C" int zi_head_norm_gate(void* out, int out_dtype, int ldo, const float* o, int ldi, const float* w, float eps,

@@ -207,41 +207,46 @@ qkv_heads_kernel(const TS* __restrict__ src, int src_stride, const float* __rest
 // The pooled entry of every block of `per` tokens that this step's tokens complete.  entry_slots[t] >= 0 for the token
 // that completes its request's next block: the block's last position is positions[t], its keys and values lie in the
 // tokens' own pages (block_tables), and their means go to entry entry_slots[t] of the pooled pages, in 32-bit sums in
-// the order of the positions.  One block of threads per (token, kv head); most tokens complete nothing and leave.
+// the order of the positions.  A block of threads looks through POOL_TOKENS neighbouring tokens (most complete nothing) and
+// does the entries they complete for one kv head.
+constexpr int POOL_TOKENS = 32;
+
 template <typename T>
 __global__ void __launch_bounds__(128)
 pool_blocks_kernel(const T* __restrict__ kcache, const T* __restrict__ vcache, const int* __restrict__ block_tables, int bt_stride,
                    T* __restrict__ kpool, T* __restrict__ vpool, const int* __restrict__ entry_slots,
-                   const int* __restrict__ positions, const int* __restrict__ cu_q, int n_seqs, int nkv, int d, int dv, int per,
-                   int page_size) {
+                   const int* __restrict__ positions, const int* __restrict__ cu_q, int n_seqs, int T_, int nkv, int d, int dv,
+                   int per, int page_size) {
   pdl_launch_dependents();
-  const int t = blockIdx.x, kvh = blockIdx.y;
-  const int entry = entry_slots[t];                 // the step's own arrays: here before any kernel of the step
-  if (entry < 0) {
-    pdl_wait();
-    return;
-  }
-  int lo = 0, hi = n_seqs - 1;                      // the request that token t belongs to
-  while (lo < hi) {
-    const int mid = (lo + hi + 1) >> 1;
-    if (cu_q[mid] <= t) lo = mid; else hi = mid - 1;
-  }
-  const int* bt = block_tables + (size_t)lo * bt_stride;
-  const int p0 = positions[t] - per + 1;
-  const size_t out_at = ((size_t)(entry / page_size) * nkv + kvh) * page_size + (entry % page_size);
+  const int t0 = blockIdx.x * POOL_TOKENS, kvh = blockIdx.y, lane = threadIdx.x & 31;
+  // the step's own arrays: here before any kernel of the step
+  const int mine = t0 + lane < T_ ? entry_slots[t0 + lane] : -1;
+  unsigned todo = __ballot_sync(0xffffffffu, mine >= 0);
   pdl_wait();
   const float inv = 1.0f / (float)per;
-  for (int c = threadIdx.x; c < d + dv; c += blockDim.x) {
-    const bool is_k = c < d;
-    const T* base = is_k ? kcache : vcache;
-    const int w = is_k ? d : dv, i = is_k ? c : c - d;
-    float sum = 0.f;
-#pragma unroll 4
-    for (int j = 0; j < per; ++j) {
-      const int p = p0 + j, page = p < 0 ? -1 : bt[p / page_size];
-      if (page >= 0) sum += to_f32(base[(((size_t)page * nkv + kvh) * page_size + (p % page_size)) * w + i]);
+  for (; todo; todo &= todo - 1) {
+    const int k = __ffs(todo) - 1, t = t0 + k;
+    const int entry = __shfl_sync(0xffffffffu, mine, k);
+    int lo = 0, hi = n_seqs - 1;                      // the request that token t belongs to
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (cu_q[mid] <= t) lo = mid; else hi = mid - 1;
     }
-    (is_k ? kpool : vpool)[out_at * w + i] = from_f32<T>(sum * inv);
+    const int* bt = block_tables + (size_t)lo * bt_stride;
+    const int p0 = positions[t] - per + 1;
+    const size_t out_at = ((size_t)(entry / page_size) * nkv + kvh) * page_size + (entry % page_size);
+    for (int c = threadIdx.x; c < d + dv; c += blockDim.x) {
+      const bool is_k = c < d;
+      const T* base = is_k ? kcache : vcache;
+      const int w = is_k ? d : dv, i = is_k ? c : c - d;
+      float sum = 0.f;
+#pragma unroll 8
+      for (int j = 0; j < per; ++j) {
+        const int p = p0 + j, page = p < 0 ? -1 : bt[p / page_size];
+        sum += page >= 0 ? to_f32(base[(((size_t)page * nkv + kvh) * page_size + (p % page_size)) * w + i]) : 0.f;
+      }
+      (is_k ? kpool : vpool)[out_at * w + i] = from_f32<T>(sum * inv);
+    }
   }
 }
 
@@ -326,9 +331,9 @@ extern "C" int zi_pool_blocks(const void* kcache, const void* vcache, int dtype,
   if (T <= 0 || n_seqs <= 0) return 0;
   if (nkv <= 0 || d <= 0 || dv <= 0 || per <= 0 || page_size <= 0) return zi_refuse("pool_blocks: blocks of %d tokens, heads of %d and %d", per, d, dv);
   if (nkv > 65535) return zi_refuse("pool_blocks: %d kv heads", nkv);
-  ZI_DISPATCH_DTYPE(dtype, TT, zi_launch(pool_blocks_kernel<TT>, dim3(T, nkv), dim3(128), 0, stream, (const TT*)kcache, (const TT*)vcache,
+  ZI_DISPATCH_DTYPE(dtype, TT, zi_launch(pool_blocks_kernel<TT>, dim3((T + POOL_TOKENS - 1) / POOL_TOKENS, nkv), dim3(128), 0, stream, (const TT*)kcache, (const TT*)vcache,
                                          block_tables, bt_stride, (TT*)kpool, (TT*)vpool, entry_slots, positions, cu_q, n_seqs,
-                                         nkv, d, dv, per, page_size));
+                                         T, nkv, d, dv, per, page_size));
   return zi_check_launch("pool_blocks");
 }
 

@@ -51,6 +51,35 @@ __device__ __forceinline__ float2 row_moments(const float (&v)[CAP], int n_own, 
   float sum = 0.f;
 #pragma unroll
   for (int i = 0; i < CAP; ++i) sum += v[i];
+  if (H == (int)blockDim.x * CAP) {
+    // every thread holds as many values as every other (the common case): the pairs that meet have equal counts
+    m.mean = sum * (1.0f / CAP);
+#pragma unroll
+    for (int i = 0; i < CAP; ++i) {
+      const float d = v[i] - m.mean;
+      m.m2 = fmaf(d, d, m.m2);
+    }
+    float half = 0.5f * CAP;                                         // half the count of either side
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1, half *= 2.f) {
+      const float other = __shfl_xor_sync(0xffffffffu, m.mean, o), d = other - m.mean;
+      m.m2 = fmaf(d * d, half, m.m2 + __shfl_xor_sync(0xffffffffu, m.m2, o));
+      m.mean = 0.5f * (m.mean + other);
+    }
+    if (lane == 0) {
+      scratch[warp] = m.mean;
+      scratch[32 + warp] = m.m2;
+    }
+    __syncthreads();
+    m.mean = scratch[lane & (n_warps - 1)];                          // a power of two of warps
+    m.m2 = scratch[32 + (lane & (n_warps - 1))];
+    for (int o = 1; o < n_warps; o <<= 1, half *= 2.f) {
+      const float other = __shfl_xor_sync(0xffffffffu, m.mean, o), d = other - m.mean;
+      m.m2 = fmaf(d * d, half, m.m2 + __shfl_xor_sync(0xffffffffu, m.m2, o));
+      m.mean = 0.5f * (m.mean + other);
+    }
+    return make_float2(m.mean, 1.0f / sqrtf(m.m2 / (float)H + eps));
+  }
   if (n_own > 0) m.mean = sum / (float)n_own;
 #pragma unroll
   for (int i = 0; i < CAP; ++i) {
@@ -105,16 +134,18 @@ sandwich_norm_kernel(float* __restrict__ h, const TA* __restrict__ a, const floa
   __shared__ float scratch[2][96];
   constexpr int CAP = NV * W;
   const int step = blockDim.x * W, c0 = threadIdx.x * W;
-  float wp[CAP];                                    // the weights come from no kernel of the step: fetched before the wait
-  if (w_post) {
+  // few values per thread (a decode step's rows): the first norm's weights, which come from no kernel of the step, are
+  // fetched before the wait; else they are read where they are used and cost no registers
+  constexpr bool EARLY = NV <= 2;
+  float wp[EARLY ? CAP : W];
+  auto fetch_w = [&](float* to, int c) {
+    if constexpr (W == 4) *reinterpret_cast<float4*>(to) = load4(w_post + c);
+    else *to = w_post[c];
+  };
+  if (EARLY && w_post) {
 #pragma unroll
     for (int i = 0; i < NV; ++i)
-#pragma unroll
-      for (int u = 0; u < W; ++u) {
-        const int c = c0 + i * step;
-        if (W == 4 && u == 0 && c < H) *reinterpret_cast<float4*>(wp + i * W) = load4(w_post + c);
-        if (W == 1 && c < H) wp[i] = w_post[c];
-      }
+      if (c0 + i * step < H) fetch_w(wp + i * W, c0 + i * step);
   }
   pdl_wait();
   const size_t src = (size_t)(rows ? rows[blockIdx.x] : blockIdx.x) * H;
@@ -157,8 +188,13 @@ sandwich_norm_kernel(float* __restrict__ h, const TA* __restrict__ a, const floa
     if (w_post) {
       const float2 st = row_moments(y, n_own, H, post_kind, post_eps, scratch[0]);
 #pragma unroll
-      for (int i = 0; i < CAP; ++i)
-        if (i < n_own) y[i] = (y[i] - st.x) * st.y * wp[i];
+      for (int i = 0; i < NV; ++i) {
+        const int c = c0 + i * step;
+        if (c >= H) continue;
+        if (!EARLY) fetch_w(wp, c);
+#pragma unroll
+        for (int u = 0; u < W; ++u) y[i * W + u] = (y[i * W + u] - st.x) * st.y * wp[(EARLY ? i * W : 0) + u];
+      }
     }
 #pragma unroll
     for (int i = 0; i < CAP; ++i)

@@ -1836,11 +1836,14 @@ def linear_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: 
 
 
 def linear_recurrence_gated(proj, lower: torch.Tensor, f_bias: Optional[torch.Tensor], state: torch.Tensor, heads: int, dim: int,
-                            vdim: int, step) -> torch.Tensor:
+                            vdim: int, step, norm_weight: Optional[torch.Tensor] = None, norm_eps: float = 0.0,
+                            out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     """The recurrence whose forget gate decides what is written, from and to ``state`` [slots, heads, dim, vdim] (float32):
     with the projection's columns [q | z | v], ``f = lower + (1 - lower) sigmoid(z + f_bias)``,
     ``S = diag(f) S + (1 - f) v^T``, ``o = S^T silu(q)``.  ``proj`` is float32 [T, heads * (2 dim + vdim)], or
-    :class:`Partials` of it whose splits the kernel adds in order.  Returns float32 [T, heads * vdim]."""
+    :class:`Partials` of it whose splits the kernel adds in order.  Returns float32 [T, heads * vdim]; with
+    ``norm_weight`` (float32 [vdim]) every head of it RMS-normed, in ``out_dtype`` (one kernel where every request
+    brings a single token)."""
     qk, hv = heads * dim, heads * vdim
     data, splits = (proj.data, proj.splits) if isinstance(proj, Partials) else (proj, 1)
     T, W = proj.shape
@@ -1849,14 +1852,26 @@ def linear_recurrence_gated(proj, lower: torch.Tensor, f_bias: Optional[torch.Te
         _need(t is None or (t.dtype == torch.float32 and t.numel() == qk and t.is_contiguous()), "the gate's vectors are float32 [heads * dim]")
     state, stride = _slot_view(state, "linear_recurrence_gated")
     _need(state[0].numel() == heads * dim * vdim, "linear_recurrence_gated: state [slots, heads, dim, vdim]")
-    out = torch.empty((T, hv), dtype=torch.float32, device=data.device)
     base = data.data_ptr()
     at = lambda cols: ctypes.c_void_p(base + 4 * cols)
+    if norm_weight is not None and step.all_decode and lib().zi_gated_decode_supported(dim, vdim) and stride % 4 == 0:
+        _need(norm_weight.dtype == torch.float32 and norm_weight.numel() == vdim and norm_weight.is_contiguous(), "the heads' norm weight is float32 [vdim]")
+        out = torch.empty((T, hv), dtype=out_dtype or torch.float32, device=data.device)
+        with _prof.region("linear recurrence (gate writes, single tokens, head norm)",
+                          lambda: _nb(data, out) + 2 * step.n_seqs * heads * dim * vdim * 4, 6 * T * heads * dim * vdim):
+            _check(lib().zi_gated_decode(
+                _ptr(out), _tag(out), out.stride(0), at(0), W, at(qk), W, at(2 * qk), W, splits, _ll(T * W), _ptr(f_bias), _ptr(lower),
+                _ptr(state), _ll(stride), heads, dim, vdim, _ptr(norm_weight), ctypes.c_float(norm_eps), _ptr(step.cu_q),
+                _ptr(step.state_slots), step.n_seqs, _stream()), "gated_decode")
+        return out
+    out = torch.empty((T, hv), dtype=torch.float32, device=data.device)
     with _prof.region("linear recurrence (gate writes)",
                       lambda: _nb(data, out) + 2 * step.n_seqs * heads * dim * vdim * 4, 6 * T * heads * dim * vdim):
         _check(lib().zi_linear_recurrence_gated(
             _ptr(out), out.stride(0), at(0), W, at(qk), W, at(2 * qk), W, splits, _ll(T * W), _ptr(f_bias), _ptr(lower), _ptr(state),
             _ll(stride), heads, dim, vdim, _ptr(step.cu_q), _ptr(step.state_slots), step.n_seqs, _stream()), "linear_recurrence_gated")
+    if norm_weight is not None:
+        return head_norm_gate(out, norm_weight, norm_eps, None, "none", heads, vdim, out_dtype or torch.float32)
     return out
 
 

@@ -123,8 +123,8 @@ class HGRN2(Mixer):
     def forward(self, x, step, cache):
         # 32-bit results of the product: the gate and the recurrence read the unrounded sums (and add its K splits)
         proj = ops.linear(x, self.w_in, out_dtype=torch.float32, allow_partials=True)
-        o = ops.linear_recurrence_gated(proj, self.lower, self.f_bias, cache.state, self.heads, self.dim, self.vdim, step)
-        y = ops.head_norm_gate(o, self.norm, self.eps, None, "none", self.heads, self.vdim, self.ctx.dtype)
+        y = ops.linear_recurrence_gated(proj, self.lower, self.f_bias, cache.state, self.heads, self.dim, self.vdim, step,
+                                        norm_weight=self.norm, norm_eps=self.eps, out_dtype=self.ctx.dtype)
         return ops.linear(y, self.w_o, out_dtype=self.ctx.dtype, allow_partials=True)
 
 
