@@ -769,3 +769,40 @@ def test_gated_recurrence_against_plain_arithmetic():
                 tol = 1e-2 if dtype == torch.bfloat16 else 2e-4
                 assert got.dtype == dtype and torch.allclose(got.float().cpu(), want, rtol=tol, atol=tol), (heads, dim, vdim)
                 assert torch.allclose(state.cpu(), ref_state, rtol=1e-4, atol=1e-4)
+
+
+@gpu
+def test_recurrence_in_tiles_against_one_walk(tmp_path, monkeypatch):
+    """Long portions cut into tiles that run side by side give what one walk over the portion gives: outputs and states,
+    portions that end at a tile's edge and just beyond, beside single tokens and short portions, from states that earlier
+    portions left; fast and slow forgetting."""
+    from zinfer_b200 import ops
+    from zinfer_b200.cache import CacheManager
+    from zinfer_b200.engine.batch import StepEntry, build_step
+
+    rows = ops.attention_prefill_tile_rows()
+    g = torch.Generator(device=DEV).manual_seed(9)
+    rnd = lambda *shape: torch.randn(*shape, generator=g, device=DEV)
+    for heads, dim, vdim, lens in ((2, 16, 24, (2 * rows, 1, 5 * rows + 1, 2, 3 * rows - 1)), (1, 64, 64, (1, 1000)), (3, 300, 8, (2 * rows + 7,)),
+                                   (2, 128, 128, (rows, 4 * rows, 1, rows + 1))):
+        m = CacheManager({}, ["s"], 16, 1, 8)
+        entries = []
+        for i, n in enumerate(lens):
+            m.add_request(i)
+            entries.append(StepEntry(i, [0] * n))
+        step = build_step(m, entries, DEV, ops.attention_tile_rows(), pf_tile_rows=rows)
+        T = step.n_tokens
+        proj = rnd(T, heads * (2 * dim + vdim))
+        lower = 0.999 * torch.rand(heads * dim, generator=g, device=DEV)
+        bias = 3.0 * rnd(heads * dim)
+        w = 1 + 0.1 * rnd(vdim)
+        state0 = rnd(9, heads, dim, vdim)
+        outs = []
+        for tiles in (False, True):
+            monkeypatch.setattr(ops, "RECURRENCE_TILES", tiles)
+            state = state0.clone()
+            y = ops.linear_recurrence_gated(proj, lower, bias, state, heads, dim, vdim, step, norm_weight=w, norm_eps=1e-5, out_dtype=torch.bfloat16)
+            outs.append((y.float(), state))
+        assert torch.allclose(outs[0][1], outs[1][1], rtol=1e-4, atol=1e-4), (heads, dim, vdim)
+        assert torch.allclose(outs[0][0], outs[1][0], rtol=2e-2, atol=2e-2), (heads, dim, vdim)
+        assert not torch.equal(outs[1][1], state0)

@@ -143,35 +143,56 @@ __device__ __forceinline__ void forget_gate(float z, float lower, float& g, floa
   k = (1.0f - lower) * down;                                   // 1 - g without cancellation
 }
 
-template <typename TQ, typename TV, int R, bool DELTA, bool GATE = false>
+// A long portion in tiles of `rows` tokens that run side by side, in three passes (CHUNK of the kernel): 1 every tile but a
+// request's last makes the state it would leave if it began from zero, and the product of its decays; a small kernel
+// then walks a request's tiles in order, S <- P S + L, and leaves each tile the state it begins with; 2 every tile runs
+// the recurrence from that state.  0: a request's tokens in one walk.
+struct RecurrenceTiles {
+  const int* tile_seq;     // request of each tile
+  const int* tile_q0;      // its first token within the request's portion
+  int rows;
+  float* states;           // [tiles][H][D][V]: L, then the state each tile begins with
+  float* decays;           // [tiles][H][D]: P
+  int only_single;         // CHUNK 0: leave out requests that bring more than one token
+};
+
+template <typename TQ, typename TV, int R, bool DELTA, bool GATE = false, int CHUNK = 0>
 __global__ void __launch_bounds__(LR_THREADS)
 linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict__ q, int ldq, const TQ* __restrict__ k,
                          int ldk, const TV* __restrict__ v, int ldv, const float* __restrict__ decay, int ldg,
                          const float* __restrict__ beta, int ldb, float q_scale, float* __restrict__ state,
                          long long slot_stride, int H, int G, int D, int V, int P, const int* __restrict__ cu_q,
-                         const int* __restrict__ state_slots, const ForgetGate fgate) {
+                         const int* __restrict__ state_slots, const ForgetGate fgate, const RecurrenceTiles tiles) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
   const int DP = P * R;                           // key channels rounded up to whole parts
   const int CW = (32 / P) * NC, CB = LR_WARPS * CW;   // columns per warp and per block
   const int BUF = 3 * TB * DP + TB * CB + TB;     // one staging buffer: q, k, g [TB][DP], v [TB][CB], beta [TB]
-  const int s = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * CB;
+  const int s = CHUNK ? tiles.tile_seq[blockIdx.x] : blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * CB;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int p = lane % P, cw = lane / P;
   const int cb = warp * CW + cw * NC, col = j0 + cb;   // this lane's first column within the block, and of the head
   const int kvh = h / (H / G);
-  const int tok0 = cu_q[s], qlen = cu_q[s + 1] - tok0;
-  if (qlen <= 0) return;
+  const int q0 = CHUNK ? tiles.tile_q0[blockIdx.x] : 0;
+  const int tok0 = cu_q[s] + q0, left = cu_q[s + 1] - tok0;
+  const int qlen = CHUNK ? min(tiles.rows, left) : left;
+  const bool last = qlen == left;
+  if (qlen <= 0 || (CHUNK == 1 && last) || (CHUNK == 0 && tiles.only_single && qlen != 1)) return;
   float* S = state + (size_t)state_slots[s] * slot_stride + (size_t)h * D * V;
+  float* ST = CHUNK ? tiles.states + ((size_t)blockIdx.x * H + h) * D * V : S;      // where this walk begins
   float Sr[NC][R];
 #pragma unroll
   for (int c = 0; c < NC; ++c)
 #pragma unroll
     for (int r = 0; r < R; ++r) {
       const int i = p * R + r;
-      Sr[c][r] = (i < D && col + c < V) ? S[(size_t)i * V + col + c] : 0.f;
+      Sr[c][r] = (CHUNK != 1 && i < D && col + c < V) ? ST[(size_t)i * V + col + c] : 0.f;
     }
+  const bool makes_decays = CHUNK == 1 && warp == 0 && blockIdx.z == 0;
+  float Pr[CHUNK == 1 ? R : 1];
+#pragma unroll
+  for (int r = 0; r < (CHUNK == 1 ? R : 1); ++r) Pr[r] = 1.f;
   // DP and CB are powers of two: shifts instead of divisions
   const int lgDP = 31 - __clz(DP), lgCB = 31 - __clz(CB), lgP = 31 - __clz(P);
   // Key channel i = p R + 4 r4 + x lies at ((r4 P + p) 4 + x) of its token's row: for one r4 the P lanes of a column
@@ -193,7 +214,7 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
       const int tt = e >> lgDP, i = e & (DP - 1);
       if (e < total && i < D) {
         const size_t row = (size_t)(tok0 + t0 + tt);
-        fq[u] = q[row * ldq + (size_t)kvh * D + i];
+        if (CHUNK != 1) fq[u] = q[row * ldq + (size_t)kvh * D + i];
         fk[u] = k[row * ldk + (size_t)kvh * D + i];
         if (!GATE) fg[u] = decay[row * ldg + (size_t)h * D + i];
       } else {
@@ -218,7 +239,7 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
           const int tt = e >> lgDP, i = e & (DP - 1);
           if (e < total && i < D) {
             const size_t row = (size_t)(tok0 + t0 + tt);
-            fq[u] += q[zo + row * ldq + (size_t)kvh * D + i];
+            if (CHUNK != 1) fq[u] += q[zo + row * ldq + (size_t)kvh * D + i];
             fk[u] += k[zo + row * ldk + (size_t)kvh * D + i];
           }
         }
@@ -237,12 +258,12 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
       if (i < D) {
         const int ch = h * D + i;
         forget_gate(kv + (fgate.bias ? fgate.bias[ch] : 0.f), fgate.lower[ch], gv, kv);
-        qv = qv * sigmoid_f32(qv);
+        if (CHUNK != 1) qv = qv * sigmoid_f32(qv);
       } else {
         kv = gv = 0.f;
       }
     }
-    buf[at] = qv * q_scale;
+    if (CHUNK != 1) buf[at] = qv * q_scale;
     buf[TB * DP + at] = kv;
     buf[2 * TB * DP + at] = gv;
   };
@@ -293,7 +314,31 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
     if (more) fetch(t0 + TB, min(TB, qlen - t0 - TB));
     const float* vs = buf + 3 * TB * DP;
     const float* bs = vs + TB * CB;
-    for (int tt = 0; tt < nt; ++tt) {
+    if constexpr (CHUNK == 1) {        // the state alone: no read-out
+      for (int tt = 0; tt < nt; ++tt) {
+        const float4* kt = reinterpret_cast<const float4*>(buf + TB * DP + tt * DP) + p;
+        const float4* gt = reinterpret_cast<const float4*>(buf + 2 * TB * DP + tt * DP) + p;
+        float vj[NC];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) vj[c] = vs[tt * CB + cb + c];
+#pragma unroll
+        for (int r4 = 0; r4 < R / 4; ++r4) {
+          const float4 g4 = gt[r4 << lgP], k4 = kt[r4 << lgP];
+#pragma unroll
+          for (int c = 0; c < NC; ++c) {
+            float* sr = Sr[c] + 4 * r4;
+            sr[0] = fmaf(g4.x, sr[0], k4.x * vj[c]);
+            sr[1] = fmaf(g4.y, sr[1], k4.y * vj[c]);
+            sr[2] = fmaf(g4.z, sr[2], k4.z * vj[c]);
+            sr[3] = fmaf(g4.w, sr[3], k4.w * vj[c]);
+          }
+          if (makes_decays) {
+            Pr[4 * r4] *= g4.x; Pr[4 * r4 + 1] *= g4.y; Pr[4 * r4 + 2] *= g4.z; Pr[4 * r4 + 3] *= g4.w;
+          }
+        }
+      }
+    }
+    for (int tt = 0; CHUNK != 1 && tt < nt; ++tt) {
       const float4* qt = reinterpret_cast<const float4*>(buf + tt * DP) + p;
       const float4* kt = reinterpret_cast<const float4*>(buf + TB * DP + tt * DP) + p;
       const float4* gt = reinterpret_cast<const float4*>(buf + 2 * TB * DP + tt * DP) + p;
@@ -338,13 +383,64 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
     __syncthreads();     // the other buffer is filled, and this one is free for the batch after it
     cur ^= 1;
   }
+  if (CHUNK == 2 && !last) return;               // the next tile has its own
+  float* SE = CHUNK == 1 ? ST : S;
 #pragma unroll
   for (int c = 0; c < NC; ++c)
 #pragma unroll
     for (int r = 0; r < R; ++r) {
       const int i = p * R + r;
-      if (i < D && col + c < V) S[(size_t)i * V + col + c] = Sr[c][r];
+      if (i < D && col + c < V) SE[(size_t)i * V + col + c] = Sr[c][r];
     }
+  if (makes_decays && cw == 0) {
+#pragma unroll
+    for (int r = 0; r < (CHUNK == 1 ? R : 1); ++r) {
+      const int i = p * R + r;
+      if (i < D) tiles.decays[((size_t)blockIdx.x * H + h) * D + i] = Pr[r];
+    }
+  }
+}
+
+// Between the two passes over a long portion's tiles: one thread per element of a head's state walks its request's tiles
+// in order.  A request's tiles may stand anywhere in the list, so each block first finds their places.
+constexpr int SCAN_THREADS = 256, SCAN_TILES = 1024;
+
+__global__ void __launch_bounds__(SCAN_THREADS)
+recurrence_scan_kernel(const RecurrenceTiles tiles, int n_tiles, const float* __restrict__ state, long long slot_stride, int H, int D,
+                       int V, const int* __restrict__ cu_q, const int* __restrict__ state_slots) {
+  pdl_launch_dependents();
+  __shared__ int at[SCAN_TILES];
+  const int s = blockIdx.x, h = blockIdx.y, e = blockIdx.z * SCAN_THREADS + threadIdx.x;
+  const int qlen = cu_q[s + 1] - cu_q[s];        // the step's own arrays: here before any kernel of the step
+  const int n = min((qlen + tiles.rows - 1) / tiles.rows, SCAN_TILES);
+  for (int t = threadIdx.x; t < n_tiles; t += SCAN_THREADS) {
+    const int c = tiles.tile_q0[t] / tiles.rows;
+    if (tiles.tile_seq[t] == s && c < n) at[c] = t;
+  }
+  __syncthreads();
+  pdl_wait();
+  if (qlen <= 1 || e >= D * V) return;           // single tokens have no tiles
+  float S = state[(size_t)state_slots[s] * slot_stride + (size_t)h * D * V + e];
+  const int i = e / V;
+  constexpr int AHEAD = 8;
+  for (int c0 = 0; c0 < n; c0 += AHEAD) {
+    float L[AHEAD], P[AHEAD];
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) {
+      const int c = c0 + u;
+      L[u] = P[u] = 0.f;
+      if (c < n - 1) {
+        L[u] = tiles.states[((size_t)at[c] * H + h) * D * V + e];
+        P[u] = tiles.decays[((size_t)at[c] * H + h) * D + i];
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) {
+      if (c0 + u >= n) break;
+      tiles.states[((size_t)at[c0 + u] * H + h) * D * V + e] = S;
+      S = fmaf(P[u], S, L[u]);
+    }
+  }
 }
 
 // ------------------------------------------- one token per request: the third form with the head norm, in one kernel
@@ -540,7 +636,8 @@ extern "C" int zi_linear_recurrence(float* out, int ldo, const void* q, int ldq,
         return zi_refuse("linear_recurrence: cannot get %zu bytes of shared memory", smem);                            \
     }                                                                                                                  \
     zi_launch(kern, dim3(grid), dim3(block), smem, stream, out, ldo, (const TQ*)q, ldq, (const TQ*)k, ldk, (const TV*)v, \
-              ldv, decay, ldg, beta, ldb, q_scale, state, slot_stride, H, G, D, V, P, cu_q, state_slots, ForgetGate{}); \
+              ldv, decay, ldg, beta, ldb, q_scale, state, slot_stride, H, G, D, V, P, cu_q, state_slots, ForgetGate{}, \
+              RecurrenceTiles{});                                                                                      \
   } while (0)
 #define ZI_LR_R(TQ, TV)                                          \
   do {                                                           \
@@ -576,8 +673,55 @@ extern "C" int zi_linear_recurrence_gated(float* out, int ldo, const float* q, i
   if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
     return zi_refuse("linear_recurrence_gated: cannot get %zu bytes of shared memory", smem);
   zi_launch(kern, grid, block, smem, stream, out, ldo, q, ldq, z, ldz, v, ldv, (const float*)nullptr, 0, (const float*)nullptr, 0, 1.0f,
-            state, slot_stride, H, H, D, V, P, cu_q, state_slots, gate);
+            state, slot_stride, H, H, D, V, P, cu_q, state_slots, gate, RecurrenceTiles{});
   return zi_check_launch("linear_recurrence_gated");
+}
+
+// Floats of workspace that the form with tiles needs.
+extern "C" long long zi_linear_recurrence_tiles_floats(int n_tiles, int H, int D, int V) { return (long long)n_tiles * H * D * (V + 1); }
+extern "C" int zi_linear_recurrence_tiles_supported(int n_tiles, int max_q_len, int rows, int D) {
+  return n_tiles > 0 && rows > 0 && D > 0 && D <= 512 && (max_q_len + rows - 1) / rows <= SCAN_TILES;
+}
+
+// The same with the long portions cut into tiles of `rows` tokens that run side by side (tile_seq, tile_q0: the step's list
+// over the requests that bring more than one token; n_single requests bring exactly one).
+extern "C" int zi_linear_recurrence_gated_tiles(float* out, int ldo, const float* q, int ldq, const float* z, int ldz, const float* v,
+                                                int ldv, int splits, long long zstride, const float* f_bias, const float* lower,
+                                                float* state, long long slot_stride, int H, int D, int V, const int* cu_q,
+                                                const int* state_slots, int n_seqs, const int* tile_seq, const int* tile_q0,
+                                                int n_tiles, int rows, int max_q_len, int n_single, float* workspace,
+                                                cudaStream_t stream) {
+  if (n_seqs <= 0) return 0;
+  if (H <= 0 || H > 65535 || V <= 0 || !zi_linear_recurrence_tiles_supported(n_tiles, max_q_len, rows, D))
+    return zi_refuse("linear_recurrence_gated_tiles: %d tiles of %d tokens, %d key channels", n_tiles, rows, D);
+  if (!lower || splits < 1 || !workspace) return zi_refuse("linear_recurrence_gated_tiles: needs the gate's lower bound and a workspace");
+  const int R = D <= 256 ? 8 : 16;
+  int P = 1;
+  while (P * R < D) P <<= 1;
+  const int CB = LR_WARPS * (32 / P) * NC;
+  const size_t smem = (size_t)2 * (3 * TB * P * R + TB * CB + TB) * sizeof(float);
+  const ForgetGate gate = {lower, f_bias, splits, zstride};
+  RecurrenceTiles tiles = {tile_seq, tile_q0, rows, workspace, workspace + (size_t)n_tiles * H * D * V, 0};
+  auto run = [&](auto kern, int blocks) {
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+      return zi_refuse("linear_recurrence_gated_tiles: cannot get %zu bytes of shared memory", smem);
+    zi_launch(kern, dim3(blocks, H, (V + CB - 1) / CB), dim3(LR_THREADS), smem, stream, out, ldo, q, ldq, z, ldz, v, ldv,
+              (const float*)nullptr, 0, (const float*)nullptr, 0, 1.0f, state, slot_stride, H, H, D, V, P, cu_q, state_slots, gate, tiles);
+    return zi_check_launch("linear_recurrence_gated_tiles");
+  };
+  int rc = R == 8 ? run(linear_recurrence_kernel<float, float, 8, false, true, 1>, n_tiles)
+                  : run(linear_recurrence_kernel<float, float, 16, false, true, 1>, n_tiles);
+  if (rc) return rc;
+  zi_launch(recurrence_scan_kernel, dim3(n_seqs, H, (D * V + SCAN_THREADS - 1) / SCAN_THREADS), dim3(SCAN_THREADS), 0, stream, tiles, n_tiles,
+            (const float*)state, slot_stride, H, D, V, cu_q, state_slots);
+  rc = zi_check_launch("linear_recurrence_gated_tiles (scan)");
+  if (rc) return rc;
+  rc = R == 8 ? run(linear_recurrence_kernel<float, float, 8, false, true, 2>, n_tiles)
+              : run(linear_recurrence_kernel<float, float, 16, false, true, 2>, n_tiles);
+  if (rc || n_single <= 0) return rc;
+  tiles.only_single = 1;
+  return R == 8 ? run(linear_recurrence_kernel<float, float, 8, false, true, 0>, n_seqs)
+                : run(linear_recurrence_kernel<float, float, 16, false, true, 0>, n_seqs);
 }
 
 // Whether the one-kernel form for single tokens takes these sizes.

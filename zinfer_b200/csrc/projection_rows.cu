@@ -209,15 +209,18 @@ qkv_heads_kernel(const TS* __restrict__ src, int src_stride, const float* __rest
 // tokens' own pages (block_tables), and their means go to entry entry_slots[t] of the pooled pages, in 32-bit sums in
 // the order of the positions.  A block of threads looks through POOL_TOKENS neighbouring tokens (most complete nothing) and
 // does the entries they complete for one kv head.
-constexpr int POOL_TOKENS = 32;
+// C: elements per access (16 bytes, or one).
+constexpr int POOL_TOKENS = 32, POOL_THREADS = 128, POOL_COLS = 16, POOL_TILE_BYTES = 32 * 1024;
 
-template <typename T>
-__global__ void __launch_bounds__(128)
+template <typename T, int C>
+__global__ void __launch_bounds__(POOL_THREADS)
 pool_blocks_kernel(const T* __restrict__ kcache, const T* __restrict__ vcache, const int* __restrict__ block_tables, int bt_stride,
                    T* __restrict__ kpool, T* __restrict__ vpool, const int* __restrict__ entry_slots,
                    const int* __restrict__ positions, const int* __restrict__ cu_q, int n_seqs, int T_, int nkv, int d, int dv,
-                   int per, int page_size) {
+                   int per, int page_size, int tile) {
   pdl_launch_dependents();
+  extern __shared__ __align__(16) float rows[];      // [tile][W]
+  const int W = d + dv;
   const int t0 = blockIdx.x * POOL_TOKENS, kvh = blockIdx.y, lane = threadIdx.x & 31;
   // the step's own arrays: here before any kernel of the step
   const int mine = t0 + lane < T_ ? entry_slots[t0 + lane] : -1;
@@ -235,17 +238,38 @@ pool_blocks_kernel(const T* __restrict__ kcache, const T* __restrict__ vcache, c
     const int* bt = block_tables + (size_t)lo * bt_stride;
     const int p0 = positions[t] - per + 1;
     const size_t out_at = ((size_t)(entry / page_size) * nkv + kvh) * page_size + (entry % page_size);
-    for (int c = threadIdx.x; c < d + dv; c += blockDim.x) {
-      const bool is_k = c < d;
-      const T* base = is_k ? kcache : vcache;
-      const int w = is_k ? d : dv, i = is_k ? c : c - d;
-      float sum = 0.f;
-#pragma unroll 8
-      for (int j = 0; j < per; ++j) {
-        const int p = p0 + j, page = p < 0 ? -1 : bt[p / page_size];
-        sum += page >= 0 ? to_f32(base[(((size_t)page * nkv + kvh) * page_size + (p % page_size)) * w + i]) : 0.f;
+    // TILE rows [key | value] at a time into shared memory, all their loads in flight together; then a thread per column
+    // adds them in the order of the positions
+    float sum[POOL_COLS];
+#pragma unroll
+    for (int u = 0; u < POOL_COLS; ++u) sum[u] = 0.f;
+    for (int j0 = 0; j0 < per; j0 += tile) {
+      const int nj = min(tile, per - j0);
+      __syncthreads();                                // the tile before is added up
+      for (int e = threadIdx.x; e < nj * (W / C); e += POOL_THREADS) {
+        const int r = e / (W / C), c = (e - r * (W / C)) * C, p = p0 + j0 + r;
+        const int page = p < 0 ? -1 : bt[p / page_size];
+        const size_t at = page < 0 ? 0 : ((size_t)page * nkv + kvh) * page_size + (p % page_size);
+        const T* src = c < d ? kcache + at * d + c : vcache + at * dv + c - d;
+        __align__(16) T v[C];
+        if constexpr (C > 1) *reinterpret_cast<uint4*>(v) = *reinterpret_cast<const uint4*>(src);
+        else v[0] = *src;
+#pragma unroll
+        for (int u = 0; u < C; ++u) rows[r * W + c + u] = page < 0 ? 0.f : to_f32(v[u]);
       }
-      (is_k ? kpool : vpool)[out_at * w + i] = from_f32<T>(sum * inv);
+      __syncthreads();
+#pragma unroll
+      for (int u = 0; u < POOL_COLS; ++u) {
+        const int c = threadIdx.x + u * POOL_THREADS;
+        if (c < W)
+          for (int r = 0; r < nj; ++r) sum[u] += rows[r * W + c];
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < POOL_COLS; ++u) {
+      const int c = threadIdx.x + u * POOL_THREADS;
+      if (c < d) kpool[out_at * d + c] = from_f32<T>(sum[u] * inv);
+      else if (c < W) vpool[out_at * dv + c - d] = from_f32<T>(sum[u] * inv);
     }
   }
 }
@@ -331,9 +355,20 @@ extern "C" int zi_pool_blocks(const void* kcache, const void* vcache, int dtype,
   if (T <= 0 || n_seqs <= 0) return 0;
   if (nkv <= 0 || d <= 0 || dv <= 0 || per <= 0 || page_size <= 0) return zi_refuse("pool_blocks: blocks of %d tokens, heads of %d and %d", per, d, dv);
   if (nkv > 65535) return zi_refuse("pool_blocks: %d kv heads", nkv);
-  ZI_DISPATCH_DTYPE(dtype, TT, zi_launch(pool_blocks_kernel<TT>, dim3((T + POOL_TOKENS - 1) / POOL_TOKENS, nkv), dim3(128), 0, stream, (const TT*)kcache, (const TT*)vcache,
-                                         block_tables, bt_stride, (TT*)kpool, (TT*)vpool, entry_slots, positions, cu_q, n_seqs,
-                                         T, nkv, d, dv, per, page_size));
+  if (d + dv > POOL_COLS * POOL_THREADS) return zi_refuse("pool_blocks: heads of %d and %d are more than this kernel holds", d, dv);
+  const int per16 = dtype == ZI_BF16 ? 8 : 4;
+  auto al16 = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+  const bool vec = d % per16 == 0 && dv % per16 == 0 && al16(kcache) && al16(vcache);
+  int tile = POOL_TILE_BYTES / (int)((d + dv) * sizeof(float));
+  tile = tile < 1 ? 1 : (tile > per ? per : tile);
+  const size_t smem = (size_t)tile * (d + dv) * sizeof(float);
+  dim3 grid((T + POOL_TOKENS - 1) / POOL_TOKENS, nkv);
+  ZI_DISPATCH_DTYPE(dtype, TT, {
+    constexpr int C = 16 / (int)sizeof(TT);
+    auto kern = vec ? pool_blocks_kernel<TT, C> : pool_blocks_kernel<TT, 1>;
+    zi_launch(kern, grid, dim3(POOL_THREADS), smem, stream, (const TT*)kcache, (const TT*)vcache, block_tables, bt_stride, (TT*)kpool,
+              (TT*)vpool, entry_slots, positions, cu_q, n_seqs, T, nkv, d, dv, per, page_size, tile);
+  });
   return zi_check_launch("pool_blocks");
 }
 

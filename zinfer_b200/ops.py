@@ -37,6 +37,7 @@ def lib() -> ctypes.CDLL:
         _LIB.zi_last_error.restype = ctypes.c_char_p
         _LIB.zi_gemm_tcgen05_plan.restype = ctypes.c_longlong
         _LIB.zi_attention_decode_workspace_floats.restype = ctypes.c_longlong
+        _LIB.zi_linear_recurrence_tiles_floats.restype = ctypes.c_longlong
     return _LIB
 
 
@@ -1835,6 +1836,9 @@ def linear_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: 
     return out
 
 
+RECURRENCE_TILES = os.environ.get("ZINFER_B200_RECURRENCE_TILES", "1") not in ("", "0")   # off: every request in one walk (comparisons)
+
+
 def linear_recurrence_gated(proj, lower: torch.Tensor, f_bias: Optional[torch.Tensor], state: torch.Tensor, heads: int, dim: int,
                             vdim: int, step, norm_weight: Optional[torch.Tensor] = None, norm_eps: float = 0.0,
                             out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
@@ -1865,11 +1869,24 @@ def linear_recurrence_gated(proj, lower: torch.Tensor, f_bias: Optional[torch.Te
                 _ptr(step.state_slots), step.n_seqs, _stream()), "gated_decode")
         return out
     out = torch.empty((T, hv), dtype=torch.float32, device=data.device)
+    tiles, rows = False, 0
+    if RECURRENCE_TILES and out_dtype == torch.bfloat16 and not step.all_decode:
+        rows = attention_prefill_tile_rows()
+        if step.max_q_len >= 2 * rows:          # and too few blocks in one walk to fill the GPU
+            tiles = (step.n_seqs - step.n_dec) * heads * max(1, vdim // 32) < 4 * _sm_count(data.device) \
+                and bool(lib().zi_linear_recurrence_tiles_supported(step.n_pf_tiles, step.max_q_len, rows, dim))
     with _prof.region("linear recurrence (gate writes)",
                       lambda: _nb(data, out) + 2 * step.n_seqs * heads * dim * vdim * 4, 6 * T * heads * dim * vdim):
-        _check(lib().zi_linear_recurrence_gated(
-            _ptr(out), out.stride(0), at(0), W, at(qk), W, at(2 * qk), W, splits, _ll(T * W), _ptr(f_bias), _ptr(lower), _ptr(state),
-            _ll(stride), heads, dim, vdim, _ptr(step.cu_q), _ptr(step.state_slots), step.n_seqs, _stream()), "linear_recurrence_gated")
+        if tiles:      # few requests with long portions: tiles of a portion side by side
+            ws = torch.empty((lib().zi_linear_recurrence_tiles_floats(step.n_pf_tiles, heads, dim, vdim),), dtype=torch.float32, device=data.device)
+            _check(lib().zi_linear_recurrence_gated_tiles(
+                _ptr(out), out.stride(0), at(0), W, at(qk), W, at(2 * qk), W, splits, _ll(T * W), _ptr(f_bias), _ptr(lower), _ptr(state),
+                _ll(stride), heads, dim, vdim, _ptr(step.cu_q), _ptr(step.state_slots), step.n_seqs, _ptr(step.pf_tile_seq),
+                _ptr(step.pf_tile_q0), step.n_pf_tiles, rows, step.max_q_len, step.n_dec, _ptr(ws), _stream()), "linear_recurrence_gated_tiles")
+        else:
+            _check(lib().zi_linear_recurrence_gated(
+                _ptr(out), out.stride(0), at(0), W, at(qk), W, at(2 * qk), W, splits, _ll(T * W), _ptr(f_bias), _ptr(lower), _ptr(state),
+                _ll(stride), heads, dim, vdim, _ptr(step.cu_q), _ptr(step.state_slots), step.n_seqs, _stream()), "linear_recurrence_gated")
     if norm_weight is not None:
         return head_norm_gate(out, norm_weight, norm_eps, None, "none", heads, vdim, out_dtype or torch.float32)
     return out
