@@ -234,13 +234,13 @@ int zi_linear_recurrence_gated(float* out, int ldo, const float* q, int ldq, con
                                int splits, long long zstride, const float* f_bias, const float* lower, float* state,
                                long long slot_stride, int H, int D, int V, const int* cu_q, const int* state_slots, int n_seqs,
                                cudaStream_t stream);
-// The same with the long portions cut into tiles of `rows` tokens that run side by side: the local states of the tiles, a
+// The same (whole rows) with the long portions cut into tiles of `rows` tokens that run side by side: q and gates, the local states of the tiles, a
 // walk over each request's tiles, the tiles again from the states they begin with.
-long long zi_linear_recurrence_tiles_floats(int n_tiles, int H, int D, int V);
+long long zi_linear_recurrence_tiles_floats(int T, int n_tiles, int H, int D, int V);
 int zi_linear_recurrence_tiles_supported(int n_tiles, int max_q_len, int rows, int D);
 int zi_linear_recurrence_gated_tiles(float* out, int ldo, const float* q, int ldq, const float* z, int ldz, const float* v, int ldv,
                                      int splits, long long zstride, const float* f_bias, const float* lower, float* state,
-                                     long long slot_stride, int H, int D, int V, const int* cu_q, const int* state_slots,
+                                     long long slot_stride, int T, int H, int D, int V, const int* cu_q, const int* state_slots,
                                      int n_seqs, const int* tile_seq, const int* tile_q0, int n_tiles, int rows, int max_q_len,
                                      int n_single, float* workspace, cudaStream_t stream);
 // The same for a step in which every request brings one token, with the RMS norm of every head (weight norm_w [V]) in the

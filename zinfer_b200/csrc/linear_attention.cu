@@ -156,8 +156,10 @@ struct RecurrenceTiles {
   int only_single;         // CHUNK 0: leave out requests that bring more than one token
 };
 
-template <typename TQ, typename TV, int R, bool DELTA, bool GATE = false, int CHUNK = 0>
-__global__ void __launch_bounds__(LR_THREADS)
+// MADE: the third form's q and gate come ready made (q, `decay`) and what is written is 1 - gate; there is no `k`.
+// (The third form is held to the registers that let several blocks share an SM.)
+template <typename TQ, typename TV, int R, bool DELTA, bool GATE = false, int CHUNK = 0, bool MADE = false>
+__global__ void __launch_bounds__(LR_THREADS, MADE ? (R > 8 ? 3 : 4) : (GATE && R <= 8 ? 2 : 1))
 linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict__ q, int ldq, const TQ* __restrict__ k,
                          int ldk, const TV* __restrict__ v, int ldv, const float* __restrict__ decay, int ldg,
                          const float* __restrict__ beta, int ldb, float q_scale, float* __restrict__ state,
@@ -168,7 +170,9 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
   extern __shared__ __align__(16) float sm[];
   const int DP = P * R;                           // key channels rounded up to whole parts
   const int CW = (32 / P) * NC, CB = LR_WARPS * CW;   // columns per warp and per block
-  const int BUF = 3 * TB * DP + TB * CB + TB;     // one staging buffer: q, k, g [TB][DP], v [TB][CB], beta [TB]
+  constexpr int PLANES = MADE ? 2 : 3;
+  const int GO = (PLANES - 1) * TB * DP, VO = PLANES * TB * DP;
+  const int BUF = VO + TB * CB + TB;     // one staging buffer: q, k (not MADE), g [TB][DP], v [TB][CB], beta [TB]
   const int s = CHUNK ? tiles.tile_seq[blockIdx.x] : blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * CB;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int p = lane % P, cw = lane / P;
@@ -215,12 +219,12 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
       if (e < total && i < D) {
         const size_t row = (size_t)(tok0 + t0 + tt);
         if (CHUNK != 1) fq[u] = q[row * ldq + (size_t)kvh * D + i];
-        fk[u] = k[row * ldk + (size_t)kvh * D + i];
+        if (!MADE) fk[u] = k[row * ldk + (size_t)kvh * D + i];
         if (!GATE) fg[u] = decay[row * ldg + (size_t)h * D + i];
       } else {
         fq[u] = from_f32<TQ>(0.f);
         fk[u] = from_f32<TQ>(0.f);
-        fg[u] = 0.f;
+        fg[u] = MADE ? 1.f : 0.f;
       }
     }
 #pragma unroll
@@ -264,8 +268,8 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
       }
     }
     if (CHUNK != 1) buf[at] = qv * q_scale;
-    buf[TB * DP + at] = kv;
-    buf[2 * TB * DP + at] = gv;
+    if (!MADE) buf[TB * DP + at] = kv;
+    buf[GO + at] = gv;
   };
   // a value that was not fetched into a register: whole, or the sum of its partial sums
   auto whole = [&](const auto* p) {
@@ -280,7 +284,7 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
     for (int u = 0; u < NPF; ++u) {
       const int e = tid + u * LR_THREADS;
       if (e < total) {
-        stage(buf, (e & ~(DP - 1)) + place(e & (DP - 1)), e & (DP - 1), to_f32(fq[u]), to_f32(fk[u]), GATE ? 0.f : fg[u]);
+        stage(buf, (e & ~(DP - 1)) + place(e & (DP - 1)), e & (DP - 1), to_f32(fq[u]), MADE ? 0.f : to_f32(fk[u]), GATE ? 0.f : fg[u]);
       }
     }
     for (int e = tid + NPF * LR_THREADS; e < total; e += LR_THREADS) {      // beyond the registers (DP > 128)
@@ -288,18 +292,19 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
       const size_t row = (size_t)(tok0 + t0 + tt);
       const bool in = i < D;
       stage(buf, (e & ~(DP - 1)) + place(i), i, in ? whole(q + row * ldq + (size_t)kvh * D + i) : 0.f,
-            in ? whole(k + row * ldk + (size_t)kvh * D + i) : 0.f, in && !GATE ? decay[row * ldg + (size_t)h * D + i] : 0.f);
+            in && !MADE ? whole(k + row * ldk + (size_t)kvh * D + i) : 0.f,
+            in && !GATE ? decay[row * ldg + (size_t)h * D + i] : (MADE ? 1.f : 0.f));
     }
 #pragma unroll
     for (int u = 0; u < NPV; ++u) {
       const int e = tid + u * LR_THREADS;
-      if (e < (nt << lgCB)) buf[3 * TB * DP + e] = to_f32(fv[u]);
+      if (e < (nt << lgCB)) buf[VO + e] = to_f32(fv[u]);
     }
     for (int e = tid + NPV * LR_THREADS; e < (nt << lgCB); e += LR_THREADS) {
       const int c = j0 + (e & (CB - 1));
-      buf[3 * TB * DP + e] = c < V ? whole(v + (size_t)(tok0 + t0 + (e >> lgCB)) * ldv + (size_t)h * V + c) : 0.f;
+      buf[VO + e] = c < V ? whole(v + (size_t)(tok0 + t0 + (e >> lgCB)) * ldv + (size_t)h * V + c) : 0.f;
     }
-    if (tid < nt) buf[3 * TB * DP + TB * CB + tid] = fb;
+    if (tid < nt) buf[VO + TB * CB + tid] = fb;
   };
   fetch(0, min(TB, qlen));
   put(0, min(TB, qlen), sm);
@@ -312,18 +317,18 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
     // buffer before the barrier at the end of this iteration
     const bool more = t0 + TB < qlen;
     if (more) fetch(t0 + TB, min(TB, qlen - t0 - TB));
-    const float* vs = buf + 3 * TB * DP;
+    const float* vs = buf + VO;
     const float* bs = vs + TB * CB;
     if constexpr (CHUNK == 1) {        // the state alone: no read-out
       for (int tt = 0; tt < nt; ++tt) {
         const float4* kt = reinterpret_cast<const float4*>(buf + TB * DP + tt * DP) + p;
-        const float4* gt = reinterpret_cast<const float4*>(buf + 2 * TB * DP + tt * DP) + p;
+        const float4* gt = reinterpret_cast<const float4*>(buf + GO + tt * DP) + p;
         float vj[NC];
 #pragma unroll
         for (int c = 0; c < NC; ++c) vj[c] = vs[tt * CB + cb + c];
 #pragma unroll
         for (int r4 = 0; r4 < R / 4; ++r4) {
-          const float4 g4 = gt[r4 << lgP], k4 = kt[r4 << lgP];
+          const float4 g4 = gt[r4 << lgP], k4 = MADE ? make_float4(1.f - g4.x, 1.f - g4.y, 1.f - g4.z, 1.f - g4.w) : kt[r4 << lgP];
 #pragma unroll
           for (int c = 0; c < NC; ++c) {
             float* sr = Sr[c] + 4 * r4;
@@ -338,7 +343,45 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
         }
       }
     }
-    for (int tt = 0; CHUNK != 1 && tt < nt; ++tt) {
+    if constexpr ((GATE || MADE) && CHUNK != 1) {       // what is written does not depend on the state: write, then read out
+      for (int tt = 0; tt < nt; ++tt) {
+        const float4* qt = reinterpret_cast<const float4*>(buf + tt * DP) + p;
+        const float4* kt = reinterpret_cast<const float4*>(buf + TB * DP + tt * DP) + p;
+        const float4* gt = reinterpret_cast<const float4*>(buf + GO + tt * DP) + p;
+        float vj[NC], b[NC];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+          vj[c] = vs[tt * CB + cb + c];
+          b[c] = 0.f;
+        }
+#pragma unroll
+        for (int r4 = 0; r4 < R / 4; ++r4) {
+          const float4 g4 = gt[r4 << lgP], q4 = qt[r4 << lgP];
+          const float4 k4 = MADE ? make_float4(1.f - g4.x, 1.f - g4.y, 1.f - g4.z, 1.f - g4.w) : kt[r4 << lgP];
+#pragma unroll
+          for (int c = 0; c < NC; ++c) {
+            float* sr = Sr[c] + 4 * r4;
+            sr[0] = fmaf(g4.x, sr[0], k4.x * vj[c]);
+            sr[1] = fmaf(g4.y, sr[1], k4.y * vj[c]);
+            sr[2] = fmaf(g4.z, sr[2], k4.z * vj[c]);
+            sr[3] = fmaf(g4.w, sr[3], k4.w * vj[c]);
+            b[c] = fmaf(sr[0], q4.x, fmaf(sr[1], q4.y, fmaf(sr[2], q4.z, fmaf(sr[3], q4.w, b[c]))));
+          }
+        }
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+          if (o < P) {
+#pragma unroll
+            for (int c = 0; c < NC; ++c) b[c] += __shfl_xor_sync(0xffffffffu, b[c], o);
+          }
+        }
+        float* po = out + (size_t)(tok0 + t0 + tt) * ldo + (size_t)h * V + col;
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+          if (p == 0 && col + c < V) po[c] = b[c];
+      }
+    }
+    for (int tt = 0; !GATE && !MADE && CHUNK != 1 && tt < nt; ++tt) {
       const float4* qt = reinterpret_cast<const float4*>(buf + tt * DP) + p;
       const float4* kt = reinterpret_cast<const float4*>(buf + TB * DP + tt * DP) + p;
       const float4* gt = reinterpret_cast<const float4*>(buf + 2 * TB * DP + tt * DP) + p;
@@ -399,6 +442,23 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
       if (i < D) tiles.decays[((size_t)blockIdx.x * H + h) * D + i] = Pr[r];
     }
   }
+}
+
+// The third form's q and gate of every token and channel, made once for both passes over a long portion's tiles.
+__global__ void make_gates_kernel(float* __restrict__ qs, float* __restrict__ gs, const float* __restrict__ q, int ldq,
+                                  const float* __restrict__ z, int ldz, const float* __restrict__ bias,
+                                  const float* __restrict__ lower, int W, size_t total) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (idx >= total) return;
+  const size_t row = idx / W;
+  const int c = (int)(idx - row * W);
+  const float x = q[row * ldq + c];
+  float g, k;
+  forget_gate(z[row * ldz + c] + (bias ? bias[c] : 0.f), lower[c], g, k);
+  qs[idx] = x * sigmoid_f32(x);
+  gs[idx] = g;
 }
 
 // Between the two passes over a long portion's tiles: one thread per element of a head's state walks its request's tiles
@@ -677,8 +737,10 @@ extern "C" int zi_linear_recurrence_gated(float* out, int ldo, const float* q, i
   return zi_check_launch("linear_recurrence_gated");
 }
 
-// Floats of workspace that the form with tiles needs.
-extern "C" long long zi_linear_recurrence_tiles_floats(int n_tiles, int H, int D, int V) { return (long long)n_tiles * H * D * (V + 1); }
+// Floats of workspace that the form with tiles needs: q and the gates of T tokens, the tiles' states, their decays.
+extern "C" long long zi_linear_recurrence_tiles_floats(int T, int n_tiles, int H, int D, int V) {
+  return 2ll * T * H * D + (long long)n_tiles * H * D * (V + 1);
+}
 extern "C" int zi_linear_recurrence_tiles_supported(int n_tiles, int max_q_len, int rows, int D) {
   return n_tiles > 0 && rows > 0 && D > 0 && D <= 512 && (max_q_len + rows - 1) / rows <= SCAN_TILES;
 }
@@ -687,41 +749,45 @@ extern "C" int zi_linear_recurrence_tiles_supported(int n_tiles, int max_q_len, 
 // over the requests that bring more than one token; n_single requests bring exactly one).
 extern "C" int zi_linear_recurrence_gated_tiles(float* out, int ldo, const float* q, int ldq, const float* z, int ldz, const float* v,
                                                 int ldv, int splits, long long zstride, const float* f_bias, const float* lower,
-                                                float* state, long long slot_stride, int H, int D, int V, const int* cu_q,
+                                                float* state, long long slot_stride, int T, int H, int D, int V, const int* cu_q,
                                                 const int* state_slots, int n_seqs, const int* tile_seq, const int* tile_q0,
                                                 int n_tiles, int rows, int max_q_len, int n_single, float* workspace,
                                                 cudaStream_t stream) {
-  if (n_seqs <= 0) return 0;
+  if (n_seqs <= 0 || T <= 0) return 0;
   if (H <= 0 || H > 65535 || V <= 0 || !zi_linear_recurrence_tiles_supported(n_tiles, max_q_len, rows, D))
     return zi_refuse("linear_recurrence_gated_tiles: %d tiles of %d tokens, %d key channels", n_tiles, rows, D);
-  if (!lower || splits < 1 || !workspace) return zi_refuse("linear_recurrence_gated_tiles: needs the gate's lower bound and a workspace");
-  const int R = D <= 256 ? 8 : 16;
+  if (!lower || splits != 1 || !workspace) return zi_refuse("linear_recurrence_gated_tiles: needs whole rows, the gate's lower bound and a workspace");
+  constexpr int R = 16;      // more rows per lane than the one-walk form: fewer lanes share a column, so fewer sums between lanes
   int P = 1;
   while (P * R < D) P <<= 1;
   const int CB = LR_WARPS * (32 / P) * NC;
-  const size_t smem = (size_t)2 * (3 * TB * P * R + TB * CB + TB) * sizeof(float);
-  const ForgetGate gate = {lower, f_bias, splits, zstride};
-  RecurrenceTiles tiles = {tile_seq, tile_q0, rows, workspace, workspace + (size_t)n_tiles * H * D * V, 0};
+  const size_t smem = (size_t)2 * (2 * TB * P * R + TB * CB + TB) * sizeof(float);
+  const ForgetGate gate = {};
+  float* qs = workspace;                                  // q and the gates, made once
+  float* gs = qs + (size_t)T * H * D;
+  float* ts = gs + (size_t)T * H * D;
+  RecurrenceTiles tiles = {tile_seq, tile_q0, rows, ts, ts + (size_t)n_tiles * H * D * V, 0};
+  const size_t total = (size_t)T * H * D;
+  zi_launch(make_gates_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, qs, gs, q, ldq, z, ldz, f_bias, lower, H * D, total);
+  int rc = zi_check_launch("linear_recurrence_gated_tiles (gates)");
+  if (rc) return rc;
   auto run = [&](auto kern, int blocks) {
     if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       return zi_refuse("linear_recurrence_gated_tiles: cannot get %zu bytes of shared memory", smem);
-    zi_launch(kern, dim3(blocks, H, (V + CB - 1) / CB), dim3(LR_THREADS), smem, stream, out, ldo, q, ldq, z, ldz, v, ldv,
-              (const float*)nullptr, 0, (const float*)nullptr, 0, 1.0f, state, slot_stride, H, H, D, V, P, cu_q, state_slots, gate, tiles);
+    zi_launch(kern, dim3(blocks, H, (V + CB - 1) / CB), dim3(LR_THREADS), smem, stream, out, ldo, (const float*)qs, H * D,
+              (const float*)nullptr, 0, v, ldv, (const float*)gs, H * D, (const float*)nullptr, 0, 1.0f, state, slot_stride, H, H, D, V, P, cu_q, state_slots, gate, tiles);
     return zi_check_launch("linear_recurrence_gated_tiles");
   };
-  int rc = R == 8 ? run(linear_recurrence_kernel<float, float, 8, false, true, 1>, n_tiles)
-                  : run(linear_recurrence_kernel<float, float, 16, false, true, 1>, n_tiles);
+  rc = run(linear_recurrence_kernel<float, float, R, false, false, 1, true>, n_tiles);
   if (rc) return rc;
   zi_launch(recurrence_scan_kernel, dim3(n_seqs, H, (D * V + SCAN_THREADS - 1) / SCAN_THREADS), dim3(SCAN_THREADS), 0, stream, tiles, n_tiles,
             (const float*)state, slot_stride, H, D, V, cu_q, state_slots);
   rc = zi_check_launch("linear_recurrence_gated_tiles (scan)");
   if (rc) return rc;
-  rc = R == 8 ? run(linear_recurrence_kernel<float, float, 8, false, true, 2>, n_tiles)
-              : run(linear_recurrence_kernel<float, float, 16, false, true, 2>, n_tiles);
+  rc = run(linear_recurrence_kernel<float, float, R, false, false, 2, true>, n_tiles);
   if (rc || n_single <= 0) return rc;
   tiles.only_single = 1;
-  return R == 8 ? run(linear_recurrence_kernel<float, float, 8, false, true, 0>, n_seqs)
-                : run(linear_recurrence_kernel<float, float, 16, false, true, 0>, n_seqs);
+  return run(linear_recurrence_kernel<float, float, R, false, false, 0, true>, n_seqs);
 }
 
 // Whether the one-kernel form for single tokens takes these sizes.

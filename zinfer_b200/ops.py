@@ -1870,7 +1870,7 @@ def linear_recurrence_gated(proj, lower: torch.Tensor, f_bias: Optional[torch.Te
         return out
     out = torch.empty((T, hv), dtype=torch.float32, device=data.device)
     tiles, rows = False, 0
-    if RECURRENCE_TILES and out_dtype == torch.bfloat16 and not step.all_decode:
+    if RECURRENCE_TILES and out_dtype == torch.bfloat16 and splits == 1 and not step.all_decode:
         rows = attention_prefill_tile_rows()
         if step.max_q_len >= 2 * rows:          # and too few blocks in one walk to fill the GPU
             tiles = (step.n_seqs - step.n_dec) * heads * max(1, vdim // 32) < 4 * _sm_count(data.device) \
@@ -1878,10 +1878,10 @@ def linear_recurrence_gated(proj, lower: torch.Tensor, f_bias: Optional[torch.Te
     with _prof.region("linear recurrence (gate writes)",
                       lambda: _nb(data, out) + 2 * step.n_seqs * heads * dim * vdim * 4, 6 * T * heads * dim * vdim):
         if tiles:      # few requests with long portions: tiles of a portion side by side
-            ws = torch.empty((lib().zi_linear_recurrence_tiles_floats(step.n_pf_tiles, heads, dim, vdim),), dtype=torch.float32, device=data.device)
+            ws = torch.empty((lib().zi_linear_recurrence_tiles_floats(T, step.n_pf_tiles, heads, dim, vdim),), dtype=torch.float32, device=data.device)
             _check(lib().zi_linear_recurrence_gated_tiles(
                 _ptr(out), out.stride(0), at(0), W, at(qk), W, at(2 * qk), W, splits, _ll(T * W), _ptr(f_bias), _ptr(lower), _ptr(state),
-                _ll(stride), heads, dim, vdim, _ptr(step.cu_q), _ptr(step.state_slots), step.n_seqs, _ptr(step.pf_tile_seq),
+                _ll(stride), T, heads, dim, vdim, _ptr(step.cu_q), _ptr(step.state_slots), step.n_seqs, _ptr(step.pf_tile_seq),
                 _ptr(step.pf_tile_q0), step.n_pf_tiles, rows, step.max_q_len, step.n_dec, _ptr(ws), _stream()), "linear_recurrence_gated_tiles")
         else:
             _check(lib().zi_linear_recurrence_gated(
