@@ -8,8 +8,8 @@ The design in short.  The embedding is scaled.  A layer norms each sublayer's in
 x <- x + N(mixer(N(x))), x <- x + N(ff(N(x))), where N takes the mean off, divides by the standard deviation and
 multiplies by a weight.  Two mixers.  ``attention``: grouped queries with biases on q, k and v, an RMS norm per
 query and key head, a rotation of each head's first dimensions in pairs (i, i + dims/2), a sliding window beside
-which every block of ``pool`` tokens that lies wholly before the window is seen as ONE key and value (the means of
-the block's keys and values), a softmax whose denominator counts one more than its keys, and values that layers
+which a block of ``pool`` tokens stands in as ONE key and value, the means of its tokens', as soon as its last token has
+left the window, a softmax whose denominator counts one more than its keys, and values that layers
 after the first mix with the first such layer's.  ``hgrn2``: a matrix-valued state per head whose forget gate f
 also decides what is written (1 - f), f bounded below per channel.  The feed-forward is dense and gated.  The
 output head is the embedding table, its logits scaled.

@@ -5,7 +5,7 @@ x <- x + N(ff(N(x))), with layer norms that have a weight and no bias (``norm1``
 embedding is scaled (``embedding.scale``) and its table, unscaled, is the output head, whose logits are multiplied by
 ``logit_scale``.  The mixers: ``attention`` (grouped queries; biases on q, k and v; an RMS norm per query and key head; a
 rotation of the head's first ``rot.dims`` dimensions; an explicit ``scale``; a window of ``mask.size`` tokens beside which
-every block of ``mask.pool`` tokens that lies wholly before the window is seen as one key and value, their means; a softmax
+each block of ``mask.pool`` tokens, once its last token has left the window, stands in as the mean key and value; a softmax
 whose denominator counts one more than its keys; with ``v_mix`` the values are mixed with those of the first such layer)
 and ``hgrn2`` (a matrix-valued state per head whose forget gate decides what is written).  The feed-forward is dense
 and gated with silu, or absent.  config.json gives every size and every constant that may differ between models; the

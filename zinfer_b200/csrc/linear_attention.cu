@@ -7,8 +7,8 @@
 //     u_t = v_t                             plain form
 //     u_t = beta_t (v_t - S^T k_t)          delta rule
 //     S <- S + k_t u_t^T ;  o_t = S^T (q_scale q_t)
-// In a third form (HGRN2: "HGRN2: Gated Linear RNNs with State Expansion", Qin et al., 2024) the forget gate also decides
-// what is written: g = l + (1 - l) sigmoid(z + b) with a lower bound l per channel, k = 1 - g, u_t = v_t, q = silu(raw q).
+// In a third form (HGRN2: "HGRN2: Gated Linear RNNs with State Expansion", Qin et al., 2024) a write is
+// what the decay leaves room for: g = l + (1 - l) sigmoid(z + b) with a lower bound l per channel, k = 1 - g, u_t = v_t, q = silu(raw q).
 // The kernel makes g, k and q from the projections as it stages them.
 // Everything here is 32-bit arithmetic.  A request's tokens of this step are rows cu_q[s] ..
 // cu_q[s+1]-1 of the flat batch and continue the request from slot state_slots[s].  Each column of S

@@ -1875,10 +1875,11 @@ def linear_recurrence_gated(proj, lower: torch.Tensor, f_bias: Optional[torch.Te
         if step.max_q_len >= 2 * rows:          # and too few blocks in one walk to fill the GPU
             tiles = (step.n_seqs - step.n_dec) * heads * max(1, vdim // 32) < 4 * _sm_count(data.device) \
                 and bool(lib().zi_linear_recurrence_tiles_supported(step.n_pf_tiles, step.max_q_len, rows, dim))
+    ws = torch.empty((lib().zi_linear_recurrence_tiles_floats(T, step.n_pf_tiles, heads, dim, vdim),), dtype=torch.float32,
+                     device=data.device) if tiles else None
     with _prof.region("linear recurrence (gate writes)",
                       lambda: _nb(data, out) + 2 * step.n_seqs * heads * dim * vdim * 4, 6 * T * heads * dim * vdim):
         if tiles:      # few requests with long portions: tiles of a portion side by side
-            ws = torch.empty((lib().zi_linear_recurrence_tiles_floats(T, step.n_pf_tiles, heads, dim, vdim),), dtype=torch.float32, device=data.device)
             _check(lib().zi_linear_recurrence_gated_tiles(
                 _ptr(out), out.stride(0), at(0), W, at(qk), W, at(2 * qk), W, splits, _ll(T * W), _ptr(f_bias), _ptr(lower), _ptr(state),
                 _ll(stride), T, heads, dim, vdim, _ptr(step.cu_q), _ptr(step.state_slots), step.n_seqs, _ptr(step.pf_tile_seq),

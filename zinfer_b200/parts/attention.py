@@ -35,10 +35,10 @@ with one gate value per output channel, ``head`` with one per head (tensor ``g``
 
 Options of the "heads" form (one product [q | k | v] with 32-bit results, one kernel that finishes the row head by
 head): ``bias: "qkv"`` adds biases to q, k and v and none to the output; ``value_mix`` {tensor, first} replaces a token's
-value by (1 - lambda) v + lambda v_first, with the scalar lambda in ``tensor`` and v_first the same token's values of the
+value v by v + lambda (v_first - v): lambda is the scalar in ``tensor``, v_first what the same token had in the
 layer whose ``first`` is true (which hands its own on, unmixed, and does not use its lambda); the mixed value is what is
-cached; ``pool`` P, with ``window`` w, lets a query at position i see, beside the window's tokens, ONE key and value for
-each block of P tokens that lies wholly before the window (b P + P - 1 <= i - w): the means of the block's keys and values as
+cached; ``pool`` P, with ``window`` w, adds to what a query at position i sees: once the last token of a block of P
+has left its window ((b + 1) P <= i - w + 1), that block stands in as ONE key and value, the means of the block's keys and values as
 the cache holds them.  Those live in pages of their own, one entry per P tokens, written with the block's last token; the
 tokens' own pages are given back once the window has passed them and their block is complete.  ``sink`` and per-head
 ``qk_norm_eps`` go with this form.

@@ -18,9 +18,9 @@ causal convolution per channel and silu; q and k are made unit vectors per head 
 times dim^(-1/2); beta = sigmoid(W_b h); g = exp(-exp(A_log_h) * softplus(W_a2 (W_a1 h) + dt_bias)) per head and key
 channel; gate sigmoid(W_g2 (W_g1 h)).  The convolutions' last taps-1 inputs are state too.
 
-:class:`HGRN2` (the form whose forget gate decides what is written; "HGRN2: Gated Linear RNNs with State Expansion",
-Qin et al., 2024, is the family): q = silu(W_q h), v = W_v h, f = l + (1 - l) sigmoid(W_f h + b) with a lower bound l
-per head and channel, g = f, k = 1 - f, u = v; no scale on q and no gate on the output.
+:class:`HGRN2` (the form that writes what its decay leaves room for; "HGRN2: Gated Linear RNNs with State Expansion",
+Qin et al., 2024, is the family): q = silu(W_q h), v = W_v h, gate f = sigmoid(z) + l (1 - sigmoid(z)) where z = W_f h + b
+and l is a floor per channel, g = f, k = 1 - f, u = v; no scale on q and no gate on the output.
 
 Decays, beta, unit norms, the recurrence, the state and the head norm are 32-bit; the projections run in the
 model's dtype.  The ranks of the low-rank pairs (a1/a2, g1/g2) are read from the tensors.
