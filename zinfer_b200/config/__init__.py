@@ -5,6 +5,7 @@ from .rogosun import RogosunConfig, rogosun_model_spec
 from .vumezen import VumezenConfig, vumezen_model_spec
 from .sepitar import SepitarConfig, sepitar_model_spec
 from .kesitar import KesitarConfig, kesitar_model_spec
+from .sumozen import SumozenConfig, sumozen_model_spec
 from .registry import (Family, UnknownArchitecture, family_for, load_config, register_family, registered,
                        unregister_family)
 
@@ -26,7 +27,11 @@ register_family(Family(name="Sepitar", model_type="sepitar", config_class=Sepita
 register_family(Family(name="Kesitar", model_type="kesitar", config_class=KesitarConfig,
                        model_spec=kesitar_model_spec), replace=True)
 
+register_family(Family(name="Sumozen", model_type="sumozen", config_class=SumozenConfig,
+                       model_spec=sumozen_model_spec), replace=True)
+
 __all__ = [
+    "SumozenConfig", "sumozen_model_spec",
     "KesitarConfig", "kesitar_model_spec",
     "SepitarConfig", "sepitar_model_spec",
     "VumezenConfig", "vumezen_model_spec",

@@ -33,6 +33,8 @@ int zi_sigmoid_gate(void* out, int ldo, const void* x, int ldx, const void* g, i
                     cudaStream_t stream);
 // act: 0 silu, 1 the tanh form of gelu
 int zi_gated_act(void* out, const void* gu, int dtype, int T, int I, int interleave, int act, cudaStream_t stream);
+int zi_gated_act_rows(void* out, const void* gu, int dtype, int T, int I, int interleave, int act, const float* row_scale,
+                      cudaStream_t stream);
 int zi_gated_act_partials(void* out, int dtype, const float* partials, int splits, long long split_stride, int T, int I,
                           int interleave, int act, cudaStream_t stream);
 int zi_residual_add_partials(float* h, const float* partials, int splits, long long split_stride, long long n,
@@ -209,8 +211,8 @@ int zi_norm_residual(float* h, const void* a, int a_dtype, const float* a_part, 
 // h += sum of up to four updates (whole or split-K partial sums, each with a multiplier) + bias; out1 = norm(h) * w1 and,
 // with w2, out2 = norm(h) * w2 (both norms share the root mean square).  With rows: picked rows, h unchanged.
 int zi_sum_norm_pair(float* h, int n_terms, const void* const* whole, const int* dtypes, const float* const* part,
-                     const int* splits, const long long* zstride, const float* scales, const float* bias, const float* w1,
-                     const float* w2, float eps, void* out1, void* out2, int out_dtype, const int* rows, int n_rows, int H,
+                     const int* splits, const long long* zstride, const float* scales, const float* const* row_scales, const float* bias,
+                     const float* w1, const float* w2, float eps, void* out1, void* out2, int out_dtype, const int* rows, int n_rows, int H,
                      cudaStream_t stream);
 int zi_cast_rows(void* out, int out_dtype, const float* h, long long n, cudaStream_t stream);
 int zi_relu2(void* x, int dtype, long long n, cudaStream_t stream);
@@ -226,7 +228,7 @@ int zi_unit_norm(float* x, int ld, int T, int heads, int d, float eps, float sca
 int zi_sigmoid_rows(float* out, int ldo, const void* x, int ldx, int dtype, int rows, int W, cudaStream_t stream);
 int zi_linear_recurrence(float* out, int ldo, const void* q, int ldq, const void* k, int ldk, int qk_dtype, const void* v,
                          int ldv, int v_dtype, const float* decay, int ldg, const float* beta, int ldb, float q_scale,
-                         float* state, long long slot_stride, int H, int G, int D, int V, int delta, const int* cu_q,
+                         float* state, long long slot_stride, int H, int G, int D, int V, int delta, int head_decay, const int* cu_q,
                          const int* state_slots, int n_seqs, cudaStream_t stream);
 // The form whose forget gate decides what is written: g = l + (1 - l) sigmoid(z + b), k = 1 - g, q = silu(raw q); q, z, v
 // float32 projections, whole (splits 1) or split-K partial sums zstride apart.
@@ -251,13 +253,31 @@ int zi_gated_decode(void* out, int out_dtype, int ldo, const float* q, int ldq, 
                     int H, int D, int V, const float* norm_w, float eps, const int* cu_q, const int* state_slots, int n_seqs,
                     cudaStream_t stream);
 int zi_head_norm_gate(void* out, int out_dtype, int ldo, const float* o, int ldi, const float* w, float eps,
-                      const void* gate, int gate_dtype, int ldgate, int act, int T, int heads, int V, cudaStream_t stream);
+                      const void* gate, int gate_dtype, int ldgate, int gate_splits, long long gate_zstride, int act, int T, int heads,
+                      int V, cudaStream_t stream);
+// (y + skip x) * silu(z), then each of `parts` equal parts of a row by its own root mean square, times w
+int zi_gated_part_norm(void* out, int out_dtype, int ldo, const float* y, int ldy, const float* x, int ldx, const float* skip, int V,
+                       const float* z, int ldz, int splits, long long zstride, const float* w, float eps, int T, int width, int parts,
+                       cudaStream_t stream);
+// Bias, short convolution, activation, unit vectors or rotation, and the place (rows or pages) of a projection's heads, with
+// the convolution's carried inputs and the steps and decays of a recurrence (conv_heads.cu)
+int zi_conv_heads_tile();
+int zi_conv_heads(const float* src, int ld, int splits, long long zstride, int T, int C, int taps, const float* kern,
+                  const float* in_bias, const float* out_bias, int act, float* tail, long long slot_stride, int n_seg,
+                  const int* segs, void* const* seg_out, const float* seg_scale, int out_dtype, float unit_eps, const float* cos_t,
+                  const float* sin_t, int n_table_pos, int rot_dims, int neighbours, const int* positions, const int* slots,
+                  int page_size, int scalars, int n_scalar, const float* a, const float* b, const float* a_log,
+                  const float* dt_bias, float* decay, float* step, const int* tile_seq, const int* tile_q0, int n_tiles,
+                  int tile_rows, const int* cu_q, const int* state_slots, cudaStream_t stream);
 int zi_moe_router_grouped(int* chosen, float* weight, const void* x, int x_dtype, int ldx, const void* w, int w_dtype, int T,
                           int K, int NR, int top, int renormalize, int score_kind, int groups, int keep, float wscale,
                           cudaStream_t stream);
 int zi_moe_route_grouped(int* chosen, float* weight, const float* logits, int T, int NR, int top, int renormalize,
                          int score_kind, int groups, int keep, float wscale, cudaStream_t stream);
 // The same two with a correction [NR] added to the scores for the choice only (null: none).
+int zi_moe_router_grouped_x(int* chosen, float* weight, const void* x, int x_dtype, int ldx, const void* w, int w_dtype,
+                            const float* correction, int T, int K, int NR, int top, int renormalize, int score_kind,
+                            int groups, int keep, float wscale, int extra, float* extra_out, cudaStream_t stream);
 int zi_moe_router_grouped_c(int* chosen, float* weight, const void* x, int x_dtype, int ldx, const void* w, int w_dtype,
                             const float* correction, int T, int K, int NR, int top, int renormalize, int score_kind,
                             int groups, int keep, float wscale, cudaStream_t stream);
@@ -306,7 +326,7 @@ int zi_moe_few_rows(void* out, int out_dtype, int ldo, const void* x, int dtype,
                     const int* row_src, const int* tile_group, const int* n_tiles_dev, int max_tiles, int N, int K,
                     int relu2, cudaStream_t stream);
 int zi_moe_align(const int* chosen, int P, int top, int E, int tile_rows, int cap_tiles, int* row_token, int* row_self,
-                 int* pair_row, int* tile_expert, int* n_tiles, cudaStream_t stream);
+                 int* pair_row, int* tile_expert, int* n_tiles, const float* weight, float* row_weight, cudaStream_t stream);
 int zi_gather_rows(void* out, const void* x, int dtype, const int* row_src, int rows, int width, int ldx,
                    cudaStream_t stream);
 int zi_moe_combine(void* out, const float* y, const void* x, int dtype, const int* chosen, const float* weight,

@@ -406,8 +406,10 @@ __device__ __forceinline__ void gate_up_columns(int i, int I, int interleave, in
   }
 }
 
-template <typename T, int ACT>
-__global__ void swiglu_kernel(T* __restrict__ out, const T* __restrict__ gu, int I, size_t total, int interleave) {
+// ROWS: gate and up of row t are multiplied by row_scale[t] first (a mixture's weight on its expert's input).
+template <typename T, int ACT, bool ROWS = false>
+__global__ void swiglu_kernel(T* __restrict__ out, const T* __restrict__ gu, int I, size_t total, int interleave,
+                              const float* __restrict__ row_scale) {
   pdl_launch_dependents();
   pdl_wait();
   size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -416,8 +418,9 @@ __global__ void swiglu_kernel(T* __restrict__ out, const T* __restrict__ gu, int
   const int i = (int)(idx - t * I);
   int gc, uc;
   gate_up_columns(i, I, interleave, gc, uc);
-  const float g = to_f32(gu[t * 2 * I + gc]);
-  const float u = to_f32(gu[t * 2 * I + uc]);
+  const float rs = ROWS ? row_scale[t] : 1.f;
+  const float g = to_f32(gu[t * 2 * I + gc]) * rs;
+  const float u = to_f32(gu[t * 2 * I + uc]) * rs;
   out[idx] = from_f32<T>(gated<ACT>(g, u));
 }
 
@@ -457,9 +460,9 @@ __global__ void swiglu_partials_kernel(T* __restrict__ out, const float* __restr
 }
 
 // Eight elements per thread (16-byte loads of bfloat16, two of float); needs I % 8 == 0.
-template <typename T, int ACT>
+template <typename T, int ACT, bool ROWS = false>
 __global__ void swiglu_vec_kernel(T* __restrict__ out, const T* __restrict__ gu, int I, size_t total_vec,
-                                  int interleave) {
+                                  int interleave, const float* __restrict__ row_scale) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -474,7 +477,12 @@ __global__ void swiglu_vec_kernel(T* __restrict__ out, const T* __restrict__ gu,
   T* o = out + t * I + i;
 #pragma unroll
   for (int k = 0; k < 8; k += 4) {
-    const float4 gv = Vec4<T>::load(g + k), uv = Vec4<T>::load(u + k);
+    float4 gv = Vec4<T>::load(g + k), uv = Vec4<T>::load(u + k);
+    if (ROWS) {
+      const float rs = row_scale[t];
+      gv = make_float4(gv.x * rs, gv.y * rs, gv.z * rs, gv.w * rs);
+      uv = make_float4(uv.x * rs, uv.y * rs, uv.z * rs, uv.w * rs);
+    }
     Vec4<T>::store(o + k, make_float4(gated<ACT>(gv.x, uv.x), gated<ACT>(gv.y, uv.y), gated<ACT>(gv.z, uv.z),
                                       gated<ACT>(gv.w, uv.w)));
   }
@@ -596,6 +604,12 @@ extern "C" int zi_gated_act_partials(void* out, int dtype, const float* partials
 
 extern "C" int zi_gated_act(void* out, const void* gu, int dtype, int T, int I, int interleave, int act,
                             cudaStream_t stream) {
+  return zi_gated_act_rows(out, gu, dtype, T, I, interleave, act, nullptr, stream);
+}
+
+// act(s_t g) * (s_t u) with a multiplier per row (null: none).
+extern "C" int zi_gated_act_rows(void* out, const void* gu, int dtype, int T, int I, int interleave, int act,
+                                 const float* row_scale, cudaStream_t stream) {
   if (interleave && (interleave % 8 || I % interleave)) return zi_refuse("swiglu: interleave %d does not fit I = %d", interleave, I);
   const size_t total = (size_t)T * I;
   if (total == 0) return 0;
@@ -604,11 +618,13 @@ extern "C" int zi_gated_act(void* out, const void* gu, int dtype, int T, int I, 
     const size_t total_vec = total / 8;
     const unsigned blocks = (unsigned)((total_vec + threads - 1) / threads);
     ZI_DISPATCH_ACT(act, ACT, ZI_DISPATCH_DTYPE(dtype, TT,
-                      zi_launch(swiglu_vec_kernel<TT, ACT>, dim3(blocks), dim3(threads), 0, stream, (TT*)out, (const TT*)gu, I, total_vec, interleave)));
+                      zi_launch(row_scale ? swiglu_vec_kernel<TT, ACT, true> : swiglu_vec_kernel<TT, ACT>, dim3(blocks), dim3(threads), 0, stream,
+                                (TT*)out, (const TT*)gu, I, total_vec, interleave, row_scale)));
     return zi_check_launch("swiglu");
   }
   const unsigned blocks = (unsigned)((total + threads - 1) / threads);
-  ZI_DISPATCH_ACT(act, ACT, ZI_DISPATCH_DTYPE(dtype, TT, zi_launch(swiglu_kernel<TT, ACT>, dim3(blocks), dim3(threads), 0, stream, (TT*)out, (const TT*)gu, I, total, interleave)));
+  ZI_DISPATCH_ACT(act, ACT, ZI_DISPATCH_DTYPE(dtype, TT, zi_launch(row_scale ? swiglu_kernel<TT, ACT, true> : swiglu_kernel<TT, ACT>, dim3(blocks), dim3(threads), 0, stream,
+                                                                    (TT*)out, (const TT*)gu, I, total, interleave, row_scale)));
   return zi_check_launch("swiglu");
 }
 
@@ -1060,11 +1076,14 @@ struct SumTerm {
   int dtype, splits;
   long long zstride;
   float scale;
+  const float* row_scale;    // [T], or null: the term of row t is multiplied by row_scale[t] as well
 };
 struct SumTerms {
   SumTerm t[4];
   int n;
 };
+
+__device__ __forceinline__ float sum_term_scale(const SumTerm& t, int row) { return t.row_scale ? t.scale * t.row_scale[row] : t.scale; }
 
 __device__ __forceinline__ float sum_term_at(const SumTerm& t, size_t at) {
   if (t.part) return operand_at((const float*)nullptr, t.part, t.splits, (size_t)t.zstride, at);
@@ -1080,8 +1099,11 @@ sum_norm_pair_kernel(float* __restrict__ h, SumTerms terms, const float* __restr
   pdl_wait();
   __shared__ float scratch[33];
   extern __shared__ float ys[];
-  const int r = blockIdx.x;
-  const size_t row = (size_t)(rows ? rows[r] : r) * H;
+  const int r = blockIdx.x, row_at = rows ? rows[r] : r;
+  const size_t row = (size_t)row_at * H;
+  float scale[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) scale[i] = i < terms.n ? sum_term_scale(terms.t[i], row_at) : 0.f;
   float ss = 0.f;
   for (int c0 = threadIdx.x; c0 < H; c0 += 4 * blockDim.x) {
     float v[4];
@@ -1091,7 +1113,9 @@ sum_norm_pair_kernel(float* __restrict__ h, SumTerms terms, const float* __restr
       v[u] = 0.f;
       if (c < H) {
         v[u] = h[row + c];
-        for (int i = 0; i < terms.n; ++i) v[u] = fmaf(terms.t[i].scale, sum_term_at(terms.t[i], row + c), v[u]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if (i < terms.n) v[u] = fmaf(scale[i], sum_term_at(terms.t[i], row + c), v[u]);
         if (bias) v[u] += bias[c];
       }
     }
@@ -1127,8 +1151,11 @@ sum_norm_pair_vec_kernel(float* __restrict__ h, SumTerms terms, const float* __r
   pdl_wait();
   __shared__ float scratch[33];
   constexpr int MAXV = 8;                 // 4-wide pieces per thread
-  const int r = blockIdx.x;
-  const size_t row = (size_t)(rows ? rows[r] : r) * H;
+  const int r = blockIdx.x, row_at = rows ? rows[r] : r;
+  const size_t row = (size_t)row_at * H;
+  float scale[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) scale[i] = i < terms.n ? sum_term_scale(terms.t[i], row_at) : 0.f;
   const bool writes_h = !rows && (terms.n > 0 || bias);
   float4 v[MAXV];
   float ss = 0.f;
@@ -1138,12 +1165,14 @@ sum_norm_pair_vec_kernel(float* __restrict__ h, SumTerms terms, const float* __r
     v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (c < H) {
       v[i] = Vec4<float>::load(h + row + c);
-      for (int t = 0; t < terms.n; ++t) {
+#pragma unroll
+      for (int t = 0; t < 4; ++t) {
+        if (t >= terms.n) break;
         const SumTerm& term = terms.t[t];
         const float4 u = term.dtype == ZI_BF16 ? Vec4<__nv_bfloat16>::load((const __nv_bfloat16*)term.whole + row + c)
                                                : Vec4<float>::load((const float*)term.whole + row + c);
-        v[i] = make_float4(fmaf(term.scale, u.x, v[i].x), fmaf(term.scale, u.y, v[i].y), fmaf(term.scale, u.z, v[i].z),
-                           fmaf(term.scale, u.w, v[i].w));
+        v[i] = make_float4(fmaf(scale[t], u.x, v[i].x), fmaf(scale[t], u.y, v[i].y), fmaf(scale[t], u.z, v[i].z),
+                           fmaf(scale[t], u.w, v[i].w));
       }
       if (bias) {
         const float4 bv = Vec4<float>::load(bias + c);
@@ -1173,8 +1202,8 @@ sum_norm_pair_vec_kernel(float* __restrict__ h, SumTerms terms, const float* __r
 
 // terms: n_terms entries of (whole, dtype, part, splits, zstride, scale), given as parallel arrays on the host.
 extern "C" int zi_sum_norm_pair(float* h, int n_terms, const void* const* whole, const int* dtypes, const float* const* part,
-                                const int* splits, const long long* zstride, const float* scales, const float* bias,
-                                const float* w1, const float* w2, float eps, void* out1, void* out2, int out_dtype,
+                                const int* splits, const long long* zstride, const float* scales,
+                                const float* const* row_scales, const float* bias, const float* w1, const float* w2, float eps, void* out1, void* out2, int out_dtype,
                                 const int* rows, int n_rows, int H, cudaStream_t stream) {
   if (n_rows <= 0 || H <= 0) return 0;
   if (n_terms < 0 || n_terms > 4) return zi_refuse("sum_norm_pair: %d updates (at most 4)", n_terms);
@@ -1184,7 +1213,7 @@ extern "C" int zi_sum_norm_pair(float* h, int n_terms, const void* const* whole,
   for (int i = 0; i < n_terms; ++i) {
     if ((whole[i] == nullptr) == (part[i] == nullptr)) return zi_refuse("sum_norm_pair: give update %d either whole or as partial sums", i);
     if (whole[i] && dtypes[i] != ZI_F32 && dtypes[i] != ZI_BF16) return zi_refuse("sum_norm_pair: unknown dtype tag %d", dtypes[i]);
-    terms.t[i] = SumTerm{whole[i], part[i], dtypes[i], splits[i], zstride[i], scales[i]};
+    terms.t[i] = SumTerm{whole[i], part[i], dtypes[i], splits[i], zstride[i], scales[i], row_scales[i]};
   }
   const size_t smem = (size_t)H * sizeof(float);
   if (smem > 200 * 1024) return zi_refuse("sum_norm_pair: rows of %d values are more than this kernel holds", H);

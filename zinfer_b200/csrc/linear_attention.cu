@@ -4,7 +4,7 @@
 //
 // The recurrence, per head, with S [D key channels, V value channels] carried per request:
 //     S <- diag(g_t) S                      the decay acts on the rows that belong to key channels
-//     u_t = v_t                             plain form
+//     u_t = v_t, or beta_t v_t              plain form, without or with a step size per token and head
 //     u_t = beta_t (v_t - S^T k_t)          delta rule
 //     S <- S + k_t u_t^T ;  o_t = S^T (q_scale q_t)
 // In a third form (HGRN2: "HGRN2: Gated Linear RNNs with State Expansion", Qin et al., 2024) a write is
@@ -164,7 +164,7 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
                          int ldk, const TV* __restrict__ v, int ldv, const float* __restrict__ decay, int ldg,
                          const float* __restrict__ beta, int ldb, float q_scale, float* __restrict__ state,
                          long long slot_stride, int H, int G, int D, int V, int P, const int* __restrict__ cu_q,
-                         const int* __restrict__ state_slots, const ForgetGate fgate, const RecurrenceTiles tiles) {
+                         const int* __restrict__ state_slots, const ForgetGate fgate, const RecurrenceTiles tiles, int gh, int gi) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
@@ -220,7 +220,7 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
         const size_t row = (size_t)(tok0 + t0 + tt);
         if (CHUNK != 1) fq[u] = q[row * ldq + (size_t)kvh * D + i];
         if (!MADE) fk[u] = k[row * ldk + (size_t)kvh * D + i];
-        if (!GATE) fg[u] = decay[row * ldg + (size_t)h * D + i];
+        if (!GATE) fg[u] = decay[row * ldg + (size_t)h * gh + i * gi];
       } else {
         fq[u] = from_f32<TQ>(0.f);
         fk[u] = from_f32<TQ>(0.f);
@@ -233,7 +233,7 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
       const int c = j0 + (e & (CB - 1));
       fv[u] = (e < (nt << lgCB) && c < V) ? v[(size_t)(tok0 + t0 + (e >> lgCB)) * ldv + (size_t)h * V + c] : from_f32<TV>(0.f);
     }
-    if (DELTA && tid < nt) fb = beta[(size_t)(tok0 + t0 + tid) * ldb + h];
+    if (!GATE && !MADE && beta && tid < nt) fb = beta[(size_t)(tok0 + t0 + tid) * ldb + h];
     if constexpr (GATE) {
       for (int z = 1; z < fgate.splits; ++z) {
         const size_t zo = (size_t)z * fgate.zstride;
@@ -293,7 +293,7 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
       const bool in = i < D;
       stage(buf, (e & ~(DP - 1)) + place(i), i, in ? whole(q + row * ldq + (size_t)kvh * D + i) : 0.f,
             in && !MADE ? whole(k + row * ldk + (size_t)kvh * D + i) : 0.f,
-            in && !GATE ? decay[row * ldg + (size_t)h * D + i] : (MADE ? 1.f : 0.f));
+            in && !GATE ? decay[row * ldg + (size_t)h * gh + i * gi] : (MADE ? 1.f : 0.f));
     }
 #pragma unroll
     for (int u = 0; u < NPV; ++u) {
@@ -416,7 +416,7 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
 #pragma unroll
       for (int c = 0; c < NC; ++c) {
         const float vj = vs[tt * CB + cb + c];
-        const float u = DELTA ? bs[tt] * (vj - a[c]) : vj;
+        const float u = bs[tt] * (DELTA ? vj - a[c] : vj);
 #pragma unroll
         for (int r = 0; r < R; ++r) Sr[c][r] = fmaf(kr[r], u, Sr[c][r]);
         if (p == 0 && col + c < V) out[(size_t)(tok0 + t0 + tt) * ldo + (size_t)h * V + col + c] = fmaf(u, kq, b[c]);
@@ -603,11 +603,11 @@ gated_decode_kernel(TO* __restrict__ out, int ldo, const float* __restrict__ q, 
 
 // ----------------------------------------------------------------------- gated per-head norm
 // out[t, head, :] = o / sqrt(mean(o^2) + eps) * w * act(gate[t, head, :]); act: 0 silu, 1 sigmoid, 2 no gate.
-// One warp per (token, head).
+// The gate may come as split-K partial sums (float32, gz apart), added in order.  One warp per (token, head).
 template <typename TG, typename TO>
 __global__ void head_norm_gate_kernel(TO* __restrict__ out, int ldo, const float* __restrict__ o, int ldi,
                                       const float* __restrict__ w, float eps, const TG* __restrict__ gate, int ldgate,
-                                      int act, int T, int heads, int V) {
+                                      int gsplits, long long gz, int act, int T, int heads, int V) {
   pdl_launch_dependents();
   pdl_wait();
   const int wi = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -619,7 +619,12 @@ __global__ void head_norm_gate_kernel(TO* __restrict__ out, int ldo, const float
   ss = warp_sum(ss);
   const float inv = 1.0f / sqrtf(ss / (float)V + eps);
   for (int i = lane; i < V; i += 32) {
-    const float g = act == 2 ? 1.f : to_f32(gate[(size_t)t * ldgate + (size_t)h * V + i]);
+    float g = 1.f;
+    if (act != 2) {
+      const TG* pg = gate + (size_t)t * ldgate + (size_t)h * V + i;
+      g = to_f32(*pg);
+      for (int z = 1; z < gsplits; ++z) g += to_f32(pg[(size_t)z * gz]);
+    }
     const float a = act == 2 ? 1.f : (act == 0 ? g * sigmoid_f32(g) : sigmoid_f32(g));
     out[(size_t)t * ldo + (size_t)h * V + i] = from_f32<TO>(p[i] * inv * w[i] * a);
   }
@@ -675,9 +680,10 @@ extern "C" int zi_sigmoid_rows(float* out, int ldo, const void* x, int ldx, int 
 extern "C" int zi_linear_recurrence(float* out, int ldo, const void* q, int ldq, const void* k, int ldk, int qk_dtype,
                                     const void* v, int ldv, int v_dtype, const float* decay, int ldg, const float* beta,
                                     int ldb, float q_scale, float* state, long long slot_stride, int H, int G, int D,
-                                    int V, int delta, const int* cu_q, const int* state_slots, int n_seqs,
+                                    int V, int delta, int head_decay, const int* cu_q, const int* state_slots, int n_seqs,
                                     cudaStream_t stream) {
   if (n_seqs <= 0) return 0;
+  const int gh = head_decay ? 1 : D, gi = head_decay ? 0 : 1;      // one decay per head, or one per key channel
   if (H <= 0 || G <= 0 || H % G) return zi_refuse("linear_recurrence: %d heads do not divide into %d key heads", H, G);
   if (D <= 0 || D > 512 || V <= 0) return zi_refuse("linear_recurrence: %d key channels (1..512), %d value channels", D, V);
   if (delta && !beta) return zi_refuse("linear_recurrence: the delta rule needs beta");
@@ -697,7 +703,7 @@ extern "C" int zi_linear_recurrence(float* out, int ldo, const void* q, int ldq,
     }                                                                                                                  \
     zi_launch(kern, dim3(grid), dim3(block), smem, stream, out, ldo, (const TQ*)q, ldq, (const TQ*)k, ldk, (const TV*)v, \
               ldv, decay, ldg, beta, ldb, q_scale, state, slot_stride, H, G, D, V, P, cu_q, state_slots, ForgetGate{}, \
-              RecurrenceTiles{});                                                                                      \
+              RecurrenceTiles{}, gh, gi);                                                                              \
   } while (0)
 #define ZI_LR_R(TQ, TV)                                          \
   do {                                                           \
@@ -733,7 +739,7 @@ extern "C" int zi_linear_recurrence_gated(float* out, int ldo, const float* q, i
   if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
     return zi_refuse("linear_recurrence_gated: cannot get %zu bytes of shared memory", smem);
   zi_launch(kern, grid, block, smem, stream, out, ldo, q, ldq, z, ldz, v, ldv, (const float*)nullptr, 0, (const float*)nullptr, 0, 1.0f,
-            state, slot_stride, H, H, D, V, P, cu_q, state_slots, gate, RecurrenceTiles{});
+            state, slot_stride, H, H, D, V, P, cu_q, state_slots, gate, RecurrenceTiles{}, D, 1);
   return zi_check_launch("linear_recurrence_gated");
 }
 
@@ -775,7 +781,7 @@ extern "C" int zi_linear_recurrence_gated_tiles(float* out, int ldo, const float
     if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       return zi_refuse("linear_recurrence_gated_tiles: cannot get %zu bytes of shared memory", smem);
     zi_launch(kern, dim3(blocks, H, (V + CB - 1) / CB), dim3(LR_THREADS), smem, stream, out, ldo, (const float*)qs, H * D,
-              (const float*)nullptr, 0, v, ldv, (const float*)gs, H * D, (const float*)nullptr, 0, 1.0f, state, slot_stride, H, H, D, V, P, cu_q, state_slots, gate, tiles);
+              (const float*)nullptr, 0, v, ldv, (const float*)gs, H * D, (const float*)nullptr, 0, 1.0f, state, slot_stride, H, H, D, V, P, cu_q, state_slots, gate, tiles, D, 1);
     return zi_check_launch("linear_recurrence_gated_tiles");
   };
   rc = run(linear_recurrence_kernel<float, float, R, false, false, 1, true>, n_tiles);
@@ -816,16 +822,67 @@ extern "C" int zi_gated_decode(void* out, int out_dtype, int ldo, const float* q
 }
 
 extern "C" int zi_head_norm_gate(void* out, int out_dtype, int ldo, const float* o, int ldi, const float* w, float eps,
-                                 const void* gate, int gate_dtype, int ldgate, int act, int T, int heads, int V,
-                                 cudaStream_t stream) {
+                                 const void* gate, int gate_dtype, int ldgate, int gate_splits, long long gate_zstride, int act,
+                                 int T, int heads, int V, cudaStream_t stream) {
   if (T <= 0 || heads <= 0) return 0;
   if (act < 0 || act > 2 || (act != 2 && !gate)) return zi_refuse("head_norm_gate: unknown gate %d", act);
   const int warps = 4;
   dim3 grid((unsigned)(((size_t)T * heads + warps - 1) / warps));
   ZI_DISPATCH_DTYPE(gate_dtype, TG, ZI_DISPATCH_DTYPE(out_dtype, TO,
       zi_launch(head_norm_gate_kernel<TG, TO>, dim3(grid), dim3(warps * 32), 0, stream, (TO*)out, ldo, o, ldi, w, eps,
-                (const TG*)gate, ldgate, act, T, heads, V)));
+                (const TG*)gate, ldgate, gate_splits, gate_zstride, act, T, heads, V)));
   return zi_check_launch("head_norm_gate");
+}
+
+// ------------------------------------------------------------------ gated norm of a row's parts
+// y' = (y + skip[c / V] * x) * silu(z); each of `parts` equal parts of the row is divided by its own root mean square and
+// multiplied by w.  skip and x may be absent; z may come as split-K partial sums.  One block per (token, part).
+namespace {
+template <typename TO>
+__global__ void __launch_bounds__(512)
+gated_part_norm_kernel(TO* __restrict__ out, int ldo, const float* __restrict__ y, int ldy, const float* __restrict__ x, int ldx,
+                       const float* __restrict__ skip, int V, const float* __restrict__ z, int ldz, int splits, long long zstride,
+                       const float* __restrict__ w, float eps, int n) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float part[];
+  __shared__ float scratch[33];
+  const size_t t = blockIdx.x;
+  const int c0 = blockIdx.y * n;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const int c = c0 + i;
+    float v = y[t * ldy + c];
+    if (skip) v = fmaf(skip[c / V], x[t * ldx + c], v);
+    float g = z[t * ldz + c];
+    for (int k = 1; k < splits; ++k) g += z[(size_t)k * zstride + t * ldz + c];
+    v *= g * sigmoid_f32(g);
+    part[i] = v;
+    ss = fmaf(v, v, ss);
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
+  for (int i = threadIdx.x; i < n; i += blockDim.x) out[t * ldo + c0 + i] = from_f32<TO>(part[i] * inv * w[c0 + i]);
+}
+}  // namespace
+
+extern "C" int zi_gated_part_norm(void* out, int out_dtype, int ldo, const float* y, int ldy, const float* x, int ldx, const float* skip,
+                                  int V, const float* z, int ldz, int splits, long long zstride, const float* w, float eps, int T,
+                                  int width, int parts, cudaStream_t stream) {
+  if (T <= 0 || width <= 0) return 0;
+  if (parts <= 0 || width % parts || parts > 65535) return zi_refuse("gated_part_norm: %d columns in %d parts", width, parts);
+  if (skip && (!x || V <= 0)) return zi_refuse("gated_part_norm: a skip needs what it multiplies");
+  if (!z || splits < 1) return zi_refuse("gated_part_norm: needs its gate");
+  const int n = width / parts;
+  const size_t smem = (size_t)n * sizeof(float);
+  if (smem > 200 * 1024) return zi_refuse("gated_part_norm: parts of %d values are more than this kernel holds", n);
+  const int threads = n >= 1024 ? 512 : (n >= 256 ? 256 : 128);
+  ZI_DISPATCH_DTYPE(out_dtype, TO, {
+    auto kern = gated_part_norm_kernel<TO>;
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+      return zi_refuse("gated_part_norm: cannot get %zu bytes of shared memory", smem);
+    zi_launch(kern, dim3(T, parts), dim3(threads), smem, stream, (TO*)out, ldo, y, ldy, x, ldx, skip, V, z, ldz, splits, zstride, w, eps, n);
+  });
+  return zi_check_launch("gated_part_norm");
 }
 
 ZI_TRACE_SETTER(linear_attention)

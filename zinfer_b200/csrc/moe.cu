@@ -255,23 +255,26 @@ moe_route_kernel(int* __restrict__ chosen, float* __restrict__ weight, const flo
 // each (23 -> 15 us for 8 tokens, 32 outputs, rows of 4,096).  32-bit multiply-adds whatever the operands' types.
 // MODE 1: the choice among groups of outputs (route_token_grouped) instead of the softmax with a correction (0);
 // MODE 2: the choice by the logits plus a bias with a softmax over the chosen (route_token_top_logits).
+// extra: rows of w behind the NR outputs that are not chosen from; sigmoid of their logits goes to extra_out [T][extra]
+// (a gate per token that shares the router's pass over the token).
 template <typename TX, typename TW, int MODE, int TOK, bool WIDE>
 __global__ void __launch_bounds__(WIDE ? 1024 : 256)
 moe_router_kernel(int* __restrict__ chosen, float* __restrict__ weight, const TX* __restrict__ x, int ldx,
                   const TW* __restrict__ w, const float* __restrict__ correction, int T, int K, int NR, int top,
-                  int renormalize, int score_kind, int groups, int keep, float wscale) {
+                  int renormalize, int score_kind, int groups, int keep, float wscale, int extra, float* __restrict__ extra_out) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float sm[];
   float* xs = sm;                        // [TOK][K]
-  float* zs = sm + (size_t)TOK * K;      // per token: [NR] logits, then [NR] scores, [NR] picks, [NR] group scores
+  const int NL = NR + extra;             // logits
+  float* zs = sm + (size_t)TOK * K;      // per token: [NL] logits, then [NR] scores, [NR] picks, [NR] group scores
   const int t0 = blockIdx.x * TOK, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   const int n_tok = min(TOK, T - t0);
   for (int i = 0; i < n_tok; ++i)
     for (int k = threadIdx.x; k < K; k += blockDim.x) xs[(size_t)i * K + k] = to_f32(x[(size_t)(t0 + i) * ldx + k]);
   __syncthreads();
   const bool vec = K % 4 == 0 && ((uintptr_t)w & 15) == 0;      // 8- or 16-byte pieces of a weight row
-  for (int j = warp; j < NR; j += warps) {
+  for (int j = warp; j < NL; j += warps) {
     const TW* wr = w + (size_t)j * K;
     float acc[TOK];
     if (vec) {
@@ -321,20 +324,22 @@ moe_router_kernel(int* __restrict__ chosen, float* __restrict__ weight, const TX
     for (int i = 0; i < TOK; ++i) {
       if (i < n_tok) {        // uniform in the block
         const float v = warp_sum(acc[i]);
-        if (lane == 0) zs[(size_t)i * 4 * NR + j] = v;
+        if (lane == 0) zs[(size_t)i * (3 * NR + NL) + j] = v;
       }
     }
   }
   __syncthreads();
   for (int i = warp; i < n_tok; i += warps) {
-    float* z = zs + (size_t)i * 4 * NR;
+    float* z = zs + (size_t)i * (3 * NR + NL);
+    float* s = z + NL;
+    for (int j = lane; j < extra; j += 32) extra_out[(size_t)(t0 + i) * extra + j] = 1.0f / (1.0f + expf(-z[NR + j]));
     if (MODE == 2)
-      route_token_top_logits(chosen, weight, z, z + NR, correction, t0 + i, NR, top, lane);     // `correction` carries the bias
+      route_token_top_logits(chosen, weight, z, s, correction, t0 + i, NR, top, lane);     // `correction` carries the bias
     else if (MODE == 1)
-      route_token_grouped(chosen, weight, z, z + NR, z + 2 * NR, z + 3 * NR, t0 + i, NR, top, renormalize, score_kind, groups,
+      route_token_grouped(chosen, weight, z, s, s + NR, s + 2 * NR, t0 + i, NR, top, renormalize, score_kind, groups,
                           keep, wscale, lane, correction);
     else
-      route_token(chosen, weight, z, z + NR, z + 2 * NR, correction, t0 + i, NR, top, renormalize, lane);
+      route_token(chosen, weight, z, s, s + NR, correction, t0 + i, NR, top, renormalize, lane);
   }
 }
 
@@ -504,13 +509,14 @@ moe_few_rows_kernel(TO* __restrict__ out, int ldo, const TX* __restrict__ x, int
 //   row_token[r]  token whose input row r multiplies (-1: padding)
 //   row_self[r]   r where the row is in use, else -1
 //   pair_row[p]   row of pair p (-1: an identity expert)
+//   row_weight[r] the pair's weight (0: padding), if asked for: the rows whose input is weighted
 //   tile_expert[i], *n_tiles     the arrays have cap_tiles tiles (at least P / tile_rows + E); rows and tiles
 //                                beyond the ones in use are marked -1 and expert 0
 __global__ void __launch_bounds__(1024)
 moe_align_kernel(const int* __restrict__ chosen, int P, int top, int E, int tile_rows, int cap_tiles,
                  int* __restrict__ row_token,
                  int* __restrict__ row_self, int* __restrict__ pair_row, int* __restrict__ tile_expert,
-                 int* __restrict__ n_tiles) {
+                 int* __restrict__ n_tiles, const float* __restrict__ weight, float* __restrict__ row_weight) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ int si[];
@@ -539,7 +545,10 @@ moe_align_kernel(const int* __restrict__ chosen, int P, int top, int E, int tile
   }
   __syncthreads();
   const int rows = cap_tiles * tile_rows;      // all rows the arrays have: a product may walk every tile
-  for (int r = threadIdx.x; r < rows; r += blockDim.x) row_token[r] = row_self[r] = -1;
+  for (int r = threadIdx.x; r < rows; r += blockDim.x) {
+    row_token[r] = row_self[r] = -1;
+    if (row_weight) row_weight[r] = 0.f;
+  }
   __syncthreads();
   for (int p = threadIdx.x; p < P; p += blockDim.x) {
     const int e = chosen[p];
@@ -548,6 +557,7 @@ moe_align_kernel(const int* __restrict__ chosen, int P, int top, int E, int tile
       r = off[e] + atomicAdd(&cursor[e], 1);
       row_token[r] = p / top;
       row_self[r] = r;
+      if (row_weight) row_weight[r] = weight[p];
     }
     pair_row[p] = r;
   }
@@ -564,7 +574,8 @@ __global__ void gather_rows_kernel(T* __restrict__ out, const T* __restrict__ x,
     out[(size_t)r * width + c] = src >= 0 ? x[(size_t)src * ldx + c] : from_f32<T>(0.f);
 }
 
-// out[t] = sum_k weight[t,k] * (expert output of pair (t,k), or x[t] for an identity expert), k ascending.
+// out[t] = sum_k weight[t,k] * (expert output of pair (t,k), or x[t] for an identity expert), k ascending; without weights
+// (the experts' inputs were weighted) the plain sum.
 template <typename T>
 __global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict__ y, const T* __restrict__ x,
                                    const int* __restrict__ chosen, const float* __restrict__ weight,
@@ -579,7 +590,7 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict_
     const size_t p = (size_t)t * top + k;
     const int e = chosen[p];
     const float v = e < E ? y[(size_t)pair_row[p] * H + c] : to_f32(x[(size_t)t * H + c]);
-    acc = fmaf(weight[p], v, acc);
+    acc = fmaf(weight ? weight[p] : 1.f, v, acc);
   }
   out[(size_t)t * H + c] = from_f32<T>(acc);
 }
@@ -620,7 +631,8 @@ extern "C" int zi_moe_route_grouped_c(int* chosen, float* weight, const float* l
 
 static int launch_moe_router(int* chosen, float* weight, const void* x, int x_dtype, int ldx, const void* w, int w_dtype,
                              const float* correction, int T, int K, int NR, int top, int renormalize, int mode,
-                             int score_kind, int groups, int keep, float wscale, cudaStream_t stream) {
+                             int score_kind, int groups, int keep, float wscale, cudaStream_t stream, int extra = 0,
+                             float* extra_out = nullptr) {
   const bool grouped = mode == 1;
   if (T <= 0) return 0;
   if (top <= 0 || top > NR) return zi_refuse("moe_router: %d of %d outputs cannot be chosen", top, NR);
@@ -633,10 +645,10 @@ static int launch_moe_router(int* chosen, float* weight, const void* x, int x_dt
   // once per token; measured on 2,048 tokens of 4,096 values and 32 outputs: 88 us with one token per block, 84 with two,
   // 103 with four, 144 with eight, whose rows leave room for one block per SM only: not kept.)
   constexpr int tok = 1;
-  const size_t smem = (size_t)tok * (K + 4 * NR) * sizeof(float);
+  const size_t smem = (size_t)tok * (K + 4 * NR + extra) * sizeof(float);
   if (smem > 200 * 1024) return zi_refuse("moe_router: rows of %d values and %d outputs are more than this kernel holds", K, NR);
   // few tokens: a warp per output, up to 32 warps, since the few blocks are bound by the latency of a warp's walk along a row
-  const int threads = T > 32 ? 256 : std::min(1024, std::max(256, 32 * NR));
+  const int threads = T > 32 ? 256 : std::min(1024, std::max(256, 32 * (NR + extra)));
   using bf = __nv_bfloat16;
 #define ZI_ROUTER_T(TX, TW, GG, WIDE)                                                                              \
   do {                                                                                                             \
@@ -644,7 +656,7 @@ static int launch_moe_router(int* chosen, float* weight, const void* x, int x_dt
     if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) \
       return zi_refuse("moe_router: cannot get %zu bytes of shared memory", smem);                                 \
     zi_launch(kern, dim3(T), dim3(threads), smem, stream, chosen, weight, (const TX*)x, ldx, (const TW*)w, correction, T, K, \
-              NR, top, renormalize, score_kind, groups, keep, wscale);                                             \
+              NR, top, renormalize, score_kind, groups, keep, wscale, extra, extra_out);                           \
   } while (0)
 #define ZI_ROUTER_G(TX, TW, GG) do { if (threads > 256) ZI_ROUTER_T(TX, TW, GG, true); else ZI_ROUTER_T(TX, TW, GG, false); } while (0)
 #define ZI_ROUTER(TX, TW) do { if (mode == 2) ZI_ROUTER_G(TX, TW, 2); else if (grouped) ZI_ROUTER_G(TX, TW, 1); else ZI_ROUTER_G(TX, TW, 0); } while (0)
@@ -679,6 +691,16 @@ extern "C" int zi_moe_router_grouped_c(int* chosen, float* weight, const void* x
                                        int score_kind, int groups, int keep, float wscale, cudaStream_t stream) {
   return launch_moe_router(chosen, weight, x, x_dtype, ldx, w, w_dtype, correction, T, K, NR, top, renormalize, 1, score_kind,
                            groups, keep, wscale, stream);
+}
+
+// The same with `extra` rows of w behind the NR outputs whose logits' sigmoids go to extra_out [T][extra].
+extern "C" int zi_moe_router_grouped_x(int* chosen, float* weight, const void* x, int x_dtype, int ldx, const void* w,
+                                       int w_dtype, const float* correction, int T, int K, int NR, int top, int renormalize,
+                                       int score_kind, int groups, int keep, float wscale, int extra, float* extra_out,
+                                       cudaStream_t stream) {
+  if (extra < 0 || (extra > 0 && !extra_out)) return zi_refuse("moe_router: %d further outputs without a place", extra);
+  return launch_moe_router(chosen, weight, x, x_dtype, ldx, w, w_dtype, correction, T, K, NR, top, renormalize, 1, score_kind,
+                           groups, keep, wscale, stream, extra, extra_out);
 }
 
 // The router's product, a bias on the logits, the `top` largest logits and the softmax over them alone, in one kernel.
@@ -734,13 +756,15 @@ extern "C" int zi_moe_few_rows(void* out, int out_dtype, int ldo, const void* x,
 }
 
 extern "C" int zi_moe_align(const int* chosen, int P, int top, int E, int tile_rows, int cap_tiles, int* row_token,
-                            int* row_self, int* pair_row, int* tile_expert, int* n_tiles, cudaStream_t stream) {
+                            int* row_self, int* pair_row, int* tile_expert, int* n_tiles, const float* weight, float* row_weight,
+                            cudaStream_t stream) {
   if (P <= 0) return 0;
+  if (row_weight && !weight) return zi_refuse("moe_align: weights per row need weights per pair");
   if (cap_tiles < (P + tile_rows - 1) / tile_rows + E) return zi_refuse("moe_align: %d tiles cannot hold %d pairs of %d experts", cap_tiles, P, E);
   const size_t smem = (size_t)(3 * E + 1) * sizeof(int);
   if (smem > 48 * 1024) return zi_refuse("moe_align: %d experts are more than this kernel holds", E);
   zi_launch(moe_align_kernel, dim3(1), dim3(1024), smem, stream, chosen, P, top, E, tile_rows, cap_tiles, row_token,
-            row_self, pair_row, tile_expert, n_tiles);
+            row_self, pair_row, tile_expert, n_tiles, weight, row_weight);
   return zi_check_launch("moe_align");
 }
 

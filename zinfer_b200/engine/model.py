@@ -39,6 +39,14 @@ def _plan_runs(spec: ModelSpec) -> list[Run]:
     return runs
 
 
+def _flat_needs(name: str, need) -> list:
+    if need is None:
+        return []
+    if isinstance(need, dict):
+        return [pair for part, n in need.items() for pair in _flat_needs(f"{name}.{part}", n)]
+    return [(name, need)]
+
+
 class DecoderModel:
     def __init__(self, spec: ModelSpec, dtype: torch.dtype, device, max_positions: Optional[int] = None):
         spec.validate()
@@ -129,15 +137,13 @@ class DecoderModel:
 
     def _needs_of(self, run: Run) -> dict:
         """The caches and states a run uses, by name.  A mixer needs one (named like the run's cache), none, or
-        several (a dictionary part -> need: a mixer of several branches; named ``<run's cache>.<part>``)."""
-        need = self.blocks[run.layer].mixer.cache_need()
-        if need is None:
-            return {}
-        if isinstance(need, dict):
-            return {f"{run.cache}.{part}": n for part, n in need.items() if n is not None}
-        return {run.cache: need}
+        several (a dictionary part -> need: a mixer of several branches; named ``<run's cache>.<part>``; a branch may
+        need several itself)."""
+        return dict(_flat_needs(run.cache, self.blocks[run.layer].mixer.cache_need()))
 
-    def _view(self, storage: CacheStorage, name: str, writes: bool, kv: dict, state: dict):
+    def _view(self, storage: CacheStorage, name: str, need, writes: bool, kv: dict, state: dict):
+        if isinstance(need, dict):     # a mixer of several branches gets its views by the branches' names
+            return {part: self._view(storage, f"{name}.{part}", n, writes, kv, state) for part, n in need.items()}
         if name in kv:
             return storage.kv_view(name, writes)
         if name in state:
@@ -150,11 +156,7 @@ class DecoderModel:
         self._embedding_view = storage.state_view(EMBEDDING_STATE) if EMBEDDING_STATE in state else None
         self._views = []
         for run in self.runs:
-            need = self.blocks[run.layer].mixer.cache_need()
-            if isinstance(need, dict):     # a mixer of several branches gets its views by the branches' names
-                self._views.append({part: self._view(storage, f"{run.cache}.{part}", run.writes, kv, state) for part in need})
-            else:
-                self._views.append(self._view(storage, run.cache, run.writes, kv, state))
+            self._views.append(self._view(storage, run.cache, self.blocks[run.layer].mixer.cache_need(), run.writes, kv, state))
 
     # ------------------------------------------------------------------ forward
     def forward(self, step, argmax: bool = False):

@@ -161,6 +161,19 @@ class Scaled:
         return self.delta.shape
 
 
+class RowScaled:
+    """An update of the residual stream whose row t is multiplied by ``rows[t]`` (float32 [T]) as it is added (a gate of one
+    number per token): ``delta`` is a tensor or :class:`Partials`."""
+
+    def __init__(self, delta, rows: torch.Tensor):
+        self.delta = delta
+        self.rows = rows
+
+    @property
+    def shape(self):
+        return self.delta.shape
+
+
 class Carried:
     """Nothing is pending: the residual stream is up to date, and ``x`` is that stream in the activations' type (a block
     that made it hands it to the next one, which may read it instead of casting the stream again)."""
@@ -185,7 +198,8 @@ class PostNormed:
 
 class Several:
     """Updates of the residual stream that are still to be added, in this order (a block whose sublayers read the
-    same stream leaves one per sublayer): each a tensor, :class:`Partials`, or either inside :class:`Scaled`.
+    same stream leaves one per sublayer): each a tensor, :class:`Partials`, either inside :class:`RowScaled`, or any of
+    these inside :class:`Scaled`.
     ``row_bias`` (float32 [width]) is a vector that is added to every row with them (an output projection's bias)."""
 
     def __init__(self, terms, row_bias: Optional[torch.Tensor] = None):
@@ -238,9 +252,15 @@ def sum_norm(h: torch.Tensor, delta, w1: torch.Tensor, eps: float, out_dtype: to
     whole, part = (ctypes.c_void_p * 4)(), (ctypes.c_void_p * 4)()
     dtypes, splits = (ctypes.c_int * 4)(), (ctypes.c_int * 4)()
     zstride, scales = (ctypes.c_longlong * 4)(), (ctypes.c_float * 4)()
+    row_scales = (ctypes.c_void_p * 4)()
     keep, nbytes = [], 0
     for i, term in enumerate(terms):
         t, scales[i] = _unscaled(term)
+        if isinstance(t, RowScaled):
+            _need(t.rows.dtype == torch.float32 and t.rows.numel() == T and t.rows.is_contiguous(), "multipliers of rows are float32, one per token")
+            row_scales[i] = t.rows.data_ptr()
+            keep.append(t.rows)
+            t = t.delta
         if isinstance(t, Partials):
             _need(tuple(t.shape) == (T, H), "an update must match the residual stream")
             part[i], splits[i], zstride[i] = t.data.data_ptr(), t.splits, T * H
@@ -255,7 +275,7 @@ def sum_norm(h: torch.Tensor, delta, w1: torch.Tensor, eps: float, out_dtype: to
     out2 = torch.empty_like(out1) if w2 is not None else None
     with _prof.region("sum of updates + norm" + (" pair" if w2 is not None else ""),
                       lambda: (2 if rows is None else 1) * n * H * 4 + nbytes + _nb(out1) * (2 if w2 is not None else 1)):
-        _check(lib().zi_sum_norm_pair(_ptr(h), n_terms, whole, dtypes, part, splits, zstride, scales, _ptr(bias), _ptr(w1),
+        _check(lib().zi_sum_norm_pair(_ptr(h), n_terms, whole, dtypes, part, splits, zstride, scales, row_scales, _ptr(bias), _ptr(w1),
                                       _ptr(w2), ctypes.c_float(eps), _ptr(out1), _ptr(out2), _tag(out1), _ptr(rows), n, H,
                                       _stream()), "sum_norm")
     return out1 if w2 is None else (out1, out2)
@@ -338,7 +358,7 @@ def add_rmsnorm(h: torch.Tensor, delta, weight: torch.Tensor, eps: float,
     ``rows`` (int32, repeats allowed) picks rows instead: the result has one row per entry,
     the norm of ``h[row] + delta[row]``, and ``h`` is left unchanged."""
     T, H = h.shape
-    if isinstance(delta, Several):      # several updates at once: the kernel that adds them all in one pass
+    if isinstance(delta, (Several, RowScaled)):      # several updates at once, or rows with multipliers: the kernel that adds them all in one pass
         _need(out is None, "several updates at once come with a new output tensor")
         return sum_norm(h, delta, weight, eps, out_dtype, rows=rows, bias=bias)
     delta, dscale = _unscaled(delta)
@@ -371,6 +391,7 @@ def residual_add(h: torch.Tensor, delta) -> None:
             residual_add(h, term)
         return
     delta, dscale = _unscaled(delta)
+    _need(not isinstance(delta, RowScaled), "residual_add: rows with multipliers go in with a norm's kernel")
     if isinstance(delta, Partials):
         delta = delta.sum(torch.float32)
     _need(h.dtype == torch.float32 and h.is_contiguous() and delta.is_contiguous() and delta.shape == h.shape,
@@ -564,16 +585,17 @@ ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
 
 
 def swiglu(gate_up, out: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
-           interleave: int = 0, activation: str = "silu") -> torch.Tensor:
+           interleave: int = 0, activation: str = "silu", row_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``act(gate) * up`` for ``gate_up`` [T, 2I]: gate then up (``interleave`` 0), or blocks
     of 2 * ``interleave`` columns holding ``interleave`` gate values and then the up values of
-    the same features.  ``activation``: ``silu`` or ``gelu_tanh`` (the tanh form of gelu)."""
+    the same features.  ``activation``: ``silu`` or ``gelu_tanh`` (the tanh form of gelu).  ``row_scale`` (float32 [T])
+    multiplies a row's gate and up values first: the two products' input was to be multiplied by it."""
     _need(activation in ACTIVATIONS, f"unknown activation {activation!r}")
     act = ACTIVATIONS[activation]
     if isinstance(gate_up, Partials):
         T, two_i = gate_up.shape
         I = two_i // 2
-        if I % 4 == 0:
+        if I % 4 == 0 and row_scale is None:
             res = torch.empty((T, I), dtype=out_dtype or torch.bfloat16, device=gate_up.data.device)
             with _prof.region("swiglu (partial sums)", lambda: _nb(res, gate_up.data)):
                 _check(lib().zi_gated_act_partials(_ptr(res), _tag(res), _ptr(gate_up.data), gate_up.splits,
@@ -582,11 +604,14 @@ def swiglu(gate_up, out: Optional[torch.Tensor] = None, out_dtype: Optional[torc
         gate_up = gate_up.sum(out_dtype or torch.bfloat16)
     T, two_i = gate_up.shape
     _need(two_i % 2 == 0 and gate_up.is_contiguous(), "swiglu input is contiguous [T, 2I]")
+    _need(row_scale is None or (row_scale.dtype == torch.float32 and row_scale.numel() == T and row_scale.is_contiguous()),
+          "multipliers of rows are float32, one per row")
     I = two_i // 2
     if out is None:
         out = torch.empty((T, I), dtype=gate_up.dtype, device=gate_up.device)
     with _prof.region("swiglu", lambda: _nb(out, gate_up)):
-        _check(lib().zi_gated_act(_ptr(out), _ptr(gate_up), _tag(gate_up), T, I, interleave, act, _stream()), "swiglu")
+        _check(lib().zi_gated_act_rows(_ptr(out), _ptr(gate_up), _tag(gate_up), T, I, interleave, act, _ptr(row_scale), _stream()),
+               "swiglu")
     return out
 
 
@@ -958,12 +983,15 @@ def linear_few_rows(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, ro
 MOE_TILE_ROWS_SMALL, MOE_TILE_ROWS, MOE_TILE_ROWS_TENSOR = 16, 64, 128
 
 
-def moe_align(chosen: torch.Tensor, experts: int, tile_rows: int):
+def moe_align(chosen: torch.Tensor, experts: int, tile_rows: int, weight: Optional[torch.Tensor] = None):
     """Lays the (token, expert) pairs out by expert in whole tiles of ``tile_rows`` rows.  Returns
     ``(row_token, row_self, pair_row, tile_expert, n_tiles)``: the token of every row (-1: padding), the
     row's own index where it is in use, the row of every pair (-1: an identity expert), the expert of
-    every tile and the number of tiles (one int32 on the device)."""
+    every tile and the number of tiles (one int32 on the device); with ``weight`` (float32 [T, top]) also the weight
+    of every row's pair (0: padding), float32 [rows]."""
     T, top = chosen.shape
+    _need(weight is None or (weight.dtype == torch.float32 and weight.shape == chosen.shape and weight.is_contiguous()),
+          "the pairs' weights are float32 [T, top]")
     P = T * top
     cap_tiles = -(-P // tile_rows) + experts
     dev = chosen.device
@@ -971,9 +999,13 @@ def moe_align(chosen: torch.Tensor, experts: int, tile_rows: int):
     n = cap_tiles * tile_rows
     row_token, row_self, pair_row = buf[:n], buf[n:2 * n], buf[2 * n:2 * n + P]
     tile_expert, n_tiles = buf[2 * n + P:2 * n + P + cap_tiles], buf[2 * n + P + cap_tiles:]
+    row_weight = torch.empty((n,), dtype=torch.float32, device=dev) if weight is not None else None
     with _prof.region("moe align", lambda: _nb(chosen) + 3 * P * 4):
         _check(lib().zi_moe_align(_ptr(_i32(chosen, "chosen")), P, top, experts, tile_rows, cap_tiles, _ptr(row_token),
-                                  _ptr(row_self), _ptr(pair_row), _ptr(tile_expert), _ptr(n_tiles), _stream()), "moe_align")
+                                  _ptr(row_self), _ptr(pair_row), _ptr(tile_expert), _ptr(n_tiles), _ptr(weight), _ptr(row_weight),
+                                 _stream()), "moe_align")
+    if weight is not None:
+        return row_token, row_self, pair_row, tile_expert, n_tiles, row_weight
     return row_token, row_self, pair_row, tile_expert, n_tiles
 
 
@@ -1014,9 +1046,10 @@ def linear_grouped_tensor(x: torch.Tensor, weight: torch.Tensor, out: torch.Tens
     return out
 
 
-def moe_combine(y: torch.Tensor, x: torch.Tensor, chosen: torch.Tensor, weight: torch.Tensor, pair_row: torch.Tensor,
+def moe_combine(y: torch.Tensor, x: torch.Tensor, chosen: torch.Tensor, weight: Optional[torch.Tensor], pair_row: torch.Tensor,
                 experts: int) -> torch.Tensor:
-    """``out[t] = sum_k weight[t, k] * (y[pair_row[t, k]] if chosen[t, k] < experts else x[t])``, k ascending."""
+    """``out[t] = sum_k weight[t, k] * (y[pair_row[t, k]] if chosen[t, k] < experts else x[t])``, k ascending; without
+    ``weight`` the plain sum (the experts' inputs were weighted)."""
     T, H = x.shape
     top = chosen.shape[1]
     _need(y.dtype == torch.float32 and y.is_contiguous() and y.shape[1] == H and x.is_contiguous(), "moe_combine: shapes")
@@ -1810,11 +1843,14 @@ def sigmoid_rows(x: torch.Tensor) -> torch.Tensor:
 
 
 def linear_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, beta: Optional[torch.Tensor],
-                      q_scale: float, state: torch.Tensor, heads: int, key_heads: int, dim: int, vdim: int, step) -> torch.Tensor:
+                      q_scale: float, state: torch.Tensor, heads: int, key_heads: int, dim: int, vdim: int, step,
+                      delta: bool = True) -> torch.Tensor:
     """Per request and head, over the step's tokens, from and to ``state`` [slots, heads, dim, vdim] (float32):
-    ``S = diag(decay_t) S``; ``u = v_t`` or, with ``beta``, ``beta_t (v_t - S^T k_t)`` (the delta rule);
+    ``S = diag(decay_t) S``; ``u = beta_t (v_t - S^T k_t)`` (the delta rule) or, with ``delta`` False or without ``beta``,
+    ``u = beta_t v_t`` (a step size; 1 without ``beta``);
     ``S += k_t u^T``; ``o_t = S^T (q_scale q_t)``.  ``q``, ``k`` [T, key_heads * dim] (head h reads key head
-    h // (heads / key_heads)), ``v`` [T, heads * vdim], ``decay`` float32 [T, heads * dim], ``beta`` float32 [T, heads];
+    h // (heads / key_heads)), ``v`` [T, heads * vdim], ``decay`` float32 [T, heads * dim] or one per head [T, heads],
+    ``beta`` float32 [T, heads];
     rows may be views of wider rows.  Returns float32 [T, heads * vdim]."""
     T = q.shape[0]
     state, stride = _slot_view(state, "linear_recurrence")
@@ -1822,16 +1858,18 @@ def linear_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: 
     _need(q.dtype == k.dtype and q.stride(1) == 1 and k.stride(1) == 1 and v.stride(1) == 1
           and q.shape[1] == key_heads * dim and k.shape[1] == key_heads * dim and v.shape[1] == heads * vdim,
           "linear_recurrence: q, k [T, key heads * dim], v [T, heads * vdim] with dense rows")
-    _need(decay.dtype == torch.float32 and decay.stride(1) == 1 and decay.shape[1] == heads * dim, "linear_recurrence: decay")
+    _need(decay.dtype == torch.float32 and decay.stride(1) == 1 and decay.shape[1] in (heads, heads * dim),
+          "linear_recurrence: decay")
     if beta is not None:
         _need(beta.dtype == torch.float32 and beta.stride(1) == 1 and beta.shape[1] == heads, "linear_recurrence: beta")
+    delta = delta and beta is not None
     out = torch.empty((T, heads * vdim), dtype=torch.float32, device=q.device)
-    with _prof.region("linear recurrence" + (" (delta rule)" if beta is not None else ""),
+    with _prof.region("linear recurrence" + (" (delta rule)" if delta else ""),
                       lambda: _nb(q, k, v, decay, out) + 2 * step.n_seqs * heads * dim * vdim * 4, 6 * T * heads * dim * vdim):
         _check(lib().zi_linear_recurrence(
             _ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _tag(q), _ptr(v), v.stride(0), _tag(v),
             _ptr(decay), decay.stride(0), _ptr(beta), beta.stride(0) if beta is not None else 0, ctypes.c_float(q_scale),
-            _ptr(state), _ll(stride), heads, key_heads, dim, vdim, 1 if beta is not None else 0, _ptr(step.cu_q),
+            _ptr(state), _ll(stride), heads, key_heads, dim, vdim, 1 if delta else 0, 1 if decay.shape[1] == heads else 0, _ptr(step.cu_q),
             _ptr(step.state_slots), step.n_seqs, _stream()), "linear_recurrence")
     return out
 
@@ -1893,21 +1931,151 @@ def linear_recurrence_gated(proj, lower: torch.Tensor, f_bias: Optional[torch.Te
     return out
 
 
-def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, eps: float, gate: Optional[torch.Tensor], gate_kind: str, heads: int,
+class Columns:
+    """Columns ``at`` .. ``at + width`` of a projection's float32 rows: of a tensor, or of :class:`Partials` whose splits the
+    consumer adds in order."""
+
+    def __init__(self, proj, at: int, width: int):
+        data = proj.data if isinstance(proj, Partials) else proj
+        _need(data.dtype == torch.float32 and data.is_contiguous() and 0 <= at and at + width <= proj.shape[1],
+              "columns of contiguous float32 rows")
+        self.data, self.at, self.width = data, at, width
+        self.splits = proj.splits if isinstance(proj, Partials) else 1
+        self.rows, self.ld = proj.shape
+        self.zstride = self.rows * self.ld
+
+    @property
+    def shape(self):
+        return (self.rows, self.width)
+
+    @property
+    def ptr(self):
+        return ctypes.c_void_p(_ptr(self.data).value + 4 * self.at)
+
+    def bytes(self) -> int:
+        return self.rows * self.width * 4 * self.splits
+
+
+class ConvSegment:
+    """Neighbouring channels of a projection that pass a short convolution: ``channels`` in heads of ``head_dim``; ``finish`` None,
+    ``unit`` (every head divided by sqrt(sum x^2 + eps), times ``scale``) or ``rotate``; ``out`` a tensor [T, >= channels] whose
+    rows take the heads (float32, or the activations' type), or pages [pages, heads, page_size, head_dim]."""
+
+    def __init__(self, channels: int, head_dim: int, out: torch.Tensor, finish: Optional[str] = None, scale: float = 1.0):
+        self.channels, self.head_dim, self.out, self.finish, self.scale = channels, head_dim, out, finish, scale
+
+
+CONV_MAX_TAPS = 17
+_FINISHES = {None: 0, "unit": 1, "rotate": 2}
+
+
+def conv_heads(u: Columns, kernel: torch.Tensor, tail: Optional[torch.Tensor], step, segments: list, in_bias: Optional[torch.Tensor] = None,
+               out_bias: Optional[torch.Tensor] = None, activation: Optional[str] = None, unit_eps: float = 0.0,
+               tables=(None, None), rot_dims: int = 0, pairing: str = "halves", slots: Optional[torch.Tensor] = None, page_size: int = 0,
+               decay=None):
+    """What follows a projection whose channels pass a causal convolution over time, in one kernel: ``in_bias`` [C] is added to
+    the projected rows ``u``; ``y_t = sum_i kernel[i] * u_(t - taps + 1 + i)`` per channel (``kernel`` float32 [taps, C], last row:
+    the current token; inputs before a request's first token of this step from ``tail`` [slots, taps-1, C], which is moved on
+    as well); ``out_bias`` and ``activation`` (None or silu); then every :class:`ConvSegment` (in the order of the channels, all C of
+    them) is finished and put where it goes.
+
+    ``decay``: (kind, a, b, a_log, dt_bias) makes the steps and decays of a recurrence from further columns of the same rows:
+    kind ``delta`` gives step = sigmoid(b), decay = exp(-exp(a_log) softplus(a + dt_bias)); kind ``ssd`` gives step =
+    softplus(a + dt_bias), decay = exp(-exp(a_log) step).  Returns (decay, step), float32 [T, heads], or None."""
+    T, C = u.shape
+    taps = kernel.shape[0]
+    _need(kernel.dtype == torch.float32 and kernel.is_contiguous() and kernel.shape[1] == C, "conv_heads: kernel float32 [taps, C]")
+    for t in (in_bias, out_bias):
+        _need(t is None or (t.dtype == torch.float32 and t.numel() == C and t.is_contiguous()), "conv_heads: biases float32 [C]")
+    stride = 0
+    if taps > 1:
+        tail, stride = _slot_view(tail, "conv_heads")
+        _need(tuple(tail.shape[1:]) == (taps - 1, C), "conv_heads: tail [slots, taps-1, C]")
+    cos, sin = tables
+    n_table = 0
+    if cos is not None:
+        _need(cos.shape == sin.shape and cos.shape[1] == rot_dims // 2 and cos.dtype == torch.float32, "rotary tables are float32 [positions, rot_dims/2]")
+        n_table = cos.shape[0]
+    _need(activation in (None, "silu") and pairing in ("halves", "neighbours"), "conv_heads: unknown activation or pairing")
+    n = len(segments)
+    ints, outs, scales = (ctypes.c_int * (5 * n))(), (ctypes.c_void_p * n)(), (ctypes.c_float * n)()
+    act_dtype = torch.float32
+    for i, s in enumerate(segments):
+        paged = s.out.dim() == 4
+        finish = s.finish if not (s.finish == "rotate" and cos is None) else None
+        dest = 2 if paged else (0 if s.out.dtype == torch.float32 else 1)
+        if paged:
+            _need(s.out.is_contiguous() and tuple(s.out.shape[1:]) == (s.channels // s.head_dim, page_size, s.head_dim), "conv_heads: pages")
+        else:
+            _need(s.out.stride(1) == 1 and s.out.shape[0] == T and s.out.shape[1] >= s.channels, "conv_heads: rows of a segment")
+        if dest:
+            act_dtype = s.out.dtype
+        # channels without a finish need no whole heads: short pieces spread them over more warps
+        d = 64 if finish is None and not paged else s.head_dim
+        ints[5 * i:5 * i + 5] = [s.channels, d, _FINISHES[finish], dest, 0 if paged else s.out.stride(0)]
+        outs[i], scales[i] = _ptr(s.out).value, s.scale
+    _need(all(s.out.dtype in (torch.float32, act_dtype) for s in segments), "conv_heads: one activations' type")
+    kind, a, b, a_log, dt_bias, dec, stp, H = 0, None, None, None, None, None, None, 0
+    if decay is not None:
+        name, a, b, a_log, dt_bias = decay
+        kind, H = {"delta": 1, "ssd": 2}[name], a.width
+        _need(all(c is None or (c.data.data_ptr() == u.data.data_ptr() and c.width == H) for c in (a, b)), "conv_heads: steps come from the same rows")
+        _need(a_log.dtype == torch.float32 and dt_bias.dtype == torch.float32 and a_log.numel() == H and dt_bias.numel() == H, "conv_heads: float32 [heads]")
+        dec = torch.empty((T, H), dtype=torch.float32, device=u.data.device)
+        stp = torch.empty_like(dec)
+    with _prof.region("convolution, heads" + (" and pages" if slots is not None else ""),
+                      lambda: u.bytes() + sum(T * s.channels * s.out.element_size() for s in segments) + 4 * step.n_seqs * (taps - 1) * C * 2,
+                      2 * T * C * taps):
+        _check(lib().zi_conv_heads(
+            u.ptr, u.ld, u.splits, _ll(u.zstride), T, C, taps, _ptr(kernel), _ptr(in_bias), _ptr(out_bias), 1 if activation == "silu" else 0,
+            _ptr(tail) if taps > 1 else None, _ll(stride), n, ints, outs, scales, F32 if act_dtype == torch.float32 else BF16,
+            ctypes.c_float(unit_eps), _ptr(cos), _ptr(sin), n_table, rot_dims if cos is not None else 0, 1 if pairing == "neighbours" else 0,
+            _ptr(step.positions), _ptr(slots), page_size, kind, H, a.ptr if a is not None else None, b.ptr if b is not None else None,
+            _ptr(a_log), _ptr(dt_bias), _ptr(dec), _ptr(stp), _ptr(step.tile_seq), _ptr(step.tile_q0), step.tile_seq.shape[0],
+            attention_tile_rows(), _ptr(step.cu_q), _ptr(step.state_slots), _stream()), "conv_heads")
+    return (dec, stp) if decay is not None else None
+
+
+def gated_part_norm(y: torch.Tensor, gate: Columns, weight: torch.Tensor, eps: float, parts: int, out_dtype: torch.dtype,
+                    skip: Optional[torch.Tensor] = None, x: Optional[torch.Tensor] = None, vdim: int = 1) -> torch.Tensor:
+    """``(y + skip * x) * silu(gate)`` for float32 ``y`` [T, width] (``skip`` float32 [width / vdim]: one per head of ``vdim`` columns; ``x``
+    float32 [T, >= width] rows), then each of ``parts`` equal parts of a row divided by its own root mean square (``eps``
+    inside the root), times ``weight`` [width]."""
+    T, W = y.shape
+    _need(y.dtype == torch.float32 and y.stride(1) == 1 and gate.shape == (T, W) and weight.dtype == torch.float32 and weight.numel() == W,
+          "gated_part_norm: shapes")
+    _need(skip is None or (skip.numel() * vdim == W and x.dtype == torch.float32 and x.stride(1) == 1 and x.shape[0] == T),
+          "gated_part_norm: a skip per head and its rows")
+    out = torch.empty((T, W), dtype=out_dtype, device=y.device)
+    with _prof.region("gated norm of parts", lambda: T * W * (4 + (4 if skip is not None else 0)) + gate.bytes() + _nb(out)):
+        _check(lib().zi_gated_part_norm(_ptr(out), _tag(out), out.stride(0), _ptr(y), y.stride(0), _ptr(x) if skip is not None else None,
+                                        x.stride(0) if skip is not None else 0, _ptr(skip), vdim, gate.ptr, gate.ld, gate.splits,
+                                        _ll(gate.zstride), _ptr(weight), ctypes.c_float(eps), T, W, parts, _stream()), "gated_part_norm")
+    return out
+
+
+def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, eps: float, gate, gate_kind: str, heads: int,
                    vdim: int, out_dtype: torch.dtype) -> torch.Tensor:
     """Every head of float32 ``o`` [T, heads * vdim] divided by its root mean square (``eps`` inside the root), times
-    ``weight`` [vdim], times ``silu(gate)`` or ``sigmoid(gate)`` (``gate`` [T, heads * vdim], rows may be views; kind
-    ``none``: no gate)."""
+    ``weight`` [vdim], times ``silu(gate)`` or ``sigmoid(gate)`` (``gate`` [T, heads * vdim], rows may be views, or
+    :class:`Columns` of a projection; kind ``none``: no gate)."""
     T = o.shape[0]
-    _need((gate is None) == (gate_kind == "none"), "head_norm_gate: a gate and its kind go together")
+    cols = gate if isinstance(gate, Columns) else None
+    if cols is not None:
+        gate = None
+        _need(cols.shape == (T, heads * vdim), "head_norm_gate: shapes")
+    _need((gate is None and cols is None) == (gate_kind == "none"), "head_norm_gate: a gate and its kind go together")
     _need(o.dtype == torch.float32 and o.is_contiguous() and (gate is None or (gate.stride(1) == 1 and gate.shape[1] == heads * vdim))
           and weight.dtype == torch.float32 and weight.numel() == vdim, "head_norm_gate: shapes")
     kinds = {"silu": 0, "sigmoid": 1, "none": 2}
     _need(gate_kind in kinds, f"head_norm_gate: unknown gate {gate_kind!r}")
     out = torch.empty((T, heads * vdim), dtype=out_dtype, device=o.device)
-    with _prof.region("head norm + gate", lambda: _nb(o, out) + (T * heads * vdim * gate.element_size() if gate is not None else 0)):
+    with _prof.region("head norm + gate", lambda: _nb(o, out) + (T * heads * vdim * gate.element_size() if gate is not None else 0)
+                      + (cols.bytes() if cols is not None else 0)):
         _check(lib().zi_head_norm_gate(_ptr(out), _tag(out), out.stride(0), _ptr(o), o.stride(0), _ptr(weight), ctypes.c_float(eps),
-                                       _ptr(gate), _tag(gate) if gate is not None else F32, gate.stride(0) if gate is not None else 0,
+                                       cols.ptr if cols is not None else _ptr(gate), _tag(gate) if gate is not None else F32,
+                                       gate.stride(0) if gate is not None else (cols.ld if cols is not None else 0),
+                                       cols.splits if cols is not None else 1, _ll(cols.zstride if cols is not None else 0),
                                        kinds[gate_kind], T, heads, vdim,
                                        _stream()), "head_norm_gate")
     return out
@@ -1915,24 +2083,26 @@ def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, eps: float, gate: Opti
 
 def moe_router_grouped(x: torch.Tensor, w_router: torch.Tensor, top: int, score: str = "sigmoid", groups: int = 1, keep: int = 1,
                        scale: float = 1.0, renormalize: bool = False,
-                       correction: Optional[torch.Tensor] = None) -> tuple[torch.Tensor, torch.Tensor]:
+                       correction: Optional[torch.Tensor] = None, extra: int = 0):
     """The router's product (32-bit multiply-adds whatever the operands' types) and :func:`moe_route_grouped` in one
-    kernel, one block per token."""
+    kernel, one block per token.  The last ``extra`` rows of ``w_router`` are not chosen from: the sigmoids of their logits
+    come back as a third result, float32 [T, extra]."""
     if correction is not None:
-        _need(correction.dtype == torch.float32 and correction.numel() == w_router.shape[0] and correction.is_contiguous(),
+        _need(correction.dtype == torch.float32 and correction.numel() == w_router.shape[0] - extra and correction.is_contiguous(),
               "the correction is float32, one value per router output")
     T, K = x.shape
-    NR = w_router.shape[0]
+    NR = w_router.shape[0] - extra
     _need(x.stride(1) == 1 and w_router.is_contiguous() and w_router.shape[1] == K, "moe_router: shapes")
+    gates = torch.empty((T, extra), dtype=torch.float32, device=x.device) if extra else None
     _need(score in ("softmax", "sigmoid"), f"unknown router score {score!r}")
     chosen = torch.empty((T, top), dtype=torch.int32, device=x.device)
     weight = torch.empty((T, top), dtype=torch.float32, device=x.device)
     with _prof.region(f"moe router (groups) N={NR} K={K}", lambda: _nb(w_router) + T * K * x.element_size(), 2 * T * NR * K):
-        _check(lib().zi_moe_router_grouped_c(_ptr(chosen), _ptr(weight), _ptr(x), _tag(x), x.stride(0), _ptr(w_router),
+        _check(lib().zi_moe_router_grouped_x(_ptr(chosen), _ptr(weight), _ptr(x), _tag(x), x.stride(0), _ptr(w_router),
                                            _tag(w_router), _ptr(correction), T, K, NR, top, 1 if renormalize else 0,
-                                           1 if score == "sigmoid" else 0, groups, keep, ctypes.c_float(scale), _stream()),
-               "moe_router_grouped")
-    return chosen, weight
+                                           1 if score == "sigmoid" else 0, groups, keep, ctypes.c_float(scale), extra, _ptr(gates),
+                                           _stream()), "moe_router_grouped")
+    return (chosen, weight, gates) if extra else (chosen, weight)
 
 
 def moe_router_top_logits(x: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Tensor], top: int):

@@ -42,6 +42,13 @@ has left its window ((b + 1) P <= i - w + 1), that block stands in as ONE key an
 the cache holds them.  Those live in pages of their own, one entry per P tokens, written with the block's last token; the
 tokens' own pages are given back once the window has passed them and their block is complete.  ``sink`` and per-head
 ``qk_norm_eps`` go with this form.
+
+The "conv" form: ``conv_taps`` n puts a causal convolution over time on every channel of q, k and v (tensors named like the
+projections plus ``.conv``, [channels, taps], last column for the current token), after the projection and its bias and before
+the rotation, without an activation; a request's last n - 1 projected values are state beside its pages.  One product
+[q | k | v] with 32-bit results, one kernel for bias, convolution, rotation (either pairing), page write and the carried
+values, the attention, the output projection.  ``bias: True``, ``softcap``, ``learned_sink``, ``distance_bias`` and
+``value_dim`` go with it.
 """
 from __future__ import annotations
 
@@ -51,7 +58,7 @@ import numpy as np
 import torch
 
 from .. import ops
-from .base import KVCacheNeed, Mixer, TensorSpec, make_part
+from .base import KVCacheNeed, Mixer, StateNeed, TensorSpec, make_part
 
 
 class GQAttention(Mixer):
@@ -107,6 +114,19 @@ class GQAttention(Mixer):
             raise ValueError(f"an output gate is per channel or per head, not {self.output_gate!r}")
         self.rows_form = bool(self.has_bias or self.whole_norm_eps is not None or self.softcap or self.learned_sink
                               or self.distance_bias or self.output_gate)
+        self.conv_taps = int(params.get("conv_taps") or 0)
+        self.conv_form = self.conv_taps > 0
+        if self.conv_form:
+            if self.conv_taps > ops.CONV_MAX_TAPS:
+                raise ValueError(f"the convolution has 1 to {ops.CONV_MAX_TAPS} taps, got {self.conv_taps}")
+            if self.qk_norm_eps is not None or self.whole_norm_eps is not None or self.output_gate or self.values_from_keys or self.keep_first \
+                    or not self.projects_kv or self.sink or params.get("bias") == "qkv" or params.get("value_mix") or params.get("pool"):
+                raise ValueError("the conv form of attention goes with none of: norms of q and k, an output gate, values from the keys, kept "
+                                 "first tokens, another layer's cache, a counted sink, the heads form's options")
+            self.rows_form = False
+            self.n_gate = 0
+            self.channels = self.nq * self.d + self.nkv * (self.d + self.dv)
+            names.setdefault("sink", "sink")
         if self.rows_form:
             if self.qk_norm_eps is not None or self.values_from_keys or self.keep_first or not self.projects_kv or self.sink:
                 raise ValueError("the rows form of attention goes with none of: per-head q/k norm, values from the keys, "
@@ -157,7 +177,10 @@ class GQAttention(Mixer):
             specs[n["v"] + ".b"] = TensorSpec((self.nkv * self.dv,), init="around_zero")
         if self.value_mix:
             specs[str(self.value_mix["tensor"])] = TensorSpec((), init="unit")
-        if self.rows_form:
+        if self.conv_form:
+            for x, rows in (("q", q), ("k", kv), ("v", self.nkv * self.dv)):
+                specs[n[x] + ".conv"] = TensorSpec((rows, self.conv_taps))
+        if self.rows_form or self.conv_form:
             if self.has_bias:
                 specs[n["q"] + ".b"] = TensorSpec((q,), init="around_zero")
                 specs[n["k"] + ".b"] = TensorSpec((kv,), init="around_zero")
@@ -193,8 +216,10 @@ class GQAttention(Mixer):
             self.row_bias = torch.cat([tensors[n[x] + ".b"].to(torch.float32) for x in ("q", "k", "v")]).contiguous()
         if self.value_mix:
             self.mix_lambda = float(tensors[str(self.value_mix["tensor"])])
-        if self.rows_form:
+        if self.rows_form or self.conv_form:
             self._bind_rows(tensors, parts)
+        if self.conv_form:
+            self.conv = torch.cat([tensors[n[x] + ".conv"].to(torch.float32) for x in ("q", "k", "v")], dim=0).t().contiguous()   # [taps, channels]
 
     def _bind_rows(self, tensors, parts):
         n = self.names
@@ -229,8 +254,11 @@ class GQAttention(Mixer):
             # a block's tokens stay until it is complete, also when the window is shorter than a block
             return {"tokens": KVCacheNeed(num_kv_heads=self.nkv, head_dim=self.d, window=max(int(self.window), self.pool), value_dim=vd),
                     "pooled": KVCacheNeed(num_kv_heads=self.nkv, head_dim=self.d, value_dim=vd, tokens_per_entry=self.pool)}
-        return KVCacheNeed(num_kv_heads=self.nkv, head_dim=self.d, window=self.window,
+        need = KVCacheNeed(num_kv_heads=self.nkv, head_dim=self.d, window=self.window,
                            value_dim=self.dv if self.dv != self.d else None, keep_first=self.keep_first)
+        if self.conv_taps > 1:     # the convolution's last inputs, oldest first
+            return {"kv": need, "conv": StateNeed((self.conv_taps - 1, self.channels), torch.float32)}
+        return need
 
     def max_positions(self):
         return None if self.position is None else getattr(self.position, "n_positions", None)
@@ -268,6 +296,28 @@ class GQAttention(Mixer):
             heads = ops.sigmoid_gate(heads, gate, out=heads, group=self.dv if self.output_gate == "head" else 1)
         return ops.linear(heads, self.w_o, out_dtype=self.ctx.dtype, allow_partials=True)
 
+    def _forward_conv(self, x, step, cache):
+        conv = None
+        if self.conv_taps > 1:
+            cache, conv = cache["kv"], cache["conv"].state
+        if not cache.writes:
+            raise ValueError("the conv form of attention fills its own cache")
+        # 32-bit results of the product: the biases and the convolution meet the unrounded sums
+        proj = ops.linear(x, self.w_rows, out_dtype=torch.float32, allow_partials=True)
+        group = step.kv_groups[cache.group]
+        tables = self.position.tables() if self.position is not None else (None, None)
+        q = torch.empty((x.shape[0], self.nq * self.d), dtype=self.ctx.dtype, device=x.device)
+        turn = "rotate" if self.position is not None else None
+        ops.conv_heads(ops.Columns(proj, 0, self.channels), self.conv, conv, step,
+                       [ops.ConvSegment(self.nq * self.d, self.d, q, turn), ops.ConvSegment(self.nkv * self.d, self.d, cache.k, turn),
+                        ops.ConvSegment(self.nkv * self.dv, self.dv, cache.v)], in_bias=self.row_bias, tables=tables,
+                       rot_dims=self.rot_dims, pairing=getattr(self.position, "pairing", "halves"), slots=group.slot_mapping,
+                       page_size=cache.page_size)
+        heads = ops.attention(q, cache.k, cache.v, group.block_tables, step, self.nq, self.nkv, self.d, cache.page_size,
+                              self.window, self.scale, value_dim=self.dv, sink_logit=self.sink_logit, softcap=self.softcap,
+                              dist_bias=self.dist_table)
+        return ops.linear(heads, self.w_o, out_dtype=self.ctx.dtype, allow_partials=True)
+
     VALUES_CARRIED = "first values"      # under this name the first mixing layer hands its values on
 
     def _forward_heads(self, x, step, cache):
@@ -298,6 +348,8 @@ class GQAttention(Mixer):
         return ops.linear(heads, self.w_o, out_dtype=self.ctx.dtype, allow_partials=True)
 
     def forward(self, x, step, cache):
+        if self.conv_form:
+            return self._forward_conv(x, step, cache)
         if self.heads_form:
             return self._forward_heads(x, step, cache)
         if self.rows_form:

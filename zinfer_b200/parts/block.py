@@ -50,17 +50,24 @@ class PreNormBlock(Block):
     def _update(self, delta):
         return delta if self.residual_scale == 1.0 else ops.Scaled(delta, self.residual_scale)
 
+    def _pending(self, out, row_bias=None):
+        """A sublayer's output as an update that is still to be added: one, or the several it handed back (two mixers side by
+        side, routed experts beside a shared one), with its output projection's bias."""
+        if not isinstance(out, tuple) and row_bias is None:
+            return self._update(out)
+        if row_bias is not None and self.residual_scale != 1.0:
+            row_bias = row_bias * self.residual_scale
+        return ops.Several([self._update(t) for t in (out if isinstance(out, tuple) else (out,))], row_bias=row_bias)
+
     def forward(self, h, pending, step, cache, bias=None):
         if self.feed_forward is not None and self.ffn_norm is None:
             raise ValueError("this arrangement needs a norm before its feed-forward")
         x = self.mixer_norm.forward(h, pending) if bias is None else self.mixer_norm.forward(h, pending, bias=bias)
-        a = self._update(self.mixer.forward(x, step, cache))
-        if getattr(self.mixer, "output_bias", None) is not None:
-            a = ops.Several([a], row_bias=self.mixer.output_bias * self.residual_scale)
+        a = self._pending(self.mixer.forward(x, step, cache), getattr(self.mixer, "output_bias", None))
         if self.feed_forward is None:
             return a
         x = self.ffn_norm.forward(h, a)
-        return self._update(self.feed_forward.forward(x))
+        return self._pending(self.feed_forward.forward(x))
 
 
 class OutputNormBlock(PreNormBlock):
@@ -87,6 +94,8 @@ class OutputNormBlock(PreNormBlock):
                 ops.residual_add(h, pending)
             x = ops.cast_rows(h, self.ctx.dtype)
         mixed = self.mixer.forward(x, step, cache)
+        if getattr(self.mixer, "output_bias", None) is not None:
+            raise ValueError("a block that norms its sublayers' outputs takes mixers without an output bias")
         a, b = mixed if isinstance(mixed, tuple) else (mixed, None)        # a mixer of two branches hands back both
         x = ops.norm_residual(h, a, self.mixer_norm.weight, self.mixer_norm.eps, self.ctx.dtype, b=b)
         if self.feed_forward is None:

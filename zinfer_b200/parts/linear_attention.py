@@ -16,7 +16,10 @@ g = sigmoid(W_a2 (W_a1 h) + b)^(1/tau), gate silu(W_g h).
 Yang et al., 2024, is the family): q, k (``kv_heads`` heads, shared by groups of value heads) and v each pass a short
 causal convolution per channel and silu; q and k are made unit vectors per head (x / sqrt(sum x^2 + 1e-6)), q also
 times dim^(-1/2); beta = sigmoid(W_b h); g = exp(-exp(A_log_h) * softplus(W_a2 (W_a1 h) + dt_bias)) per head and key
-channel; gate sigmoid(W_g2 (W_g1 h)).  The convolutions' last taps-1 inputs are state too.
+channel; gate sigmoid(W_g2 (W_g1 h)).  The convolutions' last taps-1 inputs are state too.  ``decay: "head"`` has one decay
+per head instead, g = exp(-exp(A_log_h) * softplus(W_a h + dt_bias)), and ``gate: "silu"`` a full projection's gate, silu(W_g h);
+with these one kernel makes all that the recurrence reads (convolutions, unit vectors, beta, decays) from the projection's
+32-bit rows.
 
 :class:`HGRN2` (the form that writes what its decay leaves room for; "HGRN2: Gated Linear RNNs with State Expansion",
 Qin et al., 2024, is the family): q = silu(W_q h), v = W_v h, gate f = sigmoid(z) + l (1 - sigmoid(z)) where z = W_f h + b
@@ -141,12 +144,16 @@ class GatedDeltaRule(Mixer):
         self.vdim = int(params["vdim"])
         self.taps = int(params["conv_taps"])
         self.eps = float(params["norm_eps"])
+        self.head_decay = params.get("decay", "channel") == "head"
+        if (params.get("decay", "channel"), params.get("gate", "sigmoid_low_rank")) not in (("channel", "sigmoid_low_rank"), ("head", "silu")):
+            raise ValueError("the delta rule is built with a decay per channel and a low-rank sigmoid gate, or a decay per head and a silu gate")
         self.decay_rank_hint = int(params.get("decay_rank", 16))
         self.gate_rank_hint = int(params.get("gate_rank", 16))
         if self.kv_heads <= 0 or self.heads % self.kv_heads:
             raise ValueError(f"{self.heads} heads do not divide into {self.kv_heads} query/key heads")
-        if not 1 <= self.taps <= 64:
-            raise ValueError(f"the convolution has 1 to 64 taps, got {self.taps}")
+        most = ops.CONV_MAX_TAPS if self.head_decay else 64
+        if not 1 <= self.taps <= most:
+            raise ValueError(f"the convolution has 1 to {most} taps, got {self.taps}")
         self.qk = self.kv_heads * self.dim
         self.hv = self.heads * self.vdim
         self.channels = 2 * self.qk + self.hv            # the convolved channels: q, k, v side by side
@@ -154,12 +161,18 @@ class GatedDeltaRule(Mixer):
 
     def tensor_specs(self):
         hid, hd = self.hidden, self.heads * self.dim
-        return {
+        common = {
             "q": TensorSpec((self.qk, hid)), "q.conv": TensorSpec((self.qk, self.taps)),
             "k": TensorSpec((self.qk, hid)), "k.conv": TensorSpec((self.qk, self.taps)),
             "v": TensorSpec((self.hv, hid)), "v.conv": TensorSpec((self.hv, self.taps)),
             "b": TensorSpec((self.heads, hid)), "A_log": TensorSpec((self.heads,), init="zeros"),
             "norm": TensorSpec((self.vdim,), init="norm"),
+        }
+        if self.head_decay:
+            return {**common, "a": TensorSpec((self.heads, hid)), "dt_bias": TensorSpec((self.heads,), init="zeros"),
+                    "g": TensorSpec((self.hv, hid)), "o": TensorSpec((hid, self.hv))}
+        return {
+            **common,
             "a1": TensorSpec((-1, hid), free=self.decay_rank_hint), "a2": TensorSpec((hd, -1), free=self.decay_rank_hint),
             "dt_bias": TensorSpec((hd,), init="zeros"),
             "g1": TensorSpec((-1, hid), free=self.gate_rank_hint), "g2": TensorSpec((self.hv, -1), free=self.gate_rank_hint),
@@ -167,6 +180,8 @@ class GatedDeltaRule(Mixer):
         }
 
     def bind(self, tensors):
+        if self.head_decay:
+            return self._bind_head_decay(tensors)
         for a, b in (("a1", "a2"), ("g1", "g2")):
             if tensors[a].shape[0] != tensors[b].shape[1]:
                 raise ValueError(f"{a} {list(tensors[a].shape)} and {b} {list(tensors[b].shape)} do not share a rank")
@@ -182,7 +197,33 @@ class GatedDeltaRule(Mixer):
         # one slot per request: S of every head, then the convolutions' last taps-1 inputs [taps-1, channels]
         return StateNeed((self.s_size + (self.taps - 1) * self.channels,), torch.float32)
 
+    # ---- one decay per head, a full gate: the projection's rows stay 32-bit (split-K partial sums included)
+    def _bind_head_decay(self, tensors):
+        f32 = lambda name: tensors[name].to(torch.float32).contiguous()
+        self.w_in = _cat([tensors[n] for n in ("q", "k", "v", "g", "a", "b")])       # one product feeds all six
+        self.conv = torch.cat([f32("q.conv"), f32("k.conv"), f32("v.conv")], dim=0).t().contiguous()      # [taps, channels]
+        self.a_log, self.dt_bias, self.norm = f32("A_log"), f32("dt_bias"), f32("norm")
+        self.w_o = tensors["o"].contiguous()
+
+    def _forward_head_decay(self, x, step, state):
+        C, H, qk, hv = self.channels, self.heads, self.qk, self.hv
+        proj = ops.linear(x, self.w_in, out_dtype=torch.float32, allow_partials=True)
+        cols = lambda at, n: ops.Columns(proj, at, n)
+        tail = state[:, self.s_size:].view(state.shape[0], self.taps - 1, C)
+        qkv = torch.empty((x.shape[0], C), dtype=torch.float32, device=x.device)
+        q, k, v = qkv[:, :qk], qkv[:, qk:2 * qk], qkv[:, 2 * qk:]
+        decay, beta = ops.conv_heads(
+            cols(0, C), self.conv, tail, step,
+            [ops.ConvSegment(qk, self.dim, q, "unit", self.dim ** -0.5), ops.ConvSegment(qk, self.dim, k, "unit"),
+             ops.ConvSegment(hv, self.vdim, v)], activation="silu", unit_eps=self.UNIT_EPS,
+            decay=("delta", cols(C + hv, H), cols(C + hv + H, H), self.a_log, self.dt_bias))
+        o = ops.linear_recurrence(q, k, v, decay, beta, 1.0, state[:, :self.s_size], H, self.kv_heads, self.dim, self.vdim, step)
+        y = ops.head_norm_gate(o, self.norm, self.eps, cols(C, hv), "silu", H, self.vdim, self.ctx.dtype)
+        return ops.linear(y, self.w_o, out_dtype=self.ctx.dtype, allow_partials=True)
+
     def forward(self, x, step, cache):
+        if self.head_decay:
+            return self._forward_head_decay(x, step, cache.state)
         C, H, qk = self.channels, self.heads, self.qk
         proj = ops.linear(x, self.w_in, out_dtype=self.ctx.dtype)
         state = cache.state
@@ -206,8 +247,11 @@ class GatedDeltaRule(Mixer):
 
 class ParallelMixer(Mixer):
     """Two mixers side by side on the same input: ``left_scale * left(h) + right_scale * right(h)``.  Each keeps its
-    own cache or state (``cache_need`` gives both by name).  ``forward`` hands back the two scaled updates as a pair;
-    the block adds them (inside its norm's kernel)."""
+    own caches and states (``cache_need`` gives both by name).  ``forward`` hands back the two scaled updates as a pair;
+    the block adds them (inside its norm's kernel), and with them ``output_bias``, the scaled sum of what the branches'
+    output projections add to every token."""
+
+    output_bias = None
 
     def __init__(self, params, ctx):
         super().__init__(params, ctx)
@@ -229,6 +273,9 @@ class ParallelMixer(Mixer):
         from .base import take
         self.left.bind(take(tensors, self.names[0]))
         self.right.bind(take(tensors, self.names[1]))
+        biases = [s * m.output_bias for s, m in ((self.left_scale, self.left), (self.right_scale, self.right))
+                  if getattr(m, "output_bias", None) is not None]
+        self.output_bias = sum(biases[1:], biases[0]).contiguous() if biases else None
 
     def cache_need(self):
         needs = {"left": self.left.cache_need(), "right": self.right.cache_need()}

@@ -14,7 +14,10 @@ largest scores and let only experts of the best groups be chosen; ``weight_scale
 ``activation: silu_gated`` makes an expert W_down (silu(W_gate h) * (W_up h)); ``shared`` (a feed-forward part) runs
 for every token beside the routed experts, and ``forward`` then hands back the pair (routed, shared) for the block
 to add.  ``score: top_logits`` chooses the ``top`` largest logits themselves (``router_bias``: a bias ``router.b`` on the
-logits) and weights them by the softmax over the chosen logits alone.  ``activation: clamped_gated`` makes an expert
+logits) and weights them by the softmax over the chosen logits alone.  ``weights_on: input`` multiplies an expert's INPUT by
+its weight (the output is the sum of expert(w h)): w meets the gate's and the up product's sums, since W (w h) = w (W h).
+``shared_gate`` names a tensor [1, hidden] behind the shared expert's prefix: sigmoid(W_sg h), one number per token, multiplies
+the shared expert's output as it is added to the stream; its product runs in the router's kernel.  ``activation: clamped_gated`` makes an expert
 W_down (g' sigmoid(``act_alpha`` g') (u' + 1)) with g' = min(W_gate h, ``limit``) and u' = clamp(W_up h, -limit, limit).
 
 The chosen (token, expert) pairs are laid out by expert on the device, in whole tiles, and two
@@ -73,6 +76,14 @@ class RoutedExperts(FeedForward):
         self.shared = make_part(params["shared"], ctx) if params.get("shared") is not None else None
         self.shared_name = params.get("shared_name", "shared.")
         self.gate_name = params.get("gate_name", "gate")
+        if params.get("weights_on", "output") not in ("output", "input"):
+            raise ValueError(f"experts' weights are on their outputs or their inputs, not {params['weights_on']!r}")
+        self.weighted_input = params.get("weights_on", "output") == "input"
+        self.shared_gate = params.get("shared_gate")
+        if self.weighted_input and (act != "silu_gated" or self.identity):
+            raise ValueError("weights on the experts' inputs are built for silu-gated experts without identity experts")
+        if self.shared_gate and (self.shared is None or self.top_logits or not self.general_route):
+            raise ValueError("a gate on the shared expert goes with a shared expert and sigmoid scores (or groups of experts)")
         self.outputs = self.experts + self.identity
         if not 1 <= self.top <= self.outputs:
             raise ValueError(f"{self.top} of {self.outputs} router outputs cannot be chosen")
@@ -95,10 +106,16 @@ class RoutedExperts(FeedForward):
         if self.shared is not None:
             from .base import prefixed
             specs.update(prefixed(self.shared_name, self.shared.tensor_specs()))
+        if self.shared_gate:
+            specs[self.shared_name + self.shared_gate] = TensorSpec((1, self.hidden))
         return specs
 
     def bind(self, tensors):
         self.w_router = tensors["router"].contiguous()
+        if self.shared_gate:         # one more row of the router's product
+            sg = tensors[self.shared_name + self.shared_gate]
+            both = [self.w_router, sg] if sg.dtype == self.w_router.dtype else [self.w_router.to(torch.float32), sg.to(torch.float32)]
+            self.w_router = torch.cat(both, dim=0).contiguous()
         self.correction = tensors["correction"].to(torch.float32).contiguous() if self.has_correction else None
         self.bias = tensors["router.b"].to(torch.float32).contiguous() if self.router_bias else None
         ups = [tensors[self.expert_names.format(e) + "up"] for e in range(self.experts)]
@@ -118,22 +135,43 @@ class RoutedExperts(FeedForward):
         self.w_down = torch.stack(downs).contiguous() if downs else torch.empty((0, self.hidden, self.inter), device=dev)
 
     def forward(self, x):
-        routed = self.routed(x)
+        chosen, weight, gate = self._route(x)
+        routed = self._experts(x, chosen, weight)
         if self.shared is None:
             return routed
-        return routed, self.shared.forward(x)
+        shared = self.shared.forward(x)
+        return routed, (shared if gate is None else ops.RowScaled(shared, gate))
 
-    def _act(self, mid2):
+    def _act(self, mid2, row_weight=None):
         """Between an expert's two products, where the first one's kernel has not done it: the gate."""
         if self.clamped:
             return ops.clamped_gate(mid2, self.limit, self.act_alpha, 1.0, self.ctx.dtype)
-        return ops.swiglu(mid2, out_dtype=self.ctx.dtype, activation="silu") if self.gated else mid2
+        if not self.gated:
+            return mid2
+        if row_weight is not None:
+            return ops.swiglu(mid2, out_dtype=self.ctx.dtype, activation="silu", row_scale=row_weight)
+        return ops.swiglu(mid2, out_dtype=self.ctx.dtype, activation="silu")
 
-    def routed(self, x):
-        T = x.shape[0]
-        relu2 = not self.gated
+    def _align(self, chosen, weight, tile):
+        """The pairs by expert; the weights of their rows where the experts' inputs are weighted."""
+        if not self.weighted_input:
+            return (*ops.moe_align(chosen, self.experts, tile), None)
+        return ops.moe_align(chosen, self.experts, tile, weight)
+
+    def _route(self, x):
+        """The chosen experts and their weights, and the shared expert's gate (float32 [T]) if it has one."""
+        gate = None
         if self.top_logits:
             chosen, weight = ops.moe_router_top_logits(x, self.w_router, self.bias, self.top)
+        elif self.shared_gate and self.hidden <= 32768:
+            chosen, weight, gate = ops.moe_router_grouped(x, self.w_router, self.top, self.score, self.groups, self.groups_kept,
+                                                          self.weight_scale, self.renormalize, correction=self.correction, extra=1)
+            gate = gate.view(-1)
+        elif self.shared_gate:
+            logits = ops.linear_cuda_cores(x, self.w_router, out_dtype=torch.float32)
+            chosen, weight = ops.moe_route_grouped(logits[:, :self.outputs].contiguous(), self.top, self.score, self.groups, self.groups_kept,
+                                                   self.weight_scale, self.renormalize, correction=self.correction)
+            gate = ops.sigmoid_rows(logits[:, self.outputs:]).view(-1)
         elif self.general_route and self.hidden <= 32768:
             chosen, weight = ops.moe_router_grouped(x, self.w_router, self.top, self.score, self.groups, self.groups_kept,
                                                     self.weight_scale, self.renormalize, correction=self.correction)
@@ -146,22 +184,28 @@ class RoutedExperts(FeedForward):
         else:
             logits = ops.linear_cuda_cores(x, self.w_router, out_dtype=torch.float32)     # 32-bit multiply-adds
             chosen, weight = ops.moe_route(logits, self.correction, self.top, self.renormalize)
+        return chosen, weight, gate
+
+    def _experts(self, x, chosen, weight):
+        T = x.shape[0]
+        relu2 = not self.gated
+        out_weight = None if self.weighted_input else weight
         pairs = T * self.top
         if pairs >= self.tensor_core_pairs and x.dtype == torch.bfloat16 and self.experts > 0 \
                 and ops.linear_grouped_tensor_ok(self.w_up) and ops.linear_grouped_tensor_ok(self.w_down):
             # a prompt's portion in bfloat16: the pairs' rows are gathered by expert into tiles of 128 and
             # both products run on the tensor cores
             tile = ops.MOE_TILE_ROWS_TENSOR
-            row_token, row_self, pair_row, tile_expert, n_tiles = ops.moe_align(chosen, self.experts, tile)
+            row_token, row_self, pair_row, tile_expert, n_tiles, row_weight = self._align(chosen, weight, tile)
             rows = row_token.numel()
             xs = ops.gather_rows(x, row_token)
             mid = torch.empty((rows, self.up_rows), dtype=self.ctx.dtype, device=x.device)
             ops.linear_grouped_tensor(xs, self.w_up, mid, tile_expert, relu2=relu2, pairs=pairs)
             y = torch.empty((rows, self.hidden), dtype=torch.float32, device=x.device)
-            ops.linear_grouped_tensor(self._act(mid), self.w_down, y, tile_expert, pairs=pairs)
-            return ops.moe_combine(y, x, chosen, weight, pair_row, self.experts)
+            ops.linear_grouped_tensor(self._act(mid, row_weight), self.w_down, y, tile_expert, pairs=pairs)
+            return ops.moe_combine(y, x, chosen, out_weight, pair_row, self.experts)
         tile = ops.MOE_TILE_ROWS if pairs > 16 * max(self.experts, 1) else ops.MOE_TILE_ROWS_SMALL
-        row_token, row_self, pair_row, tile_expert, n_tiles = ops.moe_align(chosen, self.experts, tile)
+        row_token, row_self, pair_row, tile_expert, n_tiles, row_weight = self._align(chosen, weight, tile)
         rows = row_token.numel()
         mid = torch.empty((rows, self.up_rows), dtype=self.ctx.dtype, device=x.device)
         y = torch.empty((rows, self.hidden), dtype=torch.float32, device=x.device)
@@ -169,8 +213,8 @@ class RoutedExperts(FeedForward):
                 and ops.linear_few_rows_ok(mid[:, :self.inter], self.w_down):
             # few rows per expert (a decode step): the experts' weights are streamed once, bound by memory
             ops.linear_few_rows(x, self.w_up, mid, row_token, tile_expert, n_tiles, relu2=relu2)
-            ops.linear_few_rows(self._act(mid), self.w_down, y, row_self, tile_expert, n_tiles)
+            ops.linear_few_rows(self._act(mid, row_weight), self.w_down, y, row_self, tile_expert, n_tiles)
         else:
             ops.linear_grouped(x, self.w_up, mid, row_token, tile_expert, n_tiles, tile, relu2=relu2)
-            ops.linear_grouped(self._act(mid), self.w_down, y, row_self, tile_expert, n_tiles, tile)
-        return ops.moe_combine(y, x, chosen, weight, pair_row, self.experts)
+            ops.linear_grouped(self._act(mid, row_weight), self.w_down, y, row_self, tile_expert, n_tiles, tile)
+        return ops.moe_combine(y, x, chosen, out_weight, pair_row, self.experts)
