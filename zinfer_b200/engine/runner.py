@@ -109,9 +109,7 @@ class ModelRunner:
         return self.manager.has_request(request_id)
 
     def add_request(self, request_id: Hashable) -> None:
-        rc = self.manager.add_request(request_id)
-        if self.storage.state:
-            self.storage.reset_slot(rc.state_slot)
+        self.manager.add_request(request_id)
 
     def end_request(self, request_id: Hashable) -> None:
         """Gives back everything the request holds."""
@@ -178,6 +176,10 @@ class ModelRunner:
         if any(e.token_src is not None for e in entries) and prev_tokens is None:
             raise StepError("an entry takes its token from the step before, but no such tokens were given")
         self.reserve(entries)
+        if self.storage.state:      # a request's first tokens find its state zero, whoever admitted it and whatever held the slot before
+            for e in entries:
+                if self.manager.length(e.request_id) == 0:
+                    self.storage.reset_slot(self.manager.requests[e.request_id].state_slot)
         if profiling.ACTIVE is not None:
             profiling.ACTIVE.begin_step()    # profiled steps launch their kernels one by one, never from a graph
         if self.graphs is not None and profiling.ACTIVE is None and self.graphs.eligible(entries):
