@@ -19,6 +19,11 @@ class Scaled:
         self.delta, self.scale = delta, float(scale)
 
 
+class RowScaled:
+    def __init__(self, delta, rows):
+        self.delta, self.rows = delta, rows
+
+
 class Several:
     def __init__(self, terms, row_bias=None):
         self.terms, self.row_bias = [], row_bias
@@ -40,6 +45,8 @@ def _terms_sum(delta):
         scale = 1.0
         if isinstance(t, Scaled):
             t, scale = t.delta, t.scale
+        if isinstance(t, RowScaled):
+            t = t.rows.view(-1, 1) * t.delta.to(torch.float32)
         v = torch.tensor(scale, dtype=torch.float32) * t.to(torch.float32)
         total = v if total is None else total + v
     return total
@@ -149,12 +156,14 @@ def linear_swiglu(x, w_interleaved, out_dtype=None, activation="silu"):
     return swiglu(linear(x, w_interleaved, out_dtype=torch.float32), interleave=64, activation=activation).to(out_dtype or x.dtype)
 
 
-def swiglu(gate_up, out=None, out_dtype=None, interleave=0, activation="silu"):
+def swiglu(gate_up, out=None, out_dtype=None, interleave=0, activation="silu", row_scale=None):
     I = gate_up.shape[1] // 2
     if interleave:
         blocks = gate_up.reshape(gate_up.shape[0], I // interleave, 2, interleave)
         gate_up = torch.cat([blocks[:, :, 0].reshape(-1, I), blocks[:, :, 1].reshape(-1, I)], dim=1)
     g, u = gate_up[:, :I].to(torch.float32), gate_up[:, I:].to(torch.float32)
+    if row_scale is not None:
+        g, u = g * row_scale.view(-1, 1), u * row_scale.view(-1, 1)
     if activation == "gelu_tanh":
         return (gelu_tanh(g) * u).to(out_dtype or gate_up.dtype)
     return (g / (1.0 + torch.exp(-g)) * u).to(out_dtype or gate_up.dtype)
@@ -267,7 +276,7 @@ def linear_few_rows_ok(x, weight):
     return False
 
 
-def moe_align(chosen, experts, tile_rows):
+def moe_align(chosen, experts, tile_rows, weight=None):
     T, top = chosen.shape
     flat = chosen.reshape(-1).tolist()
     row_token, row_self, tile_expert = [], [], []
@@ -287,6 +296,11 @@ def moe_align(chosen, experts, tile_rows):
     row_token += [-1] * (cap - len(row_token))
     row_self += [-1] * (cap - len(row_self))
     i32 = lambda v: torch.tensor(v, dtype=torch.int32)
+    if weight is not None:
+        row_weight = torch.zeros(cap, dtype=torch.float32)
+        for p, r in enumerate(pair_row):
+            row_weight[r] = weight.reshape(-1)[p]
+        return (*moe_align(chosen, experts, tile_rows), row_weight)
     return i32(row_token), i32(row_self), i32(pair_row), i32(tile_expert + [0] * (cap // tile_rows - n_tiles)), i32([n_tiles])
 
 
@@ -313,7 +327,7 @@ def moe_combine(y, x, chosen, weight, pair_row, experts):
         for k in range(top):
             e = int(chosen[t, k])
             v = y[int(pair_row[t * top + k])] if e < experts else x[t].to(torch.float32)
-            out[t] += weight[t, k] * v
+            out[t] += v if weight is None else weight[t, k] * v
     return out.to(x.dtype)
 
 
@@ -640,7 +654,9 @@ def sigmoid_rows(x):
     return torch.sigmoid(x.to(torch.float32)).contiguous()
 
 
-def linear_recurrence(q, k, v, decay, beta, q_scale, state, heads, key_heads, dim, vdim, step):
+def linear_recurrence(q, k, v, decay, beta, q_scale, state, heads, key_heads, dim, vdim, step, delta=True):
+    if decay.shape[1] == heads:
+        decay = decay.repeat_interleave(dim, dim=1)
     T = q.shape[0]
     out = torch.zeros((T, heads * vdim), dtype=torch.float32)
     rep = heads // key_heads
@@ -654,16 +670,70 @@ def linear_recurrence(q, k, v, decay, beta, q_scale, state, heads, key_heads, di
                 Sh = decay[t, h * dim:(h + 1) * dim].unsqueeze(-1) * S[h]
                 u = vf[t, h * vdim:(h + 1) * vdim]
                 if beta is not None:
-                    u = beta[t, h] * (u - Sh.T @ kk)
+                    u = beta[t, h] * (u - Sh.T @ kk if delta else u)
                 S[h] = Sh + kk.unsqueeze(-1) * u.unsqueeze(0)
                 out[t, h * vdim:(h + 1) * vdim] = S[h].T @ qq
         state[slot] = S.reshape(state[slot].shape)
     return out
 
 
+class Columns:
+    def __init__(self, proj, at, width):
+        self.value, self.width = proj[:, at:at + width], width
+        self.shape = self.value.shape
+
+
+class ConvSegment:
+    def __init__(self, channels, head_dim, out, finish=None, scale=1.0):
+        self.channels, self.head_dim, self.out, self.finish, self.scale = channels, head_dim, out, finish, scale
+
+
+def conv_heads(u, kernel, tail, step, segments, in_bias=None, out_bias=None, activation=None, unit_eps=0.0, tables=(None, None),
+               rot_dims=0, pairing="halves", slots=None, page_size=0, decay=None):
+    x = u.value.to(torch.float32) + (in_bias if in_bias is not None else 0.0)
+    taps, C = kernel.shape
+    if tail is None:
+        tail = torch.zeros((int(step.state_slots.max()) + 1, 0, C))
+    y = short_conv(x, kernel.T, tail, step, None) + (out_bias if out_bias is not None else 0.0)
+    short_conv_carry(x, taps, tail, step)
+    if activation == "silu":
+        y = y * torch.sigmoid(y)
+    at, T = 0, x.shape[0]
+    for s in segments:
+        v = y[:, at:at + s.channels].reshape(T, -1, s.head_dim)
+        at += s.channels
+        if s.finish == "unit":
+            v = s.scale * v / torch.sqrt((v * v).sum(-1, keepdim=True) + unit_eps)
+        elif s.finish == "rotate" and tables[0] is not None:
+            cos, sin = (t[step.positions.long()].unsqueeze(1) for t in tables)
+            v = (_rotate_neighbours if pairing == "neighbours" else _rotate_first)(v, cos, sin, rot_dims)
+        if s.out.dim() == 4:
+            for t in range(T):
+                slot = int(slots[t])
+                if slot >= 0:
+                    s.out[slot // page_size, :, slot % page_size] = v[t].to(s.out.dtype)
+        else:
+            s.out[:, :s.channels] = v.reshape(T, -1).to(s.out.dtype)
+    if decay is None:
+        return None
+    kind, a, b, a_log, dt_bias = decay
+    sp = torch.nn.functional.softplus(a.value.to(torch.float32) + dt_bias)
+    return torch.exp(-torch.exp(a_log) * sp), sp if kind == "ssd" else torch.sigmoid(b.value.to(torch.float32))
+
+
+def gated_part_norm(y, gate, weight, eps, parts, out_dtype, skip=None, x=None, vdim=1):
+    T, W = y.shape
+    v = y if skip is None else y + skip.repeat_interleave(vdim) * x[:, :W]
+    z = gate.value.to(torch.float32)
+    v = (v * z * torch.sigmoid(z)).reshape(T, parts, W // parts)
+    return ((v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps)).reshape(T, W) * weight).to(out_dtype)
+
+
 def head_norm_gate(o, weight, eps, gate, gate_kind, heads, vdim, out_dtype):
     T = o.shape[0]
     x = o.reshape(T, heads, vdim)
+    if isinstance(gate, Columns):
+        gate = gate.value
     if gate_kind == "none":
         return (x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * weight).reshape(T, heads * vdim).to(out_dtype)
     g = gate.to(torch.float32).reshape(T, heads, vdim)
@@ -687,7 +757,10 @@ def moe_route_grouped(logits, top, score="sigmoid", groups=1, keep=1, scale=1.0,
     return chosen.to(torch.int32), (weight * scale).to(torch.float32)
 
 
-def moe_router_grouped(x, w_router, top, score="sigmoid", groups=1, keep=1, scale=1.0, renormalize=False, correction=None):
+def moe_router_grouped(x, w_router, top, score="sigmoid", groups=1, keep=1, scale=1.0, renormalize=False, correction=None, extra=0):
+    if extra:
+        gates = torch.sigmoid(x.to(torch.float32) @ w_router[-extra:].to(torch.float32).T)
+        return (*moe_router_grouped(x, w_router[:-extra], top, score, groups, keep, scale, renormalize, correction), gates)
     return moe_route_grouped(x.to(torch.float32) @ w_router.to(torch.float32).T, top, score, groups, keep, scale, renormalize,
                              correction)
 
