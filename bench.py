@@ -27,7 +27,8 @@ Luvavik (the nearest design the engine has) and Qwen3, and ``--design vumezen`` 
 Rogosun (whose attention with a sink and routed experts beside a shared one are the nearest the engine has) and Qwen3, and
 ``--design sepitar`` for the Sepitar design, beside Vumezen, Luvavik and Qwen3, and ``--design kesitar`` for the Kesitar
 design, beside Rogosun (the nearest recurrence; its feed-forwards all dense here), Vumezen (the nearest attention) and Qwen3
-with the same feed-forward; ``--profile PATH`` adds both models' per-kernel-class times and
+with the same feed-forward, and ``--design sumozen`` for the Sumozen design, beside Rogosun (the nearest mixers and experts; experts
+in every layer here) and Qwen3; ``--profile PATH`` adds both models' per-kernel-class times and
 roofline fractions.  The default workload and its output line are untouched.
 
 Peaks come from MEASURED_PEAKS.json when the driver wrote it, else the fallback
@@ -225,6 +226,24 @@ def kesitar_shape(width: int, heads: int, dense_ff: int) -> dict:
             "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0}, "logit_scale": 1.0, "max_position_embeddings": 8192}
 
 
+def sumozen_shape(width: int, heads: int, experts: int, top: int, expert_ff: int) -> dict:
+    """A Sumozen configuration with layers the size of a real model's: Mamba-2 as wide as the model (heads of 64 channels, a
+    state of 128, two groups, four norm groups, four taps); parallel layers of attention with biases, convolutions of
+    three taps and a capped score (heads of 128, four query heads per kv head, rescaled rotation of the whole head) beside a
+    gated delta rule (heads of 128 x 256 behind convolutions of four taps); experts whose inputs are weighted beside a gated
+    shared expert in every layer.  Seven layers."""
+    g = max(1, width // 256)
+    mam = {"type": "mamba2", "mixer": {"heads": width // 64, "vdim": 64, "state": 128, "groups": 2, "norm_groups": 4, "conv": 4}}
+    par = {"type": "parallel", "mixer": {
+        "left": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "conv": 3, "softcap": 50.0,
+                 "rot": {"base": 1000000.0, "dims": 128, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}},
+        "right": {"heads": g, "kv_heads": max(1, g // 2), "dim": 128, "vdim": 256, "conv": 4}, "left_scale": 0.8, "right_scale": 0.5}}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "shared": {"ff": expert_ff}, "router": {"experts": experts, "top": top}}
+    layers = [dict(lay, mlp=moe) for lay in (mam, par, mam, mam, par, mam, par)]
+    return {"architecture": "Sumozen", "vocab": 32768, "width": width, "layers": layers, "norm": {"eps": 1e-6},
+            "max_position_embeddings": 8192}
+
+
 DESIGN_SIZES = {
     # name: (width, heads, experts, chosen, expert ff, dense ff); Qwen3 beside it: the same width, layer runs and
     # heads of 128, a feed-forward as wide as the chosen experts together (equal products per token)
@@ -317,6 +336,17 @@ def compare_designs(args) -> int:
             results[f"vumezen_{size}"] = measure(f"vumezen_{size}", VumezenConfig.from_dict(own), own["vocab"])
             other = rogosun_shape(width, heads, experts, top, eff, dff)
             results[f"rogosun_{size}"] = measure(f"rogosun_{size}", RogosunConfig.from_dict(other), other["vocab"])
+        elif args.design == "sumozen":
+            # beside Rogosun (attention beside a delta rule on the same input, linear recurrences with a matrix state, experts
+            # beside a shared one) with routed experts in every layer, and Qwen3
+            from zinfer_b200.config import RogosunConfig, SumozenConfig
+            own = sumozen_shape(width, heads, experts, top, eff)
+            results[f"sumozen_{size}"] = measure(f"sumozen_{size}", SumozenConfig.from_dict(own), own["vocab"])
+            other = rogosun_shape(width, heads, experts, top, eff, dff)
+            routed = next(lay["mlp"] for lay in other["layers"] if lay["mlp"]["kind"] == "moe")
+            for lay in other["layers"]:
+                lay["mlp"] = routed
+            results[f"rogosun_{size}"] = measure(f"rogosun_{size}", RogosunConfig.from_dict(other), other["vocab"])
         elif args.design == "sepitar":
             # beside Vumezen (blocks whose sublayers read one stream, attention with a window and a sink on the same
             # tensor-core kernels, experts beside a shared one), Luvavik (latent attention) and Qwen3
@@ -351,6 +381,7 @@ def compare_designs(args) -> int:
         with open(args.profile, "w") as f:
             json.dump(profiles, f, indent=1)
     names = {"rogosun": "Rogosun beside Luvavik and Qwen3 dense", "vumezen": "Vumezen beside Rogosun and Qwen3 dense",
+             "sumozen": "Sumozen beside Rogosun (routed experts in every layer) and Qwen3 dense",
              "sepitar": "Sepitar beside Vumezen, Luvavik and Qwen3 dense",
              "kesitar": "Kesitar beside Rogosun (dense feed-forwards), Vumezen and Qwen3 dense"}.get(
         args.design, "Luvavik beside Qwen3 dense")
@@ -377,7 +408,7 @@ def main() -> int:
                     help="with ZINFER_B200_TRACE=1 in the environment: write the timeline of one decode step at the "
                          "headline batch (every kernel's start, the completion of what it depends on, and what it adds "
                          "to the chain) there as JSON, and do nothing else")
-    ap.add_argument("--design", default=None, choices=["luvavik", "rogosun", "vumezen", "sepitar", "kesitar"],
+    ap.add_argument("--design", default=None, choices=["luvavik", "rogosun", "vumezen", "sepitar", "kesitar", "sumozen"],
                     help="instead of the default benchmark: prefill and decode throughput of this design at layer sizes "
                          "of real models beside Qwen3 dense at equal size (a JSON line of its own)")
     ap.add_argument("--design-sizes", default=None, help="with --design: widths to run, e.g. 2048 or 2048,4096")

@@ -324,12 +324,10 @@ def test_long_memory_is_real_and_a_lost_state_would_show(tmp_path, kind):
     later), so a state that is lost, reset or taken from another slot cannot pass; and a request in a used slot starts
     from nothing."""
     n = 220
-    layer = {"mamba2": U.mam(2, 16, 16, 1, 1, 3), "delta": U.par(U.att(1, 1, 8, 8, 1.0, 1), U.delta(2, 2, 8, 8, 3), 1e-3, 1.0),
+    layer = {"mamba2": U.mam(2, 16, 16, 1, 1, 3), "delta": U.par(U.att(1, 1, 8, 8, 1.0, 1), U.delta(2, 2, 64, 8, 3), 1e-3, 1.0),
              "conv": U.par(U.att(1, 1, 8, 8, 1.0, 17), U.delta(1, 1, 8, 8, 17), 1.0, 1.0)}[kind]
     cfg = U.config(67, 32, [layer])
     weights = U.make_weights(cfg, seed=51, slow=True)
-    if kind == "delta":
-        weights["l0.mix.right.b"] = (weights["l0.mix.right.b"].float() * 0.2 - 0.0).to(torch.bfloat16)
     toks = ru.make_requests(cfg["vocab"], [n], seed=8)["r0"]
     reqs = {"r0": toks, "r1": [(toks[0] + 1) % cfg["vocab"]] + toks[1:], "r2": toks[:5]}
     plain = U.plain_logits(cfg, weights, reqs)
@@ -342,24 +340,45 @@ def test_long_memory_is_real_and_a_lost_state_would_show(tmp_path, kind):
             ru.assert_close(ru.run_in_process(runner, trace), plain, what=f"memory of {kind}", argmax_frac=0.0, **TOL[dtype])
 
 
+def _far_key(dim):
+    """One attention layer whose queries all point the same way (a large bias, nothing along the rotated dimensions), and 270
+    tokens of which only number 19 has a key along it."""
+    cfg = U.config(67, 32, [U.par(U.att(2, 1, dim, dim, 1.0 / dim ** 0.5, 2, rot=(4, 1e4), softcap=25.0), U.delta(1, 1, 8, 8, 2), 1.0, 1e-3)])
+    w = U.make_weights(cfg, seed=41)
+    f = lambda n: w["l0.mix.left." + n].float()
+    q, b = f("q").view(2, dim, -1) * 0.1, f("q.b").view(2, dim) * 9.0 + 3.0
+    q[:, :4], b[:, :4] = 0.0, 0.0
+    own = torch.tensor([0.1, 1.0])
+    for n, t in (("q", q), ("q.b", b), ("q.conv", own), ("k.conv", own), ("v.conv", own)):
+        old = w["l0.mix.left." + n]
+        w["l0.mix.left." + n] = (t.reshape(old.shape) if t.numel() == old.numel() else t.expand(old.shape)).to(torch.bfloat16).contiguous()
+    k = P.model_norm(w["embed"].double(), w["l0.norm1"], 1e-5) @ w["l0.mix.left.k"].double().T + w["l0.mix.left.k.b"].double()
+    order = (k @ b.mean(0).double()).argsort(descending=True).tolist()
+    quiet, rng = order[len(order) // 2:], np.random.default_rng(7)
+    toks = [int(rng.choice(quiet)) for _ in range(270)]
+    toks[19] = order[0]
+    return cfg, w, toks
+
+
+@pytest.mark.parametrize("dim", [8, 64])
+def test_the_far_key_matters(dim):
+    """In the plain model the last positions' logits are others without the one loud token 250 tokens back."""
+    cfg, weights, toks = _far_key(dim)
+    right = P.PlainSumozen(cfg, weights).forward(toks)[-5:].numpy()
+    lost = P.PlainSumozen(cfg, weights).forward(toks[:19] + [toks[18]] + toks[20:])[-5:].numpy()
+    assert (np.abs(right - lost).max(-1) > 0.2 * np.abs(right).max(-1)).all()
+
+
 @gpu
 @pytest.mark.parametrize("dim", [8, 64])
 def test_a_single_far_key_decides(tmp_path, dim):
-    """One key 250 tokens back carries much of the last query's softmax: among the tokens that could stand at position 19
-    the test takes the one whose presence moves the last position's logits most in the plain model, and requires that
-    move to be large; an engine that lost that key could not match."""
-    cfg = U.config(67, 32, [U.par(U.att(2, 1, dim, dim, 4.0 / dim ** 0.5, 2, rot=(4, 1e6), softcap=30.0), U.delta(1, 1, 8, 8, 2), 1.0, 1e-3)])
-    weights = U.make_weights(cfg, seed=41)
-    toks = ru.make_requests(cfg["vocab"], [270], seed=7)["r0"]
-    last = lambda t: P.PlainSumozen(cfg, weights).forward(t)[-1].numpy()
-    lost = last(toks[:19] + [toks[18]] + toks[20:])
-    move = {c: np.abs(last(toks[:19] + [c] + toks[20:]) - lost).max() for c in range(0, cfg["vocab"], 5)}
-    toks[19] = max(move, key=move.get)
+    """One key 250 tokens back carries much of the last queries' softmax (the test above), on the exact kernel and on the
+    tensor-core kernels; an engine that lost that key could not match."""
+    cfg, weights, toks = _far_key(dim)
     plain = U.plain_logits(cfg, weights, {"r0": toks})
-    assert np.abs(plain["r0"][-1] - lost).max() > 0.1 * np.abs(plain["r0"][-1]).max()     # the far key matters
     for dtype in (torch.float32, torch.bfloat16):
         runner = make_runner(tmp_path, cfg, weights, dtype, DEV, page_size=16, max_tokens=288, max_requests=1)
-        for trace in (ru.trace_whole({"r0": toks}), ru.trace_tail_decode({"r0": toks}, 5)):
+        for trace in (ru.trace_whole({"r0": toks}), ru.trace_tail_decode({"r0": toks}, 5), ru.trace_portions({"r0": toks}, 2)):
             ru.assert_close(ru.run_in_process(runner, trace), plain, what="one far key", argmax_frac=0.0, **TOL[dtype])
 
 
