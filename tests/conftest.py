@@ -81,7 +81,7 @@ def cpu_kernels(monkeypatch):
                  "decay_sigmoid_root_", "decay_exp_softplus_", "unit_norm_", "sigmoid_rows", "linear_recurrence", "head_norm_gate",
                  "moe_route_grouped", "moe_router_grouped", "Several", "sum_norm", "add_rmsnorm_pair", "embed_bigram",
                  "clamped_gate", "rmsnorm_rows", "rope_table_freqs", "qkv_rows_prepare", "latent_prepare_rows", "moe_router_top_logits",
-                 "PostNormed", "PooledKeys", "RowScaled", "Columns", "ConvSegment", "conv_heads", "gated_part_norm", "sandwich_norm", "qkv_heads_prepare", "pool_blocks", "linear_recurrence_gated"):
+                 "PostNormed", "PooledKeys", "RowScaled", "Columns", "ConvSegment", "conv_heads", "head_decay_recurrence", "gated_part_norm", "sandwich_norm", "qkv_heads_prepare", "pool_blocks", "linear_recurrence_gated"):
         monkeypatch.setattr(ops, name, getattr(kernel_refs, name))
     monkeypatch.setattr(ops, "lib", lambda: None)
     monkeypatch.setattr(runner, "_require_cuda", lambda device: None)

@@ -654,9 +654,9 @@ def sigmoid_rows(x):
     return torch.sigmoid(x.to(torch.float32)).contiguous()
 
 
-def linear_recurrence(q, k, v, decay, beta, q_scale, state, heads, key_heads, dim, vdim, step, delta=True):
-    if decay.shape[1] == heads:
-        decay = decay.repeat_interleave(dim, dim=1)
+def linear_recurrence(q, k, v, decay, beta, q_scale, state, heads, key_heads, dim, vdim, step, delta=True, log_decay=None):
+    if decay is None:
+        decay = torch.exp(log_decay).repeat_interleave(dim, dim=1)
     T = q.shape[0]
     out = torch.zeros((T, heads * vdim), dtype=torch.float32)
     rep = heads // key_heads
@@ -675,6 +675,10 @@ def linear_recurrence(q, k, v, decay, beta, q_scale, state, heads, key_heads, di
                 out[t, h * vdim:(h + 1) * vdim] = S[h].T @ qq
         state[slot] = S.reshape(state[slot].shape)
     return out
+
+
+def head_decay_recurrence(q, k, v, log_decay, beta, state, heads, key_heads, dim, vdim, step, delta, fast):
+    return linear_recurrence(q, k, v, None, beta, 1.0, state, heads, key_heads, dim, vdim, step, delta=delta, log_decay=log_decay)
 
 
 class Columns:
@@ -718,7 +722,7 @@ def conv_heads(u, kernel, tail, step, segments, in_bias=None, out_bias=None, act
         return None
     kind, a, b, a_log, dt_bias = decay
     sp = torch.nn.functional.softplus(a.value.to(torch.float32) + dt_bias)
-    return torch.exp(-torch.exp(a_log) * sp), sp if kind == "ssd" else torch.sigmoid(b.value.to(torch.float32))
+    return -torch.exp(a_log) * sp, sp if kind == "ssd" else torch.sigmoid(b.value.to(torch.float32))
 
 
 def gated_part_norm(y, gate, weight, eps, parts, out_dtype, skip=None, x=None, vdim=1):

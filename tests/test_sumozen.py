@@ -615,8 +615,7 @@ def test_gated_part_norm_and_row_weights_against_plain_arithmetic():
 @pytest.mark.parametrize("D,V,heads,groups", [(16, 8, 4, 2), (24, 40, 4, 4), (130, 33, 3, 1), (64, 64, 8, 2), (128, 128, 2, 1)])
 @pytest.mark.parametrize("delta", [False, True])
 def test_recurrence_with_a_decay_per_head(D, V, heads, groups, delta):
-    """One decay and one step per head: the delta rule, and the plain form with a step size, in unequal portions, in one step
-    and cut in two (the same bits)."""
+    """One decay and one step per head: the delta rule, and the plain form with a step size, in unequal portions."""
     import kernel_refs as R
     from zinfer_b200 import ops
 
@@ -626,10 +625,45 @@ def test_recurrence_with_a_decay_per_head(D, V, heads, groups, delta):
     q, k = (0.3 * torch.randn(T, groups * D, generator=g) for _ in range(2))
     k = R.unit_norm_(k, groups, D, 1e-6)
     v = torch.randn(T, heads * V, generator=g)
-    decay, beta = 0.8 + 0.2 * torch.rand(T, heads, generator=g), torch.rand(T, heads, generator=g)
+    logs, beta = torch.log(0.8 + 0.2 * torch.rand(T, heads, generator=g)), torch.rand(T, heads, generator=g)
     state0 = torch.randn(9, heads, D, V, generator=g)
     sr, sd = state0.clone(), state0.to(DEV)
-    want = R.linear_recurrence(q, k, v, decay, beta, 0.7, sr, heads, groups, D, V, ref, delta=delta)
-    got = ops.linear_recurrence(*(t.to(DEV) for t in (q, k, v, decay, beta)), 0.7, sd, heads, groups, D, V, step, delta=delta)
+    want = R.linear_recurrence(q, k, v, None, beta, 0.7, sr, heads, groups, D, V, ref, delta=delta, log_decay=logs)
+    got = ops.linear_recurrence(q.to(DEV), k.to(DEV), v.to(DEV), None, beta.to(DEV), 0.7, sd, heads, groups, D, V, step, delta=delta, log_decay=logs.to(DEV))
     assert torch.allclose(got.cpu(), want, rtol=1e-4, atol=1e-4 * max(1.0, want.abs().max().item()))
     assert torch.allclose(sd.cpu(), sr, rtol=1e-4, atol=1e-4)
+
+
+@gpu
+@pytest.mark.parametrize("D,V,heads,groups", [(16, 8, 4, 2), (48, 48, 4, 2), (32, 32, 4, 2), (64, 64, 8, 2), (128, 256, 2, 1), (112, 33, 3, 3), (128, 64, 6, 2)])
+@pytest.mark.parametrize("delta", [False, True])
+def test_recurrence_in_chunks_against_one_walk(monkeypatch, D, V, heads, groups, delta):
+    """Long portions in chunks of 64 tokens on the tensor cores give what the walk token by token gives, outputs and states:
+    portions that end at a chunk's edge, one before and one behind it, short ones and single tokens beside them, states that
+    earlier portions left; decays from 1 down to next to nothing."""
+    from zinfer_b200 import ops
+
+    g = torch.Generator(device=DEV).manual_seed(D + V)
+    rnd = lambda *s: torch.randn(*s, generator=g, device=DEV)
+    for lens, strong in (((200, 1, 64, 65), False), ((63, 129, 2, 1), False), ((1000,), True), ((96, 128, 1, 1, 320), True)):
+        step, _ = _steps(lens)
+        T = step.n_tokens
+        rows = rnd(T, 2 * groups * D + heads * V)
+        q, k, v = rows[:, :groups * D], rows[:, groups * D:2 * groups * D], rows[:, 2 * groups * D:]
+        for x in (q, k):
+            x.copy_(torch.nn.functional.normalize(x.reshape(T, groups, D), dim=-1).reshape(T, -1))
+        logs = -torch.rand(T, heads, generator=g, device=DEV) * (0.05 if not strong else 1.0)
+        if strong:
+            logs[::7] = -30.0
+            logs[3::11] = 0.0
+        beta = torch.rand(T, heads, generator=g, device=DEV) * (1.0 if delta else 2.0)
+        state0 = rnd(9, heads, D, V)
+        outs = []
+        for chunks in (False, True):
+            monkeypatch.setattr(ops, "RECURRENCE_CHUNKS", chunks)
+            state = state0.clone()
+            o = ops.head_decay_recurrence(q, k, v, logs, beta, state, heads, groups, D, V, step, delta=delta, fast=True)
+            outs.append((o, state))
+        for a, b in zip(*outs):
+            assert torch.isfinite(b).all() and (a - b).abs().max() <= 1e-4 * max(1.0, a.abs().max().item()), (lens, (a - b).abs().max(), a.abs().max())
+        assert not torch.equal(outs[1][1], state0)

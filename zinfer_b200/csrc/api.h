@@ -228,8 +228,14 @@ int zi_unit_norm(float* x, int ld, int T, int heads, int d, float eps, float sca
 int zi_sigmoid_rows(float* out, int ldo, const void* x, int ldx, int dtype, int rows, int W, cudaStream_t stream);
 int zi_linear_recurrence(float* out, int ldo, const void* q, int ldq, const void* k, int ldk, int qk_dtype, const void* v,
                          int ldv, int v_dtype, const float* decay, int ldg, const float* beta, int ldb, float q_scale,
-                         float* state, long long slot_stride, int H, int G, int D, int V, int delta, int head_decay, const int* cu_q,
-                         const int* state_slots, int n_seqs, cudaStream_t stream);
+                         float* state, long long slot_stride, int H, int G, int D, int V, int delta, int head_decay, int only_single,
+                         const int* cu_q, const int* state_slots, int n_seqs, cudaStream_t stream);
+// Long portions of the recurrences with one decay per head, in chunks (chunked_recurrence.cu)
+int zi_chunked_recurrence_supported(int D, int V, int H, int G);
+long long zi_chunked_recurrence_workspace_floats(int T, int n_seqs, int H, int G, int D, int V, int delta);
+int zi_chunked_recurrence(float* out, int ldo, const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* logg,
+                          const float* beta, float* state, long long slot_stride, int T, int H, int G, int D, int V, int delta,
+                          const int* cu_q, const int* state_slots, int n_seqs, float* workspace, cudaStream_t stream);
 // The form whose forget gate decides what is written: g = l + (1 - l) sigmoid(z + b), k = 1 - g, q = silu(raw q); q, z, v
 // float32 projections, whole (splits 1) or split-K partial sums zstride apart.
 int zi_linear_recurrence_gated(float* out, int ldo, const float* q, int ldq, const float* z, int ldz, const float* v, int ldv,

@@ -1,0 +1,587 @@
+// Long portions of the recurrences with one decay per head and token (linear_attention.cu has the form that walks the
+// tokens one by one), in chunks of 64 tokens whose work is matrix products:
+//
+//     S <- g_t S ;  u_t = beta_t (v_t - S^T k_t) (delta rule)  or  u_t = beta_t v_t ;  S <- S + k_t u_t^T ;  o_t = S^T q_t
+//
+// With c_t = log g_1 + .. + log g_t inside a chunk that begins from S0, the chunk's updates U solve a triangular system,
+// (I + L) U = diag(beta) (V - diag(e^c) K S0) with L_ts = beta_t e^(c_t - c_s) (k_t . k_s) for s < t, so that U = U0 - W S0
+// with (I + L) [W | U0] = diag(beta) [diag(e^c) K | V]; then
+//
+//     O = diag(e^c) Q S0 + P U,  P_ts = e^(c_t - c_s) (q_t . k_s) for s <= t ;   S1 = e^(c_64) S0 + K^T diag(e^(c_64 - c)) U
+//
+// (the chunked form of "Parallelizing Linear Transformers with the Delta Rule over Sequence Length", Yang et al., 2024, and
+// of "Gated Delta Networks", Yang et al., 2024; without the delta rule W = 0 and U = diag(beta) V, the state-space duality of
+// Dao and Gu, 2024).  Three kernels:
+//   1. chunk_scores   per chunk and key head: q . k and k . k (32-bit multiply-adds), Q and K as pairs of bfloat16
+//                     values (high part and remainder: 16 bits of mantissa together), the sums c of every head
+//   2. chunk_solve    (delta rule) per chunk and head: the triangular system by forward substitution in 32-bit, a
+//                     thread per column of [W | U0]; W as pairs of bfloat16 values
+//   3. chunk_walk     per request, head and 32 value channels: the chunks in order; the products with the state on the
+//                     tensor cores (mma.sync, each operand as two bfloat16 parts, three products, 32-bit sums); the state
+//                     stays in 32-bit accumulators
+// Kernels 1 and 2 do all chunks side by side; only the third walks.  A request's chunks begin with its portion; the places of
+// its chunks in the workspace follow from cu_q alone: chunk i of request s lies at cu_q[s] / 64 + s + i.
+#include "api.h"
+#include "common.cuh"
+
+namespace {
+constexpr int CK = 64;               // tokens per chunk
+constexpr int CK_VP = 32;            // value channels per block of the walk
+constexpr int CK_PAD = 8;            // bfloat16 elements behind every row in shared memory: rows start 16 bytes further on
+using bf = __nv_bfloat16;
+
+struct Chunked {
+  const float* q;      // [T][G * D] rows, ready (unit vectors, scale)
+  const float* k;
+  const float* v;      // [T][H * V]
+  int ldq, ldk, ldv;
+  const float* logg;   // [T][H] logarithms of the decays
+  const float* beta;   // [T][H]
+  float* state;
+  long long slot_stride;
+  int H, G, D, V;
+  const int* cu_q;
+  const int* state_slots;
+  int n_seqs, slots;
+  float* out;          // [T][H * V]
+  int ldo;
+  // workspace
+  bf* qs;              // [slots][G][2][CK][D]
+  bf* ks;
+  float* qk;           // [slots][G][CK][CK]
+  float* kk;           // delta rule only
+  float* c;            // [slots][H][CK]
+  bf* w;               // [slots][H][2][CK][D]
+  float* u0;           // [slots][H][CK][V]
+};
+
+__device__ __forceinline__ bool chunk_of(const Chunked& j, int slot, int& seq, int& first, int& n) {
+  int lo = 0, hi = j.n_seqs - 1;      // the last request whose first place is at or before this one
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (j.cu_q[mid] / CK + mid <= slot) lo = mid; else hi = mid - 1;
+  }
+  seq = lo;
+  const int tok0 = j.cu_q[lo], qlen = j.cu_q[lo + 1] - tok0, i = slot - (tok0 / CK + lo);
+  first = tok0 + i * CK;
+  n = min(CK, qlen - i * CK);
+  return qlen > 1 && i >= 0 && n > 0;                 // single tokens are not done here
+}
+
+__device__ __forceinline__ void split2(float x, bf& hi, bf& lo) {
+  hi = __float2bfloat16_rn(x);
+  lo = __float2bfloat16_rn(x - __bfloat162float(hi));
+}
+__device__ __forceinline__ uint32_t pack2(bf a, bf b) {
+  const __nv_bfloat162 p = __halves2bfloat162(a, b);
+  return *reinterpret_cast<const uint32_t*>(&p);
+}
+
+// ------------------------------------------------------------------------------------------- 1. scores
+constexpr int CS_THREADS = 256, CS_PITCH = CK + 4;
+
+template <bool DELTA>
+__global__ void __launch_bounds__(CS_THREADS)
+chunk_scores_kernel(const Chunked j) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float cs[];
+  float* qt = cs;                                     // [D][CS_PITCH]: transposed, so that four tokens are one read
+  float* kt = qt + j.D * CS_PITCH;
+  const int slot = blockIdx.x, g = blockIdx.y, tid = threadIdx.x, D = j.D;
+  int seq, first, n;
+  if (!chunk_of(j, slot, seq, first, n)) {            // uniform in the block
+    pdl_wait();
+    return;
+  }
+  pdl_wait();
+  bf* qo = j.qs + ((size_t)slot * j.G + g) * 2 * CK * D;
+  bf* ko = j.ks + ((size_t)slot * j.G + g) * 2 * CK * D;
+  // a warp takes 4 tokens x 32 channels at a time: whole lines of memory, few lanes on one bank
+  for (int e = tid; e < CK * 8 * ((D + 31) / 32); e += CS_THREADS) {
+    const int unit = e >> 5, l = e & 31;
+    const int t = (unit & 15) * 4 + (l >> 3), i = (unit >> 4) * 32 + (l & 7) * 4;
+    if (i >= D) continue;
+    float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
+    if (t < n) {
+      const float* pq = j.q + (size_t)(first + t) * j.ldq + (size_t)g * D + i;
+      const float* pk = j.k + (size_t)(first + t) * j.ldk + (size_t)g * D + i;
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        a[u] = pq[u];
+        b[u] = pk[u];
+      }
+    }
+    bf ah[4], al[4], bh[4], bl[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      qt[(i + u) * CS_PITCH + t] = a[u];
+      kt[(i + u) * CS_PITCH + t] = b[u];
+      split2(a[u], ah[u], al[u]);
+      split2(b[u], bh[u], bl[u]);
+    }
+    const size_t at = (size_t)t * D + i;
+    *reinterpret_cast<uint2*>(qo + at) = make_uint2(pack2(ah[0], ah[1]), pack2(ah[2], ah[3]));
+    *reinterpret_cast<uint2*>(qo + CK * D + at) = make_uint2(pack2(al[0], al[1]), pack2(al[2], al[3]));
+    *reinterpret_cast<uint2*>(ko + at) = make_uint2(pack2(bh[0], bh[1]), pack2(bh[2], bh[3]));
+    *reinterpret_cast<uint2*>(ko + CK * D + at) = make_uint2(pack2(bl[0], bl[1]), pack2(bl[2], bl[3]));
+  }
+  // the sums of the logarithms, two tokens per lane, a warp per head of this key head's group
+  const int warp = tid >> 5, lane = tid & 31, rep = j.H / j.G;
+  for (int r = warp; r < rep; r += CS_THREADS / 32) {
+    const int h = g * rep + r;
+    float a = 2 * lane < n ? j.logg[(size_t)(first + 2 * lane) * j.H + h] : 0.f;
+    float b = 2 * lane + 1 < n ? j.logg[(size_t)(first + 2 * lane + 1) * j.H + h] : 0.f;
+    b += a;
+    float run = b;                                    // both tokens; then of all lanes up to this one
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float x = __shfl_up_sync(0xffffffffu, run, o);
+      if (lane >= o) run += x;
+    }
+    float before = __shfl_up_sync(0xffffffffu, run, 1);
+    if (lane == 0) before = 0.f;
+    float* co = j.c + ((size_t)slot * j.H + h) * CK;
+    co[2 * lane] = before + a;
+    co[2 * lane + 1] = before + b;
+  }
+  __syncthreads();
+  const int ty = tid >> 4, tx = tid & 15;             // four tokens t x four tokens s per thread
+  if (tx > ty) return;                                // s > t throughout: never read
+  float qk[4][4], kk[4][4];
+#pragma unroll
+  for (int a = 0; a < 4; ++a)
+#pragma unroll
+    for (int b = 0; b < 4; ++b) qk[a][b] = kk[a][b] = 0.f;
+  for (int i = 0; i < D; ++i) {
+    const float4 q4 = *reinterpret_cast<const float4*>(qt + i * CS_PITCH + 4 * ty);
+    const float4 s4 = *reinterpret_cast<const float4*>(kt + i * CS_PITCH + 4 * tx);
+    const float qa[4] = {q4.x, q4.y, q4.z, q4.w}, sa[4] = {s4.x, s4.y, s4.z, s4.w};
+#pragma unroll
+    for (int a = 0; a < 4; ++a)
+#pragma unroll
+      for (int b = 0; b < 4; ++b) qk[a][b] = fmaf(qa[a], sa[b], qk[a][b]);
+    if constexpr (DELTA) {
+      const float4 k4 = *reinterpret_cast<const float4*>(kt + i * CS_PITCH + 4 * ty);
+      const float ka[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+      for (int a = 0; a < 4; ++a)
+#pragma unroll
+        for (int b = 0; b < 4; ++b) kk[a][b] = fmaf(ka[a], sa[b], kk[a][b]);
+    }
+  }
+  const size_t base = ((size_t)slot * j.G + g) * CK * CK;
+#pragma unroll
+  for (int a = 0; a < 4; ++a) {
+    *reinterpret_cast<float4*>(j.qk + base + (4 * ty + a) * CK + 4 * tx) = make_float4(qk[a][0], qk[a][1], qk[a][2], qk[a][3]);
+    if constexpr (DELTA)
+      *reinterpret_cast<float4*>(j.kk + base + (4 * ty + a) * CK + 4 * tx) = make_float4(kk[a][0], kk[a][1], kk[a][2], kk[a][3]);
+  }
+}
+
+// -------------------------------------------------------------------------------- 2. the triangular system
+constexpr int SV_B = 16;             // rows per block of the substitution
+constexpr int SV_THREADS = 128, NT = SV_THREADS;      // columns per block
+
+__global__ void __launch_bounds__(SV_THREADS)
+chunk_solve_kernel(const Chunked j) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float sv[];
+  const int slot = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, D = j.D, V = j.V;
+  float* lt = sv;                                     // [s][t]: L transposed, CS_PITCH apart
+  float* bs = lt + CK * CS_PITCH;                     // beta, then beta e^c
+  float* be = bs + CK;
+  float* xs = be + CK;                                // [CK][NT]: solved rows of this block's columns
+  int seq, first, n;
+  if (!chunk_of(j, slot, seq, first, n)) {
+    pdl_wait();
+    return;
+  }
+  pdl_wait();
+  const int g = h / (j.H / j.G);
+  const float* c = j.c + ((size_t)slot * j.H + h) * CK;
+  const float* kk = j.kk + ((size_t)slot * j.G + g) * CK * CK;
+  for (int t = tid; t < CK; t += NT) {
+    const float b = t < n ? j.beta[(size_t)(first + t) * j.H + h] : 0.f;
+    bs[t] = b;
+    be[t] = b * expf(c[t]);
+  }
+  __syncthreads();
+  for (int e = tid; e < CK * CK; e += NT) {
+    const int t = e / CK, s = e - t * CK;
+    lt[s * CS_PITCH + t] = s < t ? bs[t] * expf(c[t] - c[s]) * kk[e] : 0.f;
+  }
+  __syncthreads();
+  bf* wo = j.w + ((size_t)slot * j.H + h) * 2 * CK * D;
+  float* uo = j.u0 + ((size_t)slot * j.H + h) * CK * V;
+  const int col = blockIdx.z * NT + tid;
+  const bool on = col < D + V, is_k = col < D;
+  const float* src = is_k ? j.k + (size_t)first * j.ldk + (size_t)g * D + col : j.v + (size_t)first * j.ldv + (size_t)h * V + col - D;
+  const int ld = is_k ? j.ldk : j.ldv;
+  const float* mul = is_k ? be : bs;
+  float next[SV_B];
+#pragma unroll
+  for (int r = 0; r < SV_B; ++r) next[r] = on && r < n ? src[(size_t)r * ld] : 0.f;
+#pragma unroll 1
+  for (int bi = 0; bi < CK; bi += SV_B) {
+    float acc[SV_B];
+#pragma unroll
+    for (int r = 0; r < SV_B; ++r) acc[r] = mul[bi + r] * next[r];
+    if (bi + SV_B < CK) {
+#pragma unroll
+      for (int r = 0; r < SV_B; ++r) next[r] = on && bi + SV_B + r < n ? src[(size_t)(bi + SV_B + r) * ld] : 0.f;
+    }
+#pragma unroll 4
+    for (int s = 0; s < bi; ++s) {
+      const float x = xs[s * NT + tid];
+#pragma unroll
+      for (int r = 0; r < SV_B; r += 4) {
+        const float4 l = *reinterpret_cast<const float4*>(lt + s * CS_PITCH + bi + r);
+        acc[r] = fmaf(-l.x, x, acc[r]);
+        acc[r + 1] = fmaf(-l.y, x, acc[r + 1]);
+        acc[r + 2] = fmaf(-l.z, x, acc[r + 2]);
+        acc[r + 3] = fmaf(-l.w, x, acc[r + 3]);
+      }
+    }
+#pragma unroll
+    for (int s = 0; s < SV_B; ++s) {                // rows below the diagonal only matter: L is zero above
+#pragma unroll
+      for (int r = s & ~3; r < SV_B; r += 4) {
+        const float4 l = *reinterpret_cast<const float4*>(lt + (bi + s) * CS_PITCH + bi + r);
+        if (r > s) acc[r] = fmaf(-l.x, acc[s], acc[r]);
+        if (r + 1 > s) acc[r + 1] = fmaf(-l.y, acc[s], acc[r + 1]);
+        if (r + 2 > s) acc[r + 2] = fmaf(-l.z, acc[s], acc[r + 2]);
+        if (r + 3 > s) acc[r + 3] = fmaf(-l.w, acc[s], acc[r + 3]);
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < SV_B; ++r) {
+      xs[(bi + r) * NT + tid] = acc[r];             // read by this thread only
+      if (on) {
+        if (is_k) {
+          bf hi, lo;
+          split2(acc[r], hi, lo);
+          wo[(size_t)(bi + r) * D + col] = hi;
+          wo[(size_t)CK * D + (size_t)(bi + r) * D + col] = lo;
+        } else {
+          uo[(size_t)(bi + r) * V + col - D] = acc[r];
+        }
+      }
+    }
+  }
+}
+
+// -------------------------------------------------------------------------------------------- 3. the walk
+constexpr int CW_THREADS = 256;
+
+__device__ __forceinline__ void ck_ldsm(uint32_t* r, const bf* p) {
+  const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void ck_ldsm_t(uint32_t* r, const bf* p) {
+  const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void ck_mma(float* d, const uint32_t* a, const uint32_t* b) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
+}
+// both operands in two parts; the product of the remainders is below the sums' own rounding
+__device__ __forceinline__ void ck_mma3(float* d, const uint32_t* ah, const uint32_t* al, const uint32_t* bh, const uint32_t* bl) {
+  ck_mma(d, al, bh);
+  ck_mma(d, ah, bl);
+  ck_mma(d, ah, bh);
+}
+__device__ __forceinline__ void ck_cp16(void* dst, const void* src) {
+  const uint32_t a = (uint32_t)__cvta_generic_to_shared(dst);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(a), "l"(src) : "memory");
+}
+
+__host__ __device__ constexpr size_t ck_walk_smem(int D, bool delta) {
+  const size_t tile = (size_t)2 * CK * (D + CK_PAD) * sizeof(bf);                   // Q, K or W in two parts
+  return tile * (delta ? 4 : 3) + 2 * (size_t)CK * (CK + 4) * sizeof(float) + 2 * CK * sizeof(float)
+         + (size_t)2 * D * (CK_VP + CK_PAD) * sizeof(bf) + (size_t)4 * CK * (CK_VP + CK_PAD) * sizeof(bf);
+}
+
+// Warp (row group wr of 16 tokens or key channels, column half wc of 16 value channels).
+template <bool DELTA>
+__global__ void __launch_bounds__(CW_THREADS)
+chunk_walk_kernel(const Chunked j) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) char walk_smem[];
+  const int D = j.D, DP = D + CK_PAD, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, wr = warp & 3, wc = warp >> 2;
+  constexpr int VP = CK_VP + CK_PAD, PP = CK + 4;
+  const int tile = 2 * CK * DP;                       // elements of a tile in two parts
+  bf* Q = reinterpret_cast<bf*>(walk_smem);
+  bf* K = Q + tile;                                   // twice
+  bf* W = K + 2 * tile;                               // delta rule only
+  float* P = reinterpret_cast<float*>(W + (DELTA ? tile : 0));      // q . k, twice
+  float* Cs = P + 2 * CK * PP;                        // sums of the logarithms, twice
+  bf* Ss = reinterpret_cast<bf*>(Cs + 2 * CK);        // the state, two parts of [D][VP]
+  bf* Us = Ss + 2 * D * VP;                           // U, two parts of [CK][VP]; then U e^(c_64 - c), two parts
+  const int seq = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * CK_VP;
+  const int tok0 = j.cu_q[seq], qlen = j.cu_q[seq + 1] - tok0;
+  pdl_wait();
+  if (qlen <= 1) return;                              // single tokens are not done here
+  const int g = h / (j.H / j.G), chunks = (qlen + CK - 1) / CK, slot0 = tok0 / CK + seq;
+  float* S = j.state + (size_t)j.state_slots[seq] * j.slot_stride + (size_t)h * D * j.V;
+  const int fr = lane >> 2, fc = (lane & 3) * 2;      // an accumulator's first row and column
+
+  // the rolling loads of a chunk: Q and W once, K, q . k and the sums in two buffers
+  auto load = [&](int i) {
+    const int slot = slot0 + i, buf = i & 1;
+    const size_t at = ((size_t)slot * j.G + g) * 2 * CK * D, wat = ((size_t)slot * j.H + h) * 2 * CK * D;
+    const int per_row = D / 8, pieces = 2 * CK * per_row;
+    for (int e = tid; e < pieces; e += CW_THREADS) {
+      const int r = e / per_row, x = (e - r * per_row) * 8;                          // row of both parts
+      ck_cp16(Q + r * DP + x, j.qs + at + (size_t)r * D + x);
+      ck_cp16(K + buf * tile + r * DP + x, j.ks + at + (size_t)r * D + x);
+      if (DELTA) ck_cp16(W + r * DP + x, j.w + wat + (size_t)r * D + x);
+    }
+    const float* qk = j.qk + ((size_t)slot * j.G + g) * CK * CK;
+    for (int e = tid; e < CK * CK / 4; e += CW_THREADS) {
+      const int r = e / (CK / 4), x = (e - r * (CK / 4)) * 4;
+      if (x <= r) ck_cp16(P + buf * CK * PP + r * PP + x, qk + r * CK + x);
+    }
+    if (tid < CK / 4) ck_cp16(Cs + buf * CK + tid * 4, j.c + ((size_t)slot * j.H + h) * CK + tid * 4);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  load(0);
+
+  // the state in accumulators: key channels 16 (wr + 4 m) .., value channels 16 wc + 8 n ..
+  float acc[2][2][4] = {};
+  auto each_state = [&](auto f) {
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+      if ((wr + 4 * m) * 16 >= D) continue;
+#pragma unroll
+      for (int nn = 0; nn < 2; ++nn)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int row = (wr + 4 * m) * 16 + fr + (e >> 1) * 8, col = wc * 16 + nn * 8 + fc + (e & 1);
+          f(acc[m][nn][e], row, col);
+        }
+    }
+  };
+  each_state([&](float& x, int row, int col) { x = v0 + col < j.V ? S[(size_t)row * j.V + v0 + col] : 0.f; });
+  auto share_state = [&] {                            // into shared memory, in two parts
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+      if ((wr + 4 * m) * 16 >= D) continue;
+#pragma unroll
+      for (int nn = 0; nn < 2; ++nn)
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const int row = (wr + 4 * m) * 16 + fr + (e >> 1) * 8, col = wc * 16 + nn * 8 + fc;
+          bf ah, al, bh, bl;
+          split2(acc[m][nn][e], ah, al);
+          split2(acc[m][nn][e + 1], bh, bl);
+          *reinterpret_cast<uint32_t*>(Ss + row * VP + col) = pack2(ah, bh);
+          *reinterpret_cast<uint32_t*>(Ss + D * VP + row * VP + col) = pack2(al, bl);
+        }
+    }
+  };
+  share_state();
+
+  const int lr = lane & 15, lc = (lane >> 4) * 8;     // ldmatrix: this lane's row and column offset within 16 x 16
+  for (int i = 0; i < chunks; ++i) {
+    const int n = min(CK, qlen - i * CK), first = tok0 + i * CK, buf = i & 1;
+    // what becomes U: asked for now, needed after the products with the state
+    float u[2][4];
+#pragma unroll
+    for (int nn = 0; nn < 2; ++nn)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int t = wr * 16 + fr + (e >> 1) * 8, col = v0 + wc * 16 + nn * 8 + fc + (e & 1);
+        u[nn][e] = 0.f;
+        if (t < n && col < j.V) {
+          if (DELTA) u[nn][e] = j.u0[(((size_t)(slot0 + i) * j.H + h) * CK + t) * j.V + col];
+          else u[nn][e] = j.beta[(size_t)(first + t) * j.H + h] * j.v[(size_t)(first + t) * j.ldv + (size_t)h * j.V + col];
+        }
+      }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                  // this chunk's tiles and the state are there; the chunk before is done with
+    float qs[2][4];
+#pragma unroll
+    for (int nn = 0; nn < 2; ++nn)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) qs[nn][e] = 0.f;
+    float ws[2][4];
+#pragma unroll
+    for (int nn = 0; nn < 2; ++nn)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) ws[nn][e] = 0.f;
+#pragma unroll 2
+    for (int kk = 0; kk < D; kk += 16) {
+      uint32_t bh[4], bl[4], ah[4], al[4];
+      ck_ldsm_t(bh, Ss + (kk + lr) * VP + wc * 16 + lc);
+      ck_ldsm_t(bl, Ss + D * VP + (kk + lr) * VP + wc * 16 + lc);
+      ck_ldsm(ah, Q + (wr * 16 + lr) * DP + kk + lc);
+      ck_ldsm(al, Q + CK * DP + (wr * 16 + lr) * DP + kk + lc);
+#pragma unroll
+      for (int nn = 0; nn < 2; ++nn) ck_mma3(qs[nn], ah, al, bh + 2 * nn, bl + 2 * nn);
+      if constexpr (DELTA) {
+        ck_ldsm(ah, W + (wr * 16 + lr) * DP + kk + lc);
+        ck_ldsm(al, W + CK * DP + (wr * 16 + lr) * DP + kk + lc);
+#pragma unroll
+        for (int nn = 0; nn < 2; ++nn) ck_mma3(ws[nn], ah, al, bh + 2 * nn, bl + 2 * nn);
+      }
+    }
+    const float* cs = Cs + buf * CK;
+    const float ct[2] = {cs[wr * 16 + fr], cs[wr * 16 + fr + 8]}, cend = cs[CK - 1];
+#pragma unroll
+    for (int nn = 0; nn < 2; ++nn)
+#pragma unroll
+      for (int e = 0; e < 4; e += 2) {
+        const int row = wr * 16 + fr + (e >> 1) * 8, col = wc * 16 + nn * 8 + fc;
+        const float x = DELTA ? u[nn][e] - ws[nn][e] : u[nn][e], y = DELTA ? u[nn][e + 1] - ws[nn][e + 1] : u[nn][e + 1];
+        const float f = expf(cend - ct[e >> 1]);
+        bf xh, xl, yh, yl;
+        split2(x, xh, xl);
+        split2(y, yh, yl);
+        *reinterpret_cast<uint32_t*>(Us + row * VP + col) = pack2(xh, yh);
+        *reinterpret_cast<uint32_t*>(Us + CK * VP + row * VP + col) = pack2(xl, yl);
+        split2(x * f, xh, xl);
+        split2(y * f, yh, yl);
+        *reinterpret_cast<uint32_t*>(Us + 2 * CK * VP + row * VP + col) = pack2(xh, yh);
+        *reinterpret_cast<uint32_t*>(Us + 3 * CK * VP + row * VP + col) = pack2(xl, yl);
+      }
+    __syncthreads();                                  // U is there; nobody reads Q, W and the state any more
+    if (i + 1 < chunks) load(i + 1);
+    // O = e^c Q S + P U
+    float o[2][4];
+    {
+      const float f0 = expf(ct[0]), f1 = expf(ct[1]);
+#pragma unroll
+      for (int nn = 0; nn < 2; ++nn) {
+        o[nn][0] = f0 * qs[nn][0];
+        o[nn][1] = f0 * qs[nn][1];
+        o[nn][2] = f1 * qs[nn][2];
+        o[nn][3] = f1 * qs[nn][3];
+      }
+    }
+    const float* Pb = P + buf * CK * PP;
+    for (int kb = 0; kb <= wr; ++kb) {
+      uint32_t ah[4], al[4], bh[4], bl[4];
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {                   // rows fr, fr + 8, fr, fr + 8; columns fc, fc, fc + 8, fc + 8
+        const int t = wr * 16 + fr + (x & 1) * 8, s = kb * 16 + fc + (x >> 1) * 8;
+        float p0 = 0.f, p1 = 0.f;
+        if (s <= t) p0 = Pb[t * PP + s] * expf(ct[x & 1] - cs[s]);
+        if (s + 1 <= t) p1 = Pb[t * PP + s + 1] * expf(ct[x & 1] - cs[s + 1]);
+        bf h0, l0, h1, l1;
+        split2(p0, h0, l0);
+        split2(p1, h1, l1);
+        ah[x] = pack2(h0, h1);
+        al[x] = pack2(l0, l1);
+      }
+      ck_ldsm_t(bh, Us + (kb * 16 + lr) * VP + wc * 16 + lc);
+      ck_ldsm_t(bl, Us + CK * VP + (kb * 16 + lr) * VP + wc * 16 + lc);
+#pragma unroll
+      for (int nn = 0; nn < 2; ++nn) ck_mma3(o[nn], ah, al, bh + 2 * nn, bl + 2 * nn);
+    }
+#pragma unroll
+    for (int nn = 0; nn < 2; ++nn)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int t = wr * 16 + fr + (e >> 1) * 8, col = v0 + wc * 16 + nn * 8 + fc + (e & 1);
+        if (t < n && col < j.V) j.out[(size_t)(first + t) * j.ldo + (size_t)h * j.V + col] = o[nn][e];
+      }
+    // S = e^(c_64) S + K^T U e^(c_64 - c)
+    const float fend = expf(cend);
+    const bf* Kb = K + buf * tile;
+#pragma unroll
+    for (int m = 0; m < 2; ++m)
+#pragma unroll
+      for (int nn = 0; nn < 2; ++nn)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[m][nn][e] *= fend;
+#pragma unroll
+    for (int kb = 0; kb < CK / 16; ++kb) {
+      uint32_t bh[4], bl[4];
+      ck_ldsm_t(bh, Us + 2 * CK * VP + (kb * 16 + lr) * VP + wc * 16 + lc);
+      ck_ldsm_t(bl, Us + 3 * CK * VP + (kb * 16 + lr) * VP + wc * 16 + lc);
+#pragma unroll
+      for (int m = 0; m < 2; ++m) {
+        const int c0 = (wr + 4 * m) * 16;
+        if (c0 >= D) continue;
+        // K lies by tokens: its transpose's 16 x 16 part, the halves of the tokens behind those of the channels
+        uint32_t ah[4], al[4];
+        const bf* kp = Kb + (kb * 16 + (lane & 7) + (lane >> 4) * 8) * DP + c0 + ((lane >> 3) & 1) * 8;
+        ck_ldsm_t(ah, kp);
+        ck_ldsm_t(al, kp + CK * DP);
+#pragma unroll
+        for (int nn = 0; nn < 2; ++nn) ck_mma3(acc[m][nn], ah, al, bh + 2 * nn, bl + 2 * nn);
+      }
+    }
+    if (i + 1 < chunks) share_state();
+  }
+  each_state([&](float& x, int row, int col) { if (v0 + col < j.V) S[(size_t)row * j.V + v0 + col] = x; });
+}
+
+struct ChunkPlan {
+  long long qs, qk, c, w, u0, total;     // floats
+};
+ChunkPlan chunk_plan(int slots, int H, int G, int D, int V, int delta) {
+  ChunkPlan p = {};
+  p.qs = (long long)slots * G * CK * D;                // Q, and as many for K: two bfloat16 parts are one float
+  p.qk = (long long)slots * G * CK * CK;
+  p.c = (long long)slots * H * CK;
+  p.w = delta ? (long long)slots * H * CK * D : 0;
+  p.u0 = delta ? (long long)slots * H * CK * V : 0;
+  p.total = 2 * p.qs + (delta ? 2 : 1) * p.qk + p.c + p.w + p.u0;
+  return p;
+}
+}  // namespace
+
+extern "C" int zi_chunked_recurrence_supported(int D, int V, int H, int G) {
+  return D >= 16 && D <= 128 && D % 16 == 0 && V > 0 && H > 0 && G > 0 && H % G == 0 && H <= 65535 && (V + CK_VP - 1) / CK_VP <= 65535;
+}
+extern "C" long long zi_chunked_recurrence_workspace_floats(int T, int n_seqs, int H, int G, int D, int V, int delta) {
+  return chunk_plan(T / CK + n_seqs + 1, H, G, D, V, delta).total;
+}
+
+// The portions of two tokens and more of a step; requests that bring one token are left alone.  logg: logarithms of the
+// decays, beta: step sizes, float32 [T][H]; workspace: zi_chunked_recurrence_workspace_floats, 16-byte aligned.
+extern "C" int zi_chunked_recurrence(float* out, int ldo, const float* q, int ldq, const float* k, int ldk, const float* v, int ldv,
+                                     const float* logg, const float* beta, float* state, long long slot_stride, int T, int H, int G,
+                                     int D, int V, int delta, const int* cu_q, const int* state_slots, int n_seqs, float* workspace,
+                                     cudaStream_t stream) {
+  if (T <= 0 || n_seqs <= 0) return 0;
+  if (!zi_chunked_recurrence_supported(D, V, H, G)) return zi_refuse("chunked_recurrence: %d heads (%d of keys) of %d x %d", H, G, D, V);
+  if (!workspace || ((uintptr_t)workspace & 15) || !logg || !beta) return zi_refuse("chunked_recurrence: needs decays, steps and an aligned workspace");
+  const int slots = T / CK + n_seqs + 1;
+  const ChunkPlan p = chunk_plan(slots, H, G, D, V, delta);
+  Chunked j = {};
+  j.q = q; j.k = k; j.v = v; j.ldq = ldq; j.ldk = ldk; j.ldv = ldv; j.logg = logg; j.beta = beta;
+  j.state = state; j.slot_stride = slot_stride; j.H = H; j.G = G; j.D = D; j.V = V;
+  j.cu_q = cu_q; j.state_slots = state_slots; j.n_seqs = n_seqs; j.slots = slots; j.out = out; j.ldo = ldo;
+  float* at = workspace;
+  j.qs = reinterpret_cast<bf*>(at); at += p.qs;
+  j.ks = reinterpret_cast<bf*>(at); at += p.qs;
+  j.qk = at; at += p.qk;
+  if (delta) { j.kk = at; at += p.qk; }
+  j.c = at; at += p.c;
+  if (delta) {
+    j.w = reinterpret_cast<bf*>(at); at += p.w;
+    j.u0 = at;
+  }
+  auto launch = [&](auto kern, dim3 grid, int threads, size_t smem, const char* what) {
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+      return zi_refuse("%s: cannot get %zu bytes of shared memory", what, smem);
+    zi_launch(kern, grid, dim3(threads), smem, stream, j);
+    return zi_check_launch(what);
+  };
+  const size_t score_smem = (size_t)2 * D * CS_PITCH * sizeof(float);
+  int rc = launch(delta ? chunk_scores_kernel<true> : chunk_scores_kernel<false>, dim3(slots, G), CS_THREADS, score_smem, "chunk_scores");
+  if (rc) return rc;
+  if (delta) {
+    const size_t solve_smem = ((size_t)CK * CS_PITCH + 2 * CK + (size_t)CK * NT) * sizeof(float);
+    rc = launch(chunk_solve_kernel, dim3(slots, H, (D + V + NT - 1) / NT), NT, solve_smem, "chunk_solve");
+    if (rc) return rc;
+  }
+  const dim3 grid(n_seqs, H, (V + CK_VP - 1) / CK_VP);
+  return delta ? launch(chunk_walk_kernel<true>, grid, CW_THREADS, ck_walk_smem(D, true), "chunk_walk")
+               : launch(chunk_walk_kernel<false>, grid, CW_THREADS, ck_walk_smem(D, false), "chunk_walk");
+}
+
+ZI_TRACE_SETTER(chunked_recurrence)

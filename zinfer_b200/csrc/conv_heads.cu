@@ -55,14 +55,14 @@ struct ConvJob {
   const int* cu_q;
   const int* state_slots;
   int smem_head;     // floats per token of a warp's shared memory (unit vectors only)
-  // what every token has once per head beside the channels: a step and a decay (scalars 0: nothing to do)
-  int scalars;       // 1: step = sigmoid(b), decay = exp(-exp(a_log) softplus(a + dt_bias)); 2: step = softplus(a + dt_bias), decay = exp(-exp(a_log) step)
+  // what every token has once per head beside the channels: a step and a decay's logarithm (scalars 0: nothing to do)
+  int scalars;       // 1: step = sigmoid(b), log decay = -exp(a_log) softplus(a + dt_bias); 2: step = softplus(a + dt_bias), log decay = -exp(a_log) step
   int n_scalar;      // heads
   const float* a;    // row 0, head 0 (rows as above: same pitch and splits)
   const float* b;
   const float* a_log;
   const float* dt_bias;
-  float* decay;      // [T][n_scalar]
+  float* decay;      // [T][n_scalar] logarithms
   float* step;
 };
 
@@ -94,7 +94,7 @@ conv_heads_kernel(const ConvJob j) {
       const int t = e / j.n_scalar, h = e - t * j.n_scalar;
       const size_t row = (size_t)(row0 + t);
       const float sp = conv_softplus(summed_at(j.a + row * j.ld + h, j.splits, j.zstride) + j.dt_bias[h]);
-      j.decay[row * j.n_scalar + h] = expf(-expf(j.a_log[h]) * sp);
+      j.decay[row * j.n_scalar + h] = -expf(j.a_log[h]) * sp;
       j.step[row * j.n_scalar + h] = j.scalars == 2 ? sp : 1.0f / (1.0f + expf(-summed_at(j.b + row * j.ld + h, j.splits, j.zstride)));
     }
     return;

@@ -220,7 +220,7 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
         const size_t row = (size_t)(tok0 + t0 + tt);
         if (CHUNK != 1) fq[u] = q[row * ldq + (size_t)kvh * D + i];
         if (!MADE) fk[u] = k[row * ldk + (size_t)kvh * D + i];
-        if (!GATE) fg[u] = decay[row * ldg + (size_t)h * gh + i * gi];
+        if (!GATE) fg[u] = gi ? decay[row * ldg + (size_t)h * gh + i] : expf(decay[row * ldg + h]);
       } else {
         fq[u] = from_f32<TQ>(0.f);
         fk[u] = from_f32<TQ>(0.f);
@@ -293,7 +293,7 @@ linear_recurrence_kernel(float* __restrict__ out, int ldo, const TQ* __restrict_
       const bool in = i < D;
       stage(buf, (e & ~(DP - 1)) + place(i), i, in ? whole(q + row * ldq + (size_t)kvh * D + i) : 0.f,
             in && !MADE ? whole(k + row * ldk + (size_t)kvh * D + i) : 0.f,
-            in && !GATE ? decay[row * ldg + (size_t)h * gh + i * gi] : (MADE ? 1.f : 0.f));
+            in && !GATE ? (gi ? decay[row * ldg + (size_t)h * gh + i] : expf(decay[row * ldg + h])) : (MADE ? 1.f : 0.f));
     }
 #pragma unroll
     for (int u = 0; u < NPV; ++u) {
@@ -680,10 +680,12 @@ extern "C" int zi_sigmoid_rows(float* out, int ldo, const void* x, int ldx, int 
 extern "C" int zi_linear_recurrence(float* out, int ldo, const void* q, int ldq, const void* k, int ldk, int qk_dtype,
                                     const void* v, int ldv, int v_dtype, const float* decay, int ldg, const float* beta,
                                     int ldb, float q_scale, float* state, long long slot_stride, int H, int G, int D,
-                                    int V, int delta, int head_decay, const int* cu_q, const int* state_slots, int n_seqs,
-                                    cudaStream_t stream) {
+                                    int V, int delta, int head_decay, int only_single, const int* cu_q, const int* state_slots,
+                                    int n_seqs, cudaStream_t stream) {
   if (n_seqs <= 0) return 0;
-  const int gh = head_decay ? 1 : D, gi = head_decay ? 0 : 1;      // one decay per head, or one per key channel
+  const int gh = head_decay ? 1 : D, gi = head_decay ? 0 : 1;      // one decay per head (its logarithm), or one per key channel
+  RecurrenceTiles walk = {};
+  walk.only_single = only_single;
   if (H <= 0 || G <= 0 || H % G) return zi_refuse("linear_recurrence: %d heads do not divide into %d key heads", H, G);
   if (D <= 0 || D > 512 || V <= 0) return zi_refuse("linear_recurrence: %d key channels (1..512), %d value channels", D, V);
   if (delta && !beta) return zi_refuse("linear_recurrence: the delta rule needs beta");
@@ -703,7 +705,7 @@ extern "C" int zi_linear_recurrence(float* out, int ldo, const void* q, int ldq,
     }                                                                                                                  \
     zi_launch(kern, dim3(grid), dim3(block), smem, stream, out, ldo, (const TQ*)q, ldq, (const TQ*)k, ldk, (const TV*)v, \
               ldv, decay, ldg, beta, ldb, q_scale, state, slot_stride, H, G, D, V, P, cu_q, state_slots, ForgetGate{}, \
-              RecurrenceTiles{}, gh, gi);                                                                              \
+              walk, gh, gi);                                                                                           \
   } while (0)
 #define ZI_LR_R(TQ, TV)                                          \
   do {                                                           \

@@ -38,6 +38,7 @@ def lib() -> ctypes.CDLL:
         _LIB.zi_gemm_tcgen05_plan.restype = ctypes.c_longlong
         _LIB.zi_attention_decode_workspace_floats.restype = ctypes.c_longlong
         _LIB.zi_linear_recurrence_tiles_floats.restype = ctypes.c_longlong
+        _LIB.zi_chunked_recurrence_workspace_floats.restype = ctypes.c_longlong
     return _LIB
 
 
@@ -1844,33 +1845,70 @@ def sigmoid_rows(x: torch.Tensor) -> torch.Tensor:
 
 def linear_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, beta: Optional[torch.Tensor],
                       q_scale: float, state: torch.Tensor, heads: int, key_heads: int, dim: int, vdim: int, step,
-                      delta: bool = True) -> torch.Tensor:
+                      delta: bool = True, log_decay: Optional[torch.Tensor] = None, only_single: bool = False,
+                      out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Per request and head, over the step's tokens, from and to ``state`` [slots, heads, dim, vdim] (float32):
     ``S = diag(decay_t) S``; ``u = beta_t (v_t - S^T k_t)`` (the delta rule) or, with ``delta`` False or without ``beta``,
     ``u = beta_t v_t`` (a step size; 1 without ``beta``);
     ``S += k_t u^T``; ``o_t = S^T (q_scale q_t)``.  ``q``, ``k`` [T, key_heads * dim] (head h reads key head
-    h // (heads / key_heads)), ``v`` [T, heads * vdim], ``decay`` float32 [T, heads * dim] or one per head [T, heads],
-    ``beta`` float32 [T, heads];
-    rows may be views of wider rows.  Returns float32 [T, heads * vdim]."""
+    h // (heads / key_heads)), ``v`` [T, heads * vdim], ``decay`` float32 [T, heads * dim], ``beta`` float32 [T, heads];
+    rows may be views of wider rows.  ``log_decay`` (float32 [T, heads]) in place of ``decay``: one decay per head, as its
+    logarithm.  ``only_single``: requests that bring more than one token are left alone.  Returns float32 [T, heads * vdim]."""
     T = q.shape[0]
+    per_head = decay is None
+    if per_head:
+        decay = log_decay
     state, stride = _slot_view(state, "linear_recurrence")
     _need(state[0].numel() == heads * dim * vdim, "linear_recurrence: state [slots, heads, dim, vdim]")
     _need(q.dtype == k.dtype and q.stride(1) == 1 and k.stride(1) == 1 and v.stride(1) == 1
           and q.shape[1] == key_heads * dim and k.shape[1] == key_heads * dim and v.shape[1] == heads * vdim,
           "linear_recurrence: q, k [T, key heads * dim], v [T, heads * vdim] with dense rows")
-    _need(decay.dtype == torch.float32 and decay.stride(1) == 1 and decay.shape[1] in (heads, heads * dim),
+    _need(decay.dtype == torch.float32 and decay.stride(1) == 1 and decay.shape[1] == (heads if per_head else heads * dim),
           "linear_recurrence: decay")
     if beta is not None:
         _need(beta.dtype == torch.float32 and beta.stride(1) == 1 and beta.shape[1] == heads, "linear_recurrence: beta")
     delta = delta and beta is not None
-    out = torch.empty((T, heads * vdim), dtype=torch.float32, device=q.device)
+    if out is None:
+        out = torch.empty((T, heads * vdim), dtype=torch.float32, device=q.device)
     with _prof.region("linear recurrence" + (" (delta rule)" if delta else ""),
                       lambda: _nb(q, k, v, decay, out) + 2 * step.n_seqs * heads * dim * vdim * 4, 6 * T * heads * dim * vdim):
         _check(lib().zi_linear_recurrence(
             _ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _tag(q), _ptr(v), v.stride(0), _tag(v),
             _ptr(decay), decay.stride(0), _ptr(beta), beta.stride(0) if beta is not None else 0, ctypes.c_float(q_scale),
-            _ptr(state), _ll(stride), heads, key_heads, dim, vdim, 1 if delta else 0, 1 if decay.shape[1] == heads else 0, _ptr(step.cu_q),
+            _ptr(state), _ll(stride), heads, key_heads, dim, vdim, 1 if delta else 0, 1 if per_head else 0, 1 if only_single else 0, _ptr(step.cu_q),
             _ptr(step.state_slots), step.n_seqs, _stream()), "linear_recurrence")
+    return out
+
+
+RECURRENCE_CHUNKS = os.environ.get("ZINFER_B200_RECURRENCE_CHUNKS", "1") not in ("", "0")   # off: every request in one walk (comparisons)
+RECURRENCE_CHUNK_MIN = 96     # from this many tokens in a request's portion the chunked form pays
+
+
+def head_decay_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: torch.Tensor, beta: torch.Tensor, state: torch.Tensor,
+                          heads: int, key_heads: int, dim: int, vdim: int, step, delta: bool, fast: bool) -> torch.Tensor:
+    """The recurrence with one decay per head (see :func:`linear_recurrence`; q ready, float32 operands): token by token, or,
+    where ``fast`` allows the tensor cores' products (each operand in two bfloat16 parts) and a portion is long, in chunks of
+    64 tokens, single tokens of the same step token by token.  Returns float32 [T, heads * vdim]."""
+    T = q.shape[0]
+    L = lib()
+    if not (fast and RECURRENCE_CHUNKS and step.max_q_len >= RECURRENCE_CHUNK_MIN and L.zi_chunked_recurrence_supported(dim, vdim, heads, key_heads)):
+        return linear_recurrence(q, k, v, None, beta, 1.0, state, heads, key_heads, dim, vdim, step, delta=delta, log_decay=log_decay)
+    st, stride = _slot_view(state, "head_decay_recurrence")
+    for t, cols in ((q, key_heads * dim), (k, key_heads * dim), (v, heads * vdim), (log_decay, heads), (beta, heads)):
+        _need(t.dtype == torch.float32 and t.stride(1) == 1 and tuple(t.shape) == (T, cols), "head_decay_recurrence: float32 rows")
+    _need(log_decay.is_contiguous() and beta.is_contiguous() and st[0].numel() == heads * dim * vdim, "head_decay_recurrence: state [slots, heads, dim, vdim]")
+    out = torch.empty((T, heads * vdim), dtype=torch.float32, device=q.device)
+    n = L.zi_chunked_recurrence_workspace_floats(T, step.n_seqs, heads, key_heads, dim, vdim, 1 if delta else 0)
+    ws = torch.empty((n,), dtype=torch.float32, device=q.device)
+    with _prof.region("recurrence in chunks" + (" (delta rule)" if delta else ""),
+                      lambda: _nb(q, k, v, log_decay, beta, out) + 2 * step.n_seqs * heads * dim * vdim * 4, (6 if delta else 4) * T * heads * dim * vdim):
+        _check(L.zi_chunked_recurrence(
+            _ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(log_decay), _ptr(beta), _ptr(st),
+            _ll(stride), T, heads, key_heads, dim, vdim, 1 if delta else 0, _ptr(step.cu_q), _ptr(step.state_slots), step.n_seqs, _ptr(ws),
+            _stream()), "chunked_recurrence")
+    if step.n_dec > 0:
+        linear_recurrence(q, k, v, None, beta, 1.0, state, heads, key_heads, dim, vdim, step, delta=delta, log_decay=log_decay, only_single=True,
+                          out=out)
     return out
 
 
@@ -1980,8 +2018,8 @@ def conv_heads(u: Columns, kernel: torch.Tensor, tail: Optional[torch.Tensor], s
     them) is finished and put where it goes.
 
     ``decay``: (kind, a, b, a_log, dt_bias) makes the steps and decays of a recurrence from further columns of the same rows:
-    kind ``delta`` gives step = sigmoid(b), decay = exp(-exp(a_log) softplus(a + dt_bias)); kind ``ssd`` gives step =
-    softplus(a + dt_bias), decay = exp(-exp(a_log) step).  Returns (decay, step), float32 [T, heads], or None."""
+    kind ``delta`` gives step = sigmoid(b), log decay = -exp(a_log) softplus(a + dt_bias); kind ``ssd`` gives step =
+    softplus(a + dt_bias), log decay = -exp(a_log) step.  Returns (log decay, step), float32 [T, heads], or None."""
     T, C = u.shape
     taps = kernel.shape[0]
     _need(kernel.dtype == torch.float32 and kernel.is_contiguous() and kernel.shape[1] == C, "conv_heads: kernel float32 [taps, C]")

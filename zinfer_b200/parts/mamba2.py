@@ -78,7 +78,8 @@ class Mamba2(Mixer):
         decay, dt = ops.conv_heads(cols(inner, C), self.conv, tail, step, [ops.ConvSegment(C, C, xbc)], out_bias=self.conv_bias,
                                    activation="silu", decay=("ssd", cols(inner + C, H), None, self.a_log, self.dt_bias))
         xs, B, Cs = xbc[:, :inner], xbc[:, inner:inner + bc], xbc[:, inner + bc:]
-        y = ops.linear_recurrence(Cs, B, xs, decay, dt, 1.0, state[:, :self.s_size], H, self.groups, self.dim, self.vdim, step, delta=False)
+        y = ops.head_decay_recurrence(Cs, B, xs, decay, dt, state[:, :self.s_size], H, self.groups, self.dim, self.vdim, step, delta=False,
+                                      fast=self.ctx.dtype == torch.bfloat16)
         y = ops.gated_part_norm(y, cols(0, inner), self.norm, self.eps, self.norm_groups, self.ctx.dtype, skip=self.skip, x=xs,
                                 vdim=self.vdim)
         return ops.linear(y, self.w_o, out_dtype=self.ctx.dtype, allow_partials=True)
