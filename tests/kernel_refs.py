@@ -677,8 +677,9 @@ def linear_recurrence(q, k, v, decay, beta, q_scale, state, heads, key_heads, di
     return out
 
 
-def head_decay_recurrence(q, k, v, log_decay, beta, state, heads, key_heads, dim, vdim, step, delta, fast):
-    return linear_recurrence(q, k, v, None, beta, 1.0, state, heads, key_heads, dim, vdim, step, delta=delta, log_decay=log_decay)
+def head_decay_recurrence(q, k, v, log_decay, beta, state, heads, key_heads, dim, vdim, step, delta, fast, norm=None):
+    o = linear_recurrence(q, k, v, None, beta, 1.0, state, heads, key_heads, dim, vdim, step, delta=delta, log_decay=log_decay)
+    return o if norm is None else head_norm_gate(o, norm[0], norm[1], norm[2], "silu", heads, vdim, norm[3])
 
 
 class Columns:

@@ -667,3 +667,34 @@ def test_recurrence_in_chunks_against_one_walk(monkeypatch, D, V, heads, groups,
         for a, b in zip(*outs):
             assert torch.isfinite(b).all() and (a - b).abs().max() <= 1e-4 * max(1.0, a.abs().max().item()), (lens, (a - b).abs().max(), a.abs().max())
         assert not torch.equal(outs[1][1], state0)
+
+
+@gpu
+@pytest.mark.parametrize("D,V,heads,groups", [(16, 8, 4, 2), (48, 48, 4, 2), (128, 256, 2, 1), (128, 64, 6, 2), (33, 100, 3, 3), (256, 32, 2, 2), (300, 256, 1, 1)])
+@pytest.mark.parametrize("delta", [False, True])
+def test_single_tokens_in_one_kernel(D, V, heads, groups, delta):
+    """A step of single tokens: recurrence, read-out and, where asked for, head norm and gate in one kernel, against plain
+    arithmetic; sizes that do not fit its registers take the walk."""
+    import kernel_refs as R
+    from zinfer_b200 import ops
+
+    g = torch.Generator().manual_seed(D + V)
+    rnd = lambda *s: torch.randn(*s, generator=g)
+    step, ref = _steps([1] * 7)
+    rows, proj, w = rnd(7, 2 * groups * D + heads * V), rnd(7, heads * V + 5), 1 + 0.2 * rnd(V)
+    rows[:, :2 * groups * D] /= D ** 0.5
+    logs, beta, state0 = -torch.rand(7, heads, generator=g), torch.rand(7, heads, generator=g), rnd(9, heads, D, V)
+    cut = lambda t: (t[:, :groups * D], t[:, groups * D:2 * groups * D], t[:, 2 * groups * D:])
+    for normed in (False, True):
+        sr = state0.clone()
+        want = R.head_decay_recurrence(*cut(rows), logs, beta, sr, heads, groups, D, V, ref, delta, True,
+                                       norm=(w, 1e-5, R.Columns(proj, 3, heads * V), torch.float32) if normed else None)
+        p = proj.to(DEV)
+        for src in (p, ops.Partials(torch.stack([0.5 * p, 0.5 * p]).contiguous())):
+            for dtype in (torch.float32, torch.bfloat16) if normed else (torch.float32,):
+                sd = state0.to(DEV)
+                got = ops.head_decay_recurrence(*cut(rows.to(DEV)), logs.to(DEV), beta.to(DEV), sd, heads, groups, D, V, step, delta, True,
+                                                norm=(w.to(DEV), 1e-5, ops.Columns(src, 3, heads * V), dtype) if normed else None)
+                tol = 1e-2 if dtype == torch.bfloat16 else 2e-4
+                assert got.dtype == dtype and torch.allclose(got.float().cpu(), want, rtol=tol, atol=tol * max(1.0, want.abs().max().item()))
+                assert torch.allclose(sd.cpu(), sr, rtol=1e-4, atol=1e-4)

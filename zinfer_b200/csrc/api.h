@@ -230,6 +230,12 @@ int zi_linear_recurrence(float* out, int ldo, const void* q, int ldq, const void
                          int ldv, int v_dtype, const float* decay, int ldg, const float* beta, int ldb, float q_scale,
                          float* state, long long slot_stride, int H, int G, int D, int V, int delta, int head_decay, int only_single,
                          const int* cu_q, const int* state_slots, int n_seqs, cudaStream_t stream);
+// Single tokens of the recurrences with one decay per head: recurrence, read-out, head norm and gate in one kernel
+int zi_head_decay_decode_supported(int D, int V);
+int zi_head_decay_decode(void* out, int out_dtype, int ldo, const float* q, int ldq, const float* k, int ldk, const float* v, int ldv,
+                         const float* logg, const float* beta, float* state, long long slot_stride, int H, int G, int D, int V,
+                         int delta, const float* norm_w, float eps, const float* gate, int ldgate, int gate_splits,
+                         long long gate_zstride, const int* cu_q, const int* state_slots, int n_seqs, cudaStream_t stream);
 // Long portions of the recurrences with one decay per head, in chunks (chunked_recurrence.cu)
 int zi_chunked_recurrence_supported(int D, int V, int H, int G);
 long long zi_chunked_recurrence_workspace_floats(int T, int n_seqs, int H, int G, int D, int V, int delta);

@@ -282,14 +282,18 @@ __device__ __forceinline__ void ck_ldsm_t(uint32_t* r, const bf* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
 }
 __device__ __forceinline__ void ck_mma(float* d, const uint32_t* a, const uint32_t* b) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
 }
-// both operands in two parts; the product of the remainders is below the sums' own rounding
-__device__ __forceinline__ void ck_mma3(float* d, const uint32_t* ah, const uint32_t* al, const uint32_t* bh, const uint32_t* bl) {
-  ck_mma(d, al, bh);
-  ck_mma(d, ah, bl);
-  ck_mma(d, ah, bh);
+// Two neighbouring 16 x 8 tiles, both operands in two parts; the product of the remainders is below the sums' own
+// rounding.  The tiles take turns, so that a product does not wait for the one right before it.
+__device__ __forceinline__ void ck_mma3(float (&d)[2][4], const uint32_t* ah, const uint32_t* al, const uint32_t* bh, const uint32_t* bl) {
+  ck_mma(d[0], al, bh);
+  ck_mma(d[1], al, bh + 2);
+  ck_mma(d[0], ah, bl);
+  ck_mma(d[1], ah, bl + 2);
+  ck_mma(d[0], ah, bh);
+  ck_mma(d[1], ah, bh + 2);
 }
 __device__ __forceinline__ void ck_cp16(void* dst, const void* src) {
   const uint32_t a = (uint32_t)__cvta_generic_to_shared(dst);
@@ -324,23 +328,24 @@ chunk_walk_kernel(const Chunked j) {
   if (qlen <= 1) return;                              // single tokens are not done here
   const int g = h / (j.H / j.G), chunks = (qlen + CK - 1) / CK, slot0 = tok0 / CK + seq;
   float* S = j.state + (size_t)j.state_slots[seq] * j.slot_stride + (size_t)h * D * j.V;
+  const bool pairs = j.V % 2 == 0 && j.ldv % 2 == 0 && j.ldo % 2 == 0 && ((uintptr_t)j.v & 7) == 0 && ((uintptr_t)j.out & 7) == 0;
   const int fr = lane >> 2, fc = (lane & 3) * 2;      // an accumulator's first row and column
 
   // the rolling loads of a chunk: Q and W once, K, q . k and the sums in two buffers
   auto load = [&](int i) {
     const int slot = slot0 + i, buf = i & 1;
     const size_t at = ((size_t)slot * j.G + g) * 2 * CK * D, wat = ((size_t)slot * j.H + h) * 2 * CK * D;
-    const int per_row = D / 8, pieces = 2 * CK * per_row;
-    for (int e = tid; e < pieces; e += CW_THREADS) {
-      const int r = e / per_row, x = (e - r * per_row) * 8;                          // row of both parts
+    const int x = (tid & 15) * 8;                      // 16 threads a row (D <= 128), rows of both parts
+#pragma unroll 4
+    for (int r = tid >> 4; r < 2 * CK && x < D; r += CW_THREADS / 16) {
       ck_cp16(Q + r * DP + x, j.qs + at + (size_t)r * D + x);
       ck_cp16(K + buf * tile + r * DP + x, j.ks + at + (size_t)r * D + x);
       if (DELTA) ck_cp16(W + r * DP + x, j.w + wat + (size_t)r * D + x);
     }
     const float* qk = j.qk + ((size_t)slot * j.G + g) * CK * CK;
     for (int e = tid; e < CK * CK / 4; e += CW_THREADS) {
-      const int r = e / (CK / 4), x = (e - r * (CK / 4)) * 4;
-      if (x <= r) ck_cp16(P + buf * CK * PP + r * PP + x, qk + r * CK + x);
+      const int r = e / (CK / 4), s = (e - r * (CK / 4)) * 4;
+      if (s <= r) ck_cp16(P + buf * CK * PP + r * PP + s, qk + r * CK + s);
     }
     if (tid < CK / 4) ck_cp16(Cs + buf * CK + tid * 4, j.c + ((size_t)slot * j.H + h) * CK + tid * 4);
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -386,18 +391,26 @@ chunk_walk_kernel(const Chunked j) {
   for (int i = 0; i < chunks; ++i) {
     const int n = min(CK, qlen - i * CK), first = tok0 + i * CK, buf = i & 1;
     // what becomes U: asked for now, needed after the products with the state
-    float u[2][4];
+    float u[2][4], step[2] = {1.f, 1.f};
 #pragma unroll
-    for (int nn = 0; nn < 2; ++nn)
+    for (int r = 0; r < 2; ++r) {
+      const int t = wr * 16 + fr + r * 8;
+      if (!DELTA) step[r] = t < n ? j.beta[(size_t)(first + t) * j.H + h] : 0.f;
+      const float* pu = DELTA ? j.u0 + (((size_t)(slot0 + i) * j.H + h) * CK + t) * j.V : j.v + (size_t)(first + t) * j.ldv + (size_t)h * j.V;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int t = wr * 16 + fr + (e >> 1) * 8, col = v0 + wc * 16 + nn * 8 + fc + (e & 1);
-        u[nn][e] = 0.f;
-        if (t < n && col < j.V) {
-          if (DELTA) u[nn][e] = j.u0[(((size_t)(slot0 + i) * j.H + h) * CK + t) * j.V + col];
-          else u[nn][e] = j.beta[(size_t)(first + t) * j.H + h] * j.v[(size_t)(first + t) * j.ldv + (size_t)h * j.V + col];
+      for (int nn = 0; nn < 2; ++nn) {
+        const int col = v0 + wc * 16 + nn * 8 + fc;
+        float2 x = make_float2(0.f, 0.f);
+        if (t < n && pairs && col < j.V) {
+          x = *reinterpret_cast<const float2*>(pu + col);
+        } else if (t < n) {
+          if (col < j.V) x.x = pu[col];
+          if (col + 1 < j.V) x.y = pu[col + 1];
         }
+        u[nn][2 * r] = x.x;
+        u[nn][2 * r + 1] = x.y;
       }
+    }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                  // this chunk's tiles and the state are there; the chunk before is done with
     float qs[2][4];
@@ -417,13 +430,12 @@ chunk_walk_kernel(const Chunked j) {
       ck_ldsm_t(bl, Ss + D * VP + (kk + lr) * VP + wc * 16 + lc);
       ck_ldsm(ah, Q + (wr * 16 + lr) * DP + kk + lc);
       ck_ldsm(al, Q + CK * DP + (wr * 16 + lr) * DP + kk + lc);
-#pragma unroll
-      for (int nn = 0; nn < 2; ++nn) ck_mma3(qs[nn], ah, al, bh + 2 * nn, bl + 2 * nn);
+      ck_mma3(qs, ah, al, bh, bl);
       if constexpr (DELTA) {
-        ck_ldsm(ah, W + (wr * 16 + lr) * DP + kk + lc);
-        ck_ldsm(al, W + CK * DP + (wr * 16 + lr) * DP + kk + lc);
-#pragma unroll
-        for (int nn = 0; nn < 2; ++nn) ck_mma3(ws[nn], ah, al, bh + 2 * nn, bl + 2 * nn);
+        uint32_t wh[4], wl[4];
+        ck_ldsm(wh, W + (wr * 16 + lr) * DP + kk + lc);
+        ck_ldsm(wl, W + CK * DP + (wr * 16 + lr) * DP + kk + lc);
+        ck_mma3(ws, wh, wl, bh, bl);
       }
     }
     const float* cs = Cs + buf * CK;
@@ -433,7 +445,7 @@ chunk_walk_kernel(const Chunked j) {
 #pragma unroll
       for (int e = 0; e < 4; e += 2) {
         const int row = wr * 16 + fr + (e >> 1) * 8, col = wc * 16 + nn * 8 + fc;
-        const float x = DELTA ? u[nn][e] - ws[nn][e] : u[nn][e], y = DELTA ? u[nn][e + 1] - ws[nn][e + 1] : u[nn][e + 1];
+        const float x = DELTA ? u[nn][e] - ws[nn][e] : step[e >> 1] * u[nn][e], y = DELTA ? u[nn][e + 1] - ws[nn][e + 1] : step[e >> 1] * u[nn][e + 1];
         const float f = expf(cend - ct[e >> 1]);
         bf xh, xl, yh, yl;
         split2(x, xh, xl);
@@ -476,15 +488,20 @@ chunk_walk_kernel(const Chunked j) {
       }
       ck_ldsm_t(bh, Us + (kb * 16 + lr) * VP + wc * 16 + lc);
       ck_ldsm_t(bl, Us + CK * VP + (kb * 16 + lr) * VP + wc * 16 + lc);
-#pragma unroll
-      for (int nn = 0; nn < 2; ++nn) ck_mma3(o[nn], ah, al, bh + 2 * nn, bl + 2 * nn);
+      ck_mma3(o, ah, al, bh, bl);
     }
 #pragma unroll
     for (int nn = 0; nn < 2; ++nn)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int t = wr * 16 + fr + (e >> 1) * 8, col = v0 + wc * 16 + nn * 8 + fc + (e & 1);
-        if (t < n && col < j.V) j.out[(size_t)(first + t) * j.ldo + (size_t)h * j.V + col] = o[nn][e];
+      for (int e = 0; e < 4; e += 2) {
+        const int t = wr * 16 + fr + (e >> 1) * 8, col = v0 + wc * 16 + nn * 8 + fc;
+        float* po = j.out + (size_t)(first + t) * j.ldo + (size_t)h * j.V + col;
+        if (t < n && pairs && col < j.V) {
+          *reinterpret_cast<float2*>(po) = make_float2(o[nn][e], o[nn][e + 1]);
+        } else if (t < n) {
+          if (col < j.V) po[0] = o[nn][e];
+          if (col + 1 < j.V) po[1] = o[nn][e + 1];
+        }
       }
     // S = e^(c_64) S + K^T U e^(c_64 - c)
     const float fend = expf(cend);
@@ -509,8 +526,7 @@ chunk_walk_kernel(const Chunked j) {
         const bf* kp = Kb + (kb * 16 + (lane & 7) + (lane >> 4) * 8) * DP + c0 + ((lane >> 3) & 1) * 8;
         ck_ldsm_t(ah, kp);
         ck_ldsm_t(al, kp + CK * DP);
-#pragma unroll
-        for (int nn = 0; nn < 2; ++nn) ck_mma3(acc[m][nn], ah, al, bh + 2 * nn, bl + 2 * nn);
+        ck_mma3(acc[m], ah, al, bh, bl);
       }
     }
     if (i + 1 < chunks) share_state();

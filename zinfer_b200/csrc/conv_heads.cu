@@ -99,11 +99,21 @@ conv_heads_kernel(const ConvJob j) {
     }
     return;
   }
+  // where the tile's tokens go, worked out once per block
+  __shared__ int tok_pos[CH_TILE], tok_page[CH_TILE], tok_off[CH_TILE];
+  if (threadIdx.x < nt && (j.cos_t || j.slots)) {
+    const int t = threadIdx.x, slot = j.slots ? j.slots[row0 + t] : -1, pos = j.positions[row0 + t];
+    tok_pos[t] = pos < 0 ? 0 : (pos >= j.n_table_pos ? j.n_table_pos - 1 : pos);      // the host refuses such positions
+    tok_page[t] = slot < 0 ? -1 : slot / j.page_size;
+    tok_off[t] = slot < 0 ? 0 : slot % j.page_size;
+  }
+  __syncthreads();
   const int head_all = blockIdx.y * CH_WARPS + warp;
   if (head_all >= j.heads) return;
   int si = 0;
   while (si + 1 < j.n_seg && head_all >= j.seg[si + 1].first_head) ++si;
-  const ConvSegment& g = j.seg[si];
+  const ConvSegment g = j.seg[si];
+  const int page_heads = g.dest == 2 ? g.n / g.d : 0;
   const int head = head_all - g.first_head;
   const int d = min(g.d, g.n - head * g.d);             // channels of this head
   const int ch0 = g.c0 + head * g.d;                    // its first channel
@@ -145,10 +155,9 @@ conv_heads_kernel(const ConvJob j) {
     if (g.dest == 1) {
       o = static_cast<T*>(g.out) + row * g.ldo + (size_t)head * g.d;
     } else {
-      const int slot = j.slots[row];
-      if (slot < 0) return;                             // a row that pads a captured batch
-      const int kv_heads = g.n / g.d;
-      o = static_cast<T*>(g.out) + (((size_t)(slot / j.page_size) * kv_heads + head) * j.page_size + slot % j.page_size) * g.d;
+      const int page = tok_page[t];
+      if (page < 0) return;                             // a row that pads a captured batch
+      o = static_cast<T*>(g.out) + (((size_t)page * page_heads + head) * j.page_size + tok_off[t]) * g.d;
     }
     if constexpr (PAIRS && sizeof(T) == 2) {
       if (two) {
@@ -225,9 +234,8 @@ conv_heads_kernel(const ConvJob j) {
           continue;
         }
         if (p < half) {
-          int pos = j.positions[row0 + t];
-          pos = pos < 0 ? 0 : (pos >= j.n_table_pos ? j.n_table_pos - 1 : pos);      // the host refuses such positions
-          rotate_pair(y0, y1, j.cos_t[(size_t)pos * half + p], j.sin_t[(size_t)pos * half + p]);
+          const size_t at = (size_t)tok_pos[t] * half + p;
+          rotate_pair(y0, y1, j.cos_t[at], j.sin_t[at]);
         }
         put(t, e0, e1, y0, y1, two);
       }

@@ -601,6 +601,123 @@ gated_decode_kernel(TO* __restrict__ out, int ldo, const float* __restrict__ q, 
   if (tid < V) out[(size_t)row * ldo + (size_t)h * V + tid] = from_f32<TO>(o * inv * w[tid]);
 }
 
+// ------------------------------- one token per request: a decay and a step per head, with the head norm and its gate
+// A block takes one request's token and one head; the whole head's state lies in the registers of its HD_THREADS threads
+// (rows of S in 16-byte pieces: LPR neighbouring lanes a row, HD_RD rows a thread), asked for before the kernel waits for the
+// one before it (nothing of this step has written it).  Both read-outs, S^T k and S^T q, come from one pass over the old
+// state:  o = g S^T q + (k . q) u,  u = beta (v - g S^T k) (DELTA) or beta v;  then S <- g S + k u^T is written.
+// With norm_w: o / sqrt(mean(o^2) + eps) * norm_w * silu(gate) in the activations' type; else o as it is.
+constexpr int HD_THREADS = 512, HD_RD = 8;
+
+template <typename TO, int NCV, bool DELTA>
+__global__ void __launch_bounds__(HD_THREADS)
+head_decay_decode_kernel(TO* __restrict__ out, int ldo, const float* __restrict__ q, int ldq, const float* __restrict__ k, int ldk,
+                         const float* __restrict__ v, int ldv, const float* __restrict__ logg, const float* __restrict__ beta,
+                         float* __restrict__ state, long long slot_stride, int H, int G, int D, int V, int LPR,
+                         const int* __restrict__ cu_q, const int* __restrict__ state_slots, const float* __restrict__ norm_w, float eps,
+                         const float* __restrict__ gate, int ldgate, int gsplits, long long gz) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float hd[];
+  __shared__ float scratch[33];
+  const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, kvh = h / (H / G);
+  const int slots = HD_THREADS / LPR, slot = tid / LPR, l = tid % LPR;
+  float* qs = hd;                    // [D] q and k, [V] u, then the partial sums [2][slots][V]
+  float* ks = qs + D;
+  float* us = hd + ((2 * D + 3) & ~3);
+  float* ra = us + V;
+  float* rb = ra + slots * V;
+  const int row = cu_q[s];
+  float* S = state + (size_t)state_slots[s] * slot_stride + (size_t)h * D * V;
+  float4 st[HD_RD][NCV];
+  auto col = [&](int c) { return (c * LPR + l) * 4; };
+#pragma unroll
+  for (int u = 0; u < HD_RD; ++u) {
+    const int i = slot + u * slots;
+#pragma unroll
+    for (int c = 0; c < NCV; ++c)
+      st[u][c] = i < D && col(c) < V ? *reinterpret_cast<const float4*>(S + (size_t)i * V + col(c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  pdl_wait();
+  for (int e = tid; e < 2 * D; e += HD_THREADS) {
+    if (e < D) qs[e] = q[(size_t)row * ldq + (size_t)kvh * D + e];
+    else ks[e - D] = k[(size_t)row * ldk + (size_t)kvh * D + e - D];
+  }
+  float vj = 0.f, gt = 0.f;
+  if (tid < V) {
+    vj = v[(size_t)row * ldv + (size_t)h * V + tid];
+    if (gate) {
+      const float* pg = gate + (size_t)row * ldgate + (size_t)h * V + tid;
+      gt = *pg;
+      for (int z = 1; z < gsplits; ++z) gt += pg[(size_t)z * gz];
+    }
+  }
+  const float g = expf(logg[(size_t)row * H + h]), b = beta[(size_t)row * H + h];
+  __syncthreads();
+  float kq = 0.f;                    // every warp makes it for itself, in the same order
+  for (int i = tid & 31; i < D; i += 32) kq = fmaf(ks[i], qs[i], kq);
+  kq = warp_sum(kq);
+  float4 a[NCV], o4[NCV];
+#pragma unroll
+  for (int c = 0; c < NCV; ++c) a[c] = o4[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int u = 0; u < HD_RD; ++u) {
+    const int i = slot + u * slots;
+    if (i >= D) break;
+    const float ki = ks[i], qi = qs[i];
+#pragma unroll
+    for (int c = 0; c < NCV; ++c) {
+      const float4 t = st[u][c];
+      if (DELTA) {
+        a[c].x = fmaf(ki, t.x, a[c].x);
+        a[c].y = fmaf(ki, t.y, a[c].y);
+        a[c].z = fmaf(ki, t.z, a[c].z);
+        a[c].w = fmaf(ki, t.w, a[c].w);
+      }
+      o4[c].x = fmaf(qi, t.x, o4[c].x);
+      o4[c].y = fmaf(qi, t.y, o4[c].y);
+      o4[c].z = fmaf(qi, t.z, o4[c].z);
+      o4[c].w = fmaf(qi, t.w, o4[c].w);
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < NCV; ++c)
+    if (col(c) < V) {
+      if (DELTA) *reinterpret_cast<float4*>(ra + (size_t)slot * V + col(c)) = a[c];
+      *reinterpret_cast<float4*>(rb + (size_t)slot * V + col(c)) = o4[c];
+    }
+  __syncthreads();
+  float o = 0.f;
+  if (tid < V) {                     // V <= HD_THREADS: one value channel per thread
+    float sa = 0.f;
+    for (int z = 0; z < slots; ++z) {
+      if (DELTA) sa += ra[(size_t)z * V + tid];
+      o += rb[(size_t)z * V + tid];
+    }
+    const float u = b * (DELTA ? vj - g * sa : vj);
+    us[tid] = u;
+    o = fmaf(u, kq, g * o);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int u = 0; u < HD_RD; ++u) {
+    const int i = slot + u * slots;
+    if (i >= D) break;
+    const float ki = ks[i];
+#pragma unroll
+    for (int c = 0; c < NCV; ++c) {
+      if (col(c) >= V) continue;
+      const float4 u4 = *reinterpret_cast<const float4*>(us + col(c)), t = st[u][c];
+      *reinterpret_cast<float4*>(S + (size_t)i * V + col(c)) =
+          make_float4(fmaf(g, t.x, ki * u4.x), fmaf(g, t.y, ki * u4.y), fmaf(g, t.z, ki * u4.z), fmaf(g, t.w, ki * u4.w));
+    }
+  }
+  if (norm_w) {                      // uniform
+    const float inv = 1.0f / sqrtf(block_sum(o * o, scratch) / (float)V + eps);
+    if (tid < V) o = o * inv * norm_w[tid] * (gt * sigmoid_f32(gt));
+  }
+  if (tid < V) out[(size_t)row * ldo + (size_t)h * V + tid] = from_f32<TO>(o);
+}
+
 // ----------------------------------------------------------------------- gated per-head norm
 // out[t, head, :] = o / sqrt(mean(o^2) + eps) * w * act(gate[t, head, :]); act: 0 silu, 1 sigmoid, 2 no gate.
 // The gate may come as split-K partial sums (float32, gz apart), added in order.  One warp per (token, head).
@@ -821,6 +938,42 @@ extern "C" int zi_gated_decode(void* out, int out_dtype, int ldo, const float* q
               gate, norm_w, eps);
   });
   return zi_check_launch("gated_decode");
+}
+
+static int head_decay_lanes(int V) {
+  int lpr = 8;
+  while (lpr < 32 && lpr * 4 < V) lpr <<= 1;
+  return lpr;
+}
+// Whether a head's state fits the registers of one block.
+extern "C" int zi_head_decay_decode_supported(int D, int V) {
+  return D > 0 && V > 0 && V <= 256 && V % 4 == 0 && D <= HD_RD * (HD_THREADS / head_decay_lanes(V));
+}
+
+// Every request brings one token: the recurrence with one decay and one step per head, read-out included; with norm_w the
+// head norm and its silu gate (float32 columns, whole or split-K partial sums) as well, in the activations' type.
+extern "C" int zi_head_decay_decode(void* out, int out_dtype, int ldo, const float* q, int ldq, const float* k, int ldk, const float* v,
+                                    int ldv, const float* logg, const float* beta, float* state, long long slot_stride, int H, int G,
+                                    int D, int V, int delta, const float* norm_w, float eps, const float* gate, int ldgate,
+                                    int gate_splits, long long gate_zstride, const int* cu_q, const int* state_slots, int n_seqs,
+                                    cudaStream_t stream) {
+  if (n_seqs <= 0) return 0;
+  if (!zi_head_decay_decode_supported(D, V)) return zi_refuse("head_decay_decode: %d key channels, %d value channels", D, V);
+  if (H <= 0 || H > 65535 || G <= 0 || H % G || !logg || !beta) return zi_refuse("head_decay_decode: %d heads, %d of keys", H, G);
+  if ((norm_w == nullptr) != (gate == nullptr)) return zi_refuse("head_decay_decode: a norm goes with its gate");
+  if (slot_stride % 4 || ((uintptr_t)state & 15)) return zi_refuse("head_decay_decode: the state must be 16-byte aligned");
+  const int LPR = head_decay_lanes(V);
+  const size_t smem = (size_t)(((2 * D + 3) & ~3) + V + 2 * (HD_THREADS / LPR) * V) * sizeof(float);
+  dim3 grid(n_seqs, H), block(HD_THREADS);
+  ZI_DISPATCH_DTYPE(out_dtype, TO, {
+    auto kern = V <= 128 ? (delta ? head_decay_decode_kernel<TO, 1, true> : head_decay_decode_kernel<TO, 1, false>)
+                         : (delta ? head_decay_decode_kernel<TO, 2, true> : head_decay_decode_kernel<TO, 2, false>);
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+      return zi_refuse("head_decay_decode: cannot get %zu bytes of shared memory", smem);
+    zi_launch(kern, grid, block, smem, stream, (TO*)out, ldo, q, ldq, k, ldk, v, ldv, logg, beta, state, slot_stride, H, G, D, V, LPR, cu_q,
+              state_slots, norm_w, eps, gate, ldgate, gate_splits, gate_zstride);
+  });
+  return zi_check_launch("head_decay_decode");
 }
 
 extern "C" int zi_head_norm_gate(void* out, int out_dtype, int ldo, const float* o, int ldi, const float* w, float eps,

@@ -574,6 +574,42 @@ __global__ void gather_rows_kernel(T* __restrict__ out, const T* __restrict__ x,
     out[(size_t)r * width + c] = src >= 0 ? x[(size_t)src * ldx + c] : from_f32<T>(0.f);
 }
 
+// The same in 16-byte pieces: whole rows of 4-wide columns (H % 4 == 0), rows of 8 for bfloat16 gathers (width % 8 == 0).
+template <typename T>
+__global__ void __launch_bounds__(256)
+gather_rows_vec_kernel(uint4* __restrict__ out, const T* __restrict__ x, const int* __restrict__ row_src, int pieces, int ldx) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r = blockIdx.x, src = row_src[r];
+  const uint4* xr = reinterpret_cast<const uint4*>(x + (size_t)(src >= 0 ? src : 0) * ldx);
+  for (int c = threadIdx.x; c < pieces; c += blockDim.x)
+    out[(size_t)r * pieces + c] = src >= 0 ? xr[c] : make_uint4(0u, 0u, 0u, 0u);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_combine_vec_kernel(T* __restrict__ out, const float* __restrict__ y, const T* __restrict__ x, const int* __restrict__ chosen,
+                       const float* __restrict__ weight, const int* __restrict__ pair_row, int top, int E, int H) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.y, c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (c >= H) return;
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+  for (int k = 0; k < top; ++k) {
+    const size_t p = (size_t)t * top + k;
+    const float4 v = chosen[p] < E ? load4(y + (size_t)pair_row[p] * H + c) : load4(x + (size_t)t * H + c);
+    const float w = weight ? weight[p] : 1.f;
+    acc.x = fmaf(w, v.x, acc.x);
+    acc.y = fmaf(w, v.y, acc.y);
+    acc.z = fmaf(w, v.z, acc.z);
+    acc.w = fmaf(w, v.w, acc.w);
+  }
+  __align__(8) T o[4] = {from_f32<T>(acc.x), from_f32<T>(acc.y), from_f32<T>(acc.z), from_f32<T>(acc.w)};
+  if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(out + (size_t)t * H + c) = make_float4(acc.x, acc.y, acc.z, acc.w);
+  else *reinterpret_cast<uint2*>(out + (size_t)t * H + c) = *reinterpret_cast<const uint2*>(o);
+}
+
 // out[t] = sum_k weight[t,k] * (expert output of pair (t,k), or x[t] for an identity expert), k ascending; without weights
 // (the experts' inputs were weighted) the plain sum.
 template <typename T>
@@ -771,6 +807,12 @@ extern "C" int zi_moe_align(const int* chosen, int P, int top, int E, int tile_r
 extern "C" int zi_gather_rows(void* out, const void* x, int dtype, const int* row_src, int rows, int width, int ldx,
                               cudaStream_t stream) {
   if (rows <= 0 || width <= 0) return 0;
+  const int per = dtype == ZI_BF16 ? 8 : 4;
+  if (width % per == 0 && ldx % per == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)out & 15) == 0) {
+    ZI_DISPATCH_DTYPE(dtype, TT, zi_launch(gather_rows_vec_kernel<TT>, dim3(rows), dim3(256), 0, stream, (uint4*)out, (const TT*)x, row_src,
+                                           width / per, ldx));
+    return zi_check_launch("gather_rows");
+  }
   ZI_DISPATCH_DTYPE(dtype, TT, zi_launch(gather_rows_kernel<TT>, dim3(rows), dim3(256), 0, stream, (TT*)out, (const TT*)x,
                                          row_src, width, ldx));
   return zi_check_launch("gather_rows");
@@ -780,6 +822,11 @@ extern "C" int zi_moe_combine(void* out, const float* y, const void* x, int dtyp
                               const float* weight, const int* pair_row, int T, int top, int E, int H,
                               cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (H % 4 == 0 && ((uintptr_t)y & 15) == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)out & 15) == 0) {
+    ZI_DISPATCH_DTYPE(dtype, TT, zi_launch(moe_combine_vec_kernel<TT>, dim3((H / 4 + 255) / 256, T), dim3(256), 0, stream, (TT*)out, y,
+                                           (const TT*)x, chosen, weight, pair_row, top, E, H));
+    return zi_check_launch("moe_combine");
+  }
   dim3 grid((H + 255) / 256, T);
   ZI_DISPATCH_DTYPE(dtype, TT, zi_launch(moe_combine_kernel<TT>, dim3(grid), dim3(256), 0, stream, (TT*)out, y, (const TT*)x,
                                          chosen, weight, pair_row, top, E, H));

@@ -1885,10 +1885,40 @@ RECURRENCE_CHUNK_MIN = 96     # from this many tokens in a request's portion the
 
 
 def head_decay_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: torch.Tensor, beta: torch.Tensor, state: torch.Tensor,
-                          heads: int, key_heads: int, dim: int, vdim: int, step, delta: bool, fast: bool) -> torch.Tensor:
+                          heads: int, key_heads: int, dim: int, vdim: int, step, delta: bool, fast: bool,
+                          norm: Optional[tuple] = None) -> torch.Tensor:
     """The recurrence with one decay per head (see :func:`linear_recurrence`; q ready, float32 operands): token by token, or,
     where ``fast`` allows the tensor cores' products (each operand in two bfloat16 parts) and a portion is long, in chunks of
-    64 tokens, single tokens of the same step token by token.  Returns float32 [T, heads * vdim]."""
+    64 tokens, single tokens of the same step token by token; a step of single tokens alone is one kernel.  Returns float32
+    [T, heads * vdim]; with ``norm`` = (weight [vdim], eps, gate :class:`Columns`, out_dtype) every head RMS-normed and
+    multiplied by silu(gate), in ``out_dtype``."""
+    T = q.shape[0]
+    L = lib()
+    if fast and step.all_decode and L.zi_head_decay_decode_supported(dim, vdim):
+        st, stride = _slot_view(state, "head_decay_recurrence")
+        if stride % 4 == 0 and st.data_ptr() % 16 == 0:
+            for t, cols in ((q, key_heads * dim), (k, key_heads * dim), (v, heads * vdim), (log_decay, heads), (beta, heads)):
+                _need(t.dtype == torch.float32 and t.stride(1) == 1 and tuple(t.shape) == (T, cols), "head_decay_recurrence: float32 rows")
+            _need(log_decay.is_contiguous() and beta.is_contiguous() and st[0].numel() == heads * dim * vdim, "head_decay_recurrence: state [slots, heads, dim, vdim]")
+            w, eps, gate, dt = norm if norm is not None else (None, 0.0, None, torch.float32)
+            _need(w is None or (w.dtype == torch.float32 and w.numel() == vdim and gate.shape == (T, heads * vdim)), "head_decay_recurrence: norm")
+            res = torch.empty((T, heads * vdim), dtype=dt, device=q.device)
+            with _prof.region("recurrence (single tokens" + (", delta rule" if delta else "") + (", head norm)" if w is not None else ")"),
+                              lambda: _nb(q, k, v, res) + 2 * step.n_seqs * heads * dim * vdim * 4 + (gate.bytes() if gate is not None else 0),
+                              6 * T * heads * dim * vdim):
+                _check(L.zi_head_decay_decode(
+                    _ptr(res), _tag(res), res.stride(0), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(log_decay),
+                    _ptr(beta), _ptr(st), _ll(stride), heads, key_heads, dim, vdim, 1 if delta else 0, _ptr(w), ctypes.c_float(eps),
+                    gate.ptr if gate is not None else None, gate.ld if gate is not None else 0, gate.splits if gate is not None else 1,
+                    _ll(gate.zstride if gate is not None else 0), _ptr(step.cu_q), _ptr(step.state_slots), step.n_seqs, _stream()), "head_decay_decode")
+            return res
+    out = _head_decay_walk(q, k, v, log_decay, beta, state, heads, key_heads, dim, vdim, step, delta, fast)
+    if norm is None:
+        return out
+    return head_norm_gate(out, norm[0], norm[1], norm[2], "silu", heads, vdim, norm[3])
+
+
+def _head_decay_walk(q, k, v, log_decay, beta, state, heads, key_heads, dim, vdim, step, delta, fast):
     T = q.shape[0]
     L = lib()
     if not (fast and RECURRENCE_CHUNKS and step.max_q_len >= RECURRENCE_CHUNK_MIN and L.zi_chunked_recurrence_supported(dim, vdim, heads, key_heads)):

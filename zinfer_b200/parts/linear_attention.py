@@ -217,9 +217,8 @@ class GatedDeltaRule(Mixer):
             [ops.ConvSegment(qk, self.dim, q, "unit", self.dim ** -0.5), ops.ConvSegment(qk, self.dim, k, "unit"),
              ops.ConvSegment(hv, self.vdim, v)], activation="silu", unit_eps=self.UNIT_EPS,
             decay=("delta", cols(C + hv, H), cols(C + hv + H, H), self.a_log, self.dt_bias))
-        o = ops.head_decay_recurrence(q, k, v, decay, beta, state[:, :self.s_size], H, self.kv_heads, self.dim, self.vdim, step, delta=True,
-                                      fast=self.ctx.dtype == torch.bfloat16)
-        y = ops.head_norm_gate(o, self.norm, self.eps, cols(C, hv), "silu", H, self.vdim, self.ctx.dtype)
+        y = ops.head_decay_recurrence(q, k, v, decay, beta, state[:, :self.s_size], H, self.kv_heads, self.dim, self.vdim, step, delta=True,
+                                      fast=self.ctx.dtype == torch.bfloat16, norm=(self.norm, self.eps, cols(C, hv), self.ctx.dtype))
         return ops.linear(y, self.w_o, out_dtype=self.ctx.dtype, allow_partials=True)
 
     def forward(self, x, step, cache):
