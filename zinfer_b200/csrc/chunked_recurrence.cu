@@ -11,15 +11,16 @@
 //
 // (the chunked form of "Parallelizing Linear Transformers with the Delta Rule over Sequence Length", Yang et al., 2024, and
 // of "Gated Delta Networks", Yang et al., 2024; without the delta rule W = 0 and U = diag(beta) V, the state-space duality of
-// Dao and Gu, 2024).  Three kernels:
+// Dao and Gu, 2024).  The kernels:
 //   1. chunk_scores   per chunk and key head: q . k and k . k (32-bit multiply-adds), Q and K as pairs of bfloat16
 //                     values (high part and remainder: 16 bits of mantissa together), the sums c of every head
-//   2. chunk_solve    (delta rule) per chunk and head: the triangular system by forward substitution in 32-bit, a
+//   2. chunk_weights  per chunk and head: P as pairs of bfloat16 values
+//      chunk_solve    (delta rule) per chunk and head: the triangular system by forward substitution in 32-bit, a
 //                     thread per column of [W | U0]; W as pairs of bfloat16 values
 //   3. chunk_walk     per request, head and 32 value channels: the chunks in order; the products with the state on the
 //                     tensor cores (mma.sync, each operand as two bfloat16 parts, three products, 32-bit sums); the state
 //                     stays in 32-bit accumulators
-// Kernels 1 and 2 do all chunks side by side; only the third walks.  A request's chunks begin with its portion; the places of
+// The first ones do all chunks side by side; only the last walks.  A request's chunks begin with its portion; the places of
 // its chunks in the workspace follow from cu_q alone: chunk i of request s lies at cu_q[s] / 64 + s + i.
 #include "api.h"
 #include "common.cuh"
@@ -50,7 +51,8 @@ struct Chunked {
   bf* ks;
   float* qk;           // [slots][G][CK][CK]
   float* kk;           // delta rule only
-  float* c;            // [slots][H][CK]
+  float* c;            // [slots][H][CK] sums of the logarithms, to base 2
+  bf* p;               // [slots][H][2][CK][CK] P
   bf* w;               // [slots][H][2][CK][D]
   float* u0;           // [slots][H][CK][V]
 };
@@ -78,6 +80,7 @@ __device__ __forceinline__ uint32_t pack2(bf a, bf b) {
 }
 
 // ------------------------------------------------------------------------------------------- 1. scores
+constexpr float LOG2E = 1.4426950408889634f;
 constexpr int CS_THREADS = 256, CS_PITCH = CK + 4;
 
 template <bool DELTA>
@@ -129,8 +132,8 @@ chunk_scores_kernel(const Chunked j) {
   const int warp = tid >> 5, lane = tid & 31, rep = j.H / j.G;
   for (int r = warp; r < rep; r += CS_THREADS / 32) {
     const int h = g * rep + r;
-    float a = 2 * lane < n ? j.logg[(size_t)(first + 2 * lane) * j.H + h] : 0.f;
-    float b = 2 * lane + 1 < n ? j.logg[(size_t)(first + 2 * lane + 1) * j.H + h] : 0.f;
+    float a = 2 * lane < n ? j.logg[(size_t)(first + 2 * lane) * j.H + h] * LOG2E : 0.f;
+    float b = 2 * lane + 1 < n ? j.logg[(size_t)(first + 2 * lane + 1) * j.H + h] * LOG2E : 0.f;
     b += a;
     float run = b;                                    // both tokens; then of all lanes up to this one
 #pragma unroll
@@ -178,11 +181,43 @@ chunk_scores_kernel(const Chunked j) {
   }
 }
 
-// -------------------------------------------------------------------------------- 2. the triangular system
-constexpr int SV_B = 16;             // rows per block of the substitution
-constexpr int SV_THREADS = 128, NT = SV_THREADS;      // columns per block
+// -------------------------------------------------------------------------------- 2. weights, the triangular system
+// Per chunk and head: P as pairs of bfloat16 values.
+constexpr int CP_THREADS = 256;
 
-__global__ void __launch_bounds__(SV_THREADS)
+__global__ void __launch_bounds__(CP_THREADS)
+chunk_weights_kernel(const Chunked j) {
+  pdl_launch_dependents();
+  const int slot = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+  int seq, first, n;
+  const bool on = chunk_of(j, slot, seq, first, n);
+  pdl_wait();
+  if (!on) return;
+  const int g = h / (j.H / j.G);
+  const float* c = j.c + ((size_t)slot * j.H + h) * CK;
+  const float* qk = j.qk + ((size_t)slot * j.G + g) * CK * CK;
+  bf* po = j.p + ((size_t)slot * j.H + h) * 2 * CK * CK;
+  for (int e = tid; e < CK * CK / 4; e += CP_THREADS) {
+    const int t = e / (CK / 4), s = (e - t * (CK / 4)) * 4;
+    if (s >= (t & ~15) + 16) continue;                // 16 x 16 parts above the diagonal are never read
+    const float4 q4 = s <= t ? *reinterpret_cast<const float4*>(qk + t * CK + s) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float4 c4 = *reinterpret_cast<const float4*>(c + s);
+    const float ct = c[t];
+    const float w[4] = {q4.x * exp2f(ct - c4.x), s + 1 <= t ? q4.y * exp2f(ct - c4.y) : 0.f, s + 2 <= t ? q4.z * exp2f(ct - c4.z) : 0.f,
+                        s + 3 <= t ? q4.w * exp2f(ct - c4.w) : 0.f};
+    bf hi[4], lo[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) split2(s + u <= t ? w[u] : 0.f, hi[u], lo[u]);
+    *reinterpret_cast<uint2*>(po + t * CK + s) = make_uint2(pack2(hi[0], hi[1]), pack2(hi[2], hi[3]));
+    *reinterpret_cast<uint2*>(po + CK * CK + t * CK + s) = make_uint2(pack2(lo[0], lo[1]), pack2(lo[2], lo[3]));
+  }
+}
+
+// (delta rule) Per chunk and head: [W | U0] by forward substitution, a column per thread.
+constexpr int SV_B = 16;             // rows per block of the substitution
+constexpr int NT = 128;              // columns per block
+
+__global__ void __launch_bounds__(NT)
 chunk_solve_kernel(const Chunked j) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) float sv[];
@@ -192,23 +227,21 @@ chunk_solve_kernel(const Chunked j) {
   float* be = bs + CK;
   float* xs = be + CK;                                // [CK][NT]: solved rows of this block's columns
   int seq, first, n;
-  if (!chunk_of(j, slot, seq, first, n)) {
-    pdl_wait();
-    return;
-  }
+  const bool on_chunk = chunk_of(j, slot, seq, first, n);
   pdl_wait();
+  if (!on_chunk) return;
   const int g = h / (j.H / j.G);
   const float* c = j.c + ((size_t)slot * j.H + h) * CK;
   const float* kk = j.kk + ((size_t)slot * j.G + g) * CK * CK;
   for (int t = tid; t < CK; t += NT) {
     const float b = t < n ? j.beta[(size_t)(first + t) * j.H + h] : 0.f;
     bs[t] = b;
-    be[t] = b * expf(c[t]);
+    be[t] = b * exp2f(c[t]);
   }
   __syncthreads();
   for (int e = tid; e < CK * CK; e += NT) {
-    const int t = e / CK, s = e - t * CK;
-    lt[s * CS_PITCH + t] = s < t ? bs[t] * expf(c[t] - c[s]) * kk[e] : 0.f;
+    const int s = e / CK, t = e - s * CK;
+    lt[s * CS_PITCH + t] = s < t ? bs[t] * exp2f(c[t] - c[s]) * kk[t * CK + s] : 0.f;
   }
   __syncthreads();
   bf* wo = j.w + ((size_t)slot * j.H + h) * 2 * CK * D;
@@ -243,7 +276,7 @@ chunk_solve_kernel(const Chunked j) {
       }
     }
 #pragma unroll
-    for (int s = 0; s < SV_B; ++s) {                // rows below the diagonal only matter: L is zero above
+    for (int s = 0; s < SV_B; ++s) {                  // only rows below the diagonal change
 #pragma unroll
       for (int r = s & ~3; r < SV_B; r += 4) {
         const float4 l = *reinterpret_cast<const float4*>(lt + (bi + s) * CS_PITCH + bi + r);
@@ -255,7 +288,7 @@ chunk_solve_kernel(const Chunked j) {
     }
 #pragma unroll
     for (int r = 0; r < SV_B; ++r) {
-      xs[(bi + r) * NT + tid] = acc[r];             // read by this thread only
+      xs[(bi + r) * NT + tid] = acc[r];               // read by this thread only
       if (on) {
         if (is_k) {
           bf hi, lo;
@@ -271,7 +304,9 @@ chunk_solve_kernel(const Chunked j) {
 }
 
 // -------------------------------------------------------------------------------------------- 3. the walk
-constexpr int CW_THREADS = 256;
+// Two groups of 8 warps share a chunk: the first moves the state on (W S, U, K^T U), the second reads out (Q S, P U).  In
+// both, warp (row group wr of 16 tokens or key channels, column half wc of 16 value channels).
+constexpr int CW_THREADS = 512;
 
 __device__ __forceinline__ void ck_ldsm(uint32_t* r, const bf* p) {
   const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
@@ -283,7 +318,7 @@ __device__ __forceinline__ void ck_ldsm_t(uint32_t* r, const bf* p) {
 }
 __device__ __forceinline__ void ck_mma(float* d, const uint32_t* a, const uint32_t* b) {
   asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
 }
 // Two neighbouring 16 x 8 tiles, both operands in two parts; the product of the remainders is below the sums' own
 // rounding.  The tiles take turns, so that a product does not wait for the one right before it.
@@ -300,26 +335,28 @@ __device__ __forceinline__ void ck_cp16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(a), "l"(src) : "memory");
 }
 
-__host__ __device__ constexpr size_t ck_walk_smem(int D, bool delta) {
+constexpr int CW_PP = CK + CK_PAD;   // pitch of P
+
+size_t ck_walk_smem(int D, bool delta) {
   const size_t tile = (size_t)2 * CK * (D + CK_PAD) * sizeof(bf);                   // Q, K or W in two parts
-  return tile * (delta ? 4 : 3) + 2 * (size_t)CK * (CK + 4) * sizeof(float) + 2 * CK * sizeof(float)
+  return tile * (delta ? 4 : 3) + 2 * (size_t)2 * CK * CW_PP * sizeof(bf) + 2 * CK * sizeof(float)
          + (size_t)2 * D * (CK_VP + CK_PAD) * sizeof(bf) + (size_t)4 * CK * (CK_VP + CK_PAD) * sizeof(bf);
 }
 
-// Warp (row group wr of 16 tokens or key channels, column half wc of 16 value channels).
 template <bool DELTA>
 __global__ void __launch_bounds__(CW_THREADS)
 chunk_walk_kernel(const Chunked j) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) char walk_smem[];
-  const int D = j.D, DP = D + CK_PAD, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, wr = warp & 3, wc = warp >> 2;
-  constexpr int VP = CK_VP + CK_PAD, PP = CK + 4;
-  const int tile = 2 * CK * DP;                       // elements of a tile in two parts
+  const int D = j.D, DP = D + CK_PAD, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, wr = warp & 3, wc = (warp >> 2) & 1;
+  const bool moves = warp < 8;                        // of the first group
+  constexpr int VP = CK_VP + CK_PAD;
+  const int tile = 2 * CK * DP, ptile = 2 * CK * CW_PP;       // elements of a tile in two parts
   bf* Q = reinterpret_cast<bf*>(walk_smem);
   bf* K = Q + tile;                                   // twice
   bf* W = K + 2 * tile;                               // delta rule only
-  float* P = reinterpret_cast<float*>(W + (DELTA ? tile : 0));      // q . k, twice
-  float* Cs = P + 2 * CK * PP;                        // sums of the logarithms, twice
+  bf* P = W + (DELTA ? tile : 0);                     // twice
+  float* Cs = reinterpret_cast<float*>(P + 2 * ptile);        // sums of the logarithms, twice
   bf* Ss = reinterpret_cast<bf*>(Cs + 2 * CK);        // the state, two parts of [D][VP]
   bf* Us = Ss + 2 * D * VP;                           // U, two parts of [CK][VP]; then U e^(c_64 - c), two parts
   const int seq = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * CK_VP;
@@ -330,34 +367,37 @@ chunk_walk_kernel(const Chunked j) {
   float* S = j.state + (size_t)j.state_slots[seq] * j.slot_stride + (size_t)h * D * j.V;
   const bool pairs = j.V % 2 == 0 && j.ldv % 2 == 0 && j.ldo % 2 == 0 && ((uintptr_t)j.v & 7) == 0 && ((uintptr_t)j.out & 7) == 0;
   const int fr = lane >> 2, fc = (lane & 3) * 2;      // an accumulator's first row and column
+  const int lr = lane & 15, lc = (lane >> 4) * 8;     // ldmatrix: this lane's row and column offset within 16 x 16
 
-  // the rolling loads of a chunk: Q and W once, K, q . k and the sums in two buffers
+  // the rolling loads of a chunk: Q and W once, K, P and the sums in two buffers
   auto load = [&](int i) {
     const int slot = slot0 + i, buf = i & 1;
     const size_t at = ((size_t)slot * j.G + g) * 2 * CK * D, wat = ((size_t)slot * j.H + h) * 2 * CK * D;
-    const int x = (tid & 15) * 8;                      // 16 threads a row (D <= 128), rows of both parts
-#pragma unroll 4
-    for (int r = tid >> 4; r < 2 * CK && x < D; r += CW_THREADS / 16) {
+    const int x = (tid & 15) * 8;                     // 16 threads a row (D <= 128), rows of both parts
+#pragma unroll
+    for (int r = tid >> 4; r < 2 * CK; r += CW_THREADS / 16) {
+      if (x >= D) break;
       ck_cp16(Q + r * DP + x, j.qs + at + (size_t)r * D + x);
       ck_cp16(K + buf * tile + r * DP + x, j.ks + at + (size_t)r * D + x);
       if (DELTA) ck_cp16(W + r * DP + x, j.w + wat + (size_t)r * D + x);
     }
-    const float* qk = j.qk + ((size_t)slot * j.G + g) * CK * CK;
-    for (int e = tid; e < CK * CK / 4; e += CW_THREADS) {
-      const int r = e / (CK / 4), s = (e - r * (CK / 4)) * 4;
-      if (s <= r) ck_cp16(P + buf * CK * PP + r * PP + s, qk + r * CK + s);
+    const bf* p = j.p + ((size_t)slot * j.H + h) * 2 * CK * CK;
+#pragma unroll
+    for (int r = tid >> 3; r < 2 * CK; r += CW_THREADS / 8) {
+      const int s = (tid & 7) * 8;
+      if (s < ((r & (CK - 1)) & ~15) + 16) ck_cp16(P + buf * ptile + r * CW_PP + s, p + r * CK + s);
     }
     if (tid < CK / 4) ck_cp16(Cs + buf * CK + tid * 4, j.c + ((size_t)slot * j.H + h) * CK + tid * 4);
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   load(0);
 
-  // the state in accumulators: key channels 16 (wr + 4 m) .., value channels 16 wc + 8 n ..
+  // the state in the first group's accumulators: key channels 16 (wr + 4 m) .., value channels 16 wc + 8 n ..
   float acc[2][2][4] = {};
   auto each_state = [&](auto f) {
 #pragma unroll
     for (int m = 0; m < 2; ++m) {
-      if ((wr + 4 * m) * 16 >= D) continue;
+      if (!moves || (wr + 4 * m) * 16 >= D) continue;
 #pragma unroll
       for (int nn = 0; nn < 2; ++nn)
 #pragma unroll
@@ -371,7 +411,7 @@ chunk_walk_kernel(const Chunked j) {
   auto share_state = [&] {                            // into shared memory, in two parts
 #pragma unroll
     for (int m = 0; m < 2; ++m) {
-      if ((wr + 4 * m) * 16 >= D) continue;
+      if (!moves || (wr + 4 * m) * 16 >= D) continue;
 #pragma unroll
       for (int nn = 0; nn < 2; ++nn)
 #pragma unroll
@@ -387,23 +427,23 @@ chunk_walk_kernel(const Chunked j) {
   };
   share_state();
 
-  const int lr = lane & 15, lc = (lane >> 4) * 8;     // ldmatrix: this lane's row and column offset within 16 x 16
   for (int i = 0; i < chunks; ++i) {
     const int n = min(CK, qlen - i * CK), first = tok0 + i * CK, buf = i & 1;
-    // what becomes U: asked for now, needed after the products with the state
+    const float* cs = Cs + buf * CK;
+    // what becomes U: asked for now, needed after the product with the state
     float u[2][4], step[2] = {1.f, 1.f};
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       const int t = wr * 16 + fr + r * 8;
-      if (!DELTA) step[r] = t < n ? j.beta[(size_t)(first + t) * j.H + h] : 0.f;
+      if (!DELTA) step[r] = moves && t < n ? j.beta[(size_t)(first + t) * j.H + h] : 0.f;
       const float* pu = DELTA ? j.u0 + (((size_t)(slot0 + i) * j.H + h) * CK + t) * j.V : j.v + (size_t)(first + t) * j.ldv + (size_t)h * j.V;
 #pragma unroll
       for (int nn = 0; nn < 2; ++nn) {
         const int col = v0 + wc * 16 + nn * 8 + fc;
         float2 x = make_float2(0.f, 0.f);
-        if (t < n && pairs && col < j.V) {
+        if (moves && t < n && pairs && col < j.V) {
           x = *reinterpret_cast<const float2*>(pu + col);
-        } else if (t < n) {
+        } else if (moves && t < n) {
           if (col < j.V) x.x = pu[col];
           if (col + 1 < j.V) x.y = pu[col + 1];
         }
@@ -413,138 +453,116 @@ chunk_walk_kernel(const Chunked j) {
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                  // this chunk's tiles and the state are there; the chunk before is done with
-    float qs[2][4];
-#pragma unroll
-    for (int nn = 0; nn < 2; ++nn)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) qs[nn][e] = 0.f;
-    float ws[2][4];
-#pragma unroll
-    for (int nn = 0; nn < 2; ++nn)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) ws[nn][e] = 0.f;
-#pragma unroll 2
-    for (int kk = 0; kk < D; kk += 16) {
-      uint32_t bh[4], bl[4], ah[4], al[4];
-      ck_ldsm_t(bh, Ss + (kk + lr) * VP + wc * 16 + lc);
-      ck_ldsm_t(bl, Ss + D * VP + (kk + lr) * VP + wc * 16 + lc);
-      ck_ldsm(ah, Q + (wr * 16 + lr) * DP + kk + lc);
-      ck_ldsm(al, Q + CK * DP + (wr * 16 + lr) * DP + kk + lc);
-      ck_mma3(qs, ah, al, bh, bl);
-      if constexpr (DELTA) {
-        uint32_t wh[4], wl[4];
-        ck_ldsm(wh, W + (wr * 16 + lr) * DP + kk + lc);
-        ck_ldsm(wl, W + CK * DP + (wr * 16 + lr) * DP + kk + lc);
-        ck_mma3(ws, wh, wl, bh, bl);
-      }
-    }
-    const float* cs = Cs + buf * CK;
     const float ct[2] = {cs[wr * 16 + fr], cs[wr * 16 + fr + 8]}, cend = cs[CK - 1];
-#pragma unroll
-    for (int nn = 0; nn < 2; ++nn)
-#pragma unroll
-      for (int e = 0; e < 4; e += 2) {
-        const int row = wr * 16 + fr + (e >> 1) * 8, col = wc * 16 + nn * 8 + fc;
-        const float x = DELTA ? u[nn][e] - ws[nn][e] : step[e >> 1] * u[nn][e], y = DELTA ? u[nn][e + 1] - ws[nn][e + 1] : step[e >> 1] * u[nn][e + 1];
-        const float f = expf(cend - ct[e >> 1]);
-        bf xh, xl, yh, yl;
-        split2(x, xh, xl);
-        split2(y, yh, yl);
-        *reinterpret_cast<uint32_t*>(Us + row * VP + col) = pack2(xh, yh);
-        *reinterpret_cast<uint32_t*>(Us + CK * VP + row * VP + col) = pack2(xl, yl);
-        split2(x * f, xh, xl);
-        split2(y * f, yh, yl);
-        *reinterpret_cast<uint32_t*>(Us + 2 * CK * VP + row * VP + col) = pack2(xh, yh);
-        *reinterpret_cast<uint32_t*>(Us + 3 * CK * VP + row * VP + col) = pack2(xl, yl);
-      }
-    __syncthreads();                                  // U is there; nobody reads Q, W and the state any more
-    if (i + 1 < chunks) load(i + 1);
-    // O = e^c Q S + P U
-    float o[2][4];
-    {
-      const float f0 = expf(ct[0]), f1 = expf(ct[1]);
-#pragma unroll
-      for (int nn = 0; nn < 2; ++nn) {
-        o[nn][0] = f0 * qs[nn][0];
-        o[nn][1] = f0 * qs[nn][1];
-        o[nn][2] = f1 * qs[nn][2];
-        o[nn][3] = f1 * qs[nn][3];
+    float so[2][4] = {};                              // W S, or Q S
+    if (DELTA || !moves) {
+      const bf* A = moves ? W : Q;
+#pragma unroll 4
+      for (int kk = 0; kk < D; kk += 16) {
+        uint32_t bh[4], bl[4], ah[4], al[4];
+        ck_ldsm_t(bh, Ss + (kk + lr) * VP + wc * 16 + lc);
+        ck_ldsm_t(bl, Ss + D * VP + (kk + lr) * VP + wc * 16 + lc);
+        ck_ldsm(ah, A + (wr * 16 + lr) * DP + kk + lc);
+        ck_ldsm(al, A + CK * DP + (wr * 16 + lr) * DP + kk + lc);
+        ck_mma3(so, ah, al, bh, bl);
       }
     }
-    const float* Pb = P + buf * CK * PP;
-    for (int kb = 0; kb <= wr; ++kb) {
-      uint32_t ah[4], al[4], bh[4], bl[4];
-#pragma unroll
-      for (int x = 0; x < 4; ++x) {                   // rows fr, fr + 8, fr, fr + 8; columns fc, fc, fc + 8, fc + 8
-        const int t = wr * 16 + fr + (x & 1) * 8, s = kb * 16 + fc + (x >> 1) * 8;
-        float p0 = 0.f, p1 = 0.f;
-        if (s <= t) p0 = Pb[t * PP + s] * expf(ct[x & 1] - cs[s]);
-        if (s + 1 <= t) p1 = Pb[t * PP + s + 1] * expf(ct[x & 1] - cs[s + 1]);
-        bf h0, l0, h1, l1;
-        split2(p0, h0, l0);
-        split2(p1, h1, l1);
-        ah[x] = pack2(h0, h1);
-        al[x] = pack2(l0, l1);
-      }
-      ck_ldsm_t(bh, Us + (kb * 16 + lr) * VP + wc * 16 + lc);
-      ck_ldsm_t(bl, Us + CK * VP + (kb * 16 + lr) * VP + wc * 16 + lc);
-      ck_mma3(o, ah, al, bh, bl);
-    }
-#pragma unroll
-    for (int nn = 0; nn < 2; ++nn)
-#pragma unroll
-      for (int e = 0; e < 4; e += 2) {
-        const int t = wr * 16 + fr + (e >> 1) * 8, col = v0 + wc * 16 + nn * 8 + fc;
-        float* po = j.out + (size_t)(first + t) * j.ldo + (size_t)h * j.V + col;
-        if (t < n && pairs && col < j.V) {
-          *reinterpret_cast<float2*>(po) = make_float2(o[nn][e], o[nn][e + 1]);
-        } else if (t < n) {
-          if (col < j.V) po[0] = o[nn][e];
-          if (col + 1 < j.V) po[1] = o[nn][e + 1];
-        }
-      }
-    // S = e^(c_64) S + K^T U e^(c_64 - c)
-    const float fend = expf(cend);
-    const bf* Kb = K + buf * tile;
-#pragma unroll
-    for (int m = 0; m < 2; ++m)
+    if (moves) {
+      const float f[2] = {exp2f(cend - ct[0]), exp2f(cend - ct[1])};
 #pragma unroll
       for (int nn = 0; nn < 2; ++nn)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) acc[m][nn][e] *= fend;
-#pragma unroll
-    for (int kb = 0; kb < CK / 16; ++kb) {
-      uint32_t bh[4], bl[4];
-      ck_ldsm_t(bh, Us + 2 * CK * VP + (kb * 16 + lr) * VP + wc * 16 + lc);
-      ck_ldsm_t(bl, Us + 3 * CK * VP + (kb * 16 + lr) * VP + wc * 16 + lc);
-#pragma unroll
-      for (int m = 0; m < 2; ++m) {
-        const int c0 = (wr + 4 * m) * 16;
-        if (c0 >= D) continue;
-        // K lies by tokens: its transpose's 16 x 16 part, the halves of the tokens behind those of the channels
-        uint32_t ah[4], al[4];
-        const bf* kp = Kb + (kb * 16 + (lane & 7) + (lane >> 4) * 8) * DP + c0 + ((lane >> 3) & 1) * 8;
-        ck_ldsm_t(ah, kp);
-        ck_ldsm_t(al, kp + CK * DP);
-        ck_mma3(acc[m], ah, al, bh, bl);
-      }
+        for (int e = 0; e < 4; e += 2) {
+          const int row = wr * 16 + fr + (e >> 1) * 8, col = wc * 16 + nn * 8 + fc;
+          const float x = DELTA ? u[nn][e] - so[nn][e] : step[e >> 1] * u[nn][e];
+          const float y = DELTA ? u[nn][e + 1] - so[nn][e + 1] : step[e >> 1] * u[nn][e + 1];
+          bf xh, xl, yh, yl;
+          split2(x, xh, xl);
+          split2(y, yh, yl);
+          *reinterpret_cast<uint32_t*>(Us + row * VP + col) = pack2(xh, yh);
+          *reinterpret_cast<uint32_t*>(Us + CK * VP + row * VP + col) = pack2(xl, yl);
+          split2(x * f[e >> 1], xh, xl);
+          split2(y * f[e >> 1], yh, yl);
+          *reinterpret_cast<uint32_t*>(Us + 2 * CK * VP + row * VP + col) = pack2(xh, yh);
+          *reinterpret_cast<uint32_t*>(Us + 3 * CK * VP + row * VP + col) = pack2(xl, yl);
+        }
     }
-    if (i + 1 < chunks) share_state();
+    __syncthreads();                                  // U is there; nobody reads Q, W and the state any more
+    if (i + 1 < chunks) load(i + 1);
+    if (!moves) {                                     // O = e^c Q S + P U
+      const float f[2] = {exp2f(ct[0]), exp2f(ct[1])};
+#pragma unroll
+      for (int nn = 0; nn < 2; ++nn)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) so[nn][e] *= f[e >> 1];
+      const bf* Pb = P + buf * ptile;
+#pragma unroll
+      for (int kb = 0; kb < CK / 16; ++kb) {
+        if (kb > wr) break;
+        uint32_t ah[4], al[4], bh[4], bl[4];
+        ck_ldsm(ah, Pb + (wr * 16 + lr) * CW_PP + kb * 16 + lc);
+        ck_ldsm(al, Pb + CK * CW_PP + (wr * 16 + lr) * CW_PP + kb * 16 + lc);
+        ck_ldsm_t(bh, Us + (kb * 16 + lr) * VP + wc * 16 + lc);
+        ck_ldsm_t(bl, Us + CK * VP + (kb * 16 + lr) * VP + wc * 16 + lc);
+        ck_mma3(so, ah, al, bh, bl);
+      }
+#pragma unroll
+      for (int nn = 0; nn < 2; ++nn)
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const int t = wr * 16 + fr + (e >> 1) * 8, col = v0 + wc * 16 + nn * 8 + fc;
+          float* po = j.out + (size_t)(first + t) * j.ldo + (size_t)h * j.V + col;
+          if (t < n && pairs && col < j.V) {
+            *reinterpret_cast<float2*>(po) = make_float2(so[nn][e], so[nn][e + 1]);
+          } else if (t < n) {
+            if (col < j.V) po[0] = so[nn][e];
+            if (col + 1 < j.V) po[1] = so[nn][e + 1];
+          }
+        }
+    } else {                                          // S = e^(c_64) S + K^T U e^(c_64 - c)
+      const float fend = exp2f(cend);
+      const bf* Kb = K + buf * tile;
+#pragma unroll
+      for (int m = 0; m < 2; ++m)
+#pragma unroll
+        for (int nn = 0; nn < 2; ++nn)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) acc[m][nn][e] *= fend;
+#pragma unroll
+      for (int kb = 0; kb < CK / 16; ++kb) {
+        uint32_t bh[4], bl[4];
+        ck_ldsm_t(bh, Us + 2 * CK * VP + (kb * 16 + lr) * VP + wc * 16 + lc);
+        ck_ldsm_t(bl, Us + 3 * CK * VP + (kb * 16 + lr) * VP + wc * 16 + lc);
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+          const int c0 = (wr + 4 * m) * 16;
+          if (c0 >= D) continue;
+          // K lies by tokens: its transpose's 16 x 16 part, the halves of the tokens behind those of the channels
+          uint32_t ah[4], al[4];
+          const bf* kp = Kb + (kb * 16 + (lane & 7) + (lane >> 4) * 8) * DP + c0 + ((lane >> 3) & 1) * 8;
+          ck_ldsm_t(ah, kp);
+          ck_ldsm_t(al, kp + CK * DP);
+          ck_mma3(acc[m], ah, al, bh, bl);
+        }
+      }
+      if (i + 1 < chunks) share_state();
+    }
   }
   each_state([&](float& x, int row, int col) { if (v0 + col < j.V) S[(size_t)row * j.V + v0 + col] = x; });
 }
 
 struct ChunkPlan {
-  long long qs, qk, c, w, u0, total;     // floats
+  long long qs, qk, c, p, w, u0, total;     // floats
 };
 ChunkPlan chunk_plan(int slots, int H, int G, int D, int V, int delta) {
   ChunkPlan p = {};
   p.qs = (long long)slots * G * CK * D;                // Q, and as many for K: two bfloat16 parts are one float
   p.qk = (long long)slots * G * CK * CK;
   p.c = (long long)slots * H * CK;
+  p.p = (long long)slots * H * CK * CK;
   p.w = delta ? (long long)slots * H * CK * D : 0;
   p.u0 = delta ? (long long)slots * H * CK * V : 0;
-  p.total = 2 * p.qs + (delta ? 2 : 1) * p.qk + p.c + p.w + p.u0;
+  p.total = 2 * p.qs + (delta ? 2 : 1) * p.qk + p.c + p.p + p.w + p.u0;
   return p;
 }
 }  // namespace
@@ -577,6 +595,7 @@ extern "C" int zi_chunked_recurrence(float* out, int ldo, const float* q, int ld
   j.qk = at; at += p.qk;
   if (delta) { j.kk = at; at += p.qk; }
   j.c = at; at += p.c;
+  j.p = reinterpret_cast<bf*>(at); at += p.p;
   if (delta) {
     j.w = reinterpret_cast<bf*>(at); at += p.w;
     j.u0 = at;
@@ -589,6 +608,8 @@ extern "C" int zi_chunked_recurrence(float* out, int ldo, const float* q, int ld
   };
   const size_t score_smem = (size_t)2 * D * CS_PITCH * sizeof(float);
   int rc = launch(delta ? chunk_scores_kernel<true> : chunk_scores_kernel<false>, dim3(slots, G), CS_THREADS, score_smem, "chunk_scores");
+  if (rc) return rc;
+  rc = launch(chunk_weights_kernel, dim3(slots, H), CP_THREADS, 0, "chunk_weights");
   if (rc) return rc;
   if (delta) {
     const size_t solve_smem = ((size_t)CK * CS_PITCH + 2 * CK + (size_t)CK * NT) * sizeof(float);

@@ -10,8 +10,8 @@
 // leave the last taps-1 inputs of the step there after they have read the old ones.
 //
 // The channels are cut into segments of equal heads.  A warp takes one head of one tile of up to CH_TILE tokens: a lane
-// keeps the running inputs of its two channels in registers while it walks the tile, so every input is read once (plus
-// taps-1 before the tile).  A lane's two channels are those of a rotated pair: neighbours (2i, 2i+1), or (i, i + rot/2).
+// keeps the running inputs of its channels in registers while it walks the tile, so every input is read once (plus taps-1
+// before the tile).  A lane's channels come in the pairs that a rotation turns: neighbours (2i, 2i+1), or (i, i + rot/2).
 // 32-bit arithmetic throughout.
 #include "api.h"
 #include "common.cuh"
@@ -76,12 +76,14 @@ __device__ __forceinline__ float summed_at(const float* p, int splits, long long
 }
 
 // TAPS > 0: that many taps, inputs and weights in registers; 0: any number, inputs read again for every tap.
-// PAIRS: a lane's two channels are neighbours whose addresses allow 8-byte accesses.
-template <typename T, int TAPS, bool PAIRS>
+// NP pairs of neighbouring channels per lane (2 or 1), whose addresses allow accesses of 16 (8) bytes; 0: one pair, any
+// addresses, either pairing.
+template <typename T, int TAPS, int NP>
 __global__ void __launch_bounds__(CH_WARPS * 32)
 conv_heads_kernel(const ConvJob j) {
   pdl_launch_dependents();
   extern __shared__ float held_all[];
+  constexpr int NR = NP > 0 ? NP : 1;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int seq = j.tile_seq[blockIdx.x], q0 = j.tile_q0[blockIdx.x];      // the step's own arrays: here before any kernel of the step
   const int tok0 = j.cu_q[seq], qlen = j.cu_q[seq + 1] - tok0;
@@ -119,148 +121,188 @@ conv_heads_kernel(const ConvJob j) {
   const int ch0 = g.c0 + head * g.d;                    // its first channel
   const int taps = TAPS > 0 ? TAPS : j.taps;
   const int rot = g.finish == 2 ? j.rot_dims : 0, half = rot >> 1;
-  float* tail = j.tail + (size_t)j.state_slots[seq] * j.slot_stride;
+  float* tail = j.tail + (size_t)j.state_slots[seq] * j.slot_stride + ch0;
+  const float* src = j.src + (size_t)tok0 * j.ld + ch0;
   float* held = held_all + (size_t)warp * CH_TILE * j.smem_head;
 
-  // an input of the convolution: row `at` of this request's portion (negative: carried from before the step)
-  auto input = [&](int at, int e, float bias) {
-    if (at < 0) return tail[(size_t)(taps - 1 + at) * j.C + ch0 + e];
-    return summed_at(j.src + (size_t)(tok0 + at) * j.ld + ch0 + e, j.splits, j.zstride) + bias;
-  };
-  auto input2 = [&](int at, int e, float2 bias) {
-    const float* p = at < 0 ? tail + (size_t)(taps - 1 + at) * j.C + ch0 + e : j.src + (size_t)(tok0 + at) * j.ld + ch0 + e;
-    float2 v = *reinterpret_cast<const float2*>(p);
-    if (at < 0) return v;
-    for (int z = 1; z < j.splits; ++z) {
-      const float2 u = *reinterpret_cast<const float2*>(p + (size_t)z * j.zstride);
-      v.x += u.x;
-      v.y += u.y;
-    }
-    return make_float2(v.x + bias.x, v.y + bias.y);
-  };
-  // where a finished value goes
-  auto put = [&](int t, int e0, int e1, float y0, float y1, bool two) {
-    const size_t row = (size_t)(row0 + t);
-    if (g.dest == 0) {
-      float* o = static_cast<float*>(g.out) + row * g.ldo + (size_t)head * g.d;
-      if (PAIRS && two) {
-        *reinterpret_cast<float2*>(o + e0) = make_float2(y0, y1);
-      } else {
-        o[e0] = y0;
-        if (two) o[e1] = y1;
-      }
-      return;
-    }
-    T* o;
-    if (g.dest == 1) {
-      o = static_cast<T*>(g.out) + row * g.ldo + (size_t)head * g.d;
+  // NR pairs of channels at a time: channel e0 and e1 of pair r, a place `p` (floats) at which channel e0 of the first lies
+  auto read = [&](const float* p, int e0, int e1, float2 (&v)[NR]) {
+    if constexpr (NP == 2) {
+      const float4 x = *reinterpret_cast<const float4*>(p + e0);
+      v[0] = make_float2(x.x, x.y);
+      v[1] = make_float2(x.z, x.w);
+    } else if constexpr (NP == 1) {
+      v[0] = *reinterpret_cast<const float2*>(p + e0);
     } else {
-      const int page = tok_page[t];
-      if (page < 0) return;                             // a row that pads a captured batch
-      o = static_cast<T*>(g.out) + (((size_t)page * page_heads + head) * j.page_size + tok_off[t]) * g.d;
+      v[0] = make_float2(p[e0], p[e1]);
     }
-    if constexpr (PAIRS && sizeof(T) == 2) {
-      if (two) {
-        *reinterpret_cast<__nv_bfloat162*>(o + e0) = __floats2bfloat162_rn(y0, y1);
-        return;
-      }
-    }
-    o[e0] = from_f32<T>(y0);
-    if (two) o[e1] = from_f32<T>(y1);
   };
-
-  const int np = (d + 1) >> 1;
-  for (int p = lane; p < np; p += 32) {
-    int e0 = 2 * p, e1 = 2 * p + 1;
-    if (!PAIRS && !j.neighbours && p < half) {          // (i, i + rot/2); the channels that do not turn follow in twos
+  const int units = (d + 2 * NR - 1) / (2 * NR);        // of 2 NR channels
+  for (int p = lane; p < units; p += 32) {
+    int e0 = 2 * NR * p, e1 = e0 + 1;
+    if (NP == 0 && !j.neighbours && p < half) {         // (i, i + rot/2); the channels that do not turn follow in twos
       e0 = p;
       e1 = p + half;
     }
-    const bool two = e1 < d;
+    const bool two = NP > 0 || e1 < d;
     const int f1 = two ? e1 : e0;                       // a channel that exists
-    float2 ib = make_float2(0.f, 0.f), ob = ib;
-    if (j.in_bias) ib = make_float2(j.in_bias[ch0 + e0], j.in_bias[ch0 + f1]);
-    if (j.out_bias) ob = make_float2(j.out_bias[ch0 + e0], j.out_bias[ch0 + f1]);
-    auto fetch = [&](int at) {
-      if (PAIRS) return input2(at, e0, ib);
-      return make_float2(input(at, e0, ib.x), input(at, f1, ib.y));
+    float2 ib[NR], ob[NR];
+#pragma unroll
+    for (int r = 0; r < NR; ++r) ib[r] = ob[r] = make_float2(0.f, 0.f);
+    if (j.in_bias) read(j.in_bias + ch0, e0, f1, ib);
+    if (j.out_bias) read(j.out_bias + ch0, e0, f1, ob);
+    // the inputs of row `at` of this request's portion (negative: carried from before the step)
+    auto fetch = [&](int at, float2 (&v)[NR]) {
+      if (at < 0) {
+        read(tail + (size_t)(taps - 1 + at) * j.C, e0, f1, v);
+        return;
+      }
+      const float* x = src + (size_t)at * j.ld;
+      read(x, e0, f1, v);
+      for (int z = 1; z < j.splits; ++z) {
+        float2 y[NR];
+        read(x + (size_t)z * j.zstride, e0, f1, y);
+#pragma unroll
+        for (int r = 0; r < NR; ++r) {
+          v[r].x += y[r].x;
+          v[r].y += y[r].y;
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < NR; ++r) {
+        v[r].x += ib[r].x;
+        v[r].y += ib[r].y;
+      }
     };
     constexpr int W = TAPS > 0 ? TAPS : 1;
-    float2 win[W], k[W];
+    float2 win[W][NR], k[W][NR];
     if constexpr (TAPS > 0) {
 #pragma unroll
       for (int i = 0; i < TAPS; ++i) {
-        k[i] = make_float2(j.kern[(size_t)i * j.C + ch0 + e0], j.kern[(size_t)i * j.C + ch0 + f1]);
-        if (i > 0) win[i] = fetch(q0 - TAPS + i);       // inputs before the tile; every token shifts them down by one
+        read(j.kern + (size_t)i * j.C + ch0, e0, f1, k[i]);
+        if (i > 0) fetch(q0 - TAPS + i, win[i]);        // inputs before the tile; every token shifts them down by one
       }
     }
     constexpr int AHEAD = 4;                            // tokens whose inputs are asked for together
 #pragma unroll 1
     for (int t0 = 0; t0 < nt; t0 += AHEAD) {
-      float2 in[AHEAD];
+      float2 in[AHEAD][NR];
       if constexpr (TAPS > 0) {
 #pragma unroll
-        for (int u = 0; u < AHEAD; ++u) in[u] = t0 + u < nt ? fetch(q0 + t0 + u) : make_float2(0.f, 0.f);
+        for (int u = 0; u < AHEAD; ++u) fetch(q0 + min(t0 + u, nt - 1), in[u]);
       }
 #pragma unroll
       for (int u = 0; u < AHEAD; ++u) {
         const int t = t0 + u;
         if (t >= nt) break;
-        float2 acc = make_float2(0.f, 0.f);
+        float2 y[NR];
+#pragma unroll
+        for (int r = 0; r < NR; ++r) y[r] = make_float2(0.f, 0.f);
         if constexpr (TAPS > 0) {
 #pragma unroll
-          for (int i = 0; i + 1 < TAPS; ++i) win[i] = win[i + 1];
-          win[TAPS - 1] = in[u];
+          for (int r = 0; r < NR; ++r) {
 #pragma unroll
-          for (int i = 0; i < TAPS; ++i) {
-            acc.x = fmaf(k[i].x, win[i].x, acc.x);
-            acc.y = fmaf(k[i].y, win[i].y, acc.y);
+            for (int i = 0; i + 1 < TAPS; ++i) win[i][r] = win[i + 1][r];
+            win[TAPS - 1][r] = in[u][r];
+#pragma unroll
+            for (int i = 0; i < TAPS; ++i) {
+              y[r].x = fmaf(k[i][r].x, win[i][r].x, y[r].x);
+              y[r].y = fmaf(k[i][r].y, win[i][r].y, y[r].y);
+            }
           }
         } else {
           for (int i = 0; i < taps; ++i) {
-            const float2 x = fetch(q0 + t - (taps - 1) + i);
-            acc.x = fmaf(j.kern[(size_t)i * j.C + ch0 + e0], x.x, acc.x);
-            acc.y = fmaf(j.kern[(size_t)i * j.C + ch0 + f1], x.y, acc.y);
+            float2 x[NR], kk[NR];
+            fetch(q0 + t - (taps - 1) + i, x);
+            read(j.kern + (size_t)i * j.C + ch0, e0, f1, kk);
+#pragma unroll
+            for (int r = 0; r < NR; ++r) {
+              y[r].x = fmaf(kk[r].x, x[r].x, y[r].x);
+              y[r].y = fmaf(kk[r].y, x[r].y, y[r].y);
+            }
           }
         }
-        float y0 = acc.x + ob.x, y1 = acc.y + ob.y;
-        if (j.act == 1) {
-          y0 = conv_silu(y0);
-          y1 = conv_silu(y1);
+#pragma unroll
+        for (int r = 0; r < NR; ++r) {
+          y[r].x += ob[r].x;
+          y[r].y += ob[r].y;
+          if (j.act == 1) {
+            y[r].x = conv_silu(y[r].x);
+            y[r].y = conv_silu(y[r].y);
+          }
+          if (NR * p + r < half) {
+            const size_t at = (size_t)tok_pos[t] * half + NR * p + r;
+            rotate_pair(y[r].x, y[r].y, j.cos_t[at], j.sin_t[at]);
+          }
         }
         if (g.finish == 1) {
-          held[t * j.smem_head + e0] = y0;
-          if (two) held[t * j.smem_head + e1] = y1;
+#pragma unroll
+          for (int r = 0; r < NR; ++r) {
+            held[t * j.smem_head + e0 + 2 * r] = y[r].x;
+            if (two) held[t * j.smem_head + e1 + 2 * r] = y[r].y;
+          }
           continue;
         }
-        if (p < half) {
-          const size_t at = (size_t)tok_pos[t] * half + p;
-          rotate_pair(y0, y1, j.cos_t[at], j.sin_t[at]);
+        // where it goes
+        const size_t row = (size_t)(row0 + t);
+        if (g.dest == 0) {
+          float* o = static_cast<float*>(g.out) + row * g.ldo + (size_t)head * g.d;
+          if constexpr (NP == 2) {
+            *reinterpret_cast<float4*>(o + e0) = make_float4(y[0].x, y[0].y, y[1].x, y[1].y);
+          } else if constexpr (NP == 1) {
+            *reinterpret_cast<float2*>(o + e0) = y[0];
+          } else {
+            o[e0] = y[0].x;
+            if (two) o[e1] = y[0].y;
+          }
+          continue;
         }
-        put(t, e0, e1, y0, y1, two);
+        T* o;
+        if (g.dest == 1) {
+          o = static_cast<T*>(g.out) + row * g.ldo + (size_t)head * g.d;
+        } else {
+          if (tok_page[t] < 0) continue;                // a row that pads a captured batch
+          o = static_cast<T*>(g.out) + (((size_t)tok_page[t] * page_heads + head) * j.page_size + tok_off[t]) * g.d;
+        }
+        if constexpr (NP > 0 && sizeof(T) == 2) {
+          __nv_bfloat162 b[NR];
+#pragma unroll
+          for (int r = 0; r < NR; ++r) b[r] = __floats2bfloat162_rn(y[r].x, y[r].y);
+          if constexpr (NP == 2) *reinterpret_cast<uint2*>(o + e0) = make_uint2(*reinterpret_cast<uint32_t*>(&b[0]), *reinterpret_cast<uint32_t*>(&b[1]));
+          else *reinterpret_cast<__nv_bfloat162*>(o + e0) = b[0];
+        } else {
+#pragma unroll
+          for (int r = 0; r < NR; ++r) {
+            o[e0 + 2 * r] = from_f32<T>(y[r].x);
+            if (two) o[e1 + 2 * r] = from_f32<T>(y[r].y);
+          }
+        }
       }
     }
     if (q0 == 0) {                                      // the inputs that the next step finds; ascending rows overwrite in place
-      for (int r = 0; r < taps - 1; ++r) {
-        const float2 u = fetch(qlen - (taps - 1) + r);  // from before this step: row r + qlen of the old tail
-        float* o = tail + (size_t)r * j.C + ch0;
-        o[e0] = u.x;
-        if (two) o[e1] = u.y;
+      for (int i = 0; i < taps - 1; ++i) {
+        float2 u[NR];
+        fetch(qlen - (taps - 1) + i, u);                // from before this step: row i + qlen of the old tail
+        float* o = tail + (size_t)i * j.C;
+#pragma unroll
+        for (int r = 0; r < NR; ++r) {
+          o[e0 + 2 * r] = u[r].x;
+          if (two) o[e1 + 2 * r] = u[r].y;
+        }
       }
     }
   }
   if (g.finish == 1) {
-    for (int t = 0; t < nt; ++t) {                      // a lane reads its own values only
+    __syncwarp();
+    for (int t = 0; t < nt; ++t) {
       const float* x = held + t * j.smem_head;
       float ss = 0.f;
-      for (int p = lane; p < np; p += 32) {
-        ss = fmaf(x[2 * p], x[2 * p], ss);
-        if (2 * p + 1 < d) ss = fmaf(x[2 * p + 1], x[2 * p + 1], ss);
-      }
+      for (int e = lane; e < d; e += 32) ss = fmaf(x[e], x[e], ss);
       const float inv = g.scale / sqrtf(warp_sum(ss) + j.unit_eps);
-      for (int p = lane; p < np; p += 32) {
-        const bool two = 2 * p + 1 < d;
-        put(t, 2 * p, 2 * p + 1, x[2 * p] * inv, two ? x[2 * p + 1] * inv : 0.f, two);
+      const size_t at = (size_t)(row0 + t) * g.ldo + (size_t)head * g.d;
+      for (int e = lane; e < d; e += 32) {
+        if (g.dest == 0) static_cast<float*>(g.out)[at + e] = x[e] * inv;
+        else static_cast<T*>(g.out)[at + e] = from_f32<T>(x[e] * inv);
       }
     }
   }
@@ -291,7 +333,11 @@ extern "C" int zi_conv_heads(const float* src, int ld, int splits, long long zst
   j.n_seg = n_seg;
   int c = 0, heads = 0, widest = 0;
   auto al = [](const void* p, size_t n) { return p == nullptr || ((uintptr_t)p & (n - 1)) == 0; };
-  bool pairs = ld % 2 == 0 && zstride % 2 == 0 && C % 2 == 0 && slot_stride % 2 == 0 && al(src, 8) && al(tail, 8);
+  auto fits = [&](int n) {       // accesses of n floats
+    return ld % n == 0 && zstride % n == 0 && C % n == 0 && slot_stride % n == 0 && al(src, 4 * n) && al(tail, 4 * n) && al(kern, 4 * n) &&
+           al(in_bias, 4 * n) && al(out_bias, 4 * n);
+  };
+  int np = fits(4) ? 2 : (fits(2) ? 1 : 0);      // pairs of channels per lane
   for (int i = 0; i < n_seg; ++i) {
     ConvSegment& g = j.seg[i];
     g.c0 = c;
@@ -309,7 +355,9 @@ extern "C" int zi_conv_heads(const float* src, int ld, int splits, long long zst
     if (g.finish == 2 && (!cos_t || rot_dims > g.d)) return zi_refuse("conv_heads: %d rotated dimensions of a head of %d", rot_dims, g.d);
     if (g.dest == 2 && (!slots || page_size <= 0)) return zi_refuse("conv_heads: pages need slots");
     if (g.finish == 1 && g.d > widest) widest = g.d;
-    pairs = pairs && g.d % 2 == 0 && g.n % 2 == 0 && g.ldo % 2 == 0 && al(g.out, 8) && (g.finish != 2 || neighbours);
+    if (g.finish == 1 && g.dest == 2) return zi_refuse("conv_heads: unit vectors go to rows");
+    const size_t wide = g.dest == 0 ? 4 : (out_dtype == ZI_BF16 ? 2 : 4);
+    while (np > 0 && (g.d % (2 * np) || g.n % (2 * np) || g.ldo % (2 * np) || !al(g.out, 2 * np * wide) || (g.finish == 2 && !neighbours))) --np;
     c += g.n;
     heads += (g.n + g.d - 1) / g.d;
   }
@@ -328,23 +376,23 @@ extern "C" int zi_conv_heads(const float* src, int ld, int splits, long long zst
   const int rows_of_blocks = (heads + CH_WARPS - 1) / CH_WARPS + (scalars ? 1 : 0);
   if (rows_of_blocks > 65535) return zi_refuse("conv_heads: %d heads", heads);
   dim3 grid(n_tiles, rows_of_blocks), block(CH_WARPS * 32);
-#define ZI_CH(TT, TAPS, PAIRS)                                                                                            \
+#define ZI_CH(TT, TAPS, NP)                                                                                               \
   do {                                                                                                                    \
-    auto kern_fn = conv_heads_kernel<TT, TAPS, PAIRS>;                                                                    \
+    auto kern_fn = conv_heads_kernel<TT, TAPS, NP>;                                                                       \
     if (smem > 48 * 1024 && cudaFuncSetAttribute(kern_fn, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) \
       return zi_refuse("conv_heads: cannot get %zu bytes of shared memory", smem);                                        \
     zi_launch(kern_fn, grid, block, smem, stream, j);                                                                     \
   } while (0)
-#define ZI_CH_TAPS(TT, PAIRS)                          \
+#define ZI_CH_TAPS(TT, NP)                             \
   do {                                                 \
     switch (taps) {                                    \
-      case 2: ZI_CH(TT, 2, PAIRS); break;              \
-      case 3: ZI_CH(TT, 3, PAIRS); break;              \
-      case 4: ZI_CH(TT, 4, PAIRS); break;              \
-      default: ZI_CH(TT, 0, PAIRS); break;             \
+      case 2: ZI_CH(TT, 2, NP); break;                 \
+      case 3: ZI_CH(TT, 3, NP); break;                 \
+      case 4: ZI_CH(TT, 4, NP); break;                 \
+      default: ZI_CH(TT, 0, NP); break;                \
     }                                                  \
   } while (0)
-  ZI_DISPATCH_DTYPE(out_dtype, TT, { if (pairs) ZI_CH_TAPS(TT, true); else ZI_CH_TAPS(TT, false); });
+  ZI_DISPATCH_DTYPE(out_dtype, TT, { if (np == 2) ZI_CH_TAPS(TT, 2); else if (np == 1) ZI_CH_TAPS(TT, 1); else ZI_CH_TAPS(TT, 0); });
 #undef ZI_CH_TAPS
 #undef ZI_CH
   return zi_check_launch("conv_heads");

@@ -1018,6 +1018,59 @@ gated_part_norm_kernel(TO* __restrict__ out, int ldo, const float* __restrict__ 
   const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
   for (int i = threadIdx.x; i < n; i += blockDim.x) out[t * ldo + c0 + i] = from_f32<TO>(part[i] * inv * w[c0 + i]);
 }
+
+// The same in 16-byte pieces, a part's values in registers (parts of up to 4,096 values).
+template <typename TO>
+__global__ void __launch_bounds__(256)
+gated_part_norm_vec_kernel(TO* __restrict__ out, int ldo, const float* __restrict__ y, int ldy, const float* __restrict__ x, int ldx,
+                           const float* __restrict__ skip, int V, const float* __restrict__ z, int ldz, int splits, long long zstride,
+                           const float* __restrict__ w, float eps, int n) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float scratch[33];
+  constexpr int MAXV = 4;
+  const size_t t = blockIdx.x;
+  const int c0 = blockIdx.y * n;
+  auto at = [](const float* p) { return *reinterpret_cast<const float4*>(p); };
+  float4 v[MAXV];
+  float ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < MAXV; ++u) {
+    const int i = (u * blockDim.x + threadIdx.x) * 4, c = c0 + i;
+    v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < n) {
+      v[u] = at(y + t * ldy + c);
+      if (skip) {
+        const float4 xv = at(x + t * ldx + c);
+        const float s = skip[c / V];
+        v[u] = make_float4(fmaf(s, xv.x, v[u].x), fmaf(s, xv.y, v[u].y), fmaf(s, xv.z, v[u].z), fmaf(s, xv.w, v[u].w));
+      }
+      float4 g = at(z + t * ldz + c);
+      for (int k = 1; k < splits; ++k) {
+        const float4 h = at(z + (size_t)k * zstride + t * ldz + c);
+        g = make_float4(g.x + h.x, g.y + h.y, g.z + h.z, g.w + h.w);
+      }
+      v[u] = make_float4(v[u].x * g.x * sigmoid_f32(g.x), v[u].y * g.y * sigmoid_f32(g.y), v[u].z * g.z * sigmoid_f32(g.z),
+                         v[u].w * g.w * sigmoid_f32(g.w));
+      ss = fmaf(v[u].x, v[u].x, fmaf(v[u].y, v[u].y, fmaf(v[u].z, v[u].z, fmaf(v[u].w, v[u].w, ss))));
+    }
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
+#pragma unroll
+  for (int u = 0; u < MAXV; ++u) {
+    const int i = (u * blockDim.x + threadIdx.x) * 4, c = c0 + i;
+    if (i >= n) continue;
+    const float4 wv = at(w + c);
+    const float o[4] = {v[u].x * inv * wv.x, v[u].y * inv * wv.y, v[u].z * inv * wv.z, v[u].w * inv * wv.w};
+    TO* po = out + t * ldo + c;
+    if constexpr (sizeof(TO) == 4) {
+      *reinterpret_cast<float4*>(po) = make_float4(o[0], o[1], o[2], o[3]);
+    } else {
+      __nv_bfloat162 a = __floats2bfloat162_rn(o[0], o[1]), b = __floats2bfloat162_rn(o[2], o[3]);
+      *reinterpret_cast<uint2*>(po) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+    }
+  }
+}
 }  // namespace
 
 extern "C" int zi_gated_part_norm(void* out, int out_dtype, int ldo, const float* y, int ldy, const float* x, int ldx, const float* skip,
@@ -1031,6 +1084,13 @@ extern "C" int zi_gated_part_norm(void* out, int out_dtype, int ldo, const float
   const size_t smem = (size_t)n * sizeof(float);
   if (smem > 200 * 1024) return zi_refuse("gated_part_norm: parts of %d values are more than this kernel holds", n);
   const int threads = n >= 1024 ? 512 : (n >= 256 ? 256 : 128);
+  auto al16 = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+  if (n % 4 == 0 && n <= 4096 && ldo % 4 == 0 && ldy % 4 == 0 && ldz % 4 == 0 && zstride % 4 == 0 && al16(out) && al16(y) && al16(z) && al16(w) &&
+      (!skip || (V % 4 == 0 && ldx % 4 == 0 && al16(x)))) {
+    ZI_DISPATCH_DTYPE(out_dtype, TO, zi_launch(gated_part_norm_vec_kernel<TO>, dim3(T, parts), dim3(n > 2048 ? 256 : (n > 512 ? 128 : 64)), 0,
+                                               stream, (TO*)out, ldo, y, ldy, x, ldx, skip, V, z, ldz, splits, zstride, w, eps, n));
+    return zi_check_launch("gated_part_norm");
+  }
   ZI_DISPATCH_DTYPE(out_dtype, TO, {
     auto kern = gated_part_norm_kernel<TO>;
     if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)

@@ -2079,7 +2079,7 @@ def conv_heads(u: Columns, kernel: torch.Tensor, tail: Optional[torch.Tensor], s
         if dest:
             act_dtype = s.out.dtype
         # channels without a finish need no whole heads: short pieces spread them over more warps
-        d = 64 if finish is None and not paged else s.head_dim
+        d = 128 if finish is None and not paged else s.head_dim
         ints[5 * i:5 * i + 5] = [s.channels, d, _FINISHES[finish], dest, 0 if paged else s.out.stride(0)]
         outs[i], scales[i] = _ptr(s.out).value, s.scale
     _need(all(s.out.dtype in (torch.float32, act_dtype) for s in segments), "conv_heads: one activations' type")
