@@ -79,7 +79,7 @@ __device__ __forceinline__ float summed_at(const float* p, int splits, long long
 // NP pairs of neighbouring channels per lane (2 or 1), whose addresses allow accesses of 16 (8) bytes; 0: one pair, any
 // addresses, either pairing.
 template <typename T, int TAPS, int NP>
-__global__ void __launch_bounds__(CH_WARPS * 32)
+__global__ void __launch_bounds__(CH_WARPS * 32, 4)
 conv_heads_kernel(const ConvJob j) {
   pdl_launch_dependents();
   extern __shared__ float held_all[];
