@@ -174,23 +174,6 @@ def plain_logits(cfg, weights, reqs):
     return {rid: P.PlainSumozen(cfg, weights).forward(toks).numpy() for rid, toks in reqs.items()}
 
 
-def router_margin(cfg, weights, toks):
-    """The plain model's smallest gap, over tokens and layers, between the last chosen router logit and the next."""
-    gaps, keep = [], P.choose
-
-    def spy(s, top):
-        z = sorted((torch.logit(torch.tensor(s, dtype=torch.float64))).tolist(), reverse=True)
-        if top < len(z):
-            gaps.append(z[top - 1] - z[top])
-        return keep(s, top)
-    P.choose = spy
-    try:
-        P.PlainSumozen(cfg, weights).forward(toks)
-    finally:
-        P.choose = keep
-    return min(gaps, default=float("inf"))
-
-
 def clear_requests(cfg, weights, lengths, seed, margin=0.05):
     """Requests whose routers have no close call (which rounding could decide otherwise): tokens are drawn one after the
     other, and drawn again where a choice would be close."""
